@@ -27,7 +27,8 @@ class RMSNormSpec:
     ``weight_offset``: the row is scaled by ``weight_offset + weight`` (1.0 for a weight that is stored as its
     deviation from one).  ``scale_in_fp32``: the scaling is done in fp32 before the one rounding to the compute
     dtype, y = cast(x * rsqrt(mean(x^2) + eps) * (weight_offset + weight)).  ``scalar_weight``: the stored weight
-    is a single number (a tensor without dimensions) that scales every coordinate."""
+    is a single number (a tensor without dimensions) that scales every coordinate.  ``output_scale``: one more factor
+    of the whole row, taken into the weight in fp32 at load (a final norm with it scales the logits)."""
 
     size: int
     eps: float
@@ -35,6 +36,7 @@ class RMSNormSpec:
     weight_offset: float = 0.0
     scale_in_fp32: bool = False
     scalar_weight: bool = False
+    output_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -139,6 +141,38 @@ class CappedAttentionSpec:
 
 
 @dataclass(frozen=True)
+class MixedAttentionSpec:
+    """Grouped-query causal attention inside chunks whose heads mix their scores before the softmax.
+
+    q and k heads have ``head_dim`` lanes, v heads ``value_dim``; query head h goes with key/value head
+    h // (heads / kv_heads).  With ``row_norm_eps`` not None the whole q projection of a token (all heads' lanes at
+    once) is RMS-normed with the plain weight q_norm, and the whole k projection with k_norm, before ``position``
+    rotates half-split pairs of the first lanes of each head.  score_h = ``scale`` q_h . k; with the role talk (a
+    [heads, heads] matrix T) score_h <- sum_g T[h, g] score_g.  ``chunk`` c not None: position p sees j <= p only if
+    p // c == j // c, counted from the sequence's start.  Ordinary softmax over the visible keys; norms, rotation,
+    scores and softmax are fp32.  ``names`` maps the roles q, k, v, o, q_norm, k_norm, talk to tensor names below
+    ``prefix``."""
+
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_dim: int
+    scale: float
+    position: object
+    prefix: str
+    names: Tuple[Tuple[str, str], ...]
+    row_norm_eps: Optional[float] = None
+    chunk: Optional[int] = None
+
+    def name(self, role: str) -> str:
+        return self.prefix + dict(self.names)[role]
+
+    def has(self, role: str) -> bool:
+        return role in dict(self.names)
+
+
+@dataclass(frozen=True)
 class LatentAttentionSpec:
     """Causal attention whose keys and values are up-projections of one cached latent row per position.
 
@@ -217,6 +251,30 @@ class ChannelDeltaSpec:
 
 
 @dataclass(frozen=True)
+class HeadDeltaSpec:
+    """Gated delta rule with one decay per head (a recurrent mixer with a matrix state per head).
+
+    q, k, v, their convolutions with SiLU, the unit vectors and the recurrence as in :class:`ChannelDeltaSpec`, but
+    the decay is one number per head, g = exp(-exp(A_log) softplus(a x + dt_bias)) with one row of a per head, and the
+    normed read-out is multiplied by silu(g x), g a full projection with one row per lane.  ``names`` maps the roles
+    q, k, v, q_conv, k_conv, v_conv, b, A_log, dt_bias, a, g, norm, o to tensor names below ``prefix``."""
+
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    qk_dim: int
+    v_dim: int
+    conv_taps: int
+    norm_eps: float
+    prefix: str
+    names: Tuple[Tuple[str, str], ...]
+    unit_eps: float = 1e-6
+
+    def name(self, role: str) -> str:
+        return self.prefix + dict(self.names)[role]
+
+
+@dataclass(frozen=True)
 class RoutedExpertsSpec:
     """Mixture of experts with a grouped top-k router, identity outputs and an optional shared expert.
 
@@ -228,7 +286,10 @@ class RoutedExpertsSpec:
     down(g * sigmoid(``gate_alpha`` g) * (u + 1)), g = min(gate x, ``limit``), u = clamp(up x, +-``limit``).
     ``shared_size`` > 0 adds one expert of that form (its own ``shared_limit``) for every token.
     ``scoring`` "sigmoid": the score of an output is the logistic function of its logit instead of the softmax.
-    ``expert_form`` "relu2": an expert (and the shared one) is down(max(up x, 0)^2), without gate, limit or bias.
+    ``expert_form`` "relu2": an expert (and the shared one) is down(max(up x, 0)^2), without gate, limit or bias;
+    "gated_silu": down(silu(gate x) * (up x)), without limits.
+    ``renormalise``: the chosen outputs' scores are divided by their sum (+ 1e-20) before they weigh; ``weight_scale``
+    multiplies every weight.
     ``weight_on_input``: a chosen expert's weight multiplies its input, out = sum_k expert_k(w_k x), not its output.
     Tensor names below ``prefix``: ``router``, ``correction``, ``e<i>.gate|up|down``, ``shared.gate|up|down``
     (no ``gate`` tensors for ungated experts)."""
@@ -249,6 +310,8 @@ class RoutedExpertsSpec:
     scoring: str = "softmax"
     expert_form: str = "gated_clamp"
     weight_on_input: bool = False
+    renormalise: bool = False
+    weight_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -382,16 +445,20 @@ class TokenSideInputSpec:
 
 @dataclass(frozen=True)
 class GatedMLPSpec:
-    """Dense gated feed-forward: down(act(gate(x)) * up(x)), no biases."""
+    """Dense gated feed-forward: down(act(gate(x)) * up(x)).  ``names`` maps the roles gate, up, down to tensor names
+    below ``prefix``; when it also names gate_bias, up_bias or down_bias, that projection adds the bias."""
 
     hidden_size: int
     intermediate_size: int
-    activation: str  # "silu"
+    activation: str  # "silu" or "gelu_tanh"
     prefix: str
     names: Tuple[Tuple[str, str], ...]
 
     def name(self, role: str) -> str:
         return self.prefix + dict(self.names)[role]
+
+    def has(self, role: str) -> bool:
+        return role in dict(self.names)
 
 
 @dataclass(frozen=True)
@@ -415,6 +482,25 @@ class SandwichBlockSpec:
     ffn_norm: object    # the three of the feed-forward are None together: the layer has none
     ffn: object
     ffn_post_norm: object
+
+
+@dataclass(frozen=True)
+class GatedPostNormBlockSpec:
+    """x <- x + norm1(mixer(x) * sigmoid(R1 x + r1)); x <- x + norm2(feed_forward(x) * sigmoid(R2 x + r2)): the
+    sublayers read the stream itself, and what they add is gated lane by lane by the stream and then normed.  The
+    gates' weights are [hidden, hidden] matrices with a bias (``*_gate_name``, ``*_gate_bias_name``); a gate name of
+    None leaves that gate out.  ``ffn`` None (with its norm and gate): the layer has no feed-forward.  Gates, norms and
+    sums are fp32."""
+
+    mixer: object
+    mixer_norm: object
+    ffn: object
+    ffn_norm: object
+    hidden_size: int
+    mixer_gate_name: Optional[str] = None
+    mixer_gate_bias_name: Optional[str] = None
+    ffn_gate_name: Optional[str] = None
+    ffn_gate_bias_name: Optional[str] = None
 
 
 @dataclass(frozen=True)

@@ -12,6 +12,10 @@
 // the softmax is the running-maximum form in fp32; the output accumulates in fp32.
 // Key j is visible to the query at position p iff j <= p and (window == 0 or j > p - window or j < keep):
 // with keep > 0 a windowed layer goes on seeing the first `keep` positions of its sequence.
+// With chunk c > 0 (instead of a window) the query at position p sees the keys of its own chunk of c positions only:
+// j <= p and j / c == p / c.
+// With mixed = 1 a query head has nkv * D lanes, one query of D lanes for every key head, and its score is the sum of
+// their dot products with all key heads of the position (heads that mix their scores; the values stay grouped).
 // With softcap c > 0 a score s (already times scale) becomes c tanh(s / c) before the softmax.
 // With sink = 1 the softmax has one more term, of score 0 and without a value: p_j = e^(s_j) / (1 + sum e^(s_k)).
 //
@@ -59,6 +63,8 @@ struct AttnArgs {
   float scale, softcap;
   int sink;             // 1: the softmax has one more term of score 0 and no value (one is added to its denominator)
   int keep;             // > 0 with a window: keys 0..keep-1 stay visible beyond the window
+  int chunk;            // > 0: keys of the query's own chunk of this many positions
+  int mixed;            // 1: q is [n_tokens, nq, nkv, D]; a score sums over the key heads
 };
 
 // 1 / (l + e^-m) for sums l taken relative to the maximum m: the denominator with the sink's term, without overflow.
@@ -95,7 +101,7 @@ attention_simt_kernel(AttnArgs a) {
   const int pos_lo = past + t0, pos_hi = past + t0 + nt - 1;
 
   // Key range seen by any row of the tile, cut into tiles of KT, then into splits.
-  int k_lo = a.window > 0 ? max(0, pos_lo - a.window + 1) : 0;
+  int k_lo = a.window > 0 ? max(0, pos_lo - a.window + 1) : (a.chunk > 0 ? pos_lo - pos_lo % a.chunk : 0);
   k_lo = (k_lo / KT) * KT;
   // the tiles of kept first keys that lie in front of the window's first tile come first in the walk
   const int keep_tiles = a.window > 0 && a.keep > 0 ? min((a.keep + KT - 1) / KT, k_lo / KT) : 0;
@@ -103,25 +109,31 @@ attention_simt_kernel(AttnArgs a) {
   const int per_split = (n_tiles + a.splits - 1) / a.splits;
   const int tile_begin = split * per_split, tile_end = min(n_tiles, tile_begin + per_split);
 
-  // Stage the query rows (fp32).  Row r: token t0 + r / hpb, head chunk*16 + r % hpb.
-  for (int i = tid; i < ROWS * D; i += NWARPS * 32) {
-    const int r = i / D, dd = i % D;
-    float v = 0.f;
-    if (r < nrows) {
-      const int tok = q_begin + t0 + r / hpb;
-      const int h = hk * g + chunk * 16 + r % hpb;
-      v = to_f<T>(((const T*)a.q)[((size_t)tok * a.nq + h) * D + dd]);
+  // Stage the query rows (fp32).  Row r: token t0 + r / hpb, head chunk*16 + r % hpb; with mixed heads the part of them
+  // that goes with key head kh.
+  auto stage_queries = [&](int kh) {
+    for (int i = tid; i < ROWS * D; i += NWARPS * 32) {
+      const int r = i / D, dd = i % D;
+      float v = 0.f;
+      if (r < nrows) {
+        const int tok = q_begin + t0 + r / hpb;
+        const int h = hk * g + chunk * 16 + r % hpb;
+        const size_t at = (size_t)tok * a.nq + h;
+        v = to_f<T>(((const T*)a.q)[(a.mixed ? at * a.nkv + kh : at) * D + dd]);
+      }
+      Qs[i] = v;
     }
-    Qs[i] = v;
-  }
+  };
+  if (!a.mixed) stage_queries(0);
 
   float m[RW], l[RW], acc[RW][NACC];
-  int rpos[RW];
+  int rpos[RW], rold[RW];       // position of the row's query, and the oldest key of its window or chunk
 #pragma unroll
   for (int r = 0; r < RW; ++r) {
     m[r] = -INFINITY; l[r] = 0.f;
     const int row = warp * RW + r;
     rpos[r] = row < nrows ? past + t0 + row / hpb : -1;
+    rold[r] = a.window > 0 ? rpos[r] - a.window + 1 : (a.chunk > 0 && rpos[r] >= 0 ? rpos[r] - rpos[r] % a.chunk : 0);
 #pragma unroll
     for (int i = 0; i < NACC; ++i) acc[r][i] = 0.f;
   }
@@ -129,68 +141,73 @@ attention_simt_kernel(AttnArgs a) {
   const int* pages = a.page_ids + a.page_start[seq];
   for (int tile = tile_begin; tile < tile_end; ++tile) {
     const int kbase = tile < keep_tiles ? tile * KT : k_lo + (tile - keep_tiles) * KT;
-    __syncthreads();  // previous tile fully consumed (also orders the Qs writes)
     // All KT keys of a tile lie in one page (page_size is a multiple of KT).
     const int page = pages[page_slot_of(kbase, a.page_size, a.ring_pages)];
-    const size_t base = (((size_t)page * a.nkv + hk) * a.page_size + (kbase % a.page_size)) * D;
-    const T* kp = (const T*)a.k_pool + base;
     const int nkeys = min(KT, pos_hi + 1 - kbase);
-    if (D % 8 == 0 && ((uintptr_t)kp % 16) == 0) {
-      // eight lanes of a row at a time (16-byte loads of bf16, two of floats)
-      for (int i = tid * 8; i < KT * D; i += NWARPS * 32 * 8) {
-        const int j = i / D, dd = i % D;
-        float v[8];
-        if (j < nkeys) {
-          if (sizeof(T) == 2) {
-            const uint4 raw = *(const uint4*)(kp + i);
-            const __nv_bfloat162* h2 = (const __nv_bfloat162*)&raw;
-#pragma unroll
-            for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(h2[e]); v[2 * e] = f.x; v[2 * e + 1] = f.y; }
-          } else {
-            const float4 lo = *(const float4*)(kp + i), hi = *(const float4*)(kp + i + 4);
-            v[0] = lo.x; v[1] = lo.y; v[2] = lo.z; v[3] = lo.w; v[4] = hi.x; v[5] = hi.y; v[6] = hi.z; v[7] = hi.w;
-          }
-        } else {
-#pragma unroll
-          for (int e = 0; e < 8; ++e) v[e] = 0.f;
-        }
-        *(float4*)&Ks[j * KSTR + dd] = make_float4(v[0], v[1], v[2], v[3]);
-        *(float4*)&Ks[j * KSTR + dd + 4] = make_float4(v[4], v[5], v[6], v[7]);
-      }
-    } else {
-      for (int i = tid; i < KT * D; i += NWARPS * 32) {
-        const int j = i / D, dd = i % D;
-        Ks[j * KSTR + dd] = j < nkeys ? to_f<T>(kp[i]) : 0.f;
-      }
-    }
-#if !ODI_SHARED_KV
-    const T* vp = (const T*)a.v_pool +
-                  (((size_t)page * a.nkv + hk) * a.page_size + (kbase % a.page_size)) * DV;
-    for (int i = tid; i < KT * DV; i += NWARPS * 32) Vs[i] = i / DV < nkeys ? to_f<T>(vp[i]) : 0.f;
-#endif
-    __syncthreads();
-
-    // scores: lane = key
     float s[RW];
 #pragma unroll
     for (int r = 0; r < RW; ++r) s[r] = 0.f;
-    const float* krow = Ks + lane * KSTR;
-    const float* qrow = Qs + (warp * RW) * D;
-#pragma unroll 4
-    for (int dd = 0; dd < D; dd += 4) {
-      const float4 kv = *(const float4*)(krow + dd);
+    const int kh_first = a.mixed ? 0 : hk, kh_last = a.mixed ? a.nkv - 1 : hk;
+    for (int kh = kh_first; kh <= kh_last; ++kh) {
+      __syncthreads();  // previous tile fully consumed (also orders the Qs writes)
+      if (a.mixed) stage_queries(kh);
+      const size_t base = (((size_t)page * a.nkv + kh) * a.page_size + (kbase % a.page_size)) * D;
+      const T* kp = (const T*)a.k_pool + base;
+      if (D % 8 == 0 && ((uintptr_t)kp % 16) == 0) {
+        // eight lanes of a row at a time (16-byte loads of bf16, two of floats)
+        for (int i = tid * 8; i < KT * D; i += NWARPS * 32 * 8) {
+          const int j = i / D, dd = i % D;
+          float v[8];
+          if (j < nkeys) {
+            if (sizeof(T) == 2) {
+              const uint4 raw = *(const uint4*)(kp + i);
+              const __nv_bfloat162* h2 = (const __nv_bfloat162*)&raw;
 #pragma unroll
-      for (int r = 0; r < RW; ++r) {
-        const float4 qv = *(const float4*)(qrow + r * D + dd);
-        s[r] = fmaf(qv.x, kv.x, s[r]); s[r] = fmaf(qv.y, kv.y, s[r]);
-        s[r] = fmaf(qv.z, kv.z, s[r]); s[r] = fmaf(qv.w, kv.w, s[r]);
+              for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(h2[e]); v[2 * e] = f.x; v[2 * e + 1] = f.y; }
+            } else {
+              const float4 lo = *(const float4*)(kp + i), hi = *(const float4*)(kp + i + 4);
+              v[0] = lo.x; v[1] = lo.y; v[2] = lo.z; v[3] = lo.w; v[4] = hi.x; v[5] = hi.y; v[6] = hi.z; v[7] = hi.w;
+            }
+          } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = 0.f;
+          }
+          *(float4*)&Ks[j * KSTR + dd] = make_float4(v[0], v[1], v[2], v[3]);
+          *(float4*)&Ks[j * KSTR + dd + 4] = make_float4(v[4], v[5], v[6], v[7]);
+        }
+      } else {
+        for (int i = tid; i < KT * D; i += NWARPS * 32) {
+          const int j = i / D, dd = i % D;
+          Ks[j * KSTR + dd] = j < nkeys ? to_f<T>(kp[i]) : 0.f;
+        }
+      }
+#if !ODI_SHARED_KV
+      const T* vp = (const T*)a.v_pool +
+                    (((size_t)page * a.nkv + hk) * a.page_size + (kbase % a.page_size)) * DV;
+      if (kh == kh_first)
+        for (int i = tid; i < KT * DV; i += NWARPS * 32) Vs[i] = i / DV < nkeys ? to_f<T>(vp[i]) : 0.f;
+#endif
+      __syncthreads();
+
+      // scores: lane = key
+      const float* krow = Ks + lane * KSTR;
+      const float* qrow = Qs + (warp * RW) * D;
+#pragma unroll 4
+      for (int dd = 0; dd < D; dd += 4) {
+        const float4 kv = *(const float4*)(krow + dd);
+#pragma unroll
+        for (int r = 0; r < RW; ++r) {
+          const float4 qv = *(const float4*)(qrow + r * D + dd);
+          s[r] = fmaf(qv.x, kv.x, s[r]); s[r] = fmaf(qv.y, kv.y, s[r]);
+          s[r] = fmaf(qv.z, kv.z, s[r]); s[r] = fmaf(qv.w, kv.w, s[r]);
+        }
       }
     }
     const int kj = kbase + lane;
     float* prow = Ps + (warp * RW) * KT;
 #pragma unroll
     for (int r = 0; r < RW; ++r) {
-      const bool vis = rpos[r] >= 0 && kj <= rpos[r] && (a.window == 0 || kj > rpos[r] - a.window || kj < a.keep);
+      const bool vis = rpos[r] >= 0 && kj <= rpos[r] && (kj >= rold[r] || kj < a.keep);
       float sc = s[r] * a.scale;
       if (a.softcap > 0.f) sc = a.softcap * tanhf(sc / a.softcap);
       if (!vis) sc = -INFINITY;
@@ -291,7 +308,8 @@ extern "C" int odi_attention_simt(const AttnArgs* args, int max_q_len, int n_tok
                                   cudaStream_t stream) {
   AttnArgs a = *args;
   if (a.n_seqs <= 0 || n_tokens <= 0) return 0;
-  if (a.nq % a.nkv != 0 || a.page_size % KT != 0 || a.splits < 1 || a.n_seqs > 65535 || a.keep < 0)
+  if (a.nq % a.nkv != 0 || a.page_size % KT != 0 || a.splits < 1 || a.n_seqs > 65535 || a.keep < 0 || a.chunk < 0 ||
+      (a.chunk > 0 && (a.window > 0 || a.keep > 0)) || (a.mixed && ODI_SHARED_KV))
     return ODI_ERR_UNSUPPORTED;
   const int g = a.nq / a.nkv;
   const int hpb = g < 16 ? g : 16;

@@ -51,6 +51,8 @@
 #define EPI_SWIGLU 3
 #define EPI_HEAD_PREP 4    // the rows of w are q, k and v heads of 128: per-head norm, rotation, cache write
 #define EPI_GELU 5         // bf16 out = gelu(acc), the exact (erf) form
+#define EPI_GEGLU 6        // bf16 out = gelu(acc_gate) * acc_up, the tanh form of GELU; weight rows as for EPI_SWIGLU
+#define EPI_IS_GATED(e) ((e) == EPI_SWIGLU || (e) == EPI_GEGLU)
 
 #define BM 128             // token rows per CTA (the lanes of its tensor memory); a tile has 2 * BM
 #define BN 256             // accumulator columns per tile
@@ -149,6 +151,10 @@ __host__ __device__ constexpr uint32_t instr_desc_bf16(int m, int n) {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
 }
 __device__ __forceinline__ float silu_f(float g) { return g / (1.f + __expf(-g)); }
+// 0.5 g (1 + tanh y) = g sigmoid(2 y), y = sqrt(2/pi) (g + 0.044715 g^3)
+__device__ __forceinline__ float gelu_tanh_f(float g) {
+  return g / (1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * g * g, g, g)));
+}
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f)); }
 
 // ------------------------------------------------------------------------------ the kernel
@@ -311,7 +317,7 @@ template <int EPI>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 1)
 gemm_prefill_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                          const __grid_constant__ CUtensorMap map_out, const PrefillGemmArgs a) {
-  constexpr bool GATE = EPI == EPI_SWIGLU;
+  constexpr bool GATE = EPI_IS_GATED(EPI);
   constexpr int OUT_PER_TILE = GATE ? BN / 2 : BN;      // output features a tile covers
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -470,8 +476,8 @@ gemm_prefill_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 #pragma unroll
               for (int i = 0; i < 4; ++i) {
                 const int e = 8 * q + 2 * i;
-                const float lo = GATE ? silu_f(v[e]) * u[e] : (EPI == EPI_GELU ? gelu_erf_f(v[e]) : v[e]);
-                const float hi = GATE ? silu_f(v[e + 1]) * u[e + 1] : (EPI == EPI_GELU ? gelu_erf_f(v[e + 1]) : v[e + 1]);
+                const float lo = GATE ? (EPI == EPI_GEGLU ? gelu_tanh_f(v[e]) : silu_f(v[e])) * u[e] : (EPI == EPI_GELU ? gelu_erf_f(v[e]) : v[e]);
+                const float hi = GATE ? (EPI == EPI_GEGLU ? gelu_tanh_f(v[e + 1]) : silu_f(v[e + 1])) * u[e + 1] : (EPI == EPI_GELU ? gelu_erf_f(v[e + 1]) : v[e + 1]);
                 __nv_bfloat162 pr = __floats2bfloat162_rn(lo, hi);
                 w[i] = *(uint32_t*)&pr;
               }
@@ -586,7 +592,7 @@ extern "C" int odi_gemm_prefill_bf16(const void* x, const void* w, void* out, in
                                      int* flags, int n_flags, int balance, cudaStream_t stream) {
   if (tokens <= 0 || n_out <= 0) return 0;
   if (K <= 0 || K % 8 != 0 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || status == nullptr) return ODI_ERR_UNSUPPORTED;
-  const bool gate = epi == EPI_SWIGLU, heads = epi == EPI_HEAD_PREP;
+  const bool gate = EPI_IS_GATED(epi), heads = epi == EPI_HEAD_PREP;
   if (gate ? w_rows != 2 * n_out : w_rows != n_out) return ODI_ERR_ARGUMENT;
   const bool f32 = epi == EPI_STORE_F32 || epi == EPI_RESIDUAL;
   if (!heads && (((uintptr_t)out & 15) || ((long)ldo * (f32 ? 4 : 2)) % 16 != 0)) return ODI_ERR_UNSUPPORTED;
@@ -657,6 +663,7 @@ extern "C" int odi_gemm_prefill_bf16(const void* x, const void* w, void* out, in
     case EPI_STORE_F32: return launch<EPI_STORE_F32>(mx, mw, mo, a, sms, stream);
     case EPI_RESIDUAL: return launch<EPI_RESIDUAL>(mx, mw, mo, a, sms, stream);
     case EPI_SWIGLU: return launch<EPI_SWIGLU>(mx, mw, mo, a, sms, stream);
+    case EPI_GEGLU: return launch<EPI_GEGLU>(mx, mw, mo, a, sms, stream);
     case EPI_HEAD_PREP: return launch<EPI_HEAD_PREP>(mx, mw, mo, a, sms, stream);
   }
   return ODI_ERR_ARGUMENT;

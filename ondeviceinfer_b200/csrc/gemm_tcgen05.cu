@@ -36,6 +36,7 @@
 #define EPI_SWIGLU 3       // out_bf16[token, n] = silu(acc_gate) * acc_up   (DUAL)
 #define EPI_HEAD_PREP 4    // the rows are q, k and v heads of 128: per-head norm, rotation, cache write
 #define EPI_GELU 5         // out_bf16[token, n] = gelu(acc), the exact (erf) form
+#define EPI_GEGLU 6        // out_bf16[token, n] = gelu(acc_gate) * acc_up, the tanh form of GELU   (DUAL)
 
 #define BM 128             // features per tile (UMMA M)
 #define BK 64              // k per stage: 64 bf16 = one 128-byte swizzle row
@@ -204,6 +205,10 @@ __host__ __device__ constexpr uint32_t instr_desc_bf16(int m, int n) {
 }
 
 __device__ __forceinline__ float silu_f(float g) { return g / (1.f + __expf(-g)); }
+// 0.5 g (1 + tanh y) = g sigmoid(2 y), y = sqrt(2/pi) (g + 0.044715 g^3)
+__device__ __forceinline__ float gelu_tanh_f(float g) {
+  return g / (1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * g * g, g, g)));
+}
 
 // One warp finishes one head of one token: `vals` holds the head's 128 projections (already rounded
 // to bf16), lane i takes elements 4i .. 4i+3, whose rotation partners sit in lane i ^ 16.  The
@@ -271,6 +276,7 @@ __device__ __forceinline__ float emit(const GemmArgs& a, int token, int n, float
   else if (EPI == EPI_STORE_F32) ((float*)a.out)[at] = v;
   else if (EPI == EPI_RESIDUAL) { const float r = ((float*)a.out)[at] + v; ((float*)a.out)[at] = r; return r; }
   else if (EPI == EPI_SWIGLU) ((bf16*)a.out)[at] = __float2bfloat16_rn(silu_f(v) * v2);
+  else if (EPI == EPI_GEGLU) ((bf16*)a.out)[at] = __float2bfloat16_rn(gelu_tanh_f(v) * v2);
   else if (EPI == EPI_GELU) ((bf16*)a.out)[at] = __float2bfloat16_rn(0.5f * v * (1.0f + erff(v * 0.70710678118654752440f)));
   return 0.f;
 }
@@ -899,6 +905,9 @@ static int dispatch_epi(int epi, const CUtensorMap& mw, const CUtensorMap& mx, c
     case EPI_SWIGLU:
       if constexpr (BN <= 128 && !(CLUSTER && BN > 64)) return launch<BN, true, EPI_SWIGLU, CLUSTER>(mw, mx, a, grid, stream);
       else return ODI_ERR_UNSUPPORTED;
+    case EPI_GEGLU:
+      if constexpr (BN <= 64) return launch<BN, true, EPI_GEGLU, CLUSTER>(mw, mx, a, grid, stream);
+      else return ODI_ERR_UNSUPPORTED;
   }
   return ODI_ERR_ARGUMENT;
 }
@@ -910,7 +919,7 @@ extern "C" long odi_gemm_bf16_scratch_floats(int tokens, int n_out, int bn, int 
   return tiles * splits * (dual ? 2 : 1) * bn * BM;
 }
 
-// x [tokens, K] bf16, w [w_rows, K] bf16 (for EPI_SWIGLU w holds the gate rows followed by
+// x [tokens, K] bf16, w [w_rows, K] bf16 (for EPI_SWIGLU and EPI_GEGLU w holds the gate rows followed by
 // the up rows and n_out = w_rows / 2), out [tokens, ldo]; bias: null or fp32 [w_rows], added to the product.
 // no_loads != 0: the self-test of the bounded waits (see GemmArgs); the result is invalid by design.
 // Tiles of 128 features x bn tokens, bn in {16, 32, 64, 128, 256}, K splits allowed; cluster != 0 lets 2..8 splits
@@ -930,7 +939,7 @@ extern "C" int odi_gemm_bf16(const void* x, const void* w, void* out, int tokens
   const bool clustered = cluster && splits > 1 && splits <= 8 && bn <= 64;
   if (splits > 1 && !clustered && (scratch == nullptr || tickets == nullptr)) return ODI_ERR_ARGUMENT;
   if (status == nullptr) return ODI_ERR_ARGUMENT;
-  const bool dual = epi == EPI_SWIGLU;
+  const bool dual = epi == EPI_SWIGLU || epi == EPI_GEGLU;
   if (dual && w_rows != 2 * n_out) return ODI_ERR_ARGUMENT;
   CUtensorMap mw, mx;
   int rc = make_map(&mw, w, w_rows, K, BM);

@@ -10,7 +10,7 @@
 //    order reads row `row_index[i] / index_div` of A (row i itself if row_index is null) and writes row i of C.
 //
 // Epilogues: 0 store as T, 1 store as fp32, 2 gated and clamped (W_g holds N gate rows then N up rows;
-// g = min(gate, limit), u = clamp(up, -limit, limit), C = g * sigmoid(alpha * g) * (u + 1) as T), 3 the exact
+// g = min(gate, limit), u = clamp(up, -limit, limit), C = g * sigmoid(alpha * g) * (u + up_shift) as T), 3 the exact
 // (erf) GELU of the sum as T, 4 its tanh form, 5 the square of max(sum, 0) as T.
 //
 // Tile: TM rows x 64 features per block of 256 threads, K in slices of 16 or 32 through shared memory (fp32).
@@ -41,7 +41,7 @@ struct GroupedArgs {
   const int* n_tiles;
   long long a_group_off, w_group_stride, c_group_off;
   int lda, ldw, ldc, M, N, K, groups, index_div, epi;
-  float limit, alpha;
+  float limit, alpha, up_shift;
 };
 
 // Eight consecutive elements of a row as floats (16-byte loads; the caller has checked the alignment).
@@ -173,7 +173,7 @@ grouped_gemm_kernel(GroupedArgs a) {
       if (GATED) {
         const float g = fminf(acc[0][i][j], a.limit);
         const float u = fminf(fmaxf(acc[GATED ? 1 : 0][i][j], -a.limit), a.limit);
-        ((T*)a.C)[crow + n] = from_f<T>(g / (1.f + expf(-a.alpha * g)) * (u + 1.f));
+        ((T*)a.C)[crow + n] = from_f<T>(g / (1.f + expf(-a.alpha * g)) * (u + a.up_shift));
       } else if (a.epi == 1) {
         ((float*)a.C)[crow + n] = acc[0][i][j];
       } else {
@@ -277,7 +277,7 @@ grouped_gemv_kernel(GroupedArgs a) {
         if (n >= a.N) continue;
         const float g = fminf(acc[2 * f][r], a.limit);
         const float u = fminf(fmaxf(acc[2 * f + 1][r], -a.limit), a.limit);
-        ((T*)a.C)[crow + n] = from_f<T>(g / (1.f + expf(-a.alpha * g)) * (u + 1.f));
+        ((T*)a.C)[crow + n] = from_f<T>(g / (1.f + expf(-a.alpha * g)) * (u + a.up_shift));
       }
     } else {
 #pragma unroll
@@ -436,7 +436,7 @@ grouped_gemv_walk_kernel(GroupedArgs a, int row_tiles) {
                 if (n >= a.N) continue;
                 const float g = fminf(acc[2 * f][r], a.limit);
                 const float u = fminf(fmaxf(acc[2 * f + 1][r], -a.limit), a.limit);
-                ((bf16*)a.C)[crow + n] = from_f<bf16>(g / (1.f + expf(-a.alpha * g)) * (u + 1.f));
+                ((bf16*)a.C)[crow + n] = from_f<bf16>(g / (1.f + expf(-a.alpha * g)) * (u + a.up_shift));
               }
             } else {
 #pragma unroll

@@ -1,0 +1,149 @@
+// Head preparation of an attention whose heads mix their scores before the softmax, one block per token:
+//
+//  * the RMS norm of the token's whole q projection (all heads' lanes at once) times a weight per lane, and the same of
+//    its k projection (optional);
+//  * the rotation of the first rot_dim lanes of every q and k head: lane i turns with lane i + rot_dim / 2 (optional);
+//  * the mixed queries (with `talk`, a matrix T [nq, nq]): the mixed score of head h, sum_g T[h, g] q_g . k_kv(g), is the
+//    dot product of the row [ sum_(g in group j) T[h, g] q_g ]_j with the position's whole key row [ k_j ]_j, so head h's
+//    query becomes that row of nkv * lanes lanes; without it the heads' queries as they are;
+//  * k and v to the token's row of their cache pages.
+//
+// fp32 arithmetic throughout, one rounding at the end.  Stored heads have `lanes` (`v_lanes`) lanes, zero behind the
+// head's own d (dv).
+#include "common.cuh"
+
+struct MixedPrepArgs {
+  const void* qkv;        // [n_tokens, nq d + nkv d + nkv dv] in T
+  void* q_out;            // [n_tokens, nq, nkv, lanes] with talk, else [n_tokens, nq, lanes]
+  void* k_pool;           // [pages, nkv, page_size, lanes]
+  void* v_pool;           // [pages, nkv, page_size, v_lanes]
+  const float* q_w;       // [nq d], or null: no norm
+  const float* k_w;       // [nkv d]
+  const float* talk;      // [nq, nq], or null
+  const float* cos_t;     // [n_tokens, rot_dim / 2], or null: no rotation
+  const float* sin_t;
+  const int* tok_seq;
+  const int* tok_pos;
+  const int* page_start;
+  const int* page_ids;
+  int n_tokens, nq, nkv, d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, write_kv;
+  float eps;
+};
+
+template <typename T> __device__ __forceinline__ void store2(T* p, float a, float b);
+template <> __device__ __forceinline__ void store2<float>(float* p, float a, float b) { *(float2*)p = make_float2(a, b); }
+template <> __device__ __forceinline__ void store2<bf16>(bf16* p, float a, float b) { *(__nv_bfloat162*)p = __floats2bfloat162_rn(a, b); }
+
+// REP: query heads per key head (0: any number, read from shared memory each time).
+template <typename T, int REP>
+__global__ void __launch_bounds__(256)
+mixed_prep_kernel(MixedPrepArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float smem[];
+  __shared__ float scratch[33];
+  const int d = a.d, nqd = a.nq * d, nkd = a.nkv * d, lanes = a.lanes;
+  float* qs = smem;               // [nq, d]
+  float* ks = smem + nqd;         // [nkv, d]
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const T* row = (const T*)a.qkv + (size_t)t * (nqd + nkd + a.nkv * a.dv);
+  float sq = 0.f, sk = 0.f;
+  for (int i = tid; i < nqd; i += blockDim.x) { const float v = to_f<T>(row[i]); qs[i] = v; sq = fmaf(v, v, sq); }
+  for (int i = tid; i < nkd; i += blockDim.x) { const float v = to_f<T>(row[nqd + i]); ks[i] = v; sk = fmaf(v, v, sk); }
+  if (a.q_w != nullptr) {
+    sq = block_sum(sq, scratch);
+    sk = block_sum(sk, scratch);
+    const float qi = 1.0f / sqrtf(sq / (float)nqd + a.eps), ki = 1.0f / sqrtf(sk / (float)nkd + a.eps);
+    for (int i = tid; i < nqd; i += blockDim.x) qs[i] *= qi * a.q_w[i];      // each thread's own elements
+    for (int i = tid; i < nkd; i += blockDim.x) ks[i] *= ki * a.k_w[i];
+  }
+  __syncthreads();
+  if (a.cos_t != nullptr) {
+    const int half = a.rot_dim >> 1;
+    for (int i = tid; i < (a.nq + a.nkv) * half; i += blockDim.x) {      // q heads, then k heads, lie one after the other
+      const int h = i / half, e = i % half;
+      float* x = smem + (size_t)h * d + e;
+      const float c = a.cos_t[(size_t)t * half + e], s = a.sin_t[(size_t)t * half + e];
+      const float u = x[0], v = x[half];
+      x[0] = fmaf(-v, s, u * c);
+      x[half] = fmaf(u, s, v * c);
+    }
+    __syncthreads();
+  }
+  if (a.write_kv) {
+    const int pos = a.tok_pos[t];
+    const int page = a.page_ids[a.page_start[a.tok_seq[t]] + page_slot_of(pos, a.page_size, a.ring_pages)];
+    const size_t at = (size_t)page * a.nkv * a.page_size + pos % a.page_size;
+    for (int i = tid; i < a.nkv * lanes; i += blockDim.x) {
+      const int j = i / lanes, e = i % lanes;
+      ((T*)a.k_pool)[(at + (size_t)j * a.page_size) * lanes + e] = from_f<T>(e < d ? ks[j * d + e] : 0.f);
+    }
+    for (int i = tid; i < a.nkv * a.v_lanes; i += blockDim.x) {
+      const int j = i / a.v_lanes, e = i % a.v_lanes;
+      ((T*)a.v_pool)[(at + (size_t)j * a.page_size) * a.v_lanes + e] = e < a.dv ? row[nqd + nkd + j * a.dv + e] : from_f<T>(0.f);
+    }
+  }
+  if (a.talk == nullptr) {
+    T* out = (T*)a.q_out + (size_t)t * a.nq * lanes;
+    for (int i = tid; i < a.nq * lanes; i += blockDim.x) {
+      const int h = i / lanes, e = i % lanes;
+      out[i] = from_f<T>(e < d ? qs[h * d + e] : 0.f);
+    }
+    return;
+  }
+  // two neighbouring lanes of a key head's query group a thread; its query heads' values stay in registers
+  const int width = a.nkv * lanes, rep = REP > 0 ? REP : a.nq / a.nkv;
+  T* out = (T*)a.q_out + (size_t)t * a.nq * width;
+  for (int p = tid; p < width / 2; p += blockDim.x) {
+    const int j = 2 * p / lanes, e = 2 * p % lanes;
+    const bool in0 = e < d, in1 = e + 1 < d;
+    const float* src = qs + (size_t)j * rep * d + e;
+    float q0[REP > 0 ? REP : 1], q1[REP > 0 ? REP : 1];
+    if (REP > 0) {
+#pragma unroll
+      for (int g = 0; g < REP; ++g) { q0[g] = in0 ? src[g * d] : 0.f; q1[g] = in1 ? src[g * d + 1] : 0.f; }
+    }
+    const float* T_j = a.talk + j * rep;
+    for (int h = 0; h < a.nq; ++h) {
+      float s0 = 0.f, s1 = 0.f;
+      if (REP > 0) {
+#pragma unroll
+        for (int g = 0; g < REP; ++g) { const float w = __ldg(T_j + (size_t)h * a.nq + g); s0 = fmaf(w, q0[g], s0); s1 = fmaf(w, q1[g], s1); }
+      } else {
+        for (int g = 0; g < rep; ++g) {
+          const float w = __ldg(T_j + (size_t)h * a.nq + g);
+          s0 = fmaf(w, in0 ? src[g * d] : 0.f, s0);
+          s1 = fmaf(w, in1 ? src[g * d + 1] : 0.f, s1);
+        }
+      }
+      store2<T>(out + (size_t)h * width + 2 * p, s0, s1);
+    }
+  }
+}
+
+template <typename T, int REP>
+static int launch_mixed_prep(const MixedPrepArgs& a, size_t smem, cudaStream_t stream) {
+  if (smem > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(mixed_prep_kernel<T, REP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return launch_pdl((mixed_prep_kernel<T, REP>), dim3(a.n_tokens), dim3(a.nq * a.d >= 1024 ? 256 : 128), smem, stream, a);
+}
+
+extern "C" int odi_mixed_prep(const MixedPrepArgs* args, int dtype, cudaStream_t stream) {
+  const MixedPrepArgs a = *args;
+  if (a.n_tokens <= 0) return 0;
+  if (a.nq <= 0 || a.nkv <= 0 || a.nq % a.nkv != 0 || a.d <= 0 || a.dv <= 0 || a.lanes < a.d || a.v_lanes < a.dv || a.lanes % 2 != 0 ||
+      a.rot_dim > a.d || (a.rot_dim & 1) || (a.q_w == nullptr) != (a.k_w == nullptr))
+    return ODI_ERR_ARGUMENT;
+  const size_t smem = sizeof(float) * (size_t)(a.nq + a.nkv) * a.d;
+  if (smem > 200 * 1024) return ODI_ERR_UNSUPPORTED;
+  const int rep = a.nq / a.nkv;
+#define ODI_MP(T) \
+  do { if (rep == 1) odi_rc = launch_mixed_prep<T, 1>(a, smem, stream); else if (rep == 2) odi_rc = launch_mixed_prep<T, 2>(a, smem, stream); \
+       else if (rep == 4) odi_rc = launch_mixed_prep<T, 4>(a, smem, stream); else if (rep == 8) odi_rc = launch_mixed_prep<T, 8>(a, smem, stream); \
+       else odi_rc = launch_mixed_prep<T, 0>(a, smem, stream); } while (0)
+  if (dtype == 0) ODI_MP(float); else ODI_MP(bf16);
+#undef ODI_MP
+  return launch_status();
+}

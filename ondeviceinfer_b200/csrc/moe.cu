@@ -5,7 +5,8 @@
 //           each output for itself); choice scores c = s + correction;
 //           the router outputs form `n_groups` equal groups of neighbours, a group's score is its largest c,
 //           only members of the `keep` best groups may be chosen; the `top` largest c among them are chosen
-//           (ties: the lower index); the weight of a chosen output is its s (no renormalisation).
+//           (ties: the lower index); the weight of a chosen output is its s, with `renormalise` divided by the sum of
+//           the chosen ones (+ 1e-20), times `scale`.
 //  table    routing without a router: a token's choices are row `token id` of an integer table, each with the
 //           same weight (out-of-range entries take no place).
 //  count    per (token, choice) pair whose output is a real expert: its rank among the pairs of that expert.
@@ -16,7 +17,8 @@
 //           expert's output row -- or times the token's own input for an identity output (index >= n_experts).
 //  gather   the routed tokens' input rows in the sorted order (for products that want their rows side by side).
 //  gated_clamp  the experts' activation on a [tokens, 2 F] product (gate lanes, then up lanes):
-//           g = min(gate, limit), u = clamp(up, -limit, limit), out = g * sigmoid(alpha * g) * (u + 1).
+//           g = min(gate, limit), u = clamp(up, -limit, limit), out = g * sigmoid(alpha * g) * (u + shift)
+//           (limit +inf, alpha 1 and shift 0: the SiLU gate).
 #include "common.cuh"
 
 struct RouteArgs {
@@ -26,6 +28,8 @@ struct RouteArgs {
   float* weights;           // [n_tokens, top]
   int n_tokens, n_all, n_groups, keep, top;
   int sigmoid;              // 1: the score of an output is the logistic function of its logit, not the softmax
+  int renormalise;          // 1: the chosen scores are divided by their sum + 1e-20
+  float scale;              // multiplies every weight
 };
 
 // (value, index) with "larger value, then lower index" as the order
@@ -102,6 +106,13 @@ moe_route_kernel(RouteArgs a) {
       if (found) c[i] = -INFINITY;
     }
     __syncwarp();
+  }
+  if (lane == 0 && (a.renormalise || a.scale != 1.f)) {      // this thread wrote the weights: the sum in their order
+    float* w = a.weights + (size_t)t * a.top;
+    float total = 0.f;
+    for (int k = 0; k < a.top; ++k) total += w[k];
+    const float div = a.renormalise ? total + 1e-20f : 1.f;
+    for (int k = 0; k < a.top; ++k) w[k] = w[k] / div * a.scale;
   }
 }
 
@@ -430,7 +441,7 @@ extern "C" int odi_moe_gather(const void* x, const int* perm, const int* offsets
 
 template <typename T>
 __global__ void gated_clamp_kernel(const T* __restrict__ gate_up, T* __restrict__ out, long long n, int F, float limit,
-                                   float alpha) {
+                                   float alpha, float shift) {
   pdl_launch_dependents();
   pdl_wait();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -439,12 +450,12 @@ __global__ void gated_clamp_kernel(const T* __restrict__ gate_up, T* __restrict_
   const int f = (int)(i % F);
   const float g = fminf(to_f<T>(gate_up[row * 2 * F + f]), limit);
   const float u = fminf(fmaxf(to_f<T>(gate_up[row * 2 * F + F + f]), -limit), limit);
-  out[i] = from_f<T>(g / (1.f + expf(-alpha * g)) * (u + 1.f));
+  out[i] = from_f<T>(g / (1.f + expf(-alpha * g)) * (u + shift));
 }
 
 // bf16, eight lanes a thread (F a multiple of 8, aligned rows): the same arithmetic.
 __global__ void gated_clamp_vec_kernel(const bf16* __restrict__ gate_up, bf16* __restrict__ out, long long n8, int F, float limit,
-                                       float alpha) {
+                                       float alpha, float shift) {
   pdl_launch_dependents();
   pdl_wait();
   const long long i8 = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -461,23 +472,23 @@ __global__ void gated_clamp_vec_kernel(const bf16* __restrict__ gate_up, bf16* _
     const float2 gv = __bfloat1622float2(g2[e]), uv = __bfloat1622float2(u2[e]);
     const float g0 = fminf(gv.x, limit), g1 = fminf(gv.y, limit);
     const float u0 = fminf(fmaxf(uv.x, -limit), limit), u1 = fminf(fmaxf(uv.y, -limit), limit);
-    o2[e] = __floats2bfloat162_rn(g0 / (1.f + expf(-alpha * g0)) * (u0 + 1.f), g1 / (1.f + expf(-alpha * g1)) * (u1 + 1.f));
+    o2[e] = __floats2bfloat162_rn(g0 / (1.f + expf(-alpha * g0)) * (u0 + shift), g1 / (1.f + expf(-alpha * g1)) * (u1 + shift));
   }
   *(uint4*)(out + i) = oraw;
 }
 
-extern "C" int odi_gated_clamp(const void* gate_up, void* out, int rows, int F, float limit, float alpha, int dtype,
-                               cudaStream_t stream) {
+extern "C" int odi_gated_clamp(const void* gate_up, void* out, int rows, int F, float limit, float alpha, float shift,
+                               int dtype, cudaStream_t stream) {
   const long long n = (long long)rows * F;
   if (n <= 0) return 0;
   if (dtype == 1 && F % 8 == 0 && (((uintptr_t)gate_up | (uintptr_t)out) & 15) == 0) {
     const long long n8 = n / 8;
     odi_rc = launch_pdl(gated_clamp_vec_kernel, dim3((unsigned)((n8 + 255) / 256)), dim3(256), 0, stream, (const bf16*)gate_up,
-                        (bf16*)out, n8, F, limit, alpha);
+                        (bf16*)out, n8, F, limit, alpha, shift);
     return launch_status();
   }
   const unsigned blocks = (unsigned)((n + 255) / 256);
-  if (dtype == 0) odi_rc = launch_pdl((gated_clamp_kernel<float>), dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, n, F, limit, alpha);
-  else odi_rc = launch_pdl((gated_clamp_kernel<bf16>), dim3(blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, n, F, limit, alpha);
+  if (dtype == 0) odi_rc = launch_pdl((gated_clamp_kernel<float>), dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, n, F, limit, alpha, shift);
+  else odi_rc = launch_pdl((gated_clamp_kernel<bf16>), dim3(blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, n, F, limit, alpha, shift);
   return launch_status();
 }

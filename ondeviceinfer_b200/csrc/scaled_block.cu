@@ -8,6 +8,8 @@
 //    included); fp32 arithmetic, one rounding each.
 //  * scaled_add2: x += a * s1 (+ b * s2), fp32, s1 and s2 one number per lane; optionally the new row once more in T.
 //  * weighted_sum: out = ca * a + cb * b on fp32 rows (two mixers' outputs and a factor each).
+//  * gated_norm_add: x += v / sqrt(mean(v^2) + eps) * w with v = y * sigmoid(gate) per row, fp32; optionally the new row
+//    once more in T: what a block adds whose sublayers' outputs are gated lane by lane and then normed.
 //  * gated_lookup: out[t, j] = gelu_tanh(z[t, j]) * table[ids[t], col + j] in T (fp32 arithmetic, one rounding):
 //    a gate on the stream times a row that the token id picks.
 #include "common.cuh"
@@ -141,6 +143,98 @@ extern "C" int odi_scaled_add2(float* x, const float* a, const float* s1, const 
   if (blocks > 2147483647L) return ODI_ERR_UNSUPPORTED;
   if (dtype == 0) odi_rc = launch_pdl((scaled_add2_kernel<float>), dim3((unsigned)blocks), dim3(256), 0, stream, x, a, s1, b, s2, (float*)copy, n, H);
   else odi_rc = launch_pdl((scaled_add2_kernel<bf16>), dim3((unsigned)blocks), dim3(256), 0, stream, x, a, s1, b, s2, (bf16*)copy, n, H);
+  return launch_status();
+}
+
+__device__ __forceinline__ float block_gate(float y, const float* gate, size_t i) {
+  return gate == nullptr ? y : y / (1.f + expf(-gate[i]));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ gate, const float* __restrict__ w,
+                      T* __restrict__ copy, int H, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  const size_t base = (size_t)blockIdx.x * H;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) { const float v = block_gate(y[base + i], gate, base + i); ss = fmaf(v, v, ss); }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float v = fmaf(block_gate(y[base + i], gate, base + i) * inv, w[i], x[base + i]);
+    x[base + i] = v;
+    if (copy != nullptr) copy[base + i] = from_f<T>(v);
+  }
+}
+
+// H a multiple of 4 and at most 4 * NV * threads: the gated row stays in registers between the two passes, and the
+// stream's row is requested before the sum of squares is known.
+template <typename T, int NV>
+__global__ void __launch_bounds__(512)
+gated_norm_add_vec_kernel(float4* __restrict__ x, const float4* __restrict__ y, const float4* __restrict__ gate,
+                          const float4* __restrict__ w, T* __restrict__ copy, int H4, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float scratch[33];
+  const size_t base = (size_t)blockIdx.x * H4;
+  float4 v[NV], r[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < H4) {
+      v[j] = y[base + i];
+      r[j] = x[base + i];
+      if (gate != nullptr) {
+        const float4 g = gate[base + i];
+        v[j].x /= 1.f + expf(-g.x); v[j].y /= 1.f + expf(-g.y); v[j].z /= 1.f + expf(-g.z); v[j].w /= 1.f + expf(-g.w);
+      }
+      ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)(4 * H4) + eps);
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < H4) {
+      const float4 g = w[i];
+      const float4 n = make_float4(fmaf(v[j].x * inv, g.x, r[j].x), fmaf(v[j].y * inv, g.y, r[j].y),
+                                   fmaf(v[j].z * inv, g.z, r[j].z), fmaf(v[j].w * inv, g.w, r[j].w));
+      x[base + i] = n;
+      if (copy != nullptr) {
+        if (sizeof(T) == 4) ((float4*)copy)[base + i] = n;
+        else {
+          uint2 packed;
+          *(__nv_bfloat162*)&packed.x = __floats2bfloat162_rn(n.x, n.y);
+          *(__nv_bfloat162*)&packed.y = __floats2bfloat162_rn(n.z, n.w);
+          ((uint2*)copy)[base + i] = packed;
+        }
+      }
+    }
+  }
+}
+
+extern "C" int odi_gated_norm_add(float* x, const float* y, const float* gate, const float* w, void* copy, int n, int H, float eps,
+                                  int dtype, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (H <= 0) return ODI_ERR_ARGUMENT;
+  if (H % 4 == 0 && H <= 8192 && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)copy) & 15) == 0) {
+    const int H4 = H / 4;
+    const int threads = H4 >= 1024 ? 512 : (H4 >= 256 ? 256 : (H4 >= 128 ? 128 : 64));
+    const int per = (H4 + threads - 1) / threads;
+#define ODI_GNA(T, NV) odi_rc = launch_pdl((gated_norm_add_vec_kernel<T, NV>), dim3(n), dim3(threads), 0, stream, (float4*)x, \
+    (const float4*)y, (const float4*)gate, (const float4*)w, (T*)copy, H4, eps)
+    if (dtype == 0) { if (per <= 1) ODI_GNA(float, 1); else if (per <= 2) ODI_GNA(float, 2); else ODI_GNA(float, 4); }
+    else { if (per <= 1) ODI_GNA(bf16, 1); else if (per <= 2) ODI_GNA(bf16, 2); else ODI_GNA(bf16, 4); }
+#undef ODI_GNA
+    return launch_status();
+  }
+  if (dtype == 0) odi_rc = launch_pdl((gated_norm_add_kernel<float>), dim3(n), dim3(256), 0, stream, x, y, gate, w, (float*)copy, H, eps);
+  else odi_rc = launch_pdl((gated_norm_add_kernel<bf16>), dim3(n), dim3(256), 0, stream, x, y, gate, w, (bf16*)copy, H, eps);
   return launch_status();
 }
 

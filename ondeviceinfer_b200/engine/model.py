@@ -112,6 +112,7 @@ class DecoderModel:
             hidden = self.embedding.forward(ctx)           # the fp32 residual stream [tokens, hidden]
         ctx.residual_sumsq = None          # nothing is known about the rows of `hidden` yet
         ctx.pending_residual_add = None
+        ctx.stream_copy = None
         if self.keeps_embedding:
             ctx.embedded = hidden.clone()  # a layer reads the embedding's output again; the stream changes in place
         for index, entry in enumerate(self.plan.order):
@@ -121,6 +122,8 @@ class DecoderModel:
             ctx.defers_residual_add = False
             if not getattr(layer, "finishes_residual_adds", False):
                 flush_residual_add(ctx)
+            if not getattr(layer, "renews_stream_copy", False):
+                ctx.stream_copy = None         # this layer changes the stream without renewing its copy
             with nvtx_range(f"layer_{entry.layer}"):
                 replaced = layer.forward(hidden, ctx, cache.view(index))
             if replaced is not None:           # a layer may hand back a new stream instead of changing it in place

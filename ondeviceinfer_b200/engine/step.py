@@ -49,6 +49,8 @@ class StepDescription:
     ``key_splits(rows)``      how a split-key decode kernel may cut the sequences' keys;
     ``memo(key, make)``       a value shared by all layers of the step (rotary tables and the like);
     ``residual_sumsq``        the note a residual product leaves for the norm that follows it;
+    ``stream_copy``           ``(stream, rows)``: the stream's rows in the compute dtype, left by the block that wrote them
+                              (None: nobody left any);
     ``pending_residual_add``, ``defers_residual_add``  a residual add left to the next norm, and the flag of a block
                               that finishes such adds (``parts/linear.py``, ``parts/block.py``).
 
@@ -61,7 +63,7 @@ class StepDescription:
 
     INTERFACE = ("token_ids", "tok_seq", "tok_pos", "cu_q", "past", "slots", "want_rows",
                  "n_seqs", "n_tokens", "n_want", "q_lens", "past_lens", "kv_lens", "max_q_len", "max_kv_len",
-                 "slot_list", "residual_sumsq", "pending_residual_add", "defers_residual_add",
+                 "slot_list", "residual_sumsq", "pending_residual_add", "defers_residual_add", "stream_copy",
                  "page_table", "key_splits", "memo")
 
     def __init__(self) -> None:
@@ -70,6 +72,7 @@ class StepDescription:
         self.residual_sumsq = None
         self.pending_residual_add = None       # (residual, product) that a block left to the next norm
         self.defers_residual_add = False       # set by a block that finishes such adds
+        self.stream_copy = None                # (stream, its rows in the compute dtype)
 
     def page_table(self, group_index: int) -> Tuple[torch.Tensor, torch.Tensor]:
         return self._page_tables[group_index]

@@ -280,7 +280,8 @@ def gemm_f32(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, residual: Opti
                             c_int(K), c_int(K), c_int(N), c_int(N), _stream()), "gemm_f32")
 
 
-EPI_STORE_BF16, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU, EPI_HEAD_PREP, EPI_GELU = 0, 1, 2, 3, 4, 5
+EPI_STORE_BF16, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU, EPI_HEAD_PREP, EPI_GELU, EPI_GEGLU = 0, 1, 2, 3, 4, 5, 6
+EPI_GATED = (EPI_SWIGLU, EPI_GEGLU)      # two weight rows a feature: the gate rows, then the up rows
 
 _gemm_state = {}
 
@@ -414,7 +415,8 @@ def gemm_bf16(x: Optional[torch.Tensor], w: torch.Tensor, out: Optional[torch.Te
     """Tensor-core product out = epilogue(x w^T): x [tokens, K] bf16, w [rows, K] bf16.
 
     ``EPI_STORE_BF16`` / ``EPI_STORE_F32``: out [tokens, rows]; ``EPI_RESIDUAL``: out (fp32) += product;
-    ``EPI_SWIGLU``: w holds the gate rows then the up rows, out [tokens, rows / 2] = silu(gate) * up;
+    ``EPI_SWIGLU`` / ``EPI_GEGLU``: w holds the gate rows then the up rows, out [tokens, rows / 2] = silu(gate) * up
+    resp. gelu(gate) * up (the tanh form);
     ``EPI_GELU``: out [tokens, rows] = gelu(product) in bf16 (the exact erf form).
     ``cluster``: let 2..8 K splits exchange their partials inside a thread-block cluster (else, and for
     more splits, through global scratch and a ticket).
@@ -466,15 +468,15 @@ def gemm_bf16(x: Optional[torch.Tensor], w: torch.Tensor, out: Optional[torch.Te
     _require(w, "w", torch.bfloat16, 2)
     tokens, K = x_like.shape
     w_rows = w.shape[0]
-    n_out = w_rows // 2 if epi == EPI_SWIGLU else w_rows
+    n_out = w_rows // 2 if epi in EPI_GATED else w_rows
     if epi == EPI_HEAD_PREP:
         if out is not None or head_prep is None:
             raise KernelError("EPI_HEAD_PREP takes head_prep and no out")
         if w.shape[1] != K:
             raise KernelError(f"gemm sizes disagree: x {tuple(x_like.shape)}, w {tuple(w.shape)}")
     else:
-        _require(out, "out", torch.bfloat16 if epi in (EPI_STORE_BF16, EPI_SWIGLU, EPI_GELU) else torch.float32, 2)
-        if w.shape[1] != K or out.shape != (tokens, n_out) or (epi == EPI_SWIGLU and w_rows % 2):
+        _require(out, "out", torch.bfloat16 if epi in (EPI_STORE_BF16, EPI_SWIGLU, EPI_GELU, EPI_GEGLU) else torch.float32, 2)
+        if w.shape[1] != K or out.shape != (tokens, n_out) or (epi in EPI_GATED and w_rows % 2):
             raise KernelError(f"gemm sizes disagree: x {tuple(x_like.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
     if sumsq_out is not None:
         _require(sumsq_out, "sumsq_out", torch.float32, 2)
@@ -489,7 +491,7 @@ def gemm_bf16(x: Optional[torch.Tensor], w: torch.Tensor, out: Optional[torch.Te
     lib = load_library("gemm_tcgen05")
     lib.odi_gemm_bf16_scratch_floats.restype = c_long
     need = lib.odi_gemm_bf16_scratch_floats(c_int(tokens), c_int(n_out), c_int(bn), c_int(splits),
-                                            c_int(1 if epi == EPI_SWIGLU else 0))
+                                            c_int(1 if epi in EPI_GATED else 0))
     tiles = -(-n_out // 128) * -(-tokens // bn)
     scratch, tickets, status = _gemm_buffers(w.device, need)
     if splits > 1 and tiles > tickets.numel() // 2:      # the upper half belongs to the many-token kernel's tile flags
@@ -556,17 +558,17 @@ def gemm_prefill_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tens
     _require(w, "w", torch.bfloat16, 2)
     tokens, K = x.shape
     w_rows = w.shape[0]
-    n_out = w_rows // 2 if epi == EPI_SWIGLU else w_rows
+    n_out = w_rows // 2 if epi in EPI_GATED else w_rows
     if epi == EPI_HEAD_PREP:
         if out is not None or head_prep is None or w.shape[1] != K:
             raise KernelError("EPI_HEAD_PREP takes head_prep, no out, and weights as wide as x")
         if not gemm_bf16_supported(x, w):
             raise KernelError(f"gemm_prefill_tcgen05 needs K a multiple of 8 and 16-byte aligned operands (K={K})")
     else:
-        if epi not in (EPI_STORE_BF16, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU, EPI_GELU):
+        if epi not in (EPI_STORE_BF16, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU, EPI_GELU, EPI_GEGLU):
             raise KernelError(f"gemm_prefill_bf16 has no epilogue {epi}")
-        _require(out, "out", torch.bfloat16 if epi in (EPI_STORE_BF16, EPI_SWIGLU, EPI_GELU) else torch.float32, 2)
-        if w.shape[1] != K or out.shape != (tokens, n_out) or (epi == EPI_SWIGLU and w_rows % 2):
+        _require(out, "out", torch.bfloat16 if epi in (EPI_STORE_BF16, EPI_SWIGLU, EPI_GELU, EPI_GEGLU) else torch.float32, 2)
+        if w.shape[1] != K or out.shape != (tokens, n_out) or (epi in EPI_GATED and w_rows % 2):
             raise KernelError(f"gemm sizes disagree: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
         if not gemm_prefill_supported(x, w, n_out, out.dtype):
             raise KernelError(f"gemm_prefill_tcgen05 needs K a multiple of 8, 16-byte aligned operands and output rows "
@@ -591,7 +593,8 @@ class _AttnArgs(Structure):
                 ("partial", c_void_p), ("cu_q", c_void_p), ("past", c_void_p), ("page_start", c_void_p),
                 ("page_ids", c_void_p), ("n_seqs", c_int), ("nq", c_int), ("nkv", c_int), ("page_size", c_int),
                 ("ring_pages", c_int), ("window", c_int), ("splits", c_int), ("bq", c_int),
-                ("head_chunks", c_int), ("scale", c_float), ("softcap", c_float), ("sink", c_int), ("keep", c_int)]
+                ("head_chunks", c_int), ("scale", c_float), ("softcap", c_float), ("sink", c_int), ("keep", c_int),
+                ("chunk", c_int), ("mixed", c_int)]
 
 
 SIMT_HEAD_DIMS = tuple(range(16, 513, 16))
@@ -600,11 +603,15 @@ SIMT_HEAD_DIMS = tuple(range(16, 513, 16))
 def attention_simt(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, n_seqs: int, max_q_len: int,
                    nq: int, nkv: int, d: int, page_size: int, ring_pages: int, window: int, scale: float,
                    splits: int = 1, partial: Optional[torch.Tensor] = None, dv: Optional[int] = None,
-                   shared_kv: bool = False, softcap: float = 0.0, sink: bool = False, keep: int = 0) -> None:
+                   shared_kv: bool = False, softcap: float = 0.0, sink: bool = False, keep: int = 0, chunk: int = 0,
+                   mixed: bool = False) -> None:
     """Causal GQA over the paged cache for any mixture of prompt and decode sequences.  ``softcap`` c > 0:
     scores (times ``scale``) become c tanh(score / c) before the softmax.  ``sink``: the softmax has one more
     term of score 0 and no value, p_j = exp(s_j) / (1 + sum_k exp(s_k)).  ``keep`` > 0 with a window: the first
     ``keep`` positions of a sequence stay visible beyond the window (a ring then has their pages pinned in front).
+
+    ``chunk`` c > 0 (instead of a window): position p sees the keys of its own chunk of c positions only.
+    ``mixed``: q is [tokens, nq, nkv, d] and a score is the sum over the key heads of q . k (see :func:`mixed_prep`).
 
     ``dv`` (default ``d``): width of the value rows and of the output.  ``shared_kv``: a cached row is key and
     value at once (the value is its first ``dv`` lanes; ``v_pool`` is None), as in attention over a latent
@@ -624,7 +631,7 @@ def attention_simt(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, 
             raise KernelError("attention over shared rows takes no value pool")
     else:
         _require(v_pool, "v_pool", q.dtype)
-    n_tokens = q.numel() // (nq * d)
+    n_tokens = q.numel() // (nq * d * (nkv if mixed else 1))
     if out.numel() != n_tokens * nq * dv:
         raise KernelError("q and out disagree")
     if splits > 1:
@@ -633,7 +640,7 @@ def attention_simt(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, 
             raise KernelError(f"splits={splits} needs an fp32 partial buffer of {need} elements")
     args = _AttnArgs(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(partial), _ptr(cu_q), _ptr(past),
                      _ptr(page_start), _ptr(page_ids), n_seqs, nq, nkv, page_size, ring_pages, window, splits,
-                     0, 0, scale, softcap, 1 if sink else 0, keep)
+                     0, 0, scale, softcap, 1 if sink else 0, keep, chunk, 1 if mixed else 0)
     defines = {"ODI_HEAD_DIM": d}
     if not plain:
         defines.update({"ODI_VALUE_DIM": dv, "ODI_SHARED_KV": 1 if shared_kv else 0})
@@ -933,8 +940,8 @@ def rmsnorm_scaled(x: torch.Tensor, scale: torch.Tensor, eps: float, out: torch.
                                   c_int(dtype_code(out.dtype)), _stream()), "rmsnorm_scaled")
 
 
-def gated_clamp(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: float) -> None:
-    """out = g * sigmoid(alpha * g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit), for
+def gated_clamp(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: float, up_shift: float = 1.0) -> None:
+    """out = g * sigmoid(alpha * g) * (u + up_shift) with g = min(gate, limit), u = clamp(up, -limit, limit), for
     ``gate_up`` [tokens, 2 F] (gate lanes, then up lanes)."""
     _require(gate_up, "gate_up", ndim=2)
     _require(out, "out", gate_up.dtype, 2)
@@ -943,7 +950,7 @@ def gated_clamp(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: f
         raise KernelError(f"gated_clamp sizes disagree: {tuple(gate_up.shape)} -> {tuple(out.shape)}")
     lib = load_library("moe")
     _check(lib.odi_gated_clamp(_ptr(gate_up), _ptr(out), c_int(rows), c_int(F), c_float(limit), c_float(alpha),
-                               c_int(dtype_code(out.dtype)), _stream()), "gated_clamp")
+                               c_float(up_shift), c_int(dtype_code(out.dtype)), _stream()), "gated_clamp")
 
 
 # ------------------------------------------------------------------------------ latent attention
@@ -1076,7 +1083,7 @@ class _GroupedArgs(Structure):
                 ("tile_row0", c_void_p), ("tile_rows", c_void_p), ("n_tiles", c_void_p),
                 ("a_group_off", ctypes.c_longlong), ("w_group_stride", ctypes.c_longlong), ("c_group_off", ctypes.c_longlong),
                 ("lda", c_int), ("ldw", c_int), ("ldc", c_int), ("M", c_int), ("N", c_int), ("K", c_int),
-                ("groups", c_int), ("index_div", c_int), ("epi", c_int), ("limit", c_float), ("alpha", c_float)]
+                ("groups", c_int), ("index_div", c_int), ("epi", c_int), ("limit", c_float), ("alpha", c_float), ("up_shift", c_float)]
 
 
 GROUPED_STORE, GROUPED_STORE_F32, GROUPED_GATED_CLAMP, GROUPED_GELU_ERF, GROUPED_GELU_TANH, GROUPED_RELU2 = 0, 1, 2, 3, 4, 5
@@ -1113,7 +1120,7 @@ def grouped_gemm_heads(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, *, a_c
         raise KernelError(f"grouped product sizes disagree: a {tuple(a.shape)}, w {tuple(w.shape)}, c {tuple(c.shape)}")
     args = _GroupedArgs(a.data_ptr() + a_col * a.element_size(), _ptr(w), c.data_ptr() + c_col * c.element_size(),
                         None, None, None, None, None, a_stride, N * K, c_stride, a.shape[1], K, c.shape[1], M, N, K,
-                        groups, 1, GROUPED_STORE_F32 if out_f32 else GROUPED_STORE, 0.0, 0.0)
+                        groups, 1, GROUPED_STORE_F32 if out_f32 else GROUPED_STORE, 0.0, 0.0, 0.0)
     lib = load_library("grouped_gemm")
     # up to four rows: the form that streams the weights; five to eight rows too when the inner size is long (the
     # tile form would walk it in a few blocks per head), in two row tiles; else tiles of 16 or 64 rows
@@ -1123,9 +1130,9 @@ def grouped_gemm_heads(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, *, a_c
 
 
 def grouped_gemm_routed(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, table: "RoutingTable", *, gather: bool,
-                        epi: int, limit: float = 0.0, alpha: float = 0.0) -> None:
+                        epi: int, limit: float = 0.0, alpha: float = 0.0, up_shift: float = 1.0) -> None:
     """The product of each routed row with its expert's matrix ``w[e]`` ([experts, rows, K]; with
-    ``GROUPED_GATED_CLAMP`` rows = N gate rows then N up rows).  Rows are taken in ``table``'s sorted order; with
+    ``GROUPED_GATED_CLAMP`` rows = N gate rows then N up rows, and the activation is that of :func:`gated_clamp`).  Rows are taken in ``table``'s sorted order; with
     ``gather`` row i reads ``a[perm[i] // top]`` (the token's input), else ``a[i]``; row i of ``c`` is written."""
     _require(a, "a", w.dtype, 2)
     _require(w, "w", ndim=3)
@@ -1136,7 +1143,7 @@ def grouped_gemm_routed(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, table
         raise KernelError(f"routed product sizes disagree: a {tuple(a.shape)}, w {tuple(w.shape)}, c {tuple(c.shape)}")
     args = _GroupedArgs(_ptr(a), _ptr(w), _ptr(c), _ptr(table.perm) if gather else None, _ptr(table.tile_group),
                         _ptr(table.tile_row0), _ptr(table.tile_rows), _ptr(table.n_tiles), 0, w_rows * K, 0,
-                        K, K, N, 0, N, K, experts, table.top if gather else 1, epi, limit, alpha)
+                        K, K, N, 0, N, K, experts, table.top if gather else 1, epi, limit, alpha, up_shift)
     lib = load_library("grouped_gemm")
     _check(lib.odi_grouped_gemm(byref(args), c_int(table.max_tiles), c_int(table.tm), c_int(dtype_code(w.dtype)),
                                 _stream()), "grouped_gemm")
@@ -1145,14 +1152,15 @@ def grouped_gemm_routed(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, table
 class _RouteArgs(Structure):
     _fields_ = [("logits", c_void_p), ("correction", c_void_p), ("ids", c_void_p), ("weights", c_void_p),
                 ("n_tokens", c_int), ("n_all", c_int), ("n_groups", c_int), ("keep", c_int), ("top", c_int),
-                ("sigmoid", c_int)]
+                ("sigmoid", c_int), ("renormalise", c_int), ("scale", c_float)]
 
 
 def moe_route(logits: torch.Tensor, correction: Optional[torch.Tensor], ids: torch.Tensor, weights: torch.Tensor, *,
-              n_groups: int, keep: int, sigmoid: bool = False) -> None:
+              n_groups: int, keep: int, sigmoid: bool = False, renormalise: bool = False, scale: float = 1.0) -> None:
     """Grouped top-k routing of fp32 ``logits`` [tokens, outputs] (see ``csrc/moe.cu``): ``ids`` and ``weights``
     [tokens, top] receive the chosen outputs, best first, and their scores: the softmax over the outputs, or with
-    ``sigmoid`` the logistic function of each logit for itself."""
+    ``sigmoid`` the logistic function of each logit for itself.  ``renormalise``: the chosen scores are divided by their
+    sum (+ 1e-20); ``scale`` multiplies every weight."""
     _require(logits, "logits", torch.float32, 2)
     _require(ids, "ids", torch.int32, 2)
     _require(weights, "weights", torch.float32, 2)
@@ -1164,7 +1172,7 @@ def moe_route(logits: torch.Tensor, correction: Optional[torch.Tensor], ids: tor
         if correction.numel() != n_all:
             raise KernelError("the correction has one entry per router output")
     args = _RouteArgs(_ptr(logits), _ptr(correction), _ptr(ids), _ptr(weights), n, n_all, n_groups, keep, ids.shape[1],
-                      1 if sigmoid else 0)
+                      1 if sigmoid else 0, 1 if renormalise else 0, scale)
     lib = load_library("moe")
     _check(lib.odi_moe_route(byref(args), _stream()), "moe_route")
 
@@ -1391,6 +1399,21 @@ def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> None:
                               _stream()), "activation")
 
 
+GATED_ACTIVATIONS = {"silu": -1, "gelu_tanh": 1}      # silu: silu_mul and the products' epilogues; else a kind of `activation`
+
+
+def gated_activation(gate_up: torch.Tensor, out: torch.Tensor, kind: str) -> None:
+    """out = act(gate_up[:, :F]) * gate_up[:, F:] (fp32 arithmetic, one rounding); ``kind`` one of ``ACTIVATIONS``."""
+    _require(gate_up, "gate_up", ndim=2)
+    _require(out, "out", gate_up.dtype, 2)
+    rows, F = out.shape
+    if kind not in ACTIVATIONS or gate_up.shape != (rows, 2 * F):
+        raise KernelError(f"gated activation {kind!r} on {tuple(gate_up.shape)} -> {tuple(out.shape)}")
+    lib = load_library("capped")
+    _check(lib.odi_gated_activation(_ptr(gate_up), _ptr(out), c_long(rows), c_int(F), c_int(ACTIVATIONS[kind]),
+                                    c_int(dtype_code(out.dtype)), _stream()), "gated_activation")
+
+
 def softcap(x: torch.Tensor, cap: float) -> None:
     """x <- cap * tanh(x / cap) in place (fp32)."""
     _require(x, "x", torch.float32)
@@ -1518,6 +1541,107 @@ def delta_rule(proj: torch.Tensor, decay_in: torch.Tensor, taps: torch.Tensor, a
                       eps, unit_eps)
     lib = load_library("delta", {"ODI_DELTA_DIM": d})
     _check(lib.odi_delta_rule(byref(args), c_int(dtype_code(proj.dtype)), _stream()), "delta_rule", 6 if K > 1 else 5)
+
+
+class _HeadDeltaArgs(Structure):
+    _fields_ = [("proj", c_void_p), ("ab", c_void_p), ("taps", c_void_p), ("a_log", c_void_p), ("dt_bias", c_void_p),
+                ("norm_w", c_void_p), ("conv_state", c_void_p), ("state", c_void_p), ("qk", c_void_p), ("gb", c_void_p),
+                ("o", c_void_p), ("out", c_void_p), ("cu_q", c_void_p), ("tok_seq", c_void_p), ("slots", c_void_p),
+                ("n_tokens", c_int), ("n_seqs", c_int), ("max_q_len", c_int), ("ld", c_int), ("heads", c_int),
+                ("kv_heads", c_int), ("d", c_int), ("dv", c_int), ("taps_n", c_int), ("eps", c_float), ("unit_eps", c_float)]
+
+
+HEAD_DELTA_MAX_DIM, HEAD_DELTA_MAX_TAPS = 512, 16
+
+
+def head_delta(proj: torch.Tensor, ab: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+               norm_w: torch.Tensor, conv_state: Optional[torch.Tensor], state: torch.Tensor, out: torch.Tensor, cu_q, tok_seq,
+               slots, *, n_seqs: int, max_q_len: int, heads: int, kv_heads: int, d: int, dv: int, eps: float,
+               unit_eps: float) -> None:
+    """The gated delta rule with one decay per head between its products (``csrc/delta_head.cu``): ``proj`` [tokens,
+    2 kv_heads d + 2 heads dv] = q, k and v channels before their convolutions, then the output gate's logits; ``ab``
+    fp32 [tokens, 2 heads] = the decay's inner term, then the step size's logit; ``taps`` fp32 [C, K], C = 2 kv_heads d +
+    heads dv; ``conv_state`` [slots, K - 1, C] and ``state`` [slots, heads, d, dv] are fp32 rows of the cache, advanced in
+    place over all tokens that each sequence brings (``max_q_len``: the most that one brings); ``out`` [tokens, heads dv]
+    receives the normed, gated read-outs in the dtype of ``proj``."""
+    _require(proj, "proj", ndim=2)
+    _require(ab, "ab", torch.float32, 2)
+    _require(out, "out", proj.dtype, 2)
+    n = proj.shape[0]
+    C, K = taps.shape
+    for name, t, shape in (("taps", taps, (2 * kv_heads * d + heads * dv, K)), ("a_log", a_log, (heads,)),
+                           ("dt_bias", dt_bias, (heads,)), ("norm_w", norm_w, (dv,))):
+        _require(t, name, torch.float32)
+        if tuple(t.shape) != shape:
+            raise KernelError(f"head_delta: {name} is {tuple(t.shape)}, expected {shape}")
+    _require(state, "state", torch.float32)
+    if (proj.shape[1] != C + heads * dv or ab.shape != (n, 2 * heads) or out.shape != (n, heads * dv)
+            or tuple(state.shape[1:]) != (heads, d, dv)):
+        raise KernelError(f"head_delta sizes disagree: proj {tuple(proj.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
+    if K > 1:
+        _require(conv_state, "conv_state", torch.float32)
+        if tuple(conv_state.shape[1:]) != (K - 1, C):
+            raise KernelError("head_delta: the convolution state is [slots, taps - 1, channels]")
+    dev = proj.device
+    qk = torch.empty((n, kv_heads, 2, d), dtype=torch.float32, device=dev)
+    gb = torch.empty((n, heads, 2), dtype=torch.float32, device=dev)
+    o = torch.empty((n, heads * dv), dtype=torch.float32, device=dev)
+    args = _HeadDeltaArgs(_ptr(proj), _ptr(ab), _ptr(taps), _ptr(a_log), _ptr(dt_bias), _ptr(norm_w),
+                          _ptr(conv_state if K > 1 else None), _ptr(state), _ptr(qk), _ptr(gb), _ptr(o), _ptr(out), _ptr(cu_q),
+                          _ptr(tok_seq), _ptr(slots), n, n_seqs, max_q_len, proj.shape[1], heads, kv_heads, d, dv, K, eps,
+                          unit_eps)
+    lib = load_library("delta_head")
+    _check(lib.odi_head_delta(byref(args), c_int(dtype_code(proj.dtype)), _stream()), "head_delta",
+           4 if K > 1 and max_q_len > 1 else 3)
+
+
+# ------------------------------------------------------------------------------ attention with mixed heads
+
+
+class _MixedPrepArgs(Structure):
+    _fields_ = [("qkv", c_void_p), ("q_out", c_void_p), ("k_pool", c_void_p), ("v_pool", c_void_p), ("q_w", c_void_p),
+                ("k_w", c_void_p), ("talk", c_void_p), ("cos_t", c_void_p), ("sin_t", c_void_p), ("tok_seq", c_void_p),
+                ("tok_pos", c_void_p), ("page_start", c_void_p), ("page_ids", c_void_p), ("n_tokens", c_int), ("nq", c_int),
+                ("nkv", c_int), ("d", c_int), ("dv", c_int), ("lanes", c_int), ("v_lanes", c_int), ("rot_dim", c_int),
+                ("page_size", c_int), ("ring_pages", c_int), ("write_kv", c_int), ("eps", c_float)]
+
+
+def mixed_prep(qkv, q_out, k_pool, v_pool, q_norm, k_norm, talk, cos_t, sin_t, tok_seq, tok_pos, page_start, page_ids, *,
+               nq: int, nkv: int, d: int, dv: int, lanes: int, v_lanes: int, rot_dim: int, page_size: int, ring_pages: int,
+               write_kv: bool, eps: float) -> None:
+    """Head preparation of an attention whose heads mix their scores (``csrc/mixed.cu``): from ``qkv`` [tokens, nq d +
+    nkv d + nkv dv] the RMS norms over a token's whole q and k rows (``q_norm`` fp32 [nq d], ``k_norm`` fp32 [nkv d]; both
+    None: no norm), the rotation of half-split pairs over the first ``rot_dim`` lanes of each head (``cos_t`` None: none),
+    k and v to the cache (stored heads of ``lanes`` and ``v_lanes`` lanes, zero behind the head's own), and the queries:
+    with ``talk`` (fp32 [nq, nq]) ``q_out`` [tokens, nq * nkv * lanes] holds for head h and key head j the sum of
+    talk[h, g] q_g over the query heads g of j; without it ``q_out`` is [tokens, nq * lanes]."""
+    _require(qkv, "qkv", ndim=2)
+    _require(q_out, "q_out", qkv.dtype, 2)
+    n = qkv.shape[0]
+    width = nq * lanes * (nkv if talk is not None else 1)
+    if qkv.shape[1] != (nq + nkv) * d + nkv * dv or q_out.shape != (n, width):
+        raise KernelError(f"mixed_prep sizes disagree: qkv {tuple(qkv.shape)}, q_out {tuple(q_out.shape)}, nq={nq}, nkv={nkv}, "
+                          f"d={d}, dv={dv}")
+    for name, w, size in (("q_norm", q_norm, nq * d), ("k_norm", k_norm, nkv * d), ("talk", talk, nq * nq)):
+        if w is not None:
+            _require(w, name, torch.float32)
+            if w.numel() != size:
+                raise KernelError(f"mixed_prep: {name} has {w.numel()} entries, expected {size}")
+    if write_kv:
+        _require(k_pool, "k_pool", qkv.dtype)
+        _require(v_pool, "v_pool", qkv.dtype)
+        if k_pool.shape[-1] != lanes or v_pool.shape[-1] != v_lanes:
+            raise KernelError("the cache pools do not have the heads' widths")
+    if cos_t is not None:
+        _require(cos_t, "cos_t", torch.float32, 2)
+        _require(sin_t, "sin_t", torch.float32, 2)
+        if cos_t.shape != (n, rot_dim // 2) or sin_t.shape != cos_t.shape:
+            raise KernelError("rope tables must be [tokens, rot_dim / 2]")
+    args = _MixedPrepArgs(_ptr(qkv), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(q_norm), _ptr(k_norm), _ptr(talk),
+                          _ptr(cos_t), _ptr(sin_t), _ptr(tok_seq), _ptr(tok_pos), _ptr(page_start), _ptr(page_ids), n, nq, nkv,
+                          d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, 1 if write_kv else 0, eps)
+    lib = load_library("mixed")
+    _check(lib.odi_mixed_prep(byref(args), c_int(dtype_code(qkv.dtype)), _stream()), "mixed_prep")
 
 
 # ------------------------------------------------------------------------------ sampling
@@ -1686,6 +1810,29 @@ def scaled_add2(x: torch.Tensor, a: torch.Tensor, s1: torch.Tensor, b: Optional[
     lib = load_library("scaled_block")
     _check(lib.odi_scaled_add2(_ptr(x), _ptr(a), _ptr(s1), _ptr(b), _ptr(s2), _ptr(copy), c_long(n), c_int(H),
                                c_int(0 if copy is None else dtype_code(copy.dtype)), _stream()), "scaled_add2")
+
+
+def gated_norm_add(x: torch.Tensor, y: torch.Tensor, gate: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
+                   copy: Optional[torch.Tensor] = None) -> None:
+    """x += v / sqrt(mean(v^2) + eps) * weight with v = y * sigmoid(gate) (``gate`` None: v = y), all fp32 rows
+    [tokens, H]; ``copy`` (optional, any compute dtype) receives the new rows once more."""
+    _require(x, "x", torch.float32, 2)
+    _require(y, "y", torch.float32, 2)
+    _require(weight, "weight", torch.float32, 1)
+    n, H = x.shape
+    if y.shape != (n, H) or weight.numel() != H:
+        raise KernelError("gated_norm_add sizes disagree")
+    if gate is not None:
+        _require(gate, "gate", torch.float32, 2)
+        if gate.shape != (n, H):
+            raise KernelError("gated_norm_add: the gate has the shape of y")
+    if copy is not None:
+        _require(copy, "copy", ndim=2)
+        if copy.shape != (n, H):
+            raise KernelError("gated_norm_add: the copy has the shape of x")
+    lib = load_library("scaled_block")
+    _check(lib.odi_gated_norm_add(_ptr(x), _ptr(y), _ptr(gate), _ptr(weight), _ptr(copy), c_int(n), c_int(H), c_float(eps),
+                                  c_int(0 if copy is None else dtype_code(copy.dtype)), _stream()), "gated_norm_add")
 
 
 def cast_rows(x: torch.Tensor, out: torch.Tensor) -> None:

@@ -2,6 +2,7 @@
 
 from ..config.lemesun import LemesunConfig
 from ..config.losivik import LosivikConfig
+from ..config.noganex import NoganexConfig
 from ..config.nulalorn import NulalornConfig
 from ..config.qwen3 import Qwen3Config
 from ..config.zigivik import ZigivikConfig
@@ -10,5 +11,6 @@ from ..registry import register_architecture
 register_architecture("Qwen3ForCausalLM", Qwen3Config, model_type="qwen3")
 register_architecture("Lemesun", LemesunConfig)
 register_architecture("Losivik", LosivikConfig)
+register_architecture("Noganex", NoganexConfig)
 register_architecture("Nulalorn", NulalornConfig)
 register_architecture("Zigivik", ZigivikConfig)

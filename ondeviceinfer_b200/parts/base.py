@@ -55,6 +55,10 @@ pending as ``ctx.pending_residual_add = (residual, output, weight, eps)``, which
 return a new residual stream instead of changing the one it was given (the model goes on with it), and a block that
 says ``reads_embedding = True`` finds the embedding's output as ``ctx.embedded``.
 
+Also optional: a block that has the stream's rows in the compute dtype when it ends may leave them for the next block
+as ``ctx.stream_copy = (hidden, rows)`` if it says ``renews_stream_copy = True`` (the model drops the note before any
+other block).
+
 Also optional: a mixer whose single-token kernel cuts each sequence's keys among several blocks may ask the
 context how (``ctx.key_splits(blocks_per_cut) -> (tiles_per_split, splits)``): the number of 64-key tiles
 that a block takes, as one int32 on the device that follows the step's sequences (also under graph replay,

@@ -5,7 +5,7 @@ from __future__ import annotations
 import torch
 
 from ..cache import StateNeed
-from ..config.specs import ParallelBlockSpec, PreNormBlockSpec, ReinjectSpec, SandwichBlockSpec, ScaledParallelBlockSpec
+from ..config.specs import GatedPostNormBlockSpec, ParallelBlockSpec, PreNormBlockSpec, ReinjectSpec, SandwichBlockSpec, ScaledParallelBlockSpec
 from ..weights.tensors import TensorDecl
 from .base import Part, build_part, register_part
 
@@ -150,6 +150,94 @@ class SandwichBlock(Part):
             out = self._branch(self.ffn, hidden, lambda r: self.ffn.forward(normed, ctx, r))
             ctx.pending_residual_add = (hidden, out, self.ffn_post_norm.weight, self.ffn_post_norm.spec.eps)
         ctx.residual_sumsq = None
+
+
+class GatedPostNormBlock(Part):
+    """x <- x + norm1(mixer(x) * sigmoid(R1 x + r1)); x <- x + norm2(feed_forward(x) * sigmoid(R2 x + r2)).
+
+    The sublayers and the gates' products read the stream's rows in the compute dtype; ``ops.gated_norm_add`` takes a
+    sublayer's fp32 output (a part that says ``returns_output`` returns it; any other adds into a zeroed buffer) and the
+    gate's fp32 logits, gates, norms and adds to the stream in fp32, and writes the new rows in the compute dtype for
+    whoever reads them next: the feed-forward, or the next block of this kind (``ctx.stream_copy``)."""
+
+    renews_stream_copy = True
+
+    def __init__(self, spec: GatedPostNormBlockSpec) -> None:
+        super().__init__(spec)
+        has = spec.ffn is not None
+        if has != (spec.ffn_norm is not None) or (not has and spec.ffn_gate_name is not None):
+            raise ValueError("a feed-forward comes with its norm (and perhaps its gate), or none of them")
+        self.mixer = build_part(spec.mixer)
+        self.mixer_norm = build_part(spec.mixer_norm)
+        self.ffn = build_part(spec.ffn) if has else None
+        self.ffn_norm = build_part(spec.ffn_norm) if has else None
+        for norm in (self.mixer_norm, self.ffn_norm):
+            if norm is not None and not (getattr(norm.spec, "scale_in_fp32", False) and hasattr(norm.spec, "eps")):
+                raise TypeError("the norm after a sublayer is an RMS norm that scales in fp32")
+
+    def _children(self):
+        return tuple(part for part in (self.mixer, self.mixer_norm, self.ffn, self.ffn_norm) if part is not None)
+
+    def tensor_decls(self):
+        s = self.spec
+        decls = [d for part in self._children() for d in part.tensor_decls()]
+        for weight, bias in ((s.mixer_gate_name, s.mixer_gate_bias_name), (s.ffn_gate_name, s.ffn_gate_bias_name)):
+            if weight is not None:
+                decls.append(TensorDecl(weight, (s.hidden_size, s.hidden_size)))
+                if bias is not None:
+                    decls.append(TensorDecl(bias, (s.hidden_size,)))
+        return decls
+
+    def load(self, fetch, runtime) -> None:
+        self.runtime = runtime
+        for part in self._children():
+            part.load(fetch, runtime)
+        s = self.spec
+        gate = lambda weight, bias: (None if weight is None else fetch.matrix(weight),
+                                     None if weight is None or bias is None else fetch.vector(bias))
+        self.mixer_gate = gate(s.mixer_gate_name, s.mixer_gate_bias_name)
+        self.ffn_gate = gate(s.ffn_gate_name, s.ffn_gate_bias_name)
+
+    def cache_needs(self):
+        return tuple(self.mixer.cache_needs())
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(part, "graph_safe", False) for part in self._children())
+
+    def _rows(self, hidden, ctx):
+        """The stream's rows in the compute dtype."""
+        from ..kernels import ops
+        if self.runtime.dtype == torch.float32:
+            return hidden
+        known = ctx.stream_copy
+        if known is not None and known[0] is hidden and known[1].dtype == self.runtime.dtype:
+            return known[1]
+        rows = torch.empty(hidden.shape, dtype=self.runtime.dtype, device=hidden.device)
+        ops.cast_rows(hidden, rows)
+        return rows
+
+    def _half(self, hidden, ctx, part, norm, gate, call):
+        from ..kernels import ops
+        from .linear import linear
+        x = self._rows(hidden, ctx)
+        weight, bias = gate
+        logits = None if weight is None else linear(x, weight, bias=bias, out_dtype=torch.float32)
+        out = SandwichBlock._branch(part, hidden, lambda residual: call(x, residual))
+        ctx.residual_sumsq = None
+        rows = None
+        if self.runtime.dtype != torch.float32:
+            rows = torch.empty(hidden.shape, dtype=self.runtime.dtype, device=hidden.device)
+        ops.gated_norm_add(hidden, out, logits, norm.weight, norm.spec.eps, rows)
+        ctx.stream_copy = None if rows is None else (hidden, rows)
+
+    def forward(self, hidden, ctx, view) -> None:
+        ctx.defers_residual_add = False        # the parts' own products add (or return) at once
+        self._half(hidden, ctx, self.mixer, self.mixer_norm, self.mixer_gate,
+                   lambda x, residual: self.mixer.forward(x, ctx, view, residual))
+        if self.ffn is not None:
+            self._half(hidden, ctx, self.ffn, self.ffn_norm, self.ffn_gate,
+                       lambda x, residual: self.ffn.forward(x, ctx, residual))
 
 
 class ParallelBlock(Part):
@@ -344,6 +432,7 @@ class Reinject(Part):
 
 register_part(PreNormBlockSpec, PreNormBlock)
 register_part(SandwichBlockSpec, SandwichBlock)
+register_part(GatedPostNormBlockSpec, GatedPostNormBlock)
 register_part(ParallelBlockSpec, ParallelBlock)
 register_part(ScaledParallelBlockSpec, ScaledParallelBlock)
 register_part(ReinjectSpec, Reinject)

@@ -43,13 +43,13 @@ PERSISTENT_MIN_TOKENS_FUSED, PERSISTENT_MIN_TOKENS_PLAIN = 1024, 2048
 
 
 def _persistent(tokens: int, weight: torch.Tensor, x: torch.Tensor, epi: int, biased: bool = False) -> bool:
-    n_out = weight.shape[0] // 2 if epi == ops.EPI_SWIGLU else weight.shape[0]
+    n_out = weight.shape[0] // 2 if epi in ops.EPI_GATED else weight.shape[0]
     out_dtype = torch.float32 if epi in (ops.EPI_STORE_F32, ops.EPI_RESIDUAL) else torch.bfloat16
     if PREFILL_GEMM == "library" or not ops.gemm_prefill_supported(x, weight, n_out, out_dtype):
         return False
     if PREFILL_GEMM == "own":
         return True
-    fused = biased or epi in (ops.EPI_SWIGLU, ops.EPI_RESIDUAL, ops.EPI_GELU)      # a bias is a fused epilogue too
+    fused = biased or epi in (ops.EPI_SWIGLU, ops.EPI_GEGLU, ops.EPI_RESIDUAL, ops.EPI_GELU)      # a bias is a fused epilogue too
     return tokens >= (PERSISTENT_MIN_TOKENS_FUSED if fused else PERSISTENT_MIN_TOKENS_PLAIN)
 
 
@@ -333,18 +333,25 @@ def activated_linear(x: torch.Tensor, weight: torch.Tensor, kind: str) -> torch.
     return out
 
 
-def gated_linear(x, weight_gate_up: torch.Tensor) -> torch.Tensor:
-    """silu(x Wg^T) * (x Wu^T) for ``weight_gate_up`` = gate rows followed by up rows."""
+def gated_linear(x, weight_gate_up: torch.Tensor, *, bias: Optional[torch.Tensor] = None, kind: str = "silu") -> torch.Tensor:
+    """act(x Wg^T + bg) * (x Wu^T + bu) for ``weight_gate_up`` = gate rows followed by up rows; ``kind`` "silu" or
+    "gelu_tanh", ``bias`` None or fp32 [2 I] (gate, then up)."""
     n, I = x.shape[0], weight_gate_up.shape[0] // 2
     act = torch.empty((n, I), dtype=x.dtype, device=x.device)
-    if x.dtype == torch.bfloat16 and _own(x, weight_gate_up):
-        x, norm = _operand(x, weight_gate_up, I, ops.EPI_SWIGLU)
-        ops.gemm_bf16(x, weight_gate_up, act, ops.EPI_SWIGLU, norm=norm)
+    epi = ops.EPI_SWIGLU if kind == "silu" else ops.EPI_GEGLU
+    biased = bias is not None
+    if x.dtype == torch.bfloat16 and _own(x, weight_gate_up, biased):
+        x, norm = _operand(x, weight_gate_up, I, epi)
+        ops.gemm_bf16(x, weight_gate_up, act, epi, norm=norm, bias=bias)
         return act
     if isinstance(x, NormedRows):
         x = x.materialize()
-    if x.dtype == torch.bfloat16 and _persistent(n, weight_gate_up, x, ops.EPI_SWIGLU):
-        ops.gemm_prefill_bf16(x, weight_gate_up, act, ops.EPI_SWIGLU)
+    if x.dtype == torch.bfloat16 and _persistent(n, weight_gate_up, x, epi, biased):
+        ops.gemm_prefill_bf16(x, weight_gate_up, act, epi, bias=bias)
         return act
-    ops.silu_mul(linear(x, weight_gate_up), act)
+    product = linear(x, weight_gate_up, bias=bias)
+    if kind == "silu":
+        ops.silu_mul(product, act)
+    else:
+        ops.gated_activation(product, act, kind)
     return act

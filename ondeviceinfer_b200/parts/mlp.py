@@ -12,31 +12,52 @@ from .linear import activated_linear, gated_linear, linear
 
 
 class GatedMLP(Part):
+    """down(act(gate(x)) * up(x)), act SiLU or the tanh form of GELU, with biases on the projections that the spec names
+    one for.  The gate and up matrices are concatenated at load so that one matrix product yields both (the biases join
+    its fp32 sums); the activation is taken in fp32 and rounded once, in the product's epilogue where the tensor-core
+    kernels serve it."""
+
     graph_safe = True   # no host work that depends on the step's values: may be captured in a CUDA graph
     takes_lazy_norm = True   # x may be a NormedRows: its first product makes the normed operand itself
-
-    """down(silu(gate(x)) * up(x)).  The gate and up matrices are concatenated at load so
-    that one matrix product yields both; the activation is taken in fp32 and rounded once."""
+    returns_output = True    # forward(..., residual=None) returns the fp32 output instead of adding it
 
     def __init__(self, spec: GatedMLPSpec) -> None:
         super().__init__(spec)
-        if spec.activation != "silu":
-            raise ValueError(f"activation {spec.activation!r} is not implemented (silu is)")
+        if spec.activation not in ops.GATED_ACTIVATIONS:
+            raise ValueError(f"activation {spec.activation!r} is not implemented ({sorted(ops.GATED_ACTIVATIONS)} are)")
 
     def tensor_decls(self):
         s = self.spec
-        return [TensorDecl(s.name("gate"), (s.intermediate_size, s.hidden_size)),
-                TensorDecl(s.name("up"), (s.intermediate_size, s.hidden_size)),
-                TensorDecl(s.name("down"), (s.hidden_size, s.intermediate_size))]
+        decls = [TensorDecl(s.name("gate"), (s.intermediate_size, s.hidden_size)),
+                 TensorDecl(s.name("up"), (s.intermediate_size, s.hidden_size)),
+                 TensorDecl(s.name("down"), (s.hidden_size, s.intermediate_size))]
+        sizes = (("gate_bias", s.intermediate_size), ("up_bias", s.intermediate_size), ("down_bias", s.hidden_size))
+        return decls + [TensorDecl(s.name(role), (size,)) for role, size in sizes if s.has(role)]
 
     def load(self, fetch, runtime) -> None:
         s = self.spec
         self.runtime = runtime
         self.w_gate_up = torch.cat([fetch.matrix(s.name("gate")), fetch.matrix(s.name("up"))], 0)
         self.w_down = fetch.matrix(s.name("down"))
+        self.b_gate_up = gate_up_bias(s, fetch, runtime)
+        self.b_down = fetch.vector(s.name("down_bias")) if s.has("down_bias") else None
 
-    def forward(self, x, ctx, residual) -> None:
-        linear(gated_linear(x, self.w_gate_up), self.w_down, residual=residual, track=ctx)
+    def forward(self, x, ctx, residual):
+        """Adds to ``residual`` (fp32); with ``residual`` None returns the output as a new fp32 tensor."""
+        act = gated_linear(x, self.w_gate_up, bias=self.b_gate_up, kind=self.spec.activation)
+        if residual is None:
+            return linear(act, self.w_down, bias=self.b_down, out_dtype=torch.float32)
+        linear(act, self.w_down, bias=self.b_down, residual=residual, track=ctx)
+        return None
+
+
+def gate_up_bias(s, fetch, runtime):
+    """The biases of the gate and up projections side by side (fp32; a projection without one adds zero), or None."""
+    if not (s.has("gate_bias") or s.has("up_bias")):
+        return None
+    return torch.cat([fetch.vector(s.name(role)) if s.has(role)
+                      else torch.zeros(s.intermediate_size, dtype=torch.float32, device=runtime.device)
+                      for role in ("gate_bias", "up_bias")])
 
 
 class PlainMLP(Part):
@@ -130,11 +151,7 @@ class ClampedGatedMLP(Part):
         self.runtime = runtime
         self.w_gate_up = torch.cat([fetch.matrix(s.name("gate")), fetch.matrix(s.name("up"))], 0)
         self.w_down = fetch.matrix(s.name("down"))
-        self.b_gate_up = None
-        if s.has("gate_bias") or s.has("up_bias"):       # a projection without a bias adds zero
-            self.b_gate_up = torch.cat([fetch.vector(s.name(role)) if s.has(role)
-                                        else torch.zeros(s.intermediate_size, dtype=torch.float32, device=runtime.device)
-                                        for role in ("gate_bias", "up_bias")])
+        self.b_gate_up = gate_up_bias(s, fetch, runtime)
         self.b_down = fetch.vector(s.name("down_bias")) if s.has("down_bias") else None
 
     def forward(self, x, ctx, residual):

@@ -17,7 +17,8 @@ class RMSNorm(Part):
 
     """weight * cast(x * rsqrt(mean(x^2) + eps)): statistics in fp32, cast to the compute
     dtype before the multiplication by the weight.  With ``scale_in_fp32`` the row is scaled in fp32 and
-    rounded once; ``weight_offset`` is added to the stored weight (in fp32, at load)."""
+    rounded once; ``weight_offset`` is added to the stored weight and ``output_scale``
+    multiplies the sum (in fp32, at load)."""
 
     def __init__(self, spec: RMSNormSpec) -> None:
         super().__init__(spec)
@@ -33,6 +34,8 @@ class RMSNorm(Part):
         self.weight = fetch.vector(self.spec.weight_name)
         if self.spec.weight_offset != 0.0:
             self.weight = self.weight + self.spec.weight_offset
+        if self.spec.output_scale != 1.0:
+            self.weight = self.weight * self.spec.output_scale
         if self.spec.scalar_weight:
             # one number for all coordinates: kept as it is for kernels that take it so, and laid out as a row
             # for the norm kernels that take a weight per coordinate

@@ -14,7 +14,8 @@ Steps of ``forward`` (no step waits for the host):
    an identity output;
 5. the shared expert, if any: gate/up product, the same activation with its own limit, down with the residual add.
 
-Options of the spec: sigmoid scores instead of the softmax (a flag of the routing kernel); ungated experts with the
+Options of the spec: experts (and the shared one) that are SiLU gates without limits, the same kernels with other
+constants; weights divided by their sum and multiplied by a constant (in the routing kernel); sigmoid scores instead of the softmax (a flag of the routing kernel); ungated experts with the
 squared ReLU (one up matrix per expert, the activation in the grouped product's epilogue or, after the vendor
 library's product, in ``ops.activation``); weights that multiply the experts' inputs (the rows are gathered in the
 sorted order and multiplied by their pair's weight in fp32 on the way, ``ops.moe_gather``; the combine then adds
@@ -23,13 +24,15 @@ the chosen rows unweighted).
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..config.specs import RoutedExpertsSpec
 from ..kernels import ops
 from ..weights.tensors import TensorDecl
 from .base import Part, register_part
-from .linear import linear
+from .linear import gated_linear, linear
 
 
 # From this many rows per expert on (on average) a bfloat16 step runs each expert's products through linear().
@@ -54,11 +57,15 @@ class RoutedExperts(Part):
             raise ValueError("top_k exceeds the outputs that the kept groups hold")
         if spec.scoring not in ("softmax", "sigmoid"):
             raise ValueError(f"scoring {spec.scoring!r} is not implemented (softmax and sigmoid are)")
-        if spec.expert_form not in ("gated_clamp", "relu2"):
-            raise ValueError(f"expert form {spec.expert_form!r} is not implemented (gated_clamp and relu2 are)")
+        if spec.expert_form not in ("gated_clamp", "gated_silu", "relu2"):
+            raise ValueError(f"expert form {spec.expert_form!r} is not implemented (gated_clamp, gated_silu and relu2 are)")
         if spec.weight_on_input and spec.num_identity > 0:
             raise ValueError("identity outputs take their weight on the output")
-        self.gated = spec.expert_form == "gated_clamp"
+        self.gated = spec.expert_form != "relu2"
+        # the gated activation g sigmoid(alpha g) (u + shift) of clamped g and u; SiLU times up is its form without limits
+        silu = spec.expert_form == "gated_silu"
+        self.limit, self.shared_limit = (math.inf, math.inf) if silu else (spec.limit, spec.shared_limit)
+        self.gate_alpha, self.up_shift = (1.0, 0.0) if silu else (spec.gate_alpha, 1.0)
         self.n_all = n_all
 
     def tensor_decls(self):
@@ -99,7 +106,7 @@ class RoutedExperts(Part):
         ids = torch.empty((n, s.top_k), dtype=torch.int32, device=dev)
         weights = torch.empty((n, s.top_k), dtype=torch.float32, device=dev)
         ops.moe_route(logits, self.correction, ids, weights, n_groups=s.num_groups, keep=s.keep_groups,
-                      sigmoid=s.scoring == "sigmoid")
+                      sigmoid=s.scoring == "sigmoid", renormalise=s.renormalise, scale=s.weight_scale)
         # single-token steps, a few rows per expert: the grouped product that streams weights through registers
         few_ok = ops.grouped_few_rows_ok((s.hidden_size, s.expert_size), x.dtype)
         table = ops.RoutingTable(n, s.top_k, max(s.num_experts, 1), dev, few_rows_ok=few_ok)
@@ -114,26 +121,29 @@ class RoutedExperts(Part):
             elif s.weight_on_input:
                 rows = torch.empty((table.n_pairs, s.hidden_size), dtype=x.dtype, device=dev)
                 ops.moe_gather(x, table, rows, weights)
-                ops.grouped_gemm_routed(rows, self.w_gate_up, act, table, gather=False, epi=first_epi, limit=s.limit,
-                                        alpha=s.gate_alpha)
+                ops.grouped_gemm_routed(rows, self.w_gate_up, act, table, gather=False, epi=first_epi, limit=self.limit,
+                                        alpha=self.gate_alpha, up_shift=self.up_shift)
                 ops.grouped_gemm_routed(act, self.w_down, expert_out, table, gather=False, epi=ops.GROUPED_STORE_F32)
             else:
-                ops.grouped_gemm_routed(x, self.w_gate_up, act, table, gather=True, epi=first_epi, limit=s.limit,
-                                        alpha=s.gate_alpha)
+                ops.grouped_gemm_routed(x, self.w_gate_up, act, table, gather=True, epi=first_epi, limit=self.limit,
+                                        alpha=self.gate_alpha, up_shift=self.up_shift)
                 ops.grouped_gemm_routed(act, self.w_down, expert_out, table, gather=False, epi=ops.GROUPED_STORE_F32)
         out = residual
         if residual is None:       # the caller wants the output itself: the combine assigns, the shared expert adds
             out = torch.empty((n, s.hidden_size), dtype=torch.float32, device=dev)
         ops.moe_combine(out, expert_out, x, ids, None if s.weight_on_input else weights, table, assign=residual is None)
         if s.shared_size > 0:
-            act = torch.empty((n, s.shared_size), dtype=x.dtype, device=dev)
-            self._activate(linear(x, self.w_shared_gate_up), act, s.shared_limit)
+            if s.expert_form == "gated_silu":
+                act = gated_linear(x, self.w_shared_gate_up)
+            else:
+                act = torch.empty((n, s.shared_size), dtype=x.dtype, device=dev)
+                self._activate(linear(x, self.w_shared_gate_up), act, self.shared_limit)
             linear(act, self.w_shared_down, residual=out, track=ctx if residual is not None else None)
         return None if residual is not None else out
 
     def _activate(self, product, act, limit):
         if self.gated:
-            ops.gated_clamp(product, act, limit, self.spec.gate_alpha)
+            ops.gated_clamp(product, act, limit, self.gate_alpha, self.up_shift)
         else:
             ops.activation(product, act, "relu2")
 
@@ -148,7 +158,7 @@ class RoutedExperts(Part):
             try:
                 ends = table.offsets[1:]
                 gate_up = torch._grouped_mm(rows, self.w_gate_up.transpose(1, 2), offs=ends)
-                self._activate(gate_up, act, s.limit)
+                self._activate(gate_up, act, self.limit)
                 down = torch._grouped_mm(act, self.w_down.transpose(1, 2), offs=ends)
                 ops.LAUNCHES["library"] += 2
                 return down                                   # rounded to the compute dtype; the combine widens it
@@ -161,7 +171,7 @@ class RoutedExperts(Part):
         for e in range(s.num_experts):
             lo, hi = bounds[e], bounds[e + 1]
             if hi > lo:
-                self._activate(linear(rows[lo:hi], self.w_gate_up[e]), act[lo:hi], s.limit)
+                self._activate(linear(rows[lo:hi], self.w_gate_up[e]), act[lo:hi], self.limit)
                 expert_out[lo:hi].copy_(linear(act[lo:hi], self.w_down[e], out_dtype=torch.float32))
         return expert_out
 
