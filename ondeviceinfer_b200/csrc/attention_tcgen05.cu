@@ -40,7 +40,11 @@
 //
 // Works for any q_len >= 1 on top of any cached length (query t of the step sits at position
 // past + t).  Optional: a window (the walk starts at the tile of the oldest key the CTA's rows see; the page list
-// may be a ring), and scores squashed by c tanh(score / c).  Compile with -DODI_HEAD_DIM=64 or 128.
+// may be a ring), scores squashed by c tanh(score / c), a chunk (the query at position p sees j <= p with j / chunk ==
+// p / chunk; the walk starts at the tile of the first row's chunk), and heads that mix their scores (MIXED): q is
+// [n_tokens, nq, nkv, D], a score is the sum over the key heads of q_hj . k_j, accumulated in tensor memory key head by
+// key head, so a page's key heads pass one after the other through a ring of their own (KRING slots) while the CTA's
+// query rows of all key heads stay in shared memory.  Compile with -DODI_HEAD_DIM=64 or 128.
 //
 // Every wait on an mbarrier is bounded (about two seconds of SM clock): a role that gives up
 // records a code in `status`, raises the CTA's abort flag, and all roles fall through to the
@@ -61,6 +65,8 @@
 #define BNK 64                 // keys per page / tile
 #define KB (D / 64)            // 64-wide blocks of the head size
 #define RING 2                 // K pages, and V pages, in flight
+#define SMEM_LIMIT (232448 - 512)      // what a CTA may ask for beside its barriers
+#define MIXED_KEY_RING 4       // slots of the key ring when heads mix their scores: a page's key heads take one each
 #define Q_BYTES (KB * BM * 128)
 #define KV_BYTES (KB * BNK * 128)     // one of K or V for a page
 #define HEAD_COLS 256                  // tensor-memory columns per head: S0, S1, O
@@ -91,6 +97,8 @@ struct TcAttnArgs {
   float softcap;          // c > 0: a score (times scale) becomes c tanh(score / c) before the softmax
   int sink;               // 1: the softmax has one more term, of score 0 and without a value
   int keep;               // > 0 with a window: keys 0..keep-1 stay visible beyond the window; their tiles come first in the walk
+  int chunk;              // > 0: keys of the query's own chunk of this many positions
+  int mixed;              // 1: a score sums over the key heads (q has nkv rows of D lanes a head)
 };
 
 // ------------------------------------------------------------------------------ PTX wrappers
@@ -350,15 +358,18 @@ __device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, b
   }
 }
 
-template <int TILES>
-__global__ void __launch_bounds__(64 + 128 * TILES, TILES == 1 ? 2 : 1)
+template <int TILES, bool MIXED>
+__global__ void __launch_bounds__(64 + 128 * TILES, TILES == 1 && !MIXED ? 2 : 1)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const TcAttnArgs a) {
   constexpr int TMEM_COLS = TILES * HEAD_COLS;
+  constexpr int KRING = MIXED ? MIXED_KEY_RING : RING;
+  static_assert(!MIXED || TILES == 1, "mixed heads take one head per CTA");
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-  // barriers: q_full, k_full[R], k_empty[R], v_full[R], v_empty[R], s_full[2], p_full[TILES][2], pv_done[TILES]
-  __shared__ __align__(8) uint64_t bars[1 + 4 * RING + 2 + 3 * TILES];
+  // barriers: q_full, k_full[KR], k_empty[KR], v_full[R], v_empty[R], s_full[2], p_full[TILES][2], pv_done[TILES]
+  constexpr int BARS = 1 + 2 * KRING + 2 * RING + 2 + 3 * TILES;
+  __shared__ __align__(8) uint64_t bars[BARS];
   __shared__ uint32_t tmem_base_slot;
   __shared__ int abort_flag;
 
@@ -372,7 +383,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const int past = a.past[seq];
   const int nt = min(BM, q_len - t0);
   // key tiles from the one that holds the oldest key any row of the CTA sees up to the diagonal
-  const int tile_lo = a.window > 0 ? max(0, past + t0 - a.window + 1) / BNK : 0;
+  const int first = past + t0;
+  const int tile_lo = (a.window > 0 ? max(0, first - a.window + 1) : (a.chunk > 0 ? first - first % a.chunk : 0)) / BNK;
   // in front of them the tiles of kept first keys that lie before the window's first tile
   const int keep_tiles = a.window > 0 && a.keep > 0 ? min((a.keep + BNK - 1) / BNK, tile_lo) : 0;
   const int n_tiles = keep_tiles + (past + t0 + nt + BNK - 1) / BNK - tile_lo;
@@ -380,15 +392,16 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const int* pages = a.page_ids + a.page_start[seq];
 
   const uint32_t bar0 = smem_u32(&bars[0]);
-  const uint32_t q_full = bar0, k_full = bar0 + 8, k_empty = k_full + 8 * RING, v_full = k_empty + 8 * RING,
+  const uint32_t q_full = bar0, k_full = bar0 + 8, k_empty = k_full + 8 * KRING, v_full = k_empty + 8 * KRING,
                  v_empty = v_full + 8 * RING, s_full = v_empty + 8 * RING, p_full = s_full + 16,
                  pv_done = p_full + 16 * TILES;
   uint8_t* q_smem = smem;                                    // head t at t * Q_BYTES
-  uint8_t* k_smem = smem + TILES * Q_BYTES;                  // ring of K pages
-  uint8_t* v_smem = k_smem + RING * KV_BYTES;             // ring of V pages
+  const int KH = MIXED ? a.nkv : 1;                          // key heads a score sums over
+  uint8_t* k_smem = smem + TILES * KH * Q_BYTES;             // ring of K pages
+  uint8_t* v_smem = k_smem + KRING * KV_BYTES;            // ring of V pages
 
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 1 + 4 * RING + 2 + 3 * TILES; ++i) mbar_init(bar0 + 8 * i, 1);
+    for (int i = 0; i < BARS; ++i) mbar_init(bar0 + 8 * i, 1);
     for (int b = 0; b < 2; ++b)
       for (int t = 0; t < TILES; ++t) mbar_init(p_full + 16 * t + 8 * b, 4);     // one arrival per softmax warp
     abort_flag = 0;
@@ -408,25 +421,29 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     // ---------------------------------------------------------------- TMA producer: K_0, K_1, V_0, then K_j, V_{j-1}
     if (lane == 0) {
       pdl_wait();      // queries and this step's keys/values come from the kernel before
-      mbar_expect_tx(q_full, TILES * Q_BYTES);
-      for (int t = 0; t < TILES; ++t)
+      mbar_expect_tx(q_full, TILES * KH * Q_BYTES);
+      for (int t = 0; t < TILES * KH; ++t)
         for (int kb = 0; kb < KB; ++kb)
-          tma_load_2d(smem_u32(q_smem + t * Q_BYTES + kb * BM * 128), &map_q, (head0 + t) * D + kb * 64, q_begin + t0, q_full);
+          tma_load_2d(smem_u32(q_smem + t * Q_BYTES + kb * BM * 128), &map_q, (head0 * KH + t) * D + kb * 64, q_begin + t0, q_full);
       bool ok = true;
-      auto load_page = [&](int j, const CUtensorMap* map, uint8_t* ring, uint32_t full, uint32_t empty) {
-        const int s = j % RING;
-        if (!mbar_wait(empty + 8 * s, ((uint32_t)(j / RING) & 1u) ^ 1u, abort_ptr)) { ok = false; return; }
+      // box n of a ring of `slots` slots: head `h` of page j
+      auto load_box = [&](int n, int slots, int j, int h, const CUtensorMap* map, uint8_t* ring, uint32_t full, uint32_t empty) {
+        const int s = n % slots;
+        if (!mbar_wait(empty + 8 * s, ((uint32_t)(n / slots) & 1u) ^ 1u, abort_ptr)) { ok = false; return; }
         const int entry = page_slot_of_page(tile_of(j), a.ring_pages);
-        const int row = (pages[entry] * a.nkv + hk) * BNK;
+        const int row = (pages[entry] * a.nkv + h) * BNK;
         mbar_expect_tx(full + 8 * s, KV_BYTES);
         for (int kb = 0; kb < KB; ++kb)
           tma_load_2d(smem_u32(ring + (size_t)s * KV_BYTES + kb * BNK * 128), map, kb * 64, row, full + 8 * s);
       };
+      auto load_keys = [&](int j) {
+        for (int g = 0; g < KH && ok; ++g) load_box(j * KH + g, KRING, j, MIXED ? g : hk, &map_k, k_smem, k_full, k_empty);
+      };
       // keys run one page ahead of values: a K slot is free as soon as its scores are computed
-      load_page(0, &map_k, k_smem, k_full, k_empty);
+      load_keys(0);
       for (int j = 1; j <= n_tiles && ok; ++j) {
-        if (j < n_tiles) load_page(j, &map_k, k_smem, k_full, k_empty);
-        if (ok) load_page(j - 1, &map_v, v_smem, v_full, v_empty);
+        if (j < n_tiles) load_keys(j);
+        if (ok) load_box(j - 1, RING, j - 1, hk, &map_v, v_smem, v_full, v_empty);
       }
       if (!ok) atomicCAS(a.status, 0, ATT_ERR_PRODUCER);
     }
@@ -437,22 +454,25 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       constexpr uint32_t idesc_o = idesc_bf16(BM, D, true);
       bool ok = mbar_wait(q_full, 0, abort_ptr);
       auto issue_s = [&](int j) -> bool {
-        const int s = j % RING, b = j & 1;
-        if (!mbar_wait(k_full + 8 * s, (uint32_t)(j / RING) & 1u, abort_ptr)) return false;
-        tc_fence_after();
-        const uint32_t k_addr = smem_u32(k_smem + (size_t)s * KV_BYTES);
+        const int b = j & 1;
+        for (int g = 0; g < KH; ++g) {
+          const int n = j * KH + g, s = n % KRING;
+          if (!mbar_wait(k_full + 8 * s, (uint32_t)(n / KRING) & 1u, abort_ptr)) return false;
+          tc_fence_after();
+          const uint32_t k_addr = smem_u32(k_smem + (size_t)s * KV_BYTES);
 #pragma unroll
-        for (int t = 0; t < TILES; ++t) {
+          for (int t = 0; t < TILES; ++t) {
 #pragma unroll
-          for (int kb = 0; kb < KB; ++kb) {
-            const uint64_t dq = desc_k_major(smem_u32(q_smem + t * Q_BYTES + kb * BM * 128));
-            const uint64_t dk = desc_k_major(k_addr + kb * BNK * 128);
+            for (int kb = 0; kb < KB; ++kb) {
+              const uint64_t dq = desc_k_major(smem_u32(q_smem + (t * KH + g) * Q_BYTES + kb * BM * 128));
+              const uint64_t dk = desc_k_major(k_addr + kb * BNK * 128);
 #pragma unroll
-            for (int i = 0; i < 4; ++i) umma(tmem_base + S_COL(t, b), dq + 2 * i, dk + 2 * i, idesc_s, (kb | i) ? 1u : 0u);
+              for (int i = 0; i < 4; ++i) umma(tmem_base + S_COL(t, b), dq + 2 * i, dk + 2 * i, idesc_s, (g | kb | i) ? 1u : 0u);
+            }
           }
+          if (g == KH - 1) umma_commit(s_full + 8 * b);       // the scores are done ...
+          umma_commit(k_empty + 8 * s);      // ... and the K slot is free
         }
-        umma_commit(s_full + 8 * b);       // the scores are done ...
-        umma_commit(k_empty + 8 * s);      // ... and the K slot is free
         return true;
       };
       // S_{j+1} overwrites the buffer whose first columns held P_{j-1}: it is issued after the product of
@@ -488,7 +508,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const uint32_t lane_addr = (uint32_t)(lane_group * 32) << 16;
     const float sl2 = a.softcap > 0.f ? LOG2E : a.scale * LOG2E;
     const float two_over_cap = a.softcap > 0.f ? 2.f / a.softcap : 0.f;
-    const int oldest = a.window > 0 ? pos - a.window + 1 : 0;
+    const int oldest = a.window > 0 ? pos - a.window + 1 : (a.chunk > 0 ? pos - pos % a.chunk : 0);
     // a sink is a key of score 0 and value 0 ahead of all others: the row starts from its maximum and its weight
     RowState st = {a.sink ? 0.f : -INFINITY, a.sink ? 1.f : 0.f};
     bool ok = true;
@@ -554,18 +574,24 @@ static int make_map(CUtensorMap* map, const void* base, long rows, long cols, in
 
 extern "C" int odi_attention_tcgen05_head_dim() { return D; }
 
+// Whether shared memory holds a CTA's query rows of `nkv` key heads (heads that mix their scores).
+extern "C" int odi_attention_tcgen05_fits_mixed(int nkv) {
+  return nkv > 0 && nkv <= 64 && nkv * Q_BYTES + (MIXED_KEY_RING + RING) * KV_BYTES + 1024 <= SMEM_LIMIT;
+}
+
 // q [n_tokens, nq * D] bf16; k_pool, v_pool [pool_pages, nkv, 64, D] bf16; out [n_tokens, nq * D].
 // heads_per_cta: 2 = two heads of a key/value group per CTA (needs an even group size), 1 = one, 0 = choose.
-template <int TILES>
+template <int TILES, bool MIXED>
 static int launch_attention(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnArgs& a,
                             int max_q_len, cudaStream_t stream) {
-  const int smem = TILES * Q_BYTES + 2 * RING * KV_BYTES + 1024;
-  auto kernel = attention_tcgen05_kernel<TILES>;
-  static bool configured = false;
-  if (!configured) {
+  const int smem = TILES * (MIXED ? a.nkv : 1) * Q_BYTES + ((MIXED ? MIXED_KEY_RING : RING) + RING) * KV_BYTES + 1024;
+  if (smem > SMEM_LIMIT) return ODI_ERR_UNSUPPORTED;
+  auto kernel = attention_tcgen05_kernel<TILES, MIXED>;
+  static int configured = 0;
+  if (configured < smem) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
-    configured = true;
+    configured = smem;
   }
   dim3 grid(a.nq / TILES, a.n_seqs, (max_q_len + BM - 1) / BM);
   odi_rc = launch_pdl((kernel), dim3(grid), dim3(64 + 128 * TILES), smem, stream, mq, mk, mv, a);
@@ -582,14 +608,16 @@ extern "C" int odi_attention_tcgen05(const void* q, const void* k_pool, const vo
     return ODI_ERR_UNSUPPORTED;
   if (pool_pages * a.nkv * BNK > 0x7fffffffL) return ODI_ERR_UNSUPPORTED;    // row coordinates are 32-bit
   if ((max_q_len + BM - 1) / BM > 65535) return ODI_ERR_UNSUPPORTED;
-  if (heads_per_cta < 0 || heads_per_cta > 2) return ODI_ERR_ARGUMENT;
+  if (heads_per_cta < 0 || heads_per_cta > 2 || a.chunk < 0 || (a.chunk > 0 && (a.window > 0 || a.keep > 0))) return ODI_ERR_ARGUMENT;
+  if (a.mixed && heads_per_cta == 2) return ODI_ERR_UNSUPPORTED;
   if (heads_per_cta == 2 && (a.nq / a.nkv) % 2 != 0) return ODI_ERR_ARGUMENT;
   CUtensorMap mq, mk, mv;
-  int rc = make_map(&mq, q, n_tokens, (long)a.nq * D, BM);
+  int rc = make_map(&mq, q, n_tokens, (long)a.nq * (a.mixed ? a.nkv : 1) * D, BM);
   if (rc == 0) rc = make_map(&mk, k_pool, pool_pages * a.nkv * BNK, D, BNK);
   if (rc == 0) rc = make_map(&mv, v_pool, pool_pages * a.nkv * BNK, D, BNK);
   if (rc != 0) return rc;
   if (heads_per_cta == 0) heads_per_cta = ODI_ATT_DEFAULT_HEADS_PER_CTA;
-  return heads_per_cta == 2 ? launch_attention<2>(mq, mk, mv, a, max_q_len, stream)
-                            : launch_attention<1>(mq, mk, mv, a, max_q_len, stream);
+  if (a.mixed) return launch_attention<1, true>(mq, mk, mv, a, max_q_len, stream);
+  return heads_per_cta == 2 ? launch_attention<2, false>(mq, mk, mv, a, max_q_len, stream)
+                            : launch_attention<1, false>(mq, mk, mv, a, max_q_len, stream);
 }

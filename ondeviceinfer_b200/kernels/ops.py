@@ -884,7 +884,7 @@ class _TcAttnArgs(Structure):
     _fields_ = [("out", c_void_p), ("cu_q", c_void_p), ("past", c_void_p), ("page_start", c_void_p),
                 ("page_ids", c_void_p), ("status", c_void_p), ("n_seqs", c_int), ("nq", c_int), ("nkv", c_int),
                 ("scale", c_float), ("window", c_int), ("ring_pages", c_int), ("softcap", c_float), ("sink", c_int),
-                ("keep", c_int)]
+                ("keep", c_int), ("chunk", c_int), ("mixed", c_int)]
 
 
 TCGEN05_ATTENTION_HEAD_DIMS = (64, 128)
@@ -892,11 +892,15 @@ TCGEN05_ATTENTION_HEAD_DIMS = (64, 128)
 
 def attention_tcgen05(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, n_seqs: int, max_q_len: int,
                       nq: int, nkv: int, d: int, page_size: int, scale: float, heads_per_cta: int = 0, window: int = 0,
-                      ring_pages: int = 0, softcap: float = 0.0, sink: bool = False, keep: int = 0) -> None:
+                      ring_pages: int = 0, softcap: float = 0.0, sink: bool = False, keep: int = 0, chunk: int = 0,
+                      mixed: bool = False) -> None:
     """bf16 causal GQA for prefill on tcgen05: scores and outputs in tensor memory, TMA-fed pages.
     ``sink``: one more term of score 0 and no value in the softmax.
     ``window`` > 0 keeps the last ``window`` keys visible (``ring_pages`` > 0: the page lists are rings);
     ``softcap`` c > 0 squashes the scores (times ``scale``) by c tanh(score / c).
+    ``chunk`` c > 0 (instead of a window): position p sees the keys of its own chunk of c positions only.
+    ``mixed``: q is [tokens, nq, nkv, d] and a score is the sum over the key heads of q . k (see :func:`mixed_prep`;
+    :func:`attention_tcgen05_fits_mixed` says for how many key heads).
     ``heads_per_cta``: 1, or 2 (two heads of a key/value group share a CTA and its K/V pages; needs an
     even group size), or 0 for the library's choice."""
     if d not in TCGEN05_ATTENTION_HEAD_DIMS:
@@ -905,16 +909,24 @@ def attention_tcgen05(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, 
         raise KernelError("the tcgen05 attention works on pages of 64 positions")
     for name, t in (("q", q), ("out", out), ("k_pool", k_pool), ("v_pool", v_pool)):
         _require(t, name, torch.bfloat16)
-    n_tokens = q.numel() // (nq * d)
-    if out.numel() != q.numel() or k_pool.shape != v_pool.shape or k_pool.dim() != 4:
+    n_tokens = q.numel() // (nq * d * (nkv if mixed else 1))
+    if out.numel() != n_tokens * nq * d or k_pool.shape != v_pool.shape or k_pool.dim() != 4:
         raise KernelError("attention_tcgen05: q/out or the pools disagree")
     _, _, status = _gemm_buffers(q.device, 0)
     args = _TcAttnArgs(_ptr(out), _ptr(cu_q), _ptr(past), _ptr(page_start), _ptr(page_ids), _ptr(status),
-                       n_seqs, nq, nkv, scale, window, ring_pages, softcap, 1 if sink else 0, keep)
+                       n_seqs, nq, nkv, scale, window, ring_pages, softcap, 1 if sink else 0, keep, chunk, 1 if mixed else 0)
     lib = load_library("attention_tcgen05", {"ODI_HEAD_DIM": d})
     _check(lib.odi_attention_tcgen05(_ptr(q), _ptr(k_pool), _ptr(v_pool), byref(args), c_int(n_tokens),
                                      c_int(max_q_len), c_long(k_pool.shape[0]), c_int(heads_per_cta), _stream()),
            "attention_tcgen05")
+
+
+def attention_tcgen05_fits_mixed(d: int, nkv: int) -> bool:
+    """Whether :func:`attention_tcgen05` takes ``mixed`` heads of ``d`` lanes over ``nkv`` key heads (shared memory holds
+    128 query rows of all of them)."""
+    if d not in TCGEN05_ATTENTION_HEAD_DIMS:
+        return False
+    return bool(load_library("attention_tcgen05", {"ODI_HEAD_DIM": d}).odi_attention_tcgen05_fits_mixed(c_int(nkv)))
 
 
 # ------------------------------------------------------------------------------ norms and activations in fp32
@@ -1642,6 +1654,55 @@ def mixed_prep(qkv, q_out, k_pool, v_pool, q_norm, k_norm, talk, cos_t, sin_t, t
                           d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, 1 if write_kv else 0, eps)
     lib = load_library("mixed")
     _check(lib.odi_mixed_prep(byref(args), c_int(dtype_code(qkv.dtype)), _stream()), "mixed_prep")
+
+
+class _MixedAttnArgs(Structure):
+    _fields_ = [("q", c_void_p), ("k_pool", c_void_p), ("v_pool", c_void_p), ("out", c_void_p), ("partial", c_void_p),
+                ("cu_q", c_void_p), ("past", c_void_p), ("page_start", c_void_p), ("page_ids", c_void_p), ("n_seqs", c_int),
+                ("nq", c_int), ("nkv", c_int), ("ring_pages", c_int), ("chunk", c_int), ("mixed", c_int), ("splits", c_int),
+                ("scale", c_float)]
+
+
+def attention_mixed_supported(dtype: torch.dtype, d: int, dv: int, nkv: int, mixed: bool) -> bool:
+    """Whether :func:`attention_mixed` takes these heads: bfloat16, key and value widths in steps of 16 up to 256, and
+    shared memory for 64 query rows of all key heads when the heads are mixed."""
+    if dtype != torch.bfloat16 or d % 16 or dv % 16 or not 16 <= d <= 256 or not 16 <= dv <= 256:
+        return False
+    lib = load_library("attention_mixed_mma", {"ODI_HEAD_DIM": d, "ODI_VALUE_DIM": dv})
+    return bool(lib.odi_attention_mixed_fits(c_int(nkv), c_int(1 if mixed else 0)))
+
+
+def attention_mixed(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, n_seqs: int, max_q_len: int, nq: int, nkv: int,
+                    d: int, dv: int, page_size: int, ring_pages: int, chunk: int, scale: float, mixed: bool, splits: int = 1,
+                    partial: Optional[torch.Tensor] = None) -> None:
+    """bf16 causal GQA on the tensor cores inside chunks (``chunk`` 0: none; the cache may be a ring of pages) for any
+    mixture of sequences; ``mixed``: q is [tokens, nq, nkv, d] and a score is the sum over the key heads of q . k (see
+    :func:`mixed_prep`), else [tokens, nq, d].  A step of single tokens (``max_q_len`` 1) takes the form that cuts each
+    sequence's visible keys into ``splits`` ranges; ``partial`` (fp32, tokens * nq * splits * (dv + 2)) holds their
+    results for the combine kernel."""
+    if not attention_mixed_supported(q.dtype, d, dv, nkv, mixed) or page_size != 64:
+        raise KernelError(f"attention_mixed takes bfloat16 heads in steps of 16 up to 256 and pages of 64 (d={d}, dv={dv}, nkv={nkv})")
+    for name, t in (("q", q), ("out", out), ("k_pool", k_pool), ("v_pool", v_pool)):
+        _require(t, name, torch.bfloat16)
+    n_tokens = q.numel() // (nq * d * (nkv if mixed else 1))
+    if out.numel() != n_tokens * nq * dv or k_pool.shape[-1] != d or v_pool.shape[-1] != dv:
+        raise KernelError("attention_mixed sizes disagree")
+    decode = max_q_len == 1
+    if decode and n_tokens != n_seqs:
+        raise KernelError("attention_mixed: max_q_len 1 means one token per sequence")
+    splits = splits if decode else 1
+    if splits > 1:
+        need = n_tokens * nq * splits * (dv + 2)
+        if partial is None or partial.numel() < need or partial.dtype != torch.float32:
+            raise KernelError(f"splits={splits} needs an fp32 partial buffer of {need} elements")
+    args = _MixedAttnArgs(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(partial if splits > 1 else None), _ptr(cu_q),
+                          _ptr(past), _ptr(page_start), _ptr(page_ids), n_seqs, nq, nkv, ring_pages, chunk, 1 if mixed else 0,
+                          splits, scale)
+    lib = load_library("attention_mixed_mma", {"ODI_HEAD_DIM": d, "ODI_VALUE_DIM": dv})
+    if decode:
+        _check(lib.odi_attention_mixed_decode(byref(args), _stream()), "attention_mixed (single tokens)", 2 if splits > 1 else 1)
+    else:
+        _check(lib.odi_attention_mixed(byref(args), c_int(max_q_len), _stream()), "attention_mixed")
 
 
 # ------------------------------------------------------------------------------ sampling

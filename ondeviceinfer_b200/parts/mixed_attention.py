@@ -116,15 +116,27 @@ class MixedAttention(Part):
         common = dict(n_seqs=ctx.n_seqs, nq=s.num_heads, nkv=s.num_kv_heads, d=self.lanes, page_size=PAGE_SIZE,
                       ring_pages=view.kv_group.ring_pages, chunk=s.chunk or 0, scale=s.scale, mixed=mixed)
         keys = ctx.max_kv_len if s.chunk is None else min(ctx.max_kv_len, s.chunk)
+        tensor_cores = ops.attention_mixed_supported(q.dtype, self.lanes, self.v_lanes, s.num_kv_heads, mixed)
         splits, partial = 1, None
         if ctx.max_q_len == 1:
-            # single tokens: cut the visible keys so that enough blocks run side by side
-            rows = s.num_kv_heads * ((s.num_heads // s.num_kv_heads + 15) // 16)
-            splits = max(1, min(32, 296 // max(ctx.n_seqs * rows, 1), (keys + 255) // 256))
+            # single tokens: cut the visible keys so that enough blocks run side by side (a chunk may straddle a tile more)
+            if tensor_cores:
+                rows, tiles = (s.num_heads + 15) // 16, (keys + 63) // 64 + (1 if s.chunk is not None else 0)
+            else:
+                rows, tiles = s.num_kv_heads * ((s.num_heads // s.num_kv_heads + 15) // 16), (keys + 255) // 256
+            splits = max(1, min(32, 296 // max(ctx.n_seqs * rows, 1), tiles))
             if splits > 1:
                 partial = torch.empty((ctx.n_tokens * s.num_heads * splits * (self.v_lanes + 2),), dtype=torch.float32,
                                       device=q.device)
-        ops.attention_simt(*where, max_q_len=ctx.max_q_len, window=0, dv=self.v_lanes, splits=splits, partial=partial, **common)
+        if (tensor_cores and ctx.max_q_len > TCGEN05_MIN_Q_LEN and self.lanes == self.v_lanes
+                and (ops.attention_tcgen05_fits_mixed(self.lanes, s.num_kv_heads) if mixed
+                     else self.lanes in ops.TCGEN05_ATTENTION_HEAD_DIMS)):
+            # bf16 prompts with heads of 64 or 128 lanes: scores and outputs in tensor memory
+            ops.attention_tcgen05(*where, max_q_len=ctx.max_q_len, **common)
+        elif tensor_cores:
+            ops.attention_mixed(*where, max_q_len=ctx.max_q_len, dv=self.v_lanes, splits=splits, partial=partial, **common)
+        else:
+            ops.attention_simt(*where, max_q_len=ctx.max_q_len, window=0, dv=self.v_lanes, splits=splits, partial=partial, **common)
         return o
 
 
