@@ -34,7 +34,7 @@ lengths and with temperature sampling.  One JSON line is printed:
 on the same configuration, and prints the same line with ``"impl": "reference"``.  Nothing of
 this library is imported in that arm.
 
-``--design lemesun`` (or ``nulalorn``, ``zigivik``, ``losivik``) leaves the default workload alone and measures that architecture instead: prefill and
+``--design lemesun`` (or ``nulalorn``, ``zigivik``, ``losivik``, ``noganex``) leaves the default workload alone and measures that architecture instead: prefill and
 decode throughput at layer sizes like a real model's beside the dense model of equal width, one JSON line
 (``run_design_points``).
 
@@ -646,6 +646,28 @@ def _losivik_config(width, heads, kv_heads, dim, rank, window, keep, ssm_heads, 
             "token_side": {"dim": side}, "layers": [latent, pair, latent, pair]}
 
 
+def _noganex_config(width, heads, kv_heads, dim, chunk, delta_heads, delta_kv, delta_dim, experts, top, ff, shared_ff, dense_ff, vocab):
+    """Four layers: attention with mixed heads and a dense feed-forward, the delta rule with routed experts, and both once
+    more (tensors of their own: no layer borrows, so that the weights read are those of four layers)."""
+    attention = {"type": "attention", "mlp": {"kind": "dense", "ff": dense_ff},
+                 "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": chunk},
+                           "rot": {"base": 10000.0, "dims": dim,
+                                   "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    delta = {"type": "delta",
+             "mlp": {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared_ff},
+                     "router": {"experts": experts, "top": top, "scale": 2.0}},
+             "mixer": {"heads": delta_heads, "kv_heads": delta_kv, "dim": delta_dim, "vdim": delta_dim, "conv": 4}}
+    return {"architecture": "Noganex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": [attention, delta, attention, delta]}
+
+
+NOGANEX_POINTS = {
+    "w2048": (_noganex_config(2048, 16, 4, 128, 1024, 16, 8, 128, 32, 4, 1024, 1024, 5 * 1024, 32768),
+              _dense_config(2048, 16, 5 * 1024, 4, 32768)),
+    "w4096": (_noganex_config(4096, 32, 8, 128, 1024, 32, 16, 128, 64, 6, 1536, 3072, 12288, 32768),
+              _dense_config(4096, 32, 12288, 4, 32768)),
+}
+
 LOSIVIK_POINTS = {
     "w2048": (_losivik_config(2048, 16, 4, 128, 512, 1024, 64, 32, 64, 128, 32, 4, 1024, 1024, 5 * 1024, 256, 32768),
               _dense_config(2048, 16, 5 * 1024, 4, 32768)),
@@ -712,7 +734,7 @@ def _time_parts(model, cache, slots, runs, torch):
 
 
 def run_design_points(args) -> int:
-    """``--design lemesun|nulalorn|zigivik|losivik``: prefill and decode throughput of that design at layer sizes like a real model's
+    """``--design lemesun|nulalorn|zigivik|losivik|noganex``: prefill and decode throughput of that design at layer sizes like a real model's
     (random weights), each beside the dense Qwen3 model of equal width, heads, layer executions and active
     feed-forward width, with the device time of every mixer and feed-forward call.  One JSON line; the default
     workload is untouched."""
@@ -730,7 +752,7 @@ def run_design_points(args) -> int:
     points = {}
     sampler = ClockSampler()
     sampler.start()
-    design_points = {"nulalorn": NULALORN_POINTS, "zigivik": ZIGIVIK_POINTS, "losivik": LOSIVIK_POINTS}.get(args.design, DESIGN_POINTS)
+    design_points = {"nulalorn": NULALORN_POINTS, "zigivik": ZIGIVIK_POINTS, "losivik": LOSIVIK_POINTS, "noganex": NOGANEX_POINTS}.get(args.design, DESIGN_POINTS)
     for name, configs in design_points.items():
         if args.design_points and name not in args.design_points.split(","):
             continue
@@ -815,7 +837,7 @@ def main() -> int:
     parser.add_argument("--prompt-range", default=None, metavar="LOW,HIGH",
                         help="unequal prompts: lengths uniform in [LOW, HIGH] from --seed instead of --prompt-len")
     parser.add_argument("--context", type=int, default=None, help="cache positions per sequence (default 4096, or what the prompt needs)")
-    parser.add_argument("--design", default=None, choices=["lemesun", "nulalorn", "zigivik", "losivik"],
+    parser.add_argument("--design", default=None, choices=["lemesun", "nulalorn", "zigivik", "losivik", "noganex"],
                         help="instead of the default workload: this design at real layer sizes beside the dense model of equal size")
     parser.add_argument("--design-points", default=None, help="which of the design's sizes, with commas (default: all)")
     args = parser.parse_args()

@@ -20,15 +20,17 @@
 //  prep       per token: convolution with SiLU of all channels, unit vectors, decays and step sizes; the convolution's
 //             state of a sequence that brings one token moves on in the same launch;
 //  conv_state the convolution's state of the other sequences: the last taps - 1 inputs;
+//  groups     the numbers of every group of four tokens: products of decays and of the group's vectors;
 //  rule       the recurrence: a block per (sequence, head, block of COLS value columns); a column of S lies in the
-//             registers of RS neighbouring lanes, R rows each, two columns a thread; 16 tokens of q, k, v and the
-//             decays are staged in shared memory, the next 16 by asynchronous copies meanwhile;
+//             registers of RS neighbouring lanes, R rows each (two rows in a register pair: packed fp32
+//             operations), two columns a thread; 16 tokens of q, k, v and the groups' numbers are staged in shared
+//             memory, the next 16 by asynchronous copies meanwhile;
 //  out_norm   per (token, head): o / rms(o) (eps inside the root) * weight * silu(gate), rounded once to T.
 #include "common.cuh"
 
 #define HD_MAX_TAPS 16
 #define HD_CPT 2            // value columns per thread
-#define HD_COEFS 40         // floats of a group of four tokens: see group_coefs
+#define HD_COEFS 32         // numbers of a group of four tokens: see hd_groups_kernel
 
 struct HeadDeltaArgs {
   const void* proj;       // [n_tokens, ld] in T: q (kv_heads d), k (kv_heads d), v (heads dv), gate (heads dv)
@@ -41,6 +43,7 @@ struct HeadDeltaArgs {
   float* state;           // [slots, heads, d, dv]
   float* qk;              // [n_tokens, kv_heads, 2, d] scratch: unit q (scaled), unit k
   float* gb;              // [n_tokens, heads, 2] scratch: decay, step size
+  float* coefs;           // [ceil(n_tokens / 4), heads, HD_COEFS] scratch: the groups' numbers
   float* o;               // [n_tokens, heads dv] scratch: v, then the read-outs in its place
   void* out;              // [n_tokens, heads dv] in T
   const int* cu_q;
@@ -133,42 +136,134 @@ __device__ __forceinline__ void hd_cp16(float* dst, const float* src) {
 __device__ __forceinline__ void hd_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void hd_cp_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 
-// Where a group's numbers lie: ck[i][j] = beta_i D_ij (k_j . k_i) at 4 i + j (j < i), cq[i][j] = D_ij (k_j . q_i) at
-// 16 + 4 i + j (j <= i), then G_i at 32 + i and D_3i at 36 + i.
+// A group's numbers (HD_COEFS floats): beta_i at 0, beta_i G_i at 4, G_i at 8, D_3i at 12, then beta_i D_ij (k_j . k_i) for
+// j < i at CK(i, j) and D_ij (k_j . q_i) for j <= i at CQ(i, j).  The group that starts at token t (t - q_begin a multiple
+// of 4, four tokens left) lies at slot t / 4: groups share no token, so no two share a slot.
+#define CK(i, j) (16 + (i) * ((i) - 1) / 2 + (j))
+#define CQ(i, j) (22 + (i) * ((i) + 1) / 2 + (j))
+
+// One warp per (token, key head); the warps of tokens that start no group leave.
+__global__ void __launch_bounds__(128)
+hd_groups_kernel(HeadDeltaArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float dots[4][20];           // k_j . k_i (the pairs as in CK), then k_j . q_i (as in CQ)
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const long item = (long)blockIdx.x * 4 + warp;
+  if (item >= (long)a.n_tokens * a.kv_heads) return;
+  const int t = (int)(item / a.kv_heads), kvh = (int)(item % a.kv_heads);
+  const int seq = a.tok_seq[t], q_begin = a.cu_q[seq], q_end = a.cu_q[seq + 1];
+  if (((t - q_begin) & 3) != 0 || t + 4 > q_end) return;
+  const size_t step = (size_t)a.kv_heads * 2 * a.d;
+  const float* base = a.qk + (size_t)t * step + (size_t)kvh * 2 * a.d;
+  float kk[6] = {}, kq[10] = {};
+  for (int e = lane; e < a.d; e += 32) {
+    float q[4], k[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { q[i] = base[i * step + e]; k[i] = base[i * step + a.d + e]; }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+#pragma unroll
+      for (int j = 0; j < i; ++j) kk[CK(i, j) - 16] = fmaf(k[i], k[j], kk[CK(i, j) - 16]);
+#pragma unroll
+      for (int j = 0; j <= i; ++j) kq[CQ(i, j) - 22] = fmaf(q[i], k[j], kq[CQ(i, j) - 22]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 6; ++i) { kk[i] = warp_sum(kk[i]); if (lane == 0) dots[warp][i] = kk[i]; }
+#pragma unroll
+  for (int i = 0; i < 10; ++i) { kq[i] = warp_sum(kq[i]); if (lane == 0) dots[warp][6 + i] = kq[i]; }
+  __syncwarp();
+  // lane n writes number n: which tokens it is about
+  int kind = lane >> 2, i = lane & 3, j = 0;
+  if (lane >= 22) { kind = 5; i = lane < 23 ? 0 : (lane < 25 ? 1 : (lane < 28 ? 2 : 3)); j = lane - CQ(i, 0); }
+  else if (lane >= 16) { kind = 4; i = lane < 17 ? 1 : (lane < 19 ? 2 : 3); j = lane - CK(i, 0); }
+  const int rep = a.heads / a.kv_heads;
+  for (int r = 0; r < rep; ++r) {
+    const int h = kvh * rep + r;
+    float g[4];
+#pragma unroll
+    for (int m = 0; m < 4; ++m) g[m] = a.gb[((size_t)(t + m) * a.heads + h) * 2];
+    const float beta = a.gb[((size_t)(t + i) * a.heads + h) * 2 + 1];
+    float G = 1.f, E = 1.f, D = 1.f;                // g_0 .. g_i;  g_(i+1) .. g_3;  g_(j+1) .. g_i
+#pragma unroll
+    for (int m = 0; m < 4; ++m) {
+      if (m <= i) G *= g[m]; else E *= g[m];
+      if (m > j && m <= i) D *= g[m];
+    }
+    float out = beta;
+    if (kind == 1) out = beta * G;
+    else if (kind == 2) out = G;
+    else if (kind == 3) out = E;
+    else if (kind == 4) out = beta * D * dots[warp][lane - 16];
+    else if (kind == 5) out = D * dots[warp][lane - 16];
+    a.coefs[((size_t)(t >> 2) * a.heads + h) * HD_COEFS + lane] = out;
+  }
+}
+
+// Two floats in one register pair (the packed fp32 operations of sm_100).
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+struct __align__(16) Quad { f32x2 lo, hi; };      // four neighbouring rows
+
 // RS lanes share a column, R rows each (rows 4 (rs + RS j) .. + 3); DP = RS R rows, those beyond d are zero.
 template <int RS, int R, int COLS, int TCH>
 __global__ void __launch_bounds__(COLS / HD_CPT * RS)
 hd_rule_kernel(HeadDeltaArgs a, int vec) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int DP = RS * R, NTH = COLS / HD_CPT * RS, NQ = R / 4;
-  constexpr int STAGE = TCH * (2 * DP + COLS + 2);
-  extern __shared__ __align__(16) float hd_smem[];      // two stages: qk [TCH][2][DP], v [TCH][COLS], gb [TCH][2]; then the groups' numbers
-  float* coefs = hd_smem + 2 * STAGE;                   // [TCH / 4][HD_COEFS]
+  constexpr int DP = RS * R, NTH = COLS / HD_CPT * RS, NQ = R / 4, NP = R / 2;
+  constexpr int STAGE = TCH * (2 * DP + COLS + 2) + (TCH / 4) * HD_COEFS;
+  constexpr int PER_LANE = RS >= 16 ? 1 : 16 / RS;      // of a column pair's 16 sums
+  // two stages: qk [TCH][2][DP], v [TCH][COLS], gb [TCH][2], the groups' numbers; then two places for the sums of every
+  // column pair
+  extern __shared__ __align__(16) float hd_smem[];
   const int seq = blockIdx.z, h = blockIdx.y, c0 = blockIdx.x * COLS;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int rs = tid % RS, col = (tid / RS) * HD_CPT;
+  float* sums = hd_smem + 2 * STAGE + (tid / RS) * 32;
   const int q_begin = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q_begin;
   if (q_len <= 0) return;
   const int slot = a.slots[seq], d = a.d, dv = a.dv, kvh = h / (a.heads / a.kv_heads);
   float* S_g = a.state + ((size_t)slot * a.heads + h) * d * dv;
-  float S[HD_CPT][R];
+  f32x2 S[HD_CPT][NP];                   // rows 2 p, 2 p + 1 of this lane's R in pair p
   bool live[HD_CPT];
 #pragma unroll
   for (int cc = 0; cc < HD_CPT; ++cc) live[cc] = c0 + col + cc < dv;
   const bool pair = (dv & 1) == 0;       // both columns of a thread in one 8-byte access (col is even)
 #pragma unroll
-  for (int r = 0; r < R; ++r) {
-    const int i = 4 * (rs + RS * (r >> 2)) + (r & 3);
-    const float* src = S_g + (size_t)i * dv + c0 + col;
-    if (pair) {
-      float2 v = make_float2(0.f, 0.f);
-      if (i < d && live[0]) v = *(const float2*)src;
-      S[0][r] = v.x; S[1][r] = v.y;
-    } else {
+  for (int p = 0; p < NP; ++p) {
+    float x[2][HD_CPT];
 #pragma unroll
-      for (int cc = 0; cc < HD_CPT; ++cc) S[cc][r] = (i < d && live[cc]) ? src[cc] : 0.f;
+    for (int e = 0; e < 2; ++e) {
+      const int i = 4 * (rs + RS * (p >> 1)) + 2 * (p & 1) + e;
+      const float* src = S_g + (size_t)i * dv + c0 + col;
+      if (pair) {
+        float2 v = make_float2(0.f, 0.f);
+        if (i < d && live[0]) v = *(const float2*)src;
+        x[e][0] = v.x; x[e][1] = v.y;
+      } else {
+#pragma unroll
+        for (int cc = 0; cc < HD_CPT; ++cc) x[e][cc] = (i < d && live[cc]) ? src[cc] : 0.f;
+      }
     }
+#pragma unroll
+    for (int cc = 0; cc < HD_CPT; ++cc) S[cc][p] = pack2(x[0][cc], x[1][cc]);
   }
   if (d < DP) {                          // the copies never touch the padding rows
     for (int i = tid; i < 2 * TCH * 2 * (DP - d); i += NTH) {
@@ -197,6 +292,11 @@ hd_rule_kernel(HeadDeltaArgs a, int vec) {
     }
     float* gs = vs + TCH * COLS;
     if (tid < nt * 2) hd_cp4(gs + tid, a.gb + ((size_t)(base + tid / 2) * a.heads + h) * 2 + (tid & 1));
+    float* cf = gs + TCH * 2;
+    for (int i = tid; i < nt / 4 * (HD_COEFS / 4); i += NTH) {
+      const int grp = i / (HD_COEFS / 4), e = 4 * (i % (HD_COEFS / 4));
+      hd_cp16(cf + grp * HD_COEFS + e, a.coefs + ((size_t)((base + 4 * grp) >> 2) * a.heads + h) * HD_COEFS + e);
+    }
     hd_cp_commit();
   };
 
@@ -210,38 +310,8 @@ hd_rule_kernel(HeadDeltaArgs a, int vec) {
     const float* buf = hd_smem + (size_t)(chunk & 1) * STAGE;
     const float* vs = buf + TCH * 2 * DP;
     const float* gs = vs + TCH * COLS;
+    const float* cfs = gs + TCH * 2;
     const int groups = nt / 4;
-    // the groups' numbers: a warp per pair (i, j), j <= i, of a group
-    for (int p = warp; p < groups * 10; p += NTH / 32) {
-      const int grp = p / 10, r = p % 10;
-      const int i = r < 1 ? 0 : (r < 3 ? 1 : (r < 6 ? 2 : 3)), j = r - i * (i + 1) / 2;
-      const float* ti = buf + (grp * 4 + i) * 2 * DP;
-      const float* kj = buf + (grp * 4 + j) * 2 * DP + DP;
-      float kk = 0.f, kq = 0.f;
-      for (int e = 4 * lane; e < DP; e += 128) {
-        const float4 q = *(const float4*)(ti + e), k = *(const float4*)(ti + DP + e), w = *(const float4*)(kj + e);
-        kk += k.x * w.x + k.y * w.y + k.z * w.z + k.w * w.w;
-        kq += q.x * w.x + q.y * w.y + q.z * w.z + q.w * w.w;
-      }
-      kk = warp_sum(kk);
-      kq = warp_sum(kq);
-      if (lane == 0) {
-        const float* g = gs + grp * 8;
-        float* out = coefs + grp * HD_COEFS;
-        float D = 1.f;
-        for (int m = j + 1; m <= i; ++m) D *= g[2 * m];
-        out[16 + 4 * i + j] = D * kq;
-        if (j < i) out[4 * i + j] = g[2 * i + 1] * D * kk;
-        else {
-          float G = 1.f, E = 1.f;
-          for (int m = 0; m <= i; ++m) G *= g[2 * m];
-          for (int m = i + 1; m < 4; ++m) E *= g[2 * m];
-          out[32 + i] = G;
-          out[36 + i] = E;
-        }
-      }
-    }
-    __syncthreads();
     float* o_row = a.o + (size_t)(q_begin + chunk * TCH) * a.heads * dv + (size_t)h * dv + c0 + col;
     const size_t o_step = (size_t)a.heads * dv;
     auto store = [&](int tt, const float* o) {
@@ -253,111 +323,161 @@ hd_rule_kernel(HeadDeltaArgs a, int vec) {
       }
     };
     for (int grp = 0; grp < groups; ++grp) {
-      const float* tok = buf + grp * 4 * 2 * DP;
-      const float* cf = coefs + grp * HD_COEFS;
-      float sk[4][HD_CPT] = {}, sq[4][HD_CPT] = {};
+      const float* tok = buf + grp * 4 * 2 * DP + 4 * rs;
+      float part[16];                    // S^T k_i of column cc at 4 cc + i, S^T q_i at 8 + 4 cc + i: this lane's rows
+      {
+        f32x2 acc[16];
 #pragma unroll
-      for (int j = 0; j < NQ; ++j) {
-        const int e = 4 * (rs + RS * j);
+        for (int x = 0; x < 16; ++x) acc[x] = 0ull;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float4 q = *(const float4*)(tok + i * 2 * DP + e), k = *(const float4*)(tok + i * 2 * DP + DP + e);
-#pragma unroll
-          for (int cc = 0; cc < HD_CPT; ++cc) {
-            const float* s = &S[cc][4 * j];
-            sk[i][cc] = fmaf(s[0], k.x, sk[i][cc]); sk[i][cc] = fmaf(s[1], k.y, sk[i][cc]);
-            sk[i][cc] = fmaf(s[2], k.z, sk[i][cc]); sk[i][cc] = fmaf(s[3], k.w, sk[i][cc]);
-            sq[i][cc] = fmaf(s[0], q.x, sq[i][cc]); sq[i][cc] = fmaf(s[1], q.y, sq[i][cc]);
-            sq[i][cc] = fmaf(s[2], q.z, sq[i][cc]); sq[i][cc] = fmaf(s[3], q.w, sq[i][cc]);
-          }
-        }
-      }
-#pragma unroll
-      for (int m = 1; m < RS; m <<= 1) {
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-          for (int cc = 0; cc < HD_CPT; ++cc) {
-            sk[i][cc] += __shfl_xor_sync(0xffffffffu, sk[i][cc], m);
-            sq[i][cc] += __shfl_xor_sync(0xffffffffu, sq[i][cc], m);
-          }
-      }
-      const float4 G = *(const float4*)(cf + 32), E = *(const float4*)(cf + 36);
-      const float Gi[4] = {G.x, G.y, G.z, G.w}, Ei[4] = {E.x, E.y, E.z, E.w};
-      float u[4][HD_CPT];
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float beta = gs[(grp * 4 + i) * 2 + 1];
-        const float2 v = *(const float2*)(vs + (grp * 4 + i) * COLS + col);
-        const float vv[2] = {v.x, v.y};
-        float o[HD_CPT];
-#pragma unroll
-        for (int cc = 0; cc < HD_CPT; ++cc) {
-          float x = beta * fmaf(-Gi[i], sk[i][cc], vv[cc]);
-          float y = Gi[i] * sq[i][cc];
-#pragma unroll
-          for (int j = 0; j < i; ++j) {
-            x = fmaf(-cf[4 * i + j], u[j][cc], x);
-            y = fmaf(cf[16 + 4 * i + j], u[j][cc], y);
-          }
-          u[i][cc] = x;
-          o[cc] = fmaf(cf[16 + 5 * i], x, y);
-        }
-        if (rs == 0) store(grp * 4 + i, o);
-      }
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int cc = 0; cc < HD_CPT; ++cc) u[i][cc] *= Ei[i];
-#pragma unroll
-      for (int j = 0; j < NQ; ++j) {
-        const int e = 4 * (rs + RS * j);
-        float4 k[4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) k[i] = *(const float4*)(tok + i * 2 * DP + DP + e);
-#pragma unroll
-        for (int cc = 0; cc < HD_CPT; ++cc) {
-          float* s = &S[cc][4 * j];
-          s[0] *= Gi[3]; s[1] *= Gi[3]; s[2] *= Gi[3]; s[3] *= Gi[3];
+        for (int j = 0; j < NQ; ++j) {
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            s[0] = fmaf(k[i].x, u[i][cc], s[0]); s[1] = fmaf(k[i].y, u[i][cc], s[1]);
-            s[2] = fmaf(k[i].z, u[i][cc], s[2]); s[3] = fmaf(k[i].w, u[i][cc], s[3]);
+            const Quad q = *(const Quad*)(tok + i * 2 * DP + 4 * RS * j), k = *(const Quad*)(tok + i * 2 * DP + DP + 4 * RS * j);
+#pragma unroll
+            for (int cc = 0; cc < HD_CPT; ++cc) {
+              acc[4 * cc + i] = fma2(S[cc][2 * j], k.lo, acc[4 * cc + i]);
+              acc[4 * cc + i] = fma2(S[cc][2 * j + 1], k.hi, acc[4 * cc + i]);
+              acc[8 + 4 * cc + i] = fma2(S[cc][2 * j], q.lo, acc[8 + 4 * cc + i]);
+              acc[8 + 4 * cc + i] = fma2(S[cc][2 * j + 1], q.hi, acc[8 + 4 * cc + i]);
+            }
+          }
+        }
+#pragma unroll
+        for (int x = 0; x < 16; ++x) {
+          float lo, hi;
+          unpack2(acc[x], lo, hi);
+          part[x] = lo + hi;
+        }
+      }
+      // sums over the column's lanes, each lane keeping its share of the 16; all of them through shared memory (two places
+      // in turn: a lane that is one group ahead writes the other)
+      float* place = sums + (grp & 1) * 16;
+      int width = 16;
+#pragma unroll
+      for (int m = RS >> 1; m > 0; m >>= 1) {
+        if (width > 1) {
+          width >>= 1;
+          const bool upper = (rs & m) != 0;
+#pragma unroll
+          for (int x = 0; x < 8; ++x)
+            if (x < width) {
+              const float keep = upper ? part[x + width] : part[x], send = upper ? part[x] : part[x + width];
+              part[x] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+            }
+        } else {
+          part[0] += __shfl_xor_sync(0xffffffffu, part[0], m);
+        }
+      }
+      // RS = 32: the last halving added the same sum in both lanes of a pair
+      const int first = RS >= 16 ? rs / (RS / 16) : rs * PER_LANE;
+#pragma unroll
+      for (int x = 0; x < PER_LANE; ++x) place[first + x] = part[x];
+      __syncwarp();
+      const float* cf = cfs + grp * HD_COEFS;
+      const float4 b4 = *(const float4*)cf, bG4 = *(const float4*)(cf + 4), G4 = *(const float4*)(cf + 8), E4 = *(const float4*)(cf + 12);
+      const float bi[4] = {b4.x, b4.y, b4.z, b4.w}, bG[4] = {bG4.x, bG4.y, bG4.z, bG4.w}, Gi[4] = {G4.x, G4.y, G4.z, G4.w},
+                  Ei[4] = {E4.x, E4.y, E4.z, E4.w};
+      float pairs[16];                   // the rest of the numbers, CK(1, 0) first
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const float4 v = *(const float4*)(cf + 16 + 4 * x);
+        pairs[4 * x] = v.x; pairs[4 * x + 1] = v.y; pairs[4 * x + 2] = v.z; pairs[4 * x + 3] = v.w;
+      }
+      float sk[HD_CPT][4], sq[HD_CPT][4], vv[4][HD_CPT], o[4][HD_CPT];
+#pragma unroll
+      for (int cc = 0; cc < HD_CPT; ++cc) {
+        const float4 k = *(const float4*)(place + 4 * cc), q = *(const float4*)(place + 8 + 4 * cc);
+        sk[cc][0] = k.x; sk[cc][1] = k.y; sk[cc][2] = k.z; sk[cc][3] = k.w;
+        sq[cc][0] = q.x; sq[cc][1] = q.y; sq[cc][2] = q.z; sq[cc][3] = q.w;
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float2 v = *(const float2*)(vs + (grp * 4 + i) * COLS + col);
+        vv[i][0] = v.x; vv[i][1] = v.y;
+      }
+      f32x2 uu[4][HD_CPT];               // D_3i u_i, twice
+#pragma unroll
+      for (int cc = 0; cc < HD_CPT; ++cc) {
+        float u[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          float x = fmaf(-bG[i], sk[cc][i], bi[i] * vv[i][cc]);
+          float y = Gi[i] * sq[cc][i];
+#pragma unroll
+          for (int j = 0; j < i; ++j) {
+            x = fmaf(-pairs[CK(i, j) - 16], u[j], x);
+            y = fmaf(pairs[CQ(i, j) - 16], u[j], y);
+          }
+          u[i] = x;
+          o[i][cc] = fmaf(pairs[CQ(i, i) - 16], x, y);
+          uu[i][cc] = pack2(x * Ei[i], x * Ei[i]);
+        }
+      }
+      if (rs == 0) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) store(grp * 4 + i, o[i]);
+      }
+      const f32x2 GG = pack2(Gi[3], Gi[3]);
+#pragma unroll
+      for (int j = 0; j < NQ; ++j) {
+#pragma unroll
+        for (int cc = 0; cc < HD_CPT; ++cc) { S[cc][2 * j] = mul2(S[cc][2 * j], GG); S[cc][2 * j + 1] = mul2(S[cc][2 * j + 1], GG); }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const Quad k = *(const Quad*)(tok + i * 2 * DP + DP + 4 * RS * j);
+#pragma unroll
+          for (int cc = 0; cc < HD_CPT; ++cc) {
+            S[cc][2 * j] = fma2(k.lo, uu[i][cc], S[cc][2 * j]);
+            S[cc][2 * j + 1] = fma2(k.hi, uu[i][cc], S[cc][2 * j + 1]);
           }
         }
       }
     }
     for (int tt = groups * 4; tt < nt; ++tt) {      // the tokens that are left
-      const float* tok = buf + tt * 2 * DP;
+      const float* tok = buf + tt * 2 * DP + 4 * rs;
       const float g = gs[tt * 2], beta = gs[tt * 2 + 1];
-      float dot[HD_CPT] = {}, o[HD_CPT] = {};
+      const f32x2 gg = pack2(g, g);
+      f32x2 acc[HD_CPT];
+      float dot[HD_CPT], o[HD_CPT];
+#pragma unroll
+      for (int cc = 0; cc < HD_CPT; ++cc) acc[cc] = 0ull;
 #pragma unroll
       for (int j = 0; j < NQ; ++j) {
-        const float4 k = *(const float4*)(tok + DP + 4 * (rs + RS * j));
+        const Quad k = *(const Quad*)(tok + DP + 4 * RS * j);
 #pragma unroll
         for (int cc = 0; cc < HD_CPT; ++cc) {
-          float* s = &S[cc][4 * j];
-          s[0] *= g; s[1] *= g; s[2] *= g; s[3] *= g;
-          dot[cc] += s[0] * k.x + s[1] * k.y + s[2] * k.z + s[3] * k.w;
+          S[cc][2 * j] = mul2(S[cc][2 * j], gg);
+          S[cc][2 * j + 1] = mul2(S[cc][2 * j + 1], gg);
+          acc[cc] = fma2(S[cc][2 * j], k.lo, acc[cc]);
+          acc[cc] = fma2(S[cc][2 * j + 1], k.hi, acc[cc]);
         }
       }
+#pragma unroll
+      for (int cc = 0; cc < HD_CPT; ++cc) { float lo, hi; unpack2(acc[cc], lo, hi); dot[cc] = lo + hi; acc[cc] = 0ull; }
 #pragma unroll
       for (int m = 1; m < RS; m <<= 1)
 #pragma unroll
         for (int cc = 0; cc < HD_CPT; ++cc) dot[cc] += __shfl_xor_sync(0xffffffffu, dot[cc], m);
-      float u[HD_CPT];
+      f32x2 uu[HD_CPT];
 #pragma unroll
-      for (int cc = 0; cc < HD_CPT; ++cc) u[cc] = beta * (vs[tt * COLS + col + cc] - dot[cc]);
+      for (int cc = 0; cc < HD_CPT; ++cc) {
+        const float u = beta * (vs[tt * COLS + col + cc] - dot[cc]);
+        uu[cc] = pack2(u, u);
+      }
 #pragma unroll
       for (int j = 0; j < NQ; ++j) {
-        const float4 k = *(const float4*)(tok + DP + 4 * (rs + RS * j)), q = *(const float4*)(tok + 4 * (rs + RS * j));
+        const Quad k = *(const Quad*)(tok + DP + 4 * RS * j), q = *(const Quad*)(tok + 4 * RS * j);
 #pragma unroll
         for (int cc = 0; cc < HD_CPT; ++cc) {
-          float* s = &S[cc][4 * j];
-          s[0] = fmaf(k.x, u[cc], s[0]); s[1] = fmaf(k.y, u[cc], s[1]); s[2] = fmaf(k.z, u[cc], s[2]); s[3] = fmaf(k.w, u[cc], s[3]);
-          o[cc] += s[0] * q.x + s[1] * q.y + s[2] * q.z + s[3] * q.w;
+          S[cc][2 * j] = fma2(k.lo, uu[cc], S[cc][2 * j]);
+          S[cc][2 * j + 1] = fma2(k.hi, uu[cc], S[cc][2 * j + 1]);
+          acc[cc] = fma2(S[cc][2 * j], q.lo, acc[cc]);
+          acc[cc] = fma2(S[cc][2 * j + 1], q.hi, acc[cc]);
         }
       }
+#pragma unroll
+      for (int cc = 0; cc < HD_CPT; ++cc) { float lo, hi; unpack2(acc[cc], lo, hi); o[cc] = lo + hi; }
 #pragma unroll
       for (int m = 1; m < RS; m <<= 1)
 #pragma unroll
@@ -366,14 +486,20 @@ hd_rule_kernel(HeadDeltaArgs a, int vec) {
     }
   }
 #pragma unroll
-  for (int r = 0; r < R; ++r) {
-    const int i = 4 * (rs + RS * (r >> 2)) + (r & 3);
-    if (i >= d) continue;
-    float* dst = S_g + (size_t)i * dv + c0 + col;
-    if (pair) { if (live[0]) *(float2*)dst = make_float2(S[0][r], S[1][r]); }
-    else {
+  for (int p = 0; p < NP; ++p) {
+    float x[2][HD_CPT];
 #pragma unroll
-      for (int cc = 0; cc < HD_CPT; ++cc) if (live[cc]) dst[cc] = S[cc][r];
+    for (int cc = 0; cc < HD_CPT; ++cc) unpack2(S[cc][p], x[0][cc], x[1][cc]);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int i = 4 * (rs + RS * (p >> 1)) + 2 * (p & 1) + e;
+      if (i >= d) continue;
+      float* dst = S_g + (size_t)i * dv + c0 + col;
+      if (pair) { if (live[0]) *(float2*)dst = make_float2(x[e][0], x[e][1]); }
+      else {
+#pragma unroll
+        for (int cc = 0; cc < HD_CPT; ++cc) if (live[cc]) dst[cc] = x[e][cc];
+      }
     }
   }
 }
@@ -405,7 +531,7 @@ hd_out_norm_kernel(HeadDeltaArgs a) {
 template <int RS, int R, int COLS, int TCH>
 static int launch_rule(const HeadDeltaArgs& a, cudaStream_t stream) {
   constexpr int DP = RS * R;
-  const size_t smem = sizeof(float) * (2 * (size_t)TCH * (2 * DP + COLS + 2) + (TCH / 4) * HD_COEFS);
+  constexpr size_t smem = sizeof(float) * (2 * ((size_t)TCH * (2 * DP + COLS + 2) + (TCH / 4) * HD_COEFS) + COLS / HD_CPT * 32);
   auto kernel = hd_rule_kernel<RS, R, COLS, TCH>;
   static bool configured = false;
   if (!configured) {
@@ -418,15 +544,17 @@ static int launch_rule(const HeadDeltaArgs& a, cudaStream_t stream) {
   return launch_pdl(kernel, grid, dim3(COLS / HD_CPT * RS), smem, stream, a, vec);
 }
 
-// Fewer columns a block make more blocks: a step of one long sequence has nothing else to run beside it.
-template <int RS, int R, int TCH>
-static int launch_rule_cols(const HeadDeltaArgs& a, cudaStream_t stream) {
-  const long heads = (long)a.heads * a.n_seqs;
-  if constexpr (RS >= 4) {
-    if (heads * ((a.dv + 31) / 32) < 148) return launch_rule<RS, R, 16, TCH>(a, stream);
+// DP rows: a lane takes 16 of a column's rows and a block 32 columns when that makes two blocks per multiprocessor; a
+// step of one long sequence has nothing else to run beside it, so there a lane takes 8 rows and a block 16 columns.
+template <int DP, int TCH>
+static int launch_rule_form(const HeadDeltaArgs& a, cudaStream_t stream) {
+  const bool narrow = (long)a.heads * a.n_seqs * ((a.dv + 31) / 32) < 2 * 148;
+  constexpr int WIDE = DP / 16, NARROW = DP / 8;
+  if constexpr (NARROW <= 32 && NARROW >= 4) {
+    if (narrow) return launch_rule<NARROW, 8, 16, TCH>(a, stream);
   }
-  if constexpr (RS == 1) return launch_rule<RS, R, 64, TCH>(a, stream);
-  else return launch_rule<RS, R, 32, TCH>(a, stream);
+  if constexpr (WIDE >= 2) return launch_rule<WIDE, 16, 32, TCH>(a, stream);
+  else return launch_rule<1, 16, 64, TCH>(a, stream);
 }
 
 template <typename T>
@@ -441,20 +569,23 @@ static int launch_head_delta(const HeadDeltaArgs& a, cudaStream_t stream) {
   odi_rc = launch_pdl((hd_prep_kernel<T>), dim3(a.n_tokens), dim3(256), smem, stream, a);
   if (odi_rc == 0 && a.taps_n > 1 && a.max_q_len > 1)
     odi_rc = launch_pdl((hd_conv_state_kernel<T>), dim3(a.n_seqs, (C + 255) / 256), dim3(256), 0, stream, a);
+  if (odi_rc == 0 && a.max_q_len >= 4)
+    odi_rc = launch_pdl(hd_groups_kernel, dim3((unsigned)(((long)a.n_tokens * a.kv_heads + 3) / 4)), dim3(128), 0, stream, a);
   if (odi_rc == 0) {
-    if (a.d <= 16) odi_rc = launch_rule_cols<1, 16, 16>(a, stream);
-    else if (a.d <= 32) odi_rc = launch_rule_cols<2, 16, 16>(a, stream);
-    else if (a.d <= 64) odi_rc = launch_rule_cols<4, 16, 16>(a, stream);
-    else if (a.d <= 128) odi_rc = launch_rule_cols<8, 16, 16>(a, stream);
-    else if (a.d <= 256) odi_rc = launch_rule_cols<16, 16, 16>(a, stream);
-    else odi_rc = launch_rule_cols<32, 16, 8>(a, stream);
+    if (a.d <= 16) odi_rc = launch_rule_form<16, 16>(a, stream);
+    else if (a.d <= 32) odi_rc = launch_rule_form<32, 16>(a, stream);
+    else if (a.d <= 64) odi_rc = launch_rule_form<64, 16>(a, stream);
+    else if (a.d <= 128) odi_rc = launch_rule_form<128, 16>(a, stream);
+    else if (a.d <= 256) odi_rc = launch_rule_form<256, 16>(a, stream);
+    else odi_rc = launch_rule_form<512, 8>(a, stream);
   }
   if (odi_rc == 0)
     odi_rc = launch_pdl((hd_out_norm_kernel<T>), dim3((unsigned)(((long)a.n_tokens * a.heads + 3) / 4)), dim3(128), 0, stream, a);
   return launch_status();
 }
 
-// Kernels launched by one call: 3, or 4 with a convolution state to move on after a step of several tokens.
+// Kernels launched by one call: 3, one more with a convolution state to move on after a step of several tokens, one more
+// when a sequence brings four tokens or more.
 extern "C" int odi_head_delta(const HeadDeltaArgs* args, int dtype, cudaStream_t stream) {
   const HeadDeltaArgs a = *args;
   if (a.n_tokens <= 0 || a.n_seqs <= 0) return 0;

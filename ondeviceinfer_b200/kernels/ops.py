@@ -1558,7 +1558,7 @@ def delta_rule(proj: torch.Tensor, decay_in: torch.Tensor, taps: torch.Tensor, a
 class _HeadDeltaArgs(Structure):
     _fields_ = [("proj", c_void_p), ("ab", c_void_p), ("taps", c_void_p), ("a_log", c_void_p), ("dt_bias", c_void_p),
                 ("norm_w", c_void_p), ("conv_state", c_void_p), ("state", c_void_p), ("qk", c_void_p), ("gb", c_void_p),
-                ("o", c_void_p), ("out", c_void_p), ("cu_q", c_void_p), ("tok_seq", c_void_p), ("slots", c_void_p),
+                ("coefs", c_void_p), ("o", c_void_p), ("out", c_void_p), ("cu_q", c_void_p), ("tok_seq", c_void_p), ("slots", c_void_p),
                 ("n_tokens", c_int), ("n_seqs", c_int), ("max_q_len", c_int), ("ld", c_int), ("heads", c_int),
                 ("kv_heads", c_int), ("d", c_int), ("dv", c_int), ("taps_n", c_int), ("eps", c_float), ("unit_eps", c_float)]
 
@@ -1597,14 +1597,15 @@ def head_delta(proj: torch.Tensor, ab: torch.Tensor, taps: torch.Tensor, a_log: 
     dev = proj.device
     qk = torch.empty((n, kv_heads, 2, d), dtype=torch.float32, device=dev)
     gb = torch.empty((n, heads, 2), dtype=torch.float32, device=dev)
+    coefs = torch.empty(((n + 3) // 4 if max_q_len >= 4 else 0, heads, 32), dtype=torch.float32, device=dev)
     o = torch.empty((n, heads * dv), dtype=torch.float32, device=dev)
     args = _HeadDeltaArgs(_ptr(proj), _ptr(ab), _ptr(taps), _ptr(a_log), _ptr(dt_bias), _ptr(norm_w),
-                          _ptr(conv_state if K > 1 else None), _ptr(state), _ptr(qk), _ptr(gb), _ptr(o), _ptr(out), _ptr(cu_q),
+                          _ptr(conv_state if K > 1 else None), _ptr(state), _ptr(qk), _ptr(gb), _ptr(coefs), _ptr(o), _ptr(out), _ptr(cu_q),
                           _ptr(tok_seq), _ptr(slots), n, n_seqs, max_q_len, proj.shape[1], heads, kv_heads, d, dv, K, eps,
                           unit_eps)
     lib = load_library("delta_head")
     _check(lib.odi_head_delta(byref(args), c_int(dtype_code(proj.dtype)), _stream()), "head_delta",
-           4 if K > 1 and max_q_len > 1 else 3)
+           3 + (K > 1 and max_q_len > 1) + (max_q_len >= 4))
 
 
 # ------------------------------------------------------------------------------ attention with mixed heads
