@@ -12,8 +12,9 @@
 // conflicts), so a score tile is accumulated item by item in registers and any number of key heads fits.  One block
 // barrier per item: item i + NS - 1 is requested when everybody has left item i - 1, whose place it takes.
 //
-//  prompts and portions: a block of 4 warps owns 64 consecutive query tokens of one head (16 rows per warp); their rows of
-//    all key heads stay in shared memory.
+//  prompts and portions: a block of 8 warps owns 64 consecutive query tokens of one head; a warp takes 16 rows and one half
+//    of every tile's keys, with a maximum, sum and accumulator of its own (merged at the end); the rows of all key heads
+//    stay in shared memory.
 //  single tokens: a block owns up to 16 query heads of one sequence (the rows of its MMAs) and one range of the visible
 //    keys; its 4 warps take 16 keys each of every tile, and merge in shared memory.  Rows of different value heads share
 //    the accumulator: a value head's product takes the probabilities of its own rows and zero for the others.  With
@@ -41,7 +42,8 @@
 #define KSTEPS (D / 16)
 #define DVTILES (DV / 8)
 #define LOG2E 1.4426950408889634f
-#define WARPS 4
+#define WARPS 4                     // of a single-token block
+#define PROMPT_WARPS 8
 #define RS (DV + 2)                 // floats of a partial result: weighted values, maximum, sum
 #define SMEM_LIMIT 232448
 
@@ -87,21 +89,22 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 // One page tile (64 rows of W bf16, contiguous in global memory) into shared-memory rows of 2 W + 16 bytes.
-template <int W>
+template <int W, int THREADS>
 __device__ __forceinline__ void load_tile(uint32_t dst, const bf16* src, int tid) {
   constexpr int CHUNKS = W / 8;    // 16-byte pieces per row
 #pragma unroll 4
-  for (int i = tid; i < KT * CHUNKS; i += WARPS * 32) {
+  for (int i = tid; i < KT * CHUNKS; i += THREADS) {
     const int r = i / CHUNKS, c = i % CHUNKS;
     cp_async16(dst + r * (2 * W + 16) + c * 16, src + (size_t)i * 8);
   }
 }
 
 // The block's query rows into shared memory: row r < rows from src + r * stride, `width` elements each, zeros behind.
+template <int THREADS>
 __device__ __forceinline__ void load_queries(uint8_t* dst, int rowb, const bf16* src, size_t stride, int rows, int total, int width,
                                              int tid) {
   const int pieces = width / 8;
-  for (int i = tid; i < total * pieces; i += WARPS * 32) {
+  for (int i = tid; i < total * pieces; i += THREADS) {
     const int r = i / pieces, c = i % pieces;
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
     if (r < rows) v = *(const uint4*)(src + (size_t)r * stride + c * 8);
@@ -110,7 +113,7 @@ __device__ __forceinline__ void load_queries(uint8_t* dst, int rowb, const bf16*
 }
 
 template <int NS>
-__global__ void __launch_bounds__(WARPS * 32)
+__global__ void __launch_bounds__(PROMPT_WARPS * 32)
 attention_mixed_kernel(MixedAttnArgs a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -138,10 +141,10 @@ attention_mixed_kernel(MixedAttnArgs a) {
       const uint32_t dst = ring_addr + (uint32_t)(next % NS) * STAGE_BYTES;
       if (next_part < KH) {
         const int kh = a.mixed ? next_part : hk;
-        load_tile<D>(dst, a.k_pool + ((size_t)next_page * a.nkv + kh) * KT * D, tid);
+        load_tile<D, PROMPT_WARPS * 32>(dst, a.k_pool + ((size_t)next_page * a.nkv + kh) * KT * D, tid);
         ++next_part;
       } else {
-        load_tile<DV>(dst, a.v_pool + ((size_t)next_page * a.nkv + hk) * KT * DV, tid);
+        load_tile<DV, PROMPT_WARPS * 32>(dst, a.v_pool + ((size_t)next_page * a.nkv + hk) * KT * DV, tid);
         next_part = 0;
         ++next_tile;
       }
@@ -151,36 +154,37 @@ attention_mixed_kernel(MixedAttnArgs a) {
   };
 #pragma unroll
   for (int i = 0; i < NS - 1; ++i) issue();
-  load_queries(smem, q_rowb, a.q + ((size_t)(q_begin + t0) * a.nq + head) * width, (size_t)a.nq * width, nt, 64, width, tid);
+  load_queries<PROMPT_WARPS * 32>(smem, q_rowb, a.q + ((size_t)(q_begin + t0) * a.nq + head) * width, (size_t)a.nq * width, nt, 64, width, tid);
 
-  const int r_lo = warp * 16 + (lane >> 2), r_hi = r_lo + 8;
+  const int rows0 = (warp & 3) * 16, half = warp >> 2;         // this warp's rows, and its half of a tile's keys
+  const int r_lo = rows0 + (lane >> 2), r_hi = r_lo + 8;
   const int pos_lo = p0 + r_lo, pos_hi = p0 + r_hi;
   const int old_lo = a.chunk > 0 ? pos_lo - pos_lo % a.chunk : 0, old_hi = a.chunk > 0 ? pos_hi - pos_hi % a.chunk : 0;
-  const int warp_first = p0 + warp * 16, warp_last = warp_first + 15;
+  const int warp_first = p0 + rows0, warp_last = warp_first + 15;
   const int warp_old = a.chunk > 0 ? warp_first - warp_first % a.chunk : 0;
-  const bool has_rows = warp * 16 < nt;
+  const bool has_rows = rows0 < nt;
   const float sl2 = a.scale * LOG2E;
   const int mi = lane >> 3, mr = lane & 7;
   // A fragments: (rows 0..7, k 0..7), (rows 8..15, same k), (rows 0..7, k 8..15), (rows 8..15, k 8..15)
-  const uint32_t a_base = q_addr + (warp * 16 + (mi & 1) * 8 + mr) * q_rowb + (mi >> 1) * 16;
+  const uint32_t a_base = q_addr + (rows0 + (mi & 1) * 8 + mr) * q_rowb + (mi >> 1) * 16;
 
-  float o[DVTILES][4], s[8][4];
+  float o[DVTILES][4], s[4][4];
 #pragma unroll
   for (int i = 0; i < DVTILES; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
 
-  int part = 0, kbase = tile_lo * KT;
+  int part = 0, kbase = tile_lo * KT + half * 32;            // the first of this warp's 32 keys
   for (int it = 0; it < n_items; ++it) {
     cp_async_wait<NS - 2>();
     __syncthreads();                       // item `it` is there, item it - 1 has been left
     issue();
     const uint32_t st = ring_addr + (uint32_t)(it % NS) * STAGE_BYTES;
-    const bool active = has_rows && kbase <= warp_last && kbase + KT > warp_old;
+    const bool active = has_rows && kbase <= warp_last && kbase + 32 > warp_old;
     if (part < KH) {
       if (active) {
         if (part == 0) {
 #pragma unroll
-          for (int i = 0; i < 8; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
+          for (int i = 0; i < 4; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
         }
         const uint32_t qa = a_base + part * D * 2;
 #pragma unroll
@@ -188,9 +192,9 @@ attention_mixed_kernel(MixedAttnArgs a) {
           uint32_t qf[4];
           ldmatrix_x4(qa + ks * 32, qf[0], qf[1], qf[2], qf[3]);
 #pragma unroll
-          for (int np = 0; np < 4; ++np) {
-            // matrices: (keys np*16 + 0..7, d ks*16 + 0..7), (same keys, d + 8), (keys + 8, d), (keys + 8, d + 8)
-            const int key = np * 16 + (mi >> 1) * 8 + mr, dd = ks * 16 + (mi & 1) * 8;
+          for (int np = 0; np < 2; ++np) {
+            // matrices: (the half's keys np*16 + 0..7, d ks*16 + 0..7), (same keys, d + 8), (keys + 8, d), (keys + 8, d + 8)
+            const int key = half * 32 + np * 16 + (mi >> 1) * 8 + mr, dd = ks * 16 + (mi & 1) * 8;
             uint32_t b0, b1, b2, b3;
             ldmatrix_x4(st + key * ROWB_K + dd * 2, b0, b1, b2, b3);
             mma_bf16(s[np * 2], qf, b0, b1);
@@ -204,7 +208,7 @@ attention_mixed_kernel(MixedAttnArgs a) {
     if (active) {
       float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < 4; ++i) {
         const int kj = kbase + i * 8 + (lane & 3) * 2;
         s[i][0] = (kj <= pos_lo && kj >= old_lo) ? s[i][0] * sl2 : -INFINITY;
         s[i][1] = (kj + 1 <= pos_lo && kj + 1 >= old_lo) ? s[i][1] * sl2 : -INFINITY;
@@ -223,9 +227,9 @@ attention_mixed_kernel(MixedAttnArgs a) {
       const float al_lo = exp2f(m_lo - ref_lo), al_hi = exp2f(m_hi - ref_hi);
       m_lo = mn_lo; m_hi = mn_hi;
       float sum_lo = 0.f, sum_hi = 0.f;
-      uint32_t pf[4][4];                  // P as A fragments for the 4 key steps of 16
+      uint32_t pf[2][4];                  // P as A fragments for the 2 key steps of 16
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < 4; ++i) {
         const float e0 = exp2f(s[i][0] - ref_lo), e1 = exp2f(s[i][1] - ref_lo);
         const float e2 = exp2f(s[i][2] - ref_hi), e3 = exp2f(s[i][3] - ref_hi);
         sum_lo += e0 + e1; sum_hi += e2 + e3;
@@ -236,11 +240,11 @@ attention_mixed_kernel(MixedAttnArgs a) {
 #pragma unroll
       for (int i = 0; i < DVTILES; ++i) { o[i][0] *= al_lo; o[i][1] *= al_lo; o[i][2] *= al_hi; o[i][3] *= al_hi; }
 #pragma unroll
-      for (int kk = 0; kk < 4; ++kk) {      // 16 keys per step
+      for (int kk = 0; kk < 2; ++kk) {      // 16 keys per step
 #pragma unroll
         for (int dp = 0; dp < DVTILES / 2; ++dp) {
           // matrices: (keys kk*16 + 0..7, d dp*16 + 0..7), (keys + 8, same d), (keys, d + 8), (keys + 8, d + 8)
-          const int key = kk * 16 + (mi & 1) * 8 + mr, dd = dp * 16 + (mi >> 1) * 8;
+          const int key = half * 32 + kk * 16 + (mi & 1) * 8 + mr, dd = dp * 16 + (mi >> 1) * 8;
           uint32_t b0, b1, b2, b3;
           ldmatrix_x4_trans(st + key * ROWB_V + dd * 2, b0, b1, b2, b3);
           mma_bf16(o[dp * 2], pf[kk], b0, b1);
@@ -254,17 +258,46 @@ attention_mixed_kernel(MixedAttnArgs a) {
   // the row sums live spread over the 4 lanes of a quad
   l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
   l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
-  const float inv_lo = l_lo > 0.f ? 1.f / l_lo : 0.f, inv_hi = l_hi > 0.f ? 1.f / l_hi : 0.f;
+  // the second half's results through the free ring: [row][DV + 2] floats, maxima in the log2 domain
+  cp_async_wait<0>();
+  __syncthreads();
   const int c = (lane & 3) * 2;
+  float* mg_lo = (float*)ring + (size_t)r_lo * RS;
+  float* mg_hi = (float*)ring + (size_t)r_hi * RS;
+  if (half == 1) {
+#pragma unroll
+    for (int i = 0; i < DVTILES; ++i) {
+      *(float2*)(mg_lo + i * 8 + c) = make_float2(o[i][0], o[i][1]);
+      *(float2*)(mg_hi + i * 8 + c) = make_float2(o[i][2], o[i][3]);
+    }
+    if ((lane & 3) == 0) { mg_lo[DV] = m_lo; mg_lo[DV + 1] = l_lo; mg_hi[DV] = m_hi; mg_hi[DV + 1] = l_hi; }
+  }
+  __syncthreads();
+  if (half == 1) return;
+  auto weights = [](float m0, float l0, float m1, float l1, float& w0, float& w1) {
+    const float M = fmaxf(m0, m1), ref = M == -INFINITY ? 0.f : M;
+    w0 = exp2f(m0 - ref); w1 = exp2f(m1 - ref);
+    const float l = w0 * l0 + w1 * l1, inv = l > 0.f ? 1.f / l : 0.f;
+    w0 *= inv; w1 *= inv;
+  };
+  float a_lo, b_lo, a_hi, b_hi;
+  weights(m_lo, l_lo, mg_lo[DV], mg_lo[DV + 1], a_lo, b_lo);
+  weights(m_hi, l_hi, mg_hi[DV], mg_hi[DV + 1], a_hi, b_hi);
   if (r_lo < nt) {
     bf16* dst = a.out + ((size_t)(q_begin + t0 + r_lo) * a.nq + head) * DV;
 #pragma unroll
-    for (int i = 0; i < DVTILES; ++i) *(uint32_t*)(dst + i * 8 + c) = pack_bf16(o[i][0] * inv_lo, o[i][1] * inv_lo);
+    for (int i = 0; i < DVTILES; ++i) {
+      const float2 v = *(const float2*)(mg_lo + i * 8 + c);
+      *(uint32_t*)(dst + i * 8 + c) = pack_bf16(o[i][0] * a_lo + v.x * b_lo, o[i][1] * a_lo + v.y * b_lo);
+    }
   }
   if (r_hi < nt) {
     bf16* dst = a.out + ((size_t)(q_begin + t0 + r_hi) * a.nq + head) * DV;
 #pragma unroll
-    for (int i = 0; i < DVTILES; ++i) *(uint32_t*)(dst + i * 8 + c) = pack_bf16(o[i][2] * inv_hi, o[i][3] * inv_hi);
+    for (int i = 0; i < DVTILES; ++i) {
+      const float2 v = *(const float2*)(mg_hi + i * 8 + c);
+      *(uint32_t*)(dst + i * 8 + c) = pack_bf16(o[i][2] * a_hi + v.x * b_hi, o[i][3] * a_hi + v.y * b_hi);
+    }
   }
 }
 
@@ -307,9 +340,9 @@ attention_mixed_decode_kernel(MixedAttnArgs a) {
       if (next_part == 0) next_page = pages[page_slot_of_page(next_tile, a.ring_pages)];
       const uint32_t dst = ring_addr + (uint32_t)(next % NS) * STAGE_BYTES;
       if (next_part < KH)
-        load_tile<D>(dst, a.k_pool + ((size_t)next_page * a.nkv + k_lo + next_part) * KT * D, tid);
+        load_tile<D, WARPS * 32>(dst, a.k_pool + ((size_t)next_page * a.nkv + k_lo + next_part) * KT * D, tid);
       else
-        load_tile<DV>(dst, a.v_pool + ((size_t)next_page * a.nkv + v_lo + next_part - KH) * KT * DV, tid);
+        load_tile<DV, WARPS * 32>(dst, a.v_pool + ((size_t)next_page * a.nkv + v_lo + next_part - KH) * KT * DV, tid);
       if (++next_part == per_tile) { next_part = 0; ++next_tile; }
       ++next;
     }
@@ -317,7 +350,7 @@ attention_mixed_decode_kernel(MixedAttnArgs a) {
   };
 #pragma unroll
   for (int i = 0; i < NS - 1; ++i) issue();
-  load_queries(smem, q_rowb, a.q + ((size_t)tok * a.nq + head0) * width, width, heads_here, 16, width, tid);
+  load_queries<WARPS * 32>(smem, q_rowb, a.q + ((size_t)tok * a.nq + head0) * width, width, heads_here, 16, width, tid);
 
   const int r_lo = lane >> 2, r_hi = r_lo + 8;
   const int g_lo = (head0 + r_lo) / rep, g_hi = (head0 + r_hi) / rep;      // the rows' value heads
@@ -493,10 +526,10 @@ static int check_args(const MixedAttnArgs& a) {
 }
 
 template <typename K>
-static int launch_one(K kernel, size_t smem, dim3 grid, const MixedAttnArgs& a, cudaStream_t stream) {
+static int launch_one(K kernel, int warps, size_t smem, dim3 grid, const MixedAttnArgs& a, cudaStream_t stream) {
   const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  return launch_pdl(kernel, grid, dim3(WARPS * 32), smem, stream, a);
+  return launch_pdl(kernel, grid, dim3(warps * 32), smem, stream, a);
 }
 
 // max_q_len: the longest q_len of the batch (sizes the grid).
@@ -509,8 +542,8 @@ extern "C" int odi_attention_mixed(const MixedAttnArgs* args, int max_q_len, cud
   if (q_tiles > 65535) return ODI_ERR_UNSUPPORTED;
   const dim3 grid(a.nq, a.n_seqs, q_tiles);
   const size_t q = query_bytes(a, 64);
-  if (q + 3 * STAGE_BYTES <= SMEM_LIMIT) odi_rc = launch_one(attention_mixed_kernel<3>, q + 3 * STAGE_BYTES, grid, a, stream);
-  else if (q + 2 * STAGE_BYTES <= SMEM_LIMIT) odi_rc = launch_one(attention_mixed_kernel<2>, q + 2 * STAGE_BYTES, grid, a, stream);
+  if (q + 3 * STAGE_BYTES <= SMEM_LIMIT) odi_rc = launch_one(attention_mixed_kernel<3>, PROMPT_WARPS, q + 3 * STAGE_BYTES, grid, a, stream);
+  else if (q + 2 * STAGE_BYTES <= SMEM_LIMIT) odi_rc = launch_one(attention_mixed_kernel<2>, PROMPT_WARPS, q + 2 * STAGE_BYTES, grid, a, stream);
   else return ODI_ERR_UNSUPPORTED;
   return launch_status();
 }
@@ -525,8 +558,8 @@ extern "C" int odi_attention_mixed_decode(const MixedAttnArgs* args, cudaStream_
   if (grid.y > 65535) return ODI_ERR_UNSUPPORTED;
   const size_t q = query_bytes(a, 16), m = merge_bytes();
   const size_t four = 4 * STAGE_BYTES > m ? 4 * STAGE_BYTES : m, two = 2 * STAGE_BYTES > m ? 2 * STAGE_BYTES : m;
-  if (q + four <= SMEM_LIMIT) odi_rc = launch_one(attention_mixed_decode_kernel<4>, q + four, grid, a, stream);
-  else if (q + two <= SMEM_LIMIT) odi_rc = launch_one(attention_mixed_decode_kernel<2>, q + two, grid, a, stream);
+  if (q + four <= SMEM_LIMIT) odi_rc = launch_one(attention_mixed_decode_kernel<4>, WARPS, q + four, grid, a, stream);
+  else if (q + two <= SMEM_LIMIT) odi_rc = launch_one(attention_mixed_decode_kernel<2>, WARPS, q + two, grid, a, stream);
   else return ODI_ERR_UNSUPPORTED;
   if (odi_rc == 0 && a.splits > 1) {
     const int threads = DV >= 128 ? 128 : (DV >= 64 ? 64 : 32);

@@ -35,7 +35,7 @@
 struct HeadDeltaArgs {
   const void* proj;       // [n_tokens, ld] in T: q (kv_heads d), k (kv_heads d), v (heads dv), gate (heads dv)
   const float* ab;        // [n_tokens, 2 heads]: a, then b
-  const float* taps;      // [C, taps_n], C = 2 kv_heads d + heads dv
+  const float* taps;      // [taps_n, C], C = 2 kv_heads d + heads dv; the last row weighs the current token
   const float* a_log;     // [heads]
   const float* dt_bias;   // [heads]
   const float* norm_w;    // [dv]
@@ -62,46 +62,78 @@ __device__ __forceinline__ float hd_input(const HeadDeltaArgs& a, int C, int q_b
   return a.conv_state[((size_t)slot * (a.taps_n - 1) + (a.taps_n - 1 + idx)) * C + c];
 }
 
-template <typename T>
+// V neighbouring channels at once: floats, and inputs in T (V = 4: 16- resp. 8-byte accesses).
+template <int V> __device__ __forceinline__ void hd_loadf(const float* p, float* v) {
+  if (V == 4) { const float4 x = *(const float4*)p; v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; }
+  else v[0] = p[0];
+}
+template <int V> __device__ __forceinline__ void hd_storef(float* p, const float* v) {
+  if (V == 4) *(float4*)p = make_float4(v[0], v[1], v[2], v[3]);
+  else p[0] = v[0];
+}
+template <typename T, int V> __device__ __forceinline__ void hd_loadt(const T* p, float* v) {
+  if (V == 1) { v[0] = to_f<T>(p[0]); return; }
+  if (sizeof(T) == 4) { hd_loadf<V>((const float*)p, v); return; }
+  const uint2 raw = *(const uint2*)p;
+  const float2 lo = __bfloat1622float2(*(const __nv_bfloat162*)&raw.x), hi = __bfloat1622float2(*(const __nv_bfloat162*)&raw.y);
+  v[0] = lo.x; v[1] = lo.y; v[2 % V] = hi.x; v[3 % V] = hi.y;
+}
+
+// A block takes one token and, of gridDim.y parts, a range of key heads with the heads that read them.
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
 hd_prep_kernel(HeadDeltaArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float ys[];          // [2 kv_heads d]: q and k behind the convolution
+  extern __shared__ __align__(16) float ys[];          // q and then k of the part's key heads behind the convolution
   const int t = blockIdx.x;
+  const int g0 = a.kv_heads * blockIdx.y / gridDim.y, g1 = a.kv_heads * (blockIdx.y + 1) / gridDim.y, rep = a.heads / a.kv_heads;
   const int qk_n = 2 * a.kv_heads * a.d, vn = a.heads * a.dv, C = qk_n + vn;
+  const int part_q = (g1 - g0) * a.d, part_n = 2 * part_q + (g1 - g0) * rep * a.dv;
   const int seq = a.tok_seq[t];
   const int q_begin = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q_begin, slot = a.slots[seq];
   const int li = t - q_begin, keep = a.taps_n - 1;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) {
-    float acc = 0.f;
-    for (int j = 0; j < a.taps_n; ++j) acc = fmaf(a.taps[(size_t)c * a.taps_n + j], hd_input<T>(a, C, q_begin, slot, li - keep + j, c), acc);
-    if (q_len == 1 && keep > 0) {        // this thread is the only one that reads or writes these inputs
-      float* st = a.conv_state + (size_t)slot * keep * C + c;
-      for (int j = 0; j + 1 < keep; ++j) st[(size_t)j * C] = st[(size_t)(j + 1) * C];
-      st[(size_t)(keep - 1) * C] = to_f<T>(((const T*)a.proj)[(size_t)t * a.ld + c]);
+  const T* row = (const T*)a.proj + (size_t)t * a.ld;
+  float* st = a.conv_state + (size_t)slot * keep * C;      // not followed when keep is 0
+  for (int x = threadIdx.x * V; x < part_n; x += blockDim.x * V) {
+    const bool is_v = x >= 2 * part_q;
+    const int c = is_v ? qk_n + g0 * rep * a.dv + (x - 2 * part_q) : (x < part_q ? 0 : a.kv_heads * a.d - part_q) + g0 * a.d + x;
+    float acc[V] = {}, in[V], w[V];
+    for (int j = 0; j < a.taps_n; ++j) {
+      const int back = keep - j;                            // tokens before this one
+      if (li >= back) hd_loadt<T, V>(row - (size_t)back * a.ld + c, in);
+      else hd_loadf<V>(st + (size_t)(keep + li - back) * C + c, in);
+      hd_loadf<V>(a.taps + (size_t)j * C + c, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e], in[e], acc[e]);
     }
-    const float y = acc / (1.f + expf(-acc));
-    if (c < qk_n) ys[c] = y;
-    else a.o[(size_t)t * vn + (c - qk_n)] = y;
+    if (q_len == 1 && keep > 0) {        // this thread is the only one that reads or writes these inputs; `in` is the token's own
+      float old[V];
+      for (int j = 0; j + 1 < keep; ++j) { hd_loadf<V>(st + (size_t)(j + 1) * C + c, old); hd_storef<V>(st + (size_t)j * C + c, old); }
+      hd_storef<V>(st + (size_t)(keep - 1) * C + c, in);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[e] = acc[e] / (1.f + expf(-acc[e]));
+    if (is_v) hd_storef<V>(a.o + (size_t)t * vn + (c - qk_n), acc);
+    else hd_storef<V>(ys + x, acc);
   }
-  for (int h = threadIdx.x; h < a.heads; h += blockDim.x) {
-    const float* row = a.ab + (size_t)t * 2 * a.heads;
-    const float decay = expf(-expf(a.a_log[h]) * hd_softplus(row[h] + a.dt_bias[h]));
+  for (int h = g0 * rep + threadIdx.x; h < g1 * rep; h += blockDim.x) {
+    const float* ab = a.ab + (size_t)t * 2 * a.heads;
+    const float decay = expf(-expf(a.a_log[h]) * hd_softplus(ab[h] + a.dt_bias[h]));
     float* dst = a.gb + ((size_t)t * a.heads + h) * 2;
     dst[0] = decay;
-    dst[1] = 1.f / (1.f + expf(-row[a.heads + h]));
+    dst[1] = 1.f / (1.f + expf(-ab[a.heads + h]));
   }
   __syncthreads();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
-  for (int w = warp; w < 2 * a.kv_heads; w += n_warps) {      // the q heads, then the k heads
+  for (int w = warp; w < 2 * (g1 - g0); w += n_warps) {      // the part's q heads, then its k heads
     const float* src = ys + (size_t)w * a.d;
     float ss = 0.f;
     for (int i = lane; i < a.d; i += 32) ss = fmaf(src[i], src[i], ss);
     ss = warp_sum(ss);
-    const bool is_k = w >= a.kv_heads;
+    const bool is_k = w >= g1 - g0;
     const float scale = 1.0f / sqrtf(ss + a.unit_eps) * (is_k ? 1.f : 1.0f / sqrtf((float)a.d));
-    float* dst = a.qk + (((size_t)t * a.kv_heads + (is_k ? w - a.kv_heads : w)) * 2 + (is_k ? 1 : 0)) * a.d;
+    float* dst = a.qk + (((size_t)t * a.kv_heads + g0 + (is_k ? w - (g1 - g0) : w)) * 2 + (is_k ? 1 : 0)) * a.d;
     for (int i = lane; i < a.d; i += 32) dst[i] = src[i] * scale;
   }
 }
@@ -560,13 +592,18 @@ static int launch_rule_form(const HeadDeltaArgs& a, cudaStream_t stream) {
 template <typename T>
 static int launch_head_delta(const HeadDeltaArgs& a, cudaStream_t stream) {
   const int C = 2 * a.kv_heads * a.d + a.heads * a.dv;
-  const size_t smem = sizeof(float) * 2 * (size_t)a.kv_heads * a.d;
+  // few tokens: a token's heads over several blocks
+  const int parts = a.n_tokens >= 296 ? 1 : min(a.kv_heads, (296 + a.n_tokens - 1) / a.n_tokens);
+  const size_t smem = sizeof(float) * 2 * (size_t)((a.kv_heads + parts - 1) / parts) * a.d;
+  if (smem > 200 * 1024) return ODI_ERR_UNSUPPORTED;
+  const bool vec = a.d % 4 == 0 && a.dv % 4 == 0 && a.ld % 4 == 0 &&
+                   (((uintptr_t)a.proj | (uintptr_t)a.taps | (uintptr_t)a.conv_state | (uintptr_t)a.o) & 15) == 0;
+  auto prep = vec ? hd_prep_kernel<T, 4> : hd_prep_kernel<T, 1>;
   if (smem > 48 * 1024) {
-    if (smem > 200 * 1024) return ODI_ERR_UNSUPPORTED;
-    const cudaError_t e = cudaFuncSetAttribute(hd_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t e = cudaFuncSetAttribute(prep, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  odi_rc = launch_pdl((hd_prep_kernel<T>), dim3(a.n_tokens), dim3(256), smem, stream, a);
+  odi_rc = launch_pdl(prep, dim3(a.n_tokens, parts), dim3(256), smem, stream, a);
   if (odi_rc == 0 && a.taps_n > 1 && a.max_q_len > 1)
     odi_rc = launch_pdl((hd_conv_state_kernel<T>), dim3(a.n_seqs, (C + 255) / 256), dim3(256), 0, stream, a);
   if (odi_rc == 0 && a.max_q_len >= 4)

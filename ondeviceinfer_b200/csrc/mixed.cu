@@ -30,10 +30,16 @@ struct MixedPrepArgs {
   float eps;
 };
 
-template <typename T> __device__ __forceinline__ void store2(T* p, float a, float b);
-template <> __device__ __forceinline__ void store2<float>(float* p, float a, float b) { *(float2*)p = make_float2(a, b); }
-template <> __device__ __forceinline__ void store2<bf16>(bf16* p, float a, float b) { *(__nv_bfloat162*)p = __floats2bfloat162_rn(a, b); }
+template <typename T> __device__ __forceinline__ void store4(T* p, const float* v);
+template <> __device__ __forceinline__ void store4<float>(float* p, const float* v) { *(float4*)p = make_float4(v[0], v[1], v[2], v[3]); }
+template <> __device__ __forceinline__ void store4<bf16>(bf16* p, const float* v) {
+  uint2 r;
+  *(__nv_bfloat162*)&r.x = __floats2bfloat162_rn(v[0], v[1]);
+  *(__nv_bfloat162*)&r.y = __floats2bfloat162_rn(v[2], v[3]);
+  *(uint2*)p = r;
+}
 
+// A block takes one token and, of gridDim.y parts, a range of the output's heads (the first part also writes k and v).
 // REP: query heads per key head (0: any number, read from shared memory each time).
 template <typename T, int REP>
 __global__ void __launch_bounds__(256)
@@ -70,7 +76,8 @@ mixed_prep_kernel(MixedPrepArgs a) {
     }
     __syncthreads();
   }
-  if (a.write_kv) {
+  const int h0 = a.nq * blockIdx.y / gridDim.y, h1 = a.nq * (blockIdx.y + 1) / gridDim.y;
+  if (a.write_kv && blockIdx.y == 0) {
     const int pos = a.tok_pos[t];
     const int page = a.page_ids[a.page_start[a.tok_seq[t]] + page_slot_of(pos, a.page_size, a.ring_pages)];
     const size_t at = (size_t)page * a.nkv * a.page_size + pos % a.page_size;
@@ -85,38 +92,52 @@ mixed_prep_kernel(MixedPrepArgs a) {
   }
   if (a.talk == nullptr) {
     T* out = (T*)a.q_out + (size_t)t * a.nq * lanes;
-    for (int i = tid; i < a.nq * lanes; i += blockDim.x) {
+    for (int i = h0 * lanes + tid; i < h1 * lanes; i += blockDim.x) {
       const int h = i / lanes, e = i % lanes;
       out[i] = from_f<T>(e < d ? qs[h * d + e] : 0.f);
     }
     return;
   }
-  // two neighbouring lanes of a key head's query group a thread; its query heads' values stay in registers
+  // four neighbouring lanes of a key head's query group a thread; its query heads' values stay in registers
   const int width = a.nkv * lanes, rep = REP > 0 ? REP : a.nq / a.nkv;
   T* out = (T*)a.q_out + (size_t)t * a.nq * width;
-  for (int p = tid; p < width / 2; p += blockDim.x) {
-    const int j = 2 * p / lanes, e = 2 * p % lanes;
-    const bool in0 = e < d, in1 = e + 1 < d;
+  for (int p = 4 * tid; p < width; p += 4 * blockDim.x) {
+    const int j = p / lanes, e = p % lanes;
     const float* src = qs + (size_t)j * rep * d + e;
-    float q0[REP > 0 ? REP : 1], q1[REP > 0 ? REP : 1];
+    float q[REP > 0 ? REP : 1][4];
     if (REP > 0) {
 #pragma unroll
-      for (int g = 0; g < REP; ++g) { q0[g] = in0 ? src[g * d] : 0.f; q1[g] = in1 ? src[g * d + 1] : 0.f; }
+      for (int g = 0; g < REP; ++g)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) q[g][x] = e + x < d ? src[g * d + x] : 0.f;
     }
     const float* T_j = a.talk + j * rep;
-    for (int h = 0; h < a.nq; ++h) {
-      float s0 = 0.f, s1 = 0.f;
+    for (int h = h0; h < h1; ++h) {
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
       if (REP > 0) {
+        float w[REP > 0 ? REP : 1];
+        if (REP > 0 && REP % 4 == 0) {
 #pragma unroll
-        for (int g = 0; g < REP; ++g) { const float w = __ldg(T_j + (size_t)h * a.nq + g); s0 = fmaf(w, q0[g], s0); s1 = fmaf(w, q1[g], s1); }
+          for (int g = 0; g < REP; g += 4) {
+            const float4 v = __ldg((const float4*)(T_j + (size_t)h * a.nq + g));
+            w[g] = v.x; w[(g + 1) % (REP > 0 ? REP : 1)] = v.y; w[(g + 2) % (REP > 0 ? REP : 1)] = v.z; w[(g + 3) % (REP > 0 ? REP : 1)] = v.w;
+          }
+        } else {
+#pragma unroll
+          for (int g = 0; g < REP; ++g) w[g] = __ldg(T_j + (size_t)h * a.nq + g);
+        }
+#pragma unroll
+        for (int g = 0; g < REP; ++g)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) s[x] = fmaf(w[g], q[g][x], s[x]);
       } else {
         for (int g = 0; g < rep; ++g) {
           const float w = __ldg(T_j + (size_t)h * a.nq + g);
-          s0 = fmaf(w, in0 ? src[g * d] : 0.f, s0);
-          s1 = fmaf(w, in1 ? src[g * d + 1] : 0.f, s1);
+#pragma unroll
+          for (int x = 0; x < 4; ++x) s[x] = fmaf(w, e + x < d ? src[g * d + x] : 0.f, s[x]);
         }
       }
-      store2<T>(out + (size_t)h * width + 2 * p, s0, s1);
+      store4<T>(out + (size_t)h * width + p, s);
     }
   }
 }
@@ -127,13 +148,15 @@ static int launch_mixed_prep(const MixedPrepArgs& a, size_t smem, cudaStream_t s
     const cudaError_t e = cudaFuncSetAttribute(mixed_prep_kernel<T, REP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  return launch_pdl((mixed_prep_kernel<T, REP>), dim3(a.n_tokens), dim3(a.nq * a.d >= 1024 ? 256 : 128), smem, stream, a);
+  // few tokens: a token's heads over several blocks
+  const int parts = a.n_tokens >= 296 ? 1 : min(a.nq, (296 + a.n_tokens - 1) / a.n_tokens);
+  return launch_pdl((mixed_prep_kernel<T, REP>), dim3(a.n_tokens, parts), dim3(a.nq * a.d >= 1024 ? 256 : 128), smem, stream, a);
 }
 
 extern "C" int odi_mixed_prep(const MixedPrepArgs* args, int dtype, cudaStream_t stream) {
   const MixedPrepArgs a = *args;
   if (a.n_tokens <= 0) return 0;
-  if (a.nq <= 0 || a.nkv <= 0 || a.nq % a.nkv != 0 || a.d <= 0 || a.dv <= 0 || a.lanes < a.d || a.v_lanes < a.dv || a.lanes % 2 != 0 ||
+  if (a.nq <= 0 || a.nkv <= 0 || a.nq % a.nkv != 0 || a.d <= 0 || a.dv <= 0 || a.lanes < a.d || a.v_lanes < a.dv || a.lanes % 4 != 0 || ((uintptr_t)a.talk | (uintptr_t)a.q_out) % 16 != 0 ||
       a.rot_dim > a.d || (a.rot_dim & 1) || (a.q_w == nullptr) != (a.k_w == nullptr))
     return ODI_ERR_ARGUMENT;
   const size_t smem = sizeof(float) * (size_t)(a.nq + a.nkv) * a.d;

@@ -307,8 +307,28 @@ cast_rows_kernel(const float* __restrict__ x, T* __restrict__ out, long n) {
   if (i < n) out[i] = from_f<T>(x[i]);
 }
 
+// Eight floats to bf16 a thread (n a multiple of 8, aligned).
+__global__ void __launch_bounds__(256)
+cast_rows_vec_kernel(const float4* __restrict__ x, uint4* __restrict__ out, long n8) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n8) return;
+  const float4 a = x[2 * i], b = x[2 * i + 1];
+  uint4 r;
+  *(__nv_bfloat162*)&r.x = __floats2bfloat162_rn(a.x, a.y);
+  *(__nv_bfloat162*)&r.y = __floats2bfloat162_rn(a.z, a.w);
+  *(__nv_bfloat162*)&r.z = __floats2bfloat162_rn(b.x, b.y);
+  *(__nv_bfloat162*)&r.w = __floats2bfloat162_rn(b.z, b.w);
+  out[i] = r;
+}
+
 extern "C" int odi_cast_rows(const float* x, void* out, long n, int dtype, cudaStream_t stream) {
   if (n <= 0) return 0;
+  if (dtype == 1 && n % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0 && n / 2048 < 2147483647L) {
+    odi_rc = launch_pdl(cast_rows_vec_kernel, dim3((unsigned)((n / 8 + 255) / 256)), dim3(256), 0, stream, (const float4*)x, (uint4*)out, n / 8);
+    return launch_status();
+  }
   const long blocks = (n + 255) / 256;
   if (blocks > 2147483647L) return ODI_ERR_UNSUPPORTED;
   if (dtype == 0) odi_rc = launch_pdl((cast_rows_kernel<float>), dim3((unsigned)blocks), dim3(256), 0, stream, x, (float*)out, n);

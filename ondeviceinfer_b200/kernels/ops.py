@@ -1572,16 +1572,16 @@ def head_delta(proj: torch.Tensor, ab: torch.Tensor, taps: torch.Tensor, a_log: 
                unit_eps: float) -> None:
     """The gated delta rule with one decay per head between its products (``csrc/delta_head.cu``): ``proj`` [tokens,
     2 kv_heads d + 2 heads dv] = q, k and v channels before their convolutions, then the output gate's logits; ``ab``
-    fp32 [tokens, 2 heads] = the decay's inner term, then the step size's logit; ``taps`` fp32 [C, K], C = 2 kv_heads d +
-    heads dv; ``conv_state`` [slots, K - 1, C] and ``state`` [slots, heads, d, dv] are fp32 rows of the cache, advanced in
+    fp32 [tokens, 2 heads] = the decay's inner term, then the step size's logit; ``taps`` fp32 [K, C], C = 2 kv_heads d +
+    heads dv (a row per tap, the last one the current token's); ``conv_state`` [slots, K - 1, C] and ``state`` [slots, heads, d, dv] are fp32 rows of the cache, advanced in
     place over all tokens that each sequence brings (``max_q_len``: the most that one brings); ``out`` [tokens, heads dv]
     receives the normed, gated read-outs in the dtype of ``proj``."""
     _require(proj, "proj", ndim=2)
     _require(ab, "ab", torch.float32, 2)
     _require(out, "out", proj.dtype, 2)
     n = proj.shape[0]
-    C, K = taps.shape
-    for name, t, shape in (("taps", taps, (2 * kv_heads * d + heads * dv, K)), ("a_log", a_log, (heads,)),
+    K, C = taps.shape
+    for name, t, shape in (("taps", taps, (K, 2 * kv_heads * d + heads * dv)), ("a_log", a_log, (heads,)),
                            ("dt_bias", dt_bias, (heads,)), ("norm_w", norm_w, (dv,))):
         _require(t, name, torch.float32)
         if tuple(t.shape) != shape:

@@ -57,7 +57,7 @@ class HeadDelta(Part):
         self.runtime = runtime
         self.w_in = torch.cat([fetch.matrix(s.name(r)) for r in ("q", "k", "v", "g")], 0)
         self.w_ab = torch.cat([fetch.matrix(s.name(r)) for r in ("a", "b")], 0)
-        self.taps = torch.cat([fetch.vector(s.name(r)) for r in ("q_conv", "k_conv", "v_conv")], 0)
+        self.taps = torch.cat([fetch.vector(s.name(r)) for r in ("q_conv", "k_conv", "v_conv")], 0).t().contiguous()
         self.a_log = fetch.vector(s.name("A_log"))
         self.dt_bias = fetch.vector(s.name("dt_bias"))
         self.out_norm = fetch.vector(s.name("norm"))

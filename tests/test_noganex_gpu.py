@@ -358,6 +358,7 @@ def test_delta_rule_over_cut_sequences(dtype, heads, kv_heads, d, dv, taps):
                              w["taps"].double(), w["A_log"].double(), w["dt_bias"].double(), w["norm"].double(), 1e-5)
             for p, ab in zip(projs, abs_)]
     dev = {k: t.float().cuda() for k, t in w.items()}
+    dev["taps"] = dev["taps"].t().contiguous()
     slots = [4, 0, 2]
     state = torch.zeros(6, heads, d, dv, device="cuda")
     conv_state = torch.zeros(6, taps - 1, C, device="cuda") if taps > 1 else None
@@ -402,7 +403,7 @@ def test_delta_rule_with_decays_down_to_zero_and_no_decay_at_all():
                             taps.double(), a_log.double(), a_log.double(), one.double(), 1e-5)
     state = torch.zeros(1, heads, d, dv, device="cuda")
     out = torch.empty(L, heads * dv, device="cuda")
-    ops.head_delta(proj.cuda(), ab.cuda(), taps.cuda(), a_log.cuda(), a_log.cuda(), one.cuda(), None, state, out, ints(0, L),
+    ops.head_delta(proj.cuda(), ab.cuda(), taps.t().contiguous().cuda(), a_log.cuda(), a_log.cuda(), one.cuda(), None, state, out, ints(0, L),
                    ints(*([0] * L)), ints(0), n_seqs=1, max_q_len=L, heads=heads, kv_heads=heads, d=d, dv=dv, eps=1e-5, unit_eps=1e-6)
     assert torch.isfinite(out).all()
     torch.testing.assert_close(out.cpu().double(), want, atol=5e-4, rtol=5e-4)
