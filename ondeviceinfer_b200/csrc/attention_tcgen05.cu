@@ -44,7 +44,9 @@
 // p / chunk; the walk starts at the tile of the first row's chunk), and heads that mix their scores (MIXED): q is
 // [n_tokens, nq, nkv, D], a score is the sum over the key heads of q_hj . k_j, accumulated in tensor memory key head by
 // key head, so a page's key heads pass one after the other through a ring of their own (KRING slots) while the CTA's
-// query rows of all key heads stay in shared memory.  Compile with -DODI_HEAD_DIM=64 or 128.
+// query rows of all key heads stay in shared memory.  When shared memory does not hold 128 rows of all key heads a CTA
+// takes 64 (QROWS): the products keep their 128 lanes, of which the upper half reads whatever lies behind the 64 rows and
+// is never looked at (lanes of a product do not mix), and two of the four softmax warps have nothing to do.  Compile with -DODI_HEAD_DIM=64 or 128.
 //
 // Every wait on an mbarrier is bounded (about two seconds of SM clock): a role that gives up
 // records a code in `status`, raises the CTA's abort flag, and all roles fall through to the
@@ -358,13 +360,14 @@ __device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, b
   }
 }
 
-template <int TILES, bool MIXED>
+template <int TILES, bool MIXED, int QROWS>
 __global__ void __launch_bounds__(64 + 128 * TILES, TILES == 1 && !MIXED ? 2 : 1)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const TcAttnArgs a) {
   constexpr int TMEM_COLS = TILES * HEAD_COLS;
   constexpr int KRING = MIXED ? MIXED_KEY_RING : RING;
-  static_assert(!MIXED || TILES == 1, "mixed heads take one head per CTA");
+  constexpr int Q_TILE = KB * QROWS * 128;       // the CTA's query rows of one head (of one key head when mixed)
+  static_assert((!MIXED || TILES == 1) && (QROWS == BM || (MIXED && QROWS == 64)), "mixed heads take one head per CTA");
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   // barriers: q_full, k_full[KR], k_empty[KR], v_full[R], v_empty[R], s_full[2], p_full[TILES][2], pv_done[TILES]
@@ -378,10 +381,10 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   // heads along x, sequences along y, query tiles along z from the last (the most keys) to the first
   const int seq = blockIdx.y, head0 = blockIdx.x * TILES, hk = head0 / (a.nq / a.nkv);
   const int q_begin = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q_begin;
-  const int t0 = (gridDim.z - 1 - blockIdx.z) * BM;
+  const int t0 = (gridDim.z - 1 - blockIdx.z) * QROWS;
   if (t0 >= q_len) return;                       // whole CTA: nothing allocated yet
   const int past = a.past[seq];
-  const int nt = min(BM, q_len - t0);
+  const int nt = min(QROWS, q_len - t0);
   // key tiles from the one that holds the oldest key any row of the CTA sees up to the diagonal
   const int first = past + t0;
   const int tile_lo = (a.window > 0 ? max(0, first - a.window + 1) : (a.chunk > 0 ? first - first % a.chunk : 0)) / BNK;
@@ -395,15 +398,15 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const uint32_t q_full = bar0, k_full = bar0 + 8, k_empty = k_full + 8 * KRING, v_full = k_empty + 8 * KRING,
                  v_empty = v_full + 8 * RING, s_full = v_empty + 8 * RING, p_full = s_full + 16,
                  pv_done = p_full + 16 * TILES;
-  uint8_t* q_smem = smem;                                    // head t at t * Q_BYTES
+  uint8_t* q_smem = smem;                                    // head t at t * Q_TILE
   const int KH = MIXED ? a.nkv : 1;                          // key heads a score sums over
-  uint8_t* k_smem = smem + TILES * KH * Q_BYTES;             // ring of K pages
+  uint8_t* k_smem = smem + TILES * KH * Q_TILE;              // ring of K pages
   uint8_t* v_smem = k_smem + KRING * KV_BYTES;            // ring of V pages
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < BARS; ++i) mbar_init(bar0 + 8 * i, 1);
     for (int b = 0; b < 2; ++b)
-      for (int t = 0; t < TILES; ++t) mbar_init(p_full + 16 * t + 8 * b, 4);     // one arrival per softmax warp
+      for (int t = 0; t < TILES; ++t) mbar_init(p_full + 16 * t + 8 * b, QROWS / 32);     // one arrival per softmax warp
     abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
@@ -421,10 +424,10 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     // ---------------------------------------------------------------- TMA producer: K_0, K_1, V_0, then K_j, V_{j-1}
     if (lane == 0) {
       pdl_wait();      // queries and this step's keys/values come from the kernel before
-      mbar_expect_tx(q_full, TILES * KH * Q_BYTES);
+      mbar_expect_tx(q_full, TILES * KH * Q_TILE);
       for (int t = 0; t < TILES * KH; ++t)
         for (int kb = 0; kb < KB; ++kb)
-          tma_load_2d(smem_u32(q_smem + t * Q_BYTES + kb * BM * 128), &map_q, (head0 * KH + t) * D + kb * 64, q_begin + t0, q_full);
+          tma_load_2d(smem_u32(q_smem + t * Q_TILE + kb * QROWS * 128), &map_q, (head0 * KH + t) * D + kb * 64, q_begin + t0, q_full);
       bool ok = true;
       // box n of a ring of `slots` slots: head `h` of page j
       auto load_box = [&](int n, int slots, int j, int h, const CUtensorMap* map, uint8_t* ring, uint32_t full, uint32_t empty) {
@@ -464,7 +467,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
           for (int t = 0; t < TILES; ++t) {
 #pragma unroll
             for (int kb = 0; kb < KB; ++kb) {
-              const uint64_t dq = desc_k_major(smem_u32(q_smem + (t * KH + g) * Q_BYTES + kb * BM * 128));
+              const uint64_t dq = desc_k_major(smem_u32(q_smem + (t * KH + g) * Q_TILE + kb * QROWS * 128));
               const uint64_t dk = desc_k_major(k_addr + kb * BNK * 128);
 #pragma unroll
               for (int i = 0; i < 4; ++i) umma(tmem_base + S_COL(t, b), dq + 2 * i, dk + 2 * i, idesc_s, (g | kb | i) ? 1u : 0u);
@@ -498,7 +501,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       }
       if (!ok) atomicCAS(a.status, 0, ATT_ERR_MMA);
     }
-  } else {
+  } else if (QROWS == BM || (warp & 3) * 32 < QROWS) {
     // ---------------------------------------------------------------- softmax and output (4 warps a head, a thread a row)
     const int tile = (warp - 2) >> 2;                // which of the CTA's heads
     const int head = head0 + tile;
@@ -574,26 +577,30 @@ static int make_map(CUtensorMap* map, const void* base, long rows, long cols, in
 
 extern "C" int odi_attention_tcgen05_head_dim() { return D; }
 
-// Whether shared memory holds a CTA's query rows of `nkv` key heads (heads that mix their scores).
-extern "C" int odi_attention_tcgen05_fits_mixed(int nkv) {
-  return nkv > 0 && nkv <= 64 && nkv * Q_BYTES + (MIXED_KEY_RING + RING) * KV_BYTES + 1024 <= SMEM_LIMIT;
+// Rows of a CTA (128 or 64) that shared memory holds for `nkv` key heads (heads that mix their scores); 0: too many.
+static int mixed_rows(int nkv) {
+  const long ring = (MIXED_KEY_RING + RING) * KV_BYTES + 1024;
+  if (nkv <= 0 || nkv > 64) return 0;
+  if ((long)nkv * Q_BYTES + ring <= SMEM_LIMIT) return BM;
+  return (long)nkv * (Q_BYTES / 2) + ring <= SMEM_LIMIT ? 64 : 0;
 }
+extern "C" int odi_attention_tcgen05_mixed_rows(int nkv) { return mixed_rows(nkv); }
 
 // q [n_tokens, nq * D] bf16; k_pool, v_pool [pool_pages, nkv, 64, D] bf16; out [n_tokens, nq * D].
 // heads_per_cta: 2 = two heads of a key/value group per CTA (needs an even group size), 1 = one, 0 = choose.
-template <int TILES, bool MIXED>
+template <int TILES, bool MIXED, int QROWS = BM>
 static int launch_attention(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnArgs& a,
                             int max_q_len, cudaStream_t stream) {
-  const int smem = TILES * (MIXED ? a.nkv : 1) * Q_BYTES + ((MIXED ? MIXED_KEY_RING : RING) + RING) * KV_BYTES + 1024;
+  const int smem = TILES * (MIXED ? a.nkv : 1) * (KB * QROWS * 128) + ((MIXED ? MIXED_KEY_RING : RING) + RING) * KV_BYTES + 1024;
   if (smem > SMEM_LIMIT) return ODI_ERR_UNSUPPORTED;
-  auto kernel = attention_tcgen05_kernel<TILES, MIXED>;
+  auto kernel = attention_tcgen05_kernel<TILES, MIXED, QROWS>;
   static int configured = 0;
   if (configured < smem) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
     configured = smem;
   }
-  dim3 grid(a.nq / TILES, a.n_seqs, (max_q_len + BM - 1) / BM);
+  dim3 grid(a.nq / TILES, a.n_seqs, (max_q_len + QROWS - 1) / QROWS);
   odi_rc = launch_pdl((kernel), dim3(grid), dim3(64 + 128 * TILES), smem, stream, mq, mk, mv, a);
   return launch_status();
 }
@@ -607,17 +614,21 @@ extern "C" int odi_attention_tcgen05(const void* q, const void* k_pool, const vo
   if (((uintptr_t)q & 15) || ((uintptr_t)k_pool & 15) || ((uintptr_t)v_pool & 15) || ((uintptr_t)a.out & 15))
     return ODI_ERR_UNSUPPORTED;
   if (pool_pages * a.nkv * BNK > 0x7fffffffL) return ODI_ERR_UNSUPPORTED;    // row coordinates are 32-bit
-  if ((max_q_len + BM - 1) / BM > 65535) return ODI_ERR_UNSUPPORTED;
+  if ((max_q_len + 63) / 64 > 65535) return ODI_ERR_UNSUPPORTED;
   if (heads_per_cta < 0 || heads_per_cta > 2 || a.chunk < 0 || (a.chunk > 0 && (a.window > 0 || a.keep > 0))) return ODI_ERR_ARGUMENT;
   if (a.mixed && heads_per_cta == 2) return ODI_ERR_UNSUPPORTED;
   if (heads_per_cta == 2 && (a.nq / a.nkv) % 2 != 0) return ODI_ERR_ARGUMENT;
+  const int q_rows = a.mixed ? mixed_rows(a.nkv) : BM;
+  if (q_rows == 0) return ODI_ERR_UNSUPPORTED;
   CUtensorMap mq, mk, mv;
-  int rc = make_map(&mq, q, n_tokens, (long)a.nq * (a.mixed ? a.nkv : 1) * D, BM);
+  int rc = make_map(&mq, q, n_tokens, (long)a.nq * (a.mixed ? a.nkv : 1) * D, q_rows);
   if (rc == 0) rc = make_map(&mk, k_pool, pool_pages * a.nkv * BNK, D, BNK);
   if (rc == 0) rc = make_map(&mv, v_pool, pool_pages * a.nkv * BNK, D, BNK);
   if (rc != 0) return rc;
   if (heads_per_cta == 0) heads_per_cta = ODI_ATT_DEFAULT_HEADS_PER_CTA;
-  if (a.mixed) return launch_attention<1, true>(mq, mk, mv, a, max_q_len, stream);
+  if (a.mixed)
+    return q_rows == BM ? launch_attention<1, true>(mq, mk, mv, a, max_q_len, stream)
+                        : launch_attention<1, true, 64>(mq, mk, mv, a, max_q_len, stream);
   return heads_per_cta == 2 ? launch_attention<2, false>(mq, mk, mv, a, max_q_len, stream)
                             : launch_attention<1, false>(mq, mk, mv, a, max_q_len, stream);
 }

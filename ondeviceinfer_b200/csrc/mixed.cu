@@ -28,6 +28,7 @@ struct MixedPrepArgs {
   const int* page_ids;
   int n_tokens, nq, nkv, d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, write_kv;
   float eps;
+  int stage_talk;         // set by the launcher: the matrix goes through shared memory
 };
 
 template <typename T> __device__ __forceinline__ void store4(T* p, const float* v);
@@ -51,11 +52,14 @@ mixed_prep_kernel(MixedPrepArgs a) {
   const int d = a.d, nqd = a.nq * d, nkd = a.nkv * d, lanes = a.lanes;
   float* qs = smem;               // [nq, d]
   float* ks = smem + nqd;         // [nkv, d]
+  float* ts = smem + (nqd + nkd + 3) / 4 * 4;      // the matrix, when it is staged
   const int t = blockIdx.x, tid = threadIdx.x;
   const T* row = (const T*)a.qkv + (size_t)t * (nqd + nkd + a.nkv * a.dv);
   float sq = 0.f, sk = 0.f;
   for (int i = tid; i < nqd; i += blockDim.x) { const float v = to_f<T>(row[i]); qs[i] = v; sq = fmaf(v, v, sq); }
   for (int i = tid; i < nkd; i += blockDim.x) { const float v = to_f<T>(row[nqd + i]); ks[i] = v; sk = fmaf(v, v, sk); }
+  if (a.stage_talk)
+    for (int i = tid; i < a.nq * a.nq; i += blockDim.x) ts[i] = a.talk[i];
   if (a.q_w != nullptr) {
     sq = block_sum(sq, scratch);
     sk = block_sum(sk, scratch);
@@ -101,7 +105,11 @@ mixed_prep_kernel(MixedPrepArgs a) {
   // four neighbouring lanes of a key head's query group a thread; its query heads' values stay in registers
   const int width = a.nkv * lanes, rep = REP > 0 ? REP : a.nq / a.nkv;
   T* out = (T*)a.q_out + (size_t)t * a.nq * width;
-  for (int p = 4 * tid; p < width; p += 4 * blockDim.x) {
+  // more threads than groups of four lanes: they share the heads out among themselves
+  const int spread = max(1, (int)blockDim.x * 4 / width), sub = 4 * tid / width;
+  const int begin = spread > 1 ? h0 + (h1 - h0) * sub / spread : h0, end = spread > 1 ? h0 + (h1 - h0) * (sub + 1) / spread : h1;
+  if (spread > 1 && sub >= spread) return;
+  for (int p = spread > 1 ? 4 * tid - sub * width : 4 * tid; p < width; p += spread > 1 ? width : 4 * blockDim.x) {
     const int j = p / lanes, e = p % lanes;
     const float* src = qs + (size_t)j * rep * d + e;
     float q[REP > 0 ? REP : 1][4];
@@ -111,20 +119,21 @@ mixed_prep_kernel(MixedPrepArgs a) {
 #pragma unroll
         for (int x = 0; x < 4; ++x) q[g][x] = e + x < d ? src[g * d + x] : 0.f;
     }
-    const float* T_j = a.talk + j * rep;
-    for (int h = h0; h < h1; ++h) {
+    const float* T_j = (a.stage_talk ? ts : a.talk) + j * rep;
+#pragma unroll 4
+    for (int h = begin; h < end; ++h) {
       float s[4] = {0.f, 0.f, 0.f, 0.f};
       if (REP > 0) {
         float w[REP > 0 ? REP : 1];
         if (REP > 0 && REP % 4 == 0) {
 #pragma unroll
           for (int g = 0; g < REP; g += 4) {
-            const float4 v = __ldg((const float4*)(T_j + (size_t)h * a.nq + g));
+            const float4 v = *(const float4*)(T_j + (size_t)h * a.nq + g);
             w[g] = v.x; w[(g + 1) % (REP > 0 ? REP : 1)] = v.y; w[(g + 2) % (REP > 0 ? REP : 1)] = v.z; w[(g + 3) % (REP > 0 ? REP : 1)] = v.w;
           }
         } else {
 #pragma unroll
-          for (int g = 0; g < REP; ++g) w[g] = __ldg(T_j + (size_t)h * a.nq + g);
+          for (int g = 0; g < REP; ++g) w[g] = T_j[(size_t)h * a.nq + g];
         }
 #pragma unroll
         for (int g = 0; g < REP; ++g)
@@ -132,7 +141,7 @@ mixed_prep_kernel(MixedPrepArgs a) {
           for (int x = 0; x < 4; ++x) s[x] = fmaf(w[g], q[g][x], s[x]);
       } else {
         for (int g = 0; g < rep; ++g) {
-          const float w = __ldg(T_j + (size_t)h * a.nq + g);
+          const float w = T_j[(size_t)h * a.nq + g];
 #pragma unroll
           for (int x = 0; x < 4; ++x) s[x] = fmaf(w, e + x < d ? src[g * d + x] : 0.f, s[x]);
         }
@@ -154,12 +163,13 @@ static int launch_mixed_prep(const MixedPrepArgs& a, size_t smem, cudaStream_t s
 }
 
 extern "C" int odi_mixed_prep(const MixedPrepArgs* args, int dtype, cudaStream_t stream) {
-  const MixedPrepArgs a = *args;
+  MixedPrepArgs a = *args;
   if (a.n_tokens <= 0) return 0;
   if (a.nq <= 0 || a.nkv <= 0 || a.nq % a.nkv != 0 || a.d <= 0 || a.dv <= 0 || a.lanes < a.d || a.v_lanes < a.dv || a.lanes % 4 != 0 || ((uintptr_t)a.talk | (uintptr_t)a.q_out) % 16 != 0 ||
       a.rot_dim > a.d || (a.rot_dim & 1) || (a.q_w == nullptr) != (a.k_w == nullptr))
     return ODI_ERR_ARGUMENT;
-  const size_t smem = sizeof(float) * (size_t)(a.nq + a.nkv) * a.d;
+  a.stage_talk = a.talk != nullptr && a.nq <= 64 && a.n_tokens >= 296;
+  const size_t smem = sizeof(float) * (((size_t)(a.nq + a.nkv) * a.d + 3) / 4 * 4 + (a.stage_talk ? a.nq * a.nq : 0));
   if (smem > 200 * 1024) return ODI_ERR_UNSUPPORTED;
   const int rep = a.nq / a.nkv;
 #define ODI_MP(T) \

@@ -900,7 +900,7 @@ def attention_tcgen05(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, 
     ``softcap`` c > 0 squashes the scores (times ``scale``) by c tanh(score / c).
     ``chunk`` c > 0 (instead of a window): position p sees the keys of its own chunk of c positions only.
     ``mixed``: q is [tokens, nq, nkv, d] and a score is the sum over the key heads of q . k (see :func:`mixed_prep`;
-    :func:`attention_tcgen05_fits_mixed` says for how many key heads).
+    :func:`attention_tcgen05_mixed_rows` says for how many key heads).
     ``heads_per_cta``: 1, or 2 (two heads of a key/value group share a CTA and its K/V pages; needs an
     even group size), or 0 for the library's choice."""
     if d not in TCGEN05_ATTENTION_HEAD_DIMS:
@@ -921,12 +921,12 @@ def attention_tcgen05(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, 
            "attention_tcgen05")
 
 
-def attention_tcgen05_fits_mixed(d: int, nkv: int) -> bool:
-    """Whether :func:`attention_tcgen05` takes ``mixed`` heads of ``d`` lanes over ``nkv`` key heads (shared memory holds
-    128 query rows of all of them)."""
+def attention_tcgen05_mixed_rows(d: int, nkv: int) -> int:
+    """Query rows of a CTA of :func:`attention_tcgen05` for ``mixed`` heads of ``d`` lanes over ``nkv`` key heads: 128, 64
+    when shared memory does not hold 128 of all of them, 0 when it does not hold 64 either."""
     if d not in TCGEN05_ATTENTION_HEAD_DIMS:
-        return False
-    return bool(load_library("attention_tcgen05", {"ODI_HEAD_DIM": d}).odi_attention_tcgen05_fits_mixed(c_int(nkv)))
+        return 0
+    return int(load_library("attention_tcgen05", {"ODI_HEAD_DIM": d}).odi_attention_tcgen05_mixed_rows(c_int(nkv)))
 
 
 # ------------------------------------------------------------------------------ norms and activations in fp32
@@ -1616,7 +1616,7 @@ class _MixedPrepArgs(Structure):
                 ("k_w", c_void_p), ("talk", c_void_p), ("cos_t", c_void_p), ("sin_t", c_void_p), ("tok_seq", c_void_p),
                 ("tok_pos", c_void_p), ("page_start", c_void_p), ("page_ids", c_void_p), ("n_tokens", c_int), ("nq", c_int),
                 ("nkv", c_int), ("d", c_int), ("dv", c_int), ("lanes", c_int), ("v_lanes", c_int), ("rot_dim", c_int),
-                ("page_size", c_int), ("ring_pages", c_int), ("write_kv", c_int), ("eps", c_float)]
+                ("page_size", c_int), ("ring_pages", c_int), ("write_kv", c_int), ("eps", c_float), ("stage_talk", c_int)]
 
 
 def mixed_prep(qkv, q_out, k_pool, v_pool, q_norm, k_norm, talk, cos_t, sin_t, tok_seq, tok_pos, page_start, page_ids, *,
@@ -1652,7 +1652,7 @@ def mixed_prep(qkv, q_out, k_pool, v_pool, q_norm, k_norm, talk, cos_t, sin_t, t
             raise KernelError("rope tables must be [tokens, rot_dim / 2]")
     args = _MixedPrepArgs(_ptr(qkv), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(q_norm), _ptr(k_norm), _ptr(talk),
                           _ptr(cos_t), _ptr(sin_t), _ptr(tok_seq), _ptr(tok_pos), _ptr(page_start), _ptr(page_ids), n, nq, nkv,
-                          d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, 1 if write_kv else 0, eps)
+                          d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, 1 if write_kv else 0, eps, 0)
     lib = load_library("mixed")
     _check(lib.odi_mixed_prep(byref(args), c_int(dtype_code(qkv.dtype)), _stream()), "mixed_prep")
 

@@ -129,7 +129,7 @@ class MixedAttention(Part):
                 partial = torch.empty((ctx.n_tokens * s.num_heads * splits * (self.v_lanes + 2),), dtype=torch.float32,
                                       device=q.device)
         if (tensor_cores and ctx.max_q_len > TCGEN05_MIN_Q_LEN and self.lanes == self.v_lanes
-                and (ops.attention_tcgen05_fits_mixed(self.lanes, s.num_kv_heads) if mixed
+                and (ops.attention_tcgen05_mixed_rows(self.lanes, s.num_kv_heads) > 0 if mixed
                      else self.lanes in ops.TCGEN05_ATTENTION_HEAD_DIMS)):
             # bf16 prompts with heads of 64 or 128 lanes: scores and outputs in tensor memory
             ops.attention_tcgen05(*where, max_q_len=ctx.max_q_len, **common)

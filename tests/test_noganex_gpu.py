@@ -292,10 +292,12 @@ def test_attention_inside_chunks(kind, dtype, mixed, chunk, L, T, ring, splits):
 
 
 @pytest.mark.parametrize("kind", ["cores", "tensor", "tensor memory"])
-def test_attention_of_unequal_sequences_in_one_launch(kind):
-    """Sequences of other lengths and pasts beside each other, heads of 128 lanes, more key heads than the ring has slots."""
+@pytest.mark.parametrize("nq,nkv,d", [(8, 4, 128), (6, 3, 64), (8, 8, 128), (12, 6, 128), (16, 16, 64)])
+def test_attention_of_unequal_sequences_in_one_launch(kind, nq, nkv, d):
+    """Sequences of other lengths and pasts beside each other, with few and with many key heads (which fill the key ring
+    several times a page, and leave room for 128 or for 64 query rows of all of them)."""
     gen = torch.Generator().manual_seed(3)
-    nq, nkv, d, chunk, dtype = 8, 4, 128, 100, torch.bfloat16
+    chunk, dtype = 100, torch.bfloat16
     runs, pasts = [70, 1, 200, 33], [0, 99, 40, 300]
     seqs, qs, pools = [], [], []
     for T, past in zip(runs, pasts):
@@ -331,8 +333,8 @@ def test_widths_that_the_tensor_core_forms_refuse():
     assert ops.attention_mixed_supported(torch.bfloat16, 128, 128, 7, True)
     assert not ops.attention_mixed_supported(torch.bfloat16, 128, 128, 64, True)
     assert ops.attention_mixed_supported(torch.bfloat16, 128, 128, 64, False)
-    assert ops.attention_tcgen05_fits_mixed(128, 4) and not ops.attention_tcgen05_fits_mixed(128, 5)
-    assert ops.attention_tcgen05_fits_mixed(64, 8) and not ops.attention_tcgen05_fits_mixed(48, 1)
+    assert [ops.attention_tcgen05_mixed_rows(128, n) for n in (1, 4, 5, 8, 9)] == [128, 128, 64, 64, 0]
+    assert [ops.attention_tcgen05_mixed_rows(64, n) for n in (8, 16, 32)] == [128, 64, 0] and ops.attention_tcgen05_mixed_rows(48, 1) == 0
 
 
 # ----------------------------------------------------------------------------- the delta rule
