@@ -99,13 +99,24 @@ hd_prep_kernel(HeadDeltaArgs a) {
     const bool is_v = x >= 2 * part_q;
     const int c = is_v ? qk_n + g0 * rep * a.dv + (x - 2 * part_q) : (x < part_q ? 0 : a.kv_heads * a.d - part_q) + g0 * a.d + x;
     float acc[V] = {}, in[V], w[V];
-    for (int j = 0; j < a.taps_n; ++j) {
-      const int back = keep - j;                            // tokens before this one
-      if (li >= back) hd_loadt<T, V>(row - (size_t)back * a.ld + c, in);
-      else hd_loadf<V>(st + (size_t)(keep + li - back) * C + c, in);
-      hd_loadf<V>(a.taps + (size_t)j * C + c, w);
+    if (li >= keep) {                    // every input is one of the step's own: no branch between the loads
+      const T* src = row - (size_t)keep * a.ld + c;
+#pragma unroll 4
+      for (int j = 0; j < a.taps_n; ++j) {
+        hd_loadt<T, V>(src + (size_t)j * a.ld, in);
+        hd_loadf<V>(a.taps + (size_t)j * C + c, w);
 #pragma unroll
-      for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e], in[e], acc[e]);
+        for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e], in[e], acc[e]);
+      }
+    } else {
+      for (int j = 0; j < a.taps_n; ++j) {
+        const int back = keep - j;                          // tokens before this one
+        if (li >= back) hd_loadt<T, V>(row - (size_t)back * a.ld + c, in);
+        else hd_loadf<V>(st + (size_t)(keep + li - back) * C + c, in);
+        hd_loadf<V>(a.taps + (size_t)j * C + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc[e] = fmaf(w[e], in[e], acc[e]);
+      }
     }
     if (q_len == 1 && keep > 0) {        // this thread is the only one that reads or writes these inputs; `in` is the token's own
       float old[V];
@@ -537,7 +548,7 @@ hd_rule_kernel(HeadDeltaArgs a, int vec) {
 }
 
 // One warp per (token, head).
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(128)
 hd_out_norm_kernel(HeadDeltaArgs a) {
   pdl_launch_dependents();
@@ -549,11 +560,32 @@ hd_out_norm_kernel(HeadDeltaArgs a) {
   const int h = (int)(item % a.heads);
   const float* o = a.o + item * a.dv;
   const T* gate = (const T*)a.proj + t * a.ld + 2 * a.kv_heads * a.d + a.heads * a.dv + (size_t)h * a.dv;
+  T* out = (T*)a.out + item * a.dv;
   float ss = 0.f;
+  if (V == 4 && a.dv <= 128) {           // the row in one piece a lane
+    const bool in = 4 * lane < a.dv;
+    float v[V] = {}, z[V] = {}, w[V] = {};
+    if (in) { hd_loadf<V>(o + 4 * lane, v); hd_loadt<T, V>(gate + 4 * lane, z); hd_loadf<V>(a.norm_w + 4 * lane, w); }
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
+    ss = warp_sum(ss);
+    const float inv = 1.0f / sqrtf(ss / (float)a.dv + a.eps);
+    if (in) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = v[e] * inv * w[e] * (z[e] / (1.f + expf(-z[e])));
+      if (sizeof(T) == 4) hd_storef<V>((float*)out + 4 * lane, v);
+      else {
+        uint2 r;
+        *(__nv_bfloat162*)&r.x = __floats2bfloat162_rn(v[0], v[1 % V]);
+        *(__nv_bfloat162*)&r.y = __floats2bfloat162_rn(v[2 % V], v[3 % V]);
+        *(uint2*)((bf16*)out + 4 * lane) = r;
+      }
+    }
+    return;
+  }
   for (int i = lane; i < a.dv; i += 32) ss = fmaf(o[i], o[i], ss);
   ss = warp_sum(ss);
   const float inv = 1.0f / sqrtf(ss / (float)a.dv + a.eps);
-  T* out = (T*)a.out + item * a.dv;
   for (int i = lane; i < a.dv; i += 32) {
     const float z = to_f<T>(gate[i]);
     out[i] = from_f<T>(o[i] * inv * a.norm_w[i] * (z / (1.f + expf(-z))));
@@ -624,7 +656,7 @@ static int launch_head_delta(const HeadDeltaArgs& a, cudaStream_t stream) {
     else odi_rc = launch_rule_form<512, 8>(a, stream);
   }
   if (odi_rc == 0)
-    odi_rc = launch_pdl((hd_out_norm_kernel<T>), dim3((unsigned)(((long)a.n_tokens * a.heads + 3) / 4)), dim3(128), 0, stream, a);
+    odi_rc = launch_pdl((vec && ((uintptr_t)a.out | (uintptr_t)a.norm_w) % 16 == 0 ? hd_out_norm_kernel<T, 4> : hd_out_norm_kernel<T, 1>), dim3((unsigned)(((long)a.n_tokens * a.heads + 3) / 4)), dim3(128), 0, stream, a);
   return launch_status();
 }
 

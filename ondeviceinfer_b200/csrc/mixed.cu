@@ -28,7 +28,7 @@ struct MixedPrepArgs {
   const int* page_ids;
   int n_tokens, nq, nkv, d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, write_kv;
   float eps;
-  int stage_talk;         // set by the launcher: the matrix goes through shared memory
+  int stage_talk, vec;    // set by the launcher: the matrix goes through shared memory; rows in pieces of 16 bytes
 };
 
 template <typename T> __device__ __forceinline__ void store4(T* p, const float* v);
@@ -38,6 +38,19 @@ template <> __device__ __forceinline__ void store4<bf16>(bf16* p, const float* v
   *(__nv_bfloat162*)&r.x = __floats2bfloat162_rn(v[0], v[1]);
   *(__nv_bfloat162*)&r.y = __floats2bfloat162_rn(v[2], v[3]);
   *(uint2*)p = r;
+}
+
+// Eight neighbouring elements as floats (16-byte accesses; the caller has checked the alignment).
+template <typename T> __device__ __forceinline__ void load8(const T* p, float* v);
+template <> __device__ __forceinline__ void load8<float>(const float* p, float* v) {
+  const float4 a = *(const float4*)p, b = *(const float4*)(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> __device__ __forceinline__ void load8<bf16>(const bf16* p, float* v) {
+  const uint4 raw = *(const uint4*)p;
+  const __nv_bfloat162* h = (const __nv_bfloat162*)&raw;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
 }
 
 // A block takes one token and, of gridDim.y parts, a range of the output's heads (the first part also writes k and v).
@@ -56,16 +69,41 @@ mixed_prep_kernel(MixedPrepArgs a) {
   const int t = blockIdx.x, tid = threadIdx.x;
   const T* row = (const T*)a.qkv + (size_t)t * (nqd + nkd + a.nkv * a.dv);
   float sq = 0.f, sk = 0.f;
-  for (int i = tid; i < nqd; i += blockDim.x) { const float v = to_f<T>(row[i]); qs[i] = v; sq = fmaf(v, v, sq); }
-  for (int i = tid; i < nkd; i += blockDim.x) { const float v = to_f<T>(row[nqd + i]); ks[i] = v; sk = fmaf(v, v, sk); }
+  if (a.vec) {          // q and k lie side by side; no piece of eight straddles them
+#pragma unroll 4
+    for (int i = 8 * tid; i < nqd + nkd; i += 8 * blockDim.x) {
+      float v[8], ss = 0.f;
+      load8<T>(row + i, v);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+      *(float4*)(smem + i) = make_float4(v[0], v[1], v[2], v[3]);
+      *(float4*)(smem + i + 4) = make_float4(v[4], v[5], v[6], v[7]);
+      if (i < nqd) sq += ss; else sk += ss;
+    }
+  } else {
+    for (int i = tid; i < nqd; i += blockDim.x) { const float v = to_f<T>(row[i]); qs[i] = v; sq = fmaf(v, v, sq); }
+    for (int i = tid; i < nkd; i += blockDim.x) { const float v = to_f<T>(row[nqd + i]); ks[i] = v; sk = fmaf(v, v, sk); }
+  }
   if (a.stage_talk)
     for (int i = tid; i < a.nq * a.nq; i += blockDim.x) ts[i] = a.talk[i];
   if (a.q_w != nullptr) {
     sq = block_sum(sq, scratch);
     sk = block_sum(sk, scratch);
     const float qi = 1.0f / sqrtf(sq / (float)nqd + a.eps), ki = 1.0f / sqrtf(sk / (float)nkd + a.eps);
-    for (int i = tid; i < nqd; i += blockDim.x) qs[i] *= qi * a.q_w[i];      // each thread's own elements
-    for (int i = tid; i < nkd; i += blockDim.x) ks[i] *= ki * a.k_w[i];
+    if (a.vec) {        // each thread's own elements
+#pragma unroll 4
+      for (int i = 8 * tid; i < nqd + nkd; i += 8 * blockDim.x) {
+        const bool is_q = i < nqd;
+        float w[8];
+        load8<float>(is_q ? a.q_w + i : a.k_w + (i - nqd), w);
+        const float r = is_q ? qi : ki;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) smem[i + e] *= r * w[e];
+      }
+    } else {
+      for (int i = tid; i < nqd; i += blockDim.x) qs[i] *= qi * a.q_w[i];
+      for (int i = tid; i < nkd; i += blockDim.x) ks[i] *= ki * a.k_w[i];
+    }
   }
   __syncthreads();
   if (a.cos_t != nullptr) {
@@ -169,6 +207,8 @@ extern "C" int odi_mixed_prep(const MixedPrepArgs* args, int dtype, cudaStream_t
       a.rot_dim > a.d || (a.rot_dim & 1) || (a.q_w == nullptr) != (a.k_w == nullptr))
     return ODI_ERR_ARGUMENT;
   a.stage_talk = a.talk != nullptr && a.nq <= 64 && a.n_tokens >= 296;
+  a.vec = a.nq * a.d % 8 == 0 && a.nkv * a.d % 8 == 0 && a.nkv * a.dv % 8 == 0 &&
+          ((uintptr_t)a.qkv | (uintptr_t)a.q_w | (uintptr_t)a.k_w) % 16 == 0;
   const size_t smem = sizeof(float) * (((size_t)(a.nq + a.nkv) * a.d + 3) / 4 * 4 + (a.stage_talk ? a.nq * a.nq : 0));
   if (smem > 200 * 1024) return ODI_ERR_UNSUPPORTED;
   const int rep = a.nq / a.nkv;

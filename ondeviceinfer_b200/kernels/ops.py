@@ -1616,7 +1616,7 @@ class _MixedPrepArgs(Structure):
                 ("k_w", c_void_p), ("talk", c_void_p), ("cos_t", c_void_p), ("sin_t", c_void_p), ("tok_seq", c_void_p),
                 ("tok_pos", c_void_p), ("page_start", c_void_p), ("page_ids", c_void_p), ("n_tokens", c_int), ("nq", c_int),
                 ("nkv", c_int), ("d", c_int), ("dv", c_int), ("lanes", c_int), ("v_lanes", c_int), ("rot_dim", c_int),
-                ("page_size", c_int), ("ring_pages", c_int), ("write_kv", c_int), ("eps", c_float), ("stage_talk", c_int)]
+                ("page_size", c_int), ("ring_pages", c_int), ("write_kv", c_int), ("eps", c_float), ("stage_talk", c_int), ("vec", c_int)]
 
 
 def mixed_prep(qkv, q_out, k_pool, v_pool, q_norm, k_norm, talk, cos_t, sin_t, tok_seq, tok_pos, page_start, page_ids, *,
@@ -1652,7 +1652,7 @@ def mixed_prep(qkv, q_out, k_pool, v_pool, q_norm, k_norm, talk, cos_t, sin_t, t
             raise KernelError("rope tables must be [tokens, rot_dim / 2]")
     args = _MixedPrepArgs(_ptr(qkv), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(q_norm), _ptr(k_norm), _ptr(talk),
                           _ptr(cos_t), _ptr(sin_t), _ptr(tok_seq), _ptr(tok_pos), _ptr(page_start), _ptr(page_ids), n, nq, nkv,
-                          d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, 1 if write_kv else 0, eps, 0)
+                          d, dv, lanes, v_lanes, rot_dim, page_size, ring_pages, 1 if write_kv else 0, eps, 0, 0)
     lib = load_library("mixed")
     _check(lib.odi_mixed_prep(byref(args), c_int(dtype_code(qkv.dtype)), _stream()), "mixed_prep")
 
