@@ -429,24 +429,27 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         for (int kb = 0; kb < KB; ++kb)
           tma_load_2d(smem_u32(q_smem + t * Q_TILE + kb * QROWS * 128), &map_q, (head0 * KH + t) * D + kb * 64, q_begin + t0, q_full);
       bool ok = true;
-      // box n of a ring of `slots` slots: head `h` of page j
-      auto load_box = [&](int n, int slots, int j, int h, const CUtensorMap* map, uint8_t* ring, uint32_t full, uint32_t empty) {
+      // where page j of the walk lies (looked up once a page: this one thread requests everything)
+      auto page_of = [&](int j) { return pages[page_slot_of_page(tile_of(j), a.ring_pages)]; };
+      int key_page = page_of(0);
+      // box n of a ring of `slots` slots: head `h` of `page`
+      auto load_box = [&](int n, int slots, int page, int h, const CUtensorMap* map, uint8_t* ring, uint32_t full, uint32_t empty) {
         const int s = n % slots;
         if (!mbar_wait(empty + 8 * s, ((uint32_t)(n / slots) & 1u) ^ 1u, abort_ptr)) { ok = false; return; }
-        const int entry = page_slot_of_page(tile_of(j), a.ring_pages);
-        const int row = (pages[entry] * a.nkv + h) * BNK;
+        const int row = (page * a.nkv + h) * BNK;
         mbar_expect_tx(full + 8 * s, KV_BYTES);
         for (int kb = 0; kb < KB; ++kb)
           tma_load_2d(smem_u32(ring + (size_t)s * KV_BYTES + kb * BNK * 128), map, kb * 64, row, full + 8 * s);
       };
       auto load_keys = [&](int j) {
-        for (int g = 0; g < KH && ok; ++g) load_box(j * KH + g, KRING, j, MIXED ? g : hk, &map_k, k_smem, k_full, k_empty);
+        for (int g = 0; g < KH && ok; ++g) load_box(j * KH + g, KRING, key_page, MIXED ? g : hk, &map_k, k_smem, k_full, k_empty);
       };
       // keys run one page ahead of values: a K slot is free as soon as its scores are computed
       load_keys(0);
       for (int j = 1; j <= n_tiles && ok; ++j) {
-        if (j < n_tiles) load_keys(j);
-        if (ok) load_box(j - 1, RING, j - 1, hk, &map_v, v_smem, v_full, v_empty);
+        const int value_page = key_page;
+        if (j < n_tiles) { key_page = page_of(j); load_keys(j); }
+        if (ok) load_box(j - 1, RING, value_page, hk, &map_v, v_smem, v_full, v_empty);
       }
       if (!ok) atomicCAS(a.status, 0, ATT_ERR_PRODUCER);
     }
