@@ -615,12 +615,23 @@ static int launch_rule(const HeadDeltaArgs& a, cudaStream_t stream) {
   return launch_pdl(kernel, grid, dim3(COLS / HD_CPT * RS), smem, stream, a, vec);
 }
 
-// DP rows: a lane takes 16 of a column's rows and a block 32 columns when that makes two blocks per multiprocessor; a
-// step of one long sequence has nothing else to run beside it, so there a lane takes 8 rows and a block 16 columns.
+// DP rows.  A lane takes 16 of a column's rows and a block 32 columns when that makes two blocks per multiprocessor.  A
+// step of one long sequence has nothing else to run beside it, and its time is its tokens' chain of instructions: there
+// a lane takes 8 rows and a block 16 columns, and when such blocks leave multiprocessors idle 4 rows (and 8 columns).
+// Measured, 2,048 tokens of one sequence, heads of 128 x 128, the whole mixer between its products, us: 16 heads 531 with 8
+// rows, 473 with 4; 32 heads 696 and 724; 8 heads 518, 457, and 405 with 8 columns
+// (heads of 64 x 64 lose with 8 columns: 419 and 473).
 template <int DP, int TCH>
 static int launch_rule_form(const HeadDeltaArgs& a, cudaStream_t stream) {
-  const bool narrow = (long)a.heads * a.n_seqs * ((a.dv + 31) / 32) < 2 * 148;
-  constexpr int WIDE = DP / 16, NARROW = DP / 8;
+  const long heads = (long)a.heads * a.n_seqs;
+  const bool narrow = heads * ((a.dv + 31) / 32) < 2 * 148, few = heads * ((a.dv + 15) / 16) <= 148;
+  constexpr int WIDE = DP / 16, NARROW = DP / 8, NARROWEST = DP / 4;
+  if constexpr (NARROWEST == 32) {
+    if (narrow && few && heads * ((a.dv + 7) / 8) <= 148) return launch_rule<NARROWEST, 4, 8, TCH>(a, stream);
+  }
+  if constexpr (NARROWEST <= 32 && NARROWEST >= 4) {
+    if (narrow && few) return launch_rule<NARROWEST, 4, 16, TCH>(a, stream);
+  }
   if constexpr (NARROW <= 32 && NARROW >= 4) {
     if (narrow) return launch_rule<NARROW, 8, 16, TCH>(a, stream);
   }

@@ -342,7 +342,9 @@ def test_widths_that_the_tensor_core_forms_refuse():
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("heads,kv_heads,d,dv,taps", [(4, 2, 32, 48, 3), (3, 1, 10, 7, 1), (6, 3, 24, 40, 4), (2, 2, 64, 33, 2), (4, 1, 128, 64, 4),
-                                                      (1, 1, 130, 5, 16), (2, 1, 300, 16, 2), (2, 2, 16, 128, 5)])
+                                                      (1, 1, 130, 5, 16), (2, 1, 300, 16, 2), (2, 2, 16, 128, 5),
+                                                      (10, 5, 128, 96, 3), (12, 4, 60, 130, 2), (40, 8, 120, 64, 2), (30, 30, 20, 90, 3),
+                                                      (40, 4, 250, 64, 2)])
 def test_delta_rule_over_cut_sequences(dtype, heads, kv_heads, d, dv, taps):
     """Three sequences cut into unequal runs (one token, fewer tokens than taps, groups of four with and without tokens
     left over, more than a staged chunk), stepped together with the state carried in slots of their own, against the
