@@ -40,6 +40,21 @@ class RMSNormSpec:
 
 
 @dataclass(frozen=True)
+class LayerNormSpec:
+    """y = cast((x - mean) / sqrt(var + eps) * weight + bias), var the mean of the squared deviations; everything in
+    fp32 with one rounding at the end.  ``streams`` s > 1: the rows given to the norm hold s parallel streams of
+    ``size`` lanes side by side, which it sums first.  ``output_scale``: one more factor of the whole row, taken into
+    weight and bias in fp32 at load (a final norm with it scales the logits)."""
+
+    size: int
+    eps: float
+    weight_name: str
+    bias_name: str
+    streams: int = 1
+    output_scale: float = 1.0
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotary position encoding over the first ``rotary_dim`` lanes of a head: lane i turns with lane
     i + rotary_dim / 2 (half-split), or, with ``interleaved``, lane 2i with lane 2i + 1; the angle of pair i at
@@ -50,7 +65,8 @@ class RotarySpec:
     n(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta) the index of the pair that makes t turns over
     ``original`` positions, lo = max(floor(n(fast)), 0), hi = min(ceil(n(slow)), rotary_dim - 1) and
     s_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency is s_i f_i / factor + (1 - s_i) f_i, and cos and
-    sin are both multiplied by 0.1 ln(factor) + 1."""
+    sin are both multiplied by 0.1 ln(factor) + 1.
+    ``linear_factor``: every frequency is divided by it (and all of them are made in double from theta)."""
 
     head_dim: int
     theta: float
@@ -58,6 +74,7 @@ class RotarySpec:
     interleaved: bool = False
     scaling: Optional[Tuple[float, float, float, float]] = None
     index_ramp: Optional[Tuple[float, float, float, float]] = None
+    linear_factor: Optional[float] = None
 
     @property
     def dim(self) -> int:
@@ -112,8 +129,15 @@ class CappedAttentionSpec:
     (``value_dim`` == ``head_dim``).
     ``keep_first`` k > 0 (with a window): keys 0..k-1 of a sequence stay visible beyond the window, at their true
     positions: position p sees j <= p with p - j < w or j < k.
-    ``names`` maps the roles q, k, v, o to tensor names below ``prefix``; when it also names q_bias or k_bias, that
-    projection adds the [out] bias of that name; when it names q_norm and k_norm (with ``unit_norm_eps``), every
+    ``q_temperature`` = (coef, every): after norm and rotation the query at position p is multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1).
+    ``bias_rows`` B > 0: rel[bucket(p - j), head] is added to the score (after scale and cap), rel the stored
+    [B, heads] table of the role rel: bucket(n) = n for n < B / 2, else
+    min(B - 1, B / 2 + floor(ln(n / (B / 2)) / ln(``bias_reach`` / (B / 2)) (B - B / 2))).
+    ``gate`` "head" or "lane": the attention's output is multiplied by sigmoid(W_g x) (role g) before the output
+    projection, one number per head resp. per lane of the heads.
+    ``names`` maps the roles q, k, v, o to tensor names below ``prefix``; when it also names q_bias, k_bias or v_bias,
+    that projection adds the [out] bias of that name; when it names q_norm and k_norm (with ``unit_norm_eps``), every
     query resp. key head is multiplied, after the division, by that [head_dim] weight, which the heads share (an RMS
     norm per head with a plain weight)."""
 
@@ -132,6 +156,10 @@ class CappedAttentionSpec:
     sink: bool = False
     values_are_keys: bool = False
     keep_first: int = 0
+    q_temperature: Optional[Tuple[float, int]] = None
+    bias_rows: int = 0
+    bias_reach: float = 0.0
+    gate: Optional[str] = None
 
     def name(self, role: str) -> str:
         return self.prefix + dict(self.names)[role]
@@ -335,7 +363,8 @@ class TableExpertsSpec:
 
 @dataclass(frozen=True)
 class MLPSpec:
-    """Dense feed-forward without a gate: down(act(up(x))), no biases; ``activation`` "gelu_erf" or "gelu_tanh"."""
+    """Dense feed-forward without a gate: down(act(up(x))), no biases; ``activation`` "gelu_erf", "gelu_tanh" or
+    "relu2" (the square of max(x, 0))."""
 
     hidden_size: int
     intermediate_size: int
@@ -408,6 +437,31 @@ class StateSpaceSpec:
     norm_eps: float
     prefix: str
     names: Tuple[Tuple[str, str], ...]
+
+    def name(self, role: str) -> str:
+        return self.prefix + dict(self.names)[role]
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """Linear attention with a fixed decay per head (a recurrent mixer with a matrix state per head).
+
+    q = W_q x and k = W_k x (``num_heads`` heads of ``qk_dim`` lanes) are rotated by ``position`` (half-split or
+    neighbouring pairs), k is then multiplied by qk_dim^-1/2; v = W_v x (heads of ``v_dim``).  Per head and token:
+    S <- ``decay``_h S + k v^T; o = S^T q.  With ``norm_eps`` not None every head's o is divided by
+    sqrt(mean of its squares + eps).  The heads side by side are multiplied by silu(W_g x) and projected by o.  The
+    state is fp32 and carried from token to token; so is everything between the projections.  ``names`` maps the
+    roles q, k, v, g, o to tensor names below ``prefix``."""
+
+    hidden_size: int
+    num_heads: int
+    qk_dim: int
+    v_dim: int
+    decay: Tuple[float, ...]
+    position: object
+    prefix: str
+    names: Tuple[Tuple[str, str], ...]
+    norm_eps: Optional[float] = None
 
     def name(self, role: str) -> str:
         return self.prefix + dict(self.names)[role]
@@ -539,6 +593,27 @@ class ScaledParallelBlockSpec:
 
 
 @dataclass(frozen=True)
+class StreamMixBlockSpec:
+    """Several parallel residual streams that every sublayer reads as a weighted sum and mixes anew (hyper-connections):
+    u = sum_s in[s] x_s; y = sublayer(norm(u)); then, all streams at once from the old ones,
+    x_t <- sum_s mix[s, t] x_s + ``residual_mult`` * out[t] * y; once for the mixer and once for the feed-forward.  The
+    stream tensor is [tokens, ``streams`` * hidden], streams side by side.  ``mixer_names`` and ``ffn_names`` are the
+    tensor names (in, out, mix) with shapes [streams], [streams], [streams, streams] ([from, to]); None stands for
+    the plain residual sum x <- x + ``residual_mult`` * y of one stream (in, out and mix all one).  ``ffn`` None (with
+    its norm and names): the layer has no feed-forward.  Norms and streams are fp32."""
+
+    mixer_norm: object
+    mixer: object
+    ffn_norm: object
+    ffn: object
+    hidden_size: int
+    streams: int = 1
+    residual_mult: float = 1.0
+    mixer_names: Optional[Tuple[str, str, str]] = None
+    ffn_names: Optional[Tuple[str, str, str]] = None
+
+
+@dataclass(frozen=True)
 class ReinjectSpec:
     """A step between layers that keeps no cache: h <- W [h ; e] + steps[index], with e the output of the
     embedding, W [hidden, 2 hidden] (the columns of h first) and ``steps`` [``num_steps``, hidden].  It opens a
@@ -569,7 +644,8 @@ class OrderEntry:
 class EmbeddingSpec:
     """Token embedding: hidden[t] = table[token[t]] * ``scale``; with ``sinusoid_base`` b an absolute position
     vector is added, entry 2i = sin(p b^(-2i / hidden_size)), entry 2i + 1 = the cosine of the same angle, p the
-    token's position in its sequence (fp32); with ``norm`` (a norm spec) the rows then pass that norm, in fp32."""
+    token's position in its sequence (fp32); with ``norm`` (a norm spec) the rows then pass that norm, in fp32.
+    ``streams`` s > 1: a token's row is written s times side by side (the parallel streams all start equal)."""
 
     vocab_size: int
     hidden_size: int
@@ -577,6 +653,7 @@ class EmbeddingSpec:
     norm: object = None
     scale: float = 1.0
     sinusoid_base: Optional[float] = None
+    streams: int = 1
 
 
 @dataclass(frozen=True)

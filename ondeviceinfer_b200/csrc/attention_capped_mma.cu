@@ -9,9 +9,11 @@
 //
 //   score = q . k * scale;  with softcap c > 0: score <- c tanh(score / c);  with sink = 1 the softmax has one more
 //   term, of score 0 and without a value: p_j = e^(s_j) / (1 + sum_k e^(s_k));
+//   with a distance bias its entry for p - j is added behind scale and cap;
 //   key j is visible to the query at position p iff j <= p and (window == 0 or j > p - window or j < keep): with
 //   keep > 0 a windowed layer goes on seeing the first `keep` positions of its sequence; their tiles come first in
 //   a block's walk, then the tiles of the window.
+// The finished heads may go to rows of their own width, times a constant and a gate (HeadOut).
 //
 // Key and value tiles (64 positions x D resp. DV bf16, contiguous in a page) are copied with cp.async, double
 // buffered, one block barrier per tile, into rows padded by 16 bytes so that ldmatrix reads are free of bank
@@ -54,7 +56,16 @@ struct CappedAttnArgs {
   float scale, softcap;
   int sink;               // 1: the softmax has one more term, of score 0 and without a value
   int keep;               // > 0 with a window: keys 0..keep-1 stay visible beyond the window
+  HeadOut ho;
+  DistanceBias rel;
+  int rel_staged;         // 1: the prompt kernel keeps its head's biases in shared memory (set by the launcher)
 };
+
+// A head's biases in shared memory, in log2 units: entry REL_PAD + n is that of distance n, with REL_PAD copies of the last
+// one behind (keys up to a tile in front of the table's end) and as many entries in front, so that a tile's 64 distances are
+// read without clamping each.
+#define REL_PAD 64
+#define REL_STAGED_MAX 8192
 
 // 1 / (l + 2^-m) for row sums l taken relative to the maximum m (log2 domain): the denominator with the sink's
 // term, without overflow; zero for a row that saw no key.
@@ -111,6 +122,13 @@ __device__ __forceinline__ float shape_score(float s, float scale, float cap, fl
   return s * LOG2E;
 }
 
+// The factor of two neighbouring lanes of a finished head.
+__device__ __forceinline__ float2 out_factors(const HeadOut& o, size_t tok, int head, int lane) {
+  if (o.gate != nullptr && !o.gate_per_head) return make_float2(head_out_factor<bf16>(o, tok, head, DV, lane), head_out_factor<bf16>(o, tok, head, DV, lane + 1));
+  const float f = head_out_factor<bf16>(o, tok, head, DV, lane);
+  return make_float2(f, f);
+}
+
 __global__ void __launch_bounds__(WARPS * 32)
 attention_capped_kernel(CappedAttnArgs a) {
   pdl_launch_dependents();
@@ -156,6 +174,13 @@ attention_capped_kernel(CappedAttnArgs a) {
   for (int i = 0; i < DVTILES; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
   const float two_over_cap = a.softcap > 0.f ? 2.f / a.softcap : 0.f;
+  const float* rel_g = a.rel.table != nullptr ? a.rel.table + (size_t)head * a.rel.n : nullptr;
+  float* rel_s = (float*)(smem + STAGES * (K_BYTES + V_BYTES));
+  const bool has_rel = rel_g != nullptr;
+  const float rel_far = has_rel ? rel_g[a.rel.n - 1] * LOG2E : 0.f;
+  if (has_rel && a.rel_staged)          // the first tile's barrier orders these writes before the reads
+    for (int i = tid; i < a.rel.n + 2 * REL_PAD; i += WARPS * 32)
+      rel_s[i] = rel_g[min(max(i - REL_PAD, 0), a.rel.n - 1)] * LOG2E;
 
   auto issue = [&](int w) {
     uint8_t* st = smem + (size_t)(w % STAGES) * (K_BYTES + V_BYTES);
@@ -192,15 +217,49 @@ attention_capped_kernel(CappedAttnArgs a) {
           mma_bf16(s[np * 2 + 1], qf[ks], b2, b3);
         }
       }
-      // scale, cap, mask, running maximum (log2 domain)
+      // scale, cap, bias, mask, running maximum (log2 domain)
+      if (has_rel) {
+        const float pre = a.softcap > 0.f ? 1.f : a.scale;
+        if (a.softcap > 0.f) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[i][e] = a.softcap * (1.f - __fdividef(2.f, __expf(s[i][e] * a.scale * two_over_cap) + 1.f));
+        }
+        if (warp_first - (kbase + KT - 1) >= a.rel.n - 1) {          // every pair is beyond the table's last distance
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[i][e] = fmaf(s[i][e], pre * LOG2E, rel_far);
+        } else if (a.rel_staged) {
+          const int last = a.rel.n - 1 + REL_PAD, k0 = kbase + (lane & 3) * 2;
+          // distances of this lane's first key, no farther than the copies reach; those behind the diagonal are masked below
+          const float* b_lo = rel_s + REL_PAD + min(max(pos_lo - k0, 0), last - 1);
+          const float* b_hi = rel_s + REL_PAD + min(max(pos_hi - k0, 0), last - 1);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            s[i][0] = fmaf(s[i][0], pre * LOG2E, b_lo[-8 * i]); s[i][1] = fmaf(s[i][1], pre * LOG2E, b_lo[-8 * i - 1]);
+            s[i][2] = fmaf(s[i][2], pre * LOG2E, b_hi[-8 * i]); s[i][3] = fmaf(s[i][3], pre * LOG2E, b_hi[-8 * i - 1]);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int dist = (e < 2 ? pos_lo : pos_hi) - (kbase + i * 8 + (lane & 3) * 2 + (e & 1));
+              s[i][e] = fmaf(s[i][e], pre * LOG2E, rel_g[min(max(dist, 0), a.rel.n - 1)] * LOG2E);
+            }
+        }
+      }
+      auto shaped = [&](float x) { return has_rel ? x : shape_score(x, a.scale, a.softcap, two_over_cap); };
       float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int kj = kbase + i * 8 + (lane & 3) * 2;
-        s[i][0] = (kj <= pos_lo && (kj >= old_lo || kj < a.keep)) ? shape_score(s[i][0], a.scale, a.softcap, two_over_cap) : -INFINITY;
-        s[i][1] = (kj + 1 <= pos_lo && (kj + 1 >= old_lo || kj + 1 < a.keep)) ? shape_score(s[i][1], a.scale, a.softcap, two_over_cap) : -INFINITY;
-        s[i][2] = (kj <= pos_hi && (kj >= old_hi || kj < a.keep)) ? shape_score(s[i][2], a.scale, a.softcap, two_over_cap) : -INFINITY;
-        s[i][3] = (kj + 1 <= pos_hi && (kj + 1 >= old_hi || kj + 1 < a.keep)) ? shape_score(s[i][3], a.scale, a.softcap, two_over_cap) : -INFINITY;
+        s[i][0] = (kj <= pos_lo && (kj >= old_lo || kj < a.keep)) ? shaped(s[i][0]) : -INFINITY;
+        s[i][1] = (kj + 1 <= pos_lo && (kj + 1 >= old_lo || kj + 1 < a.keep)) ? shaped(s[i][1]) : -INFINITY;
+        s[i][2] = (kj <= pos_hi && (kj >= old_hi || kj < a.keep)) ? shaped(s[i][2]) : -INFINITY;
+        s[i][3] = (kj + 1 <= pos_hi && (kj + 1 >= old_hi || kj + 1 < a.keep)) ? shaped(s[i][3]) : -INFINITY;
         mx_lo = fmaxf(mx_lo, fmaxf(s[i][0], s[i][1]));
         mx_hi = fmaxf(mx_hi, fmaxf(s[i][2], s[i][3]));
       }
@@ -249,14 +308,22 @@ attention_capped_kernel(CappedAttnArgs a) {
   if (a.sink) { inv_lo = sink_inverse_log2(m_lo, l_lo); inv_hi = sink_inverse_log2(m_hi, l_hi); }
   const int c = (lane & 3) * 2;
   if (r_lo < nt) {
-    bf16* dst = a.out + ((size_t)(q_begin + t0 + r_lo) * a.nq + head) * DV;
+    const size_t tok = q_begin + t0 + r_lo;
+    bf16* dst = a.out + tok * a.ho.out_ld + head * DV;
 #pragma unroll
-    for (int i = 0; i < DVTILES; ++i) *(uint32_t*)(dst + i * 8 + c) = pack_bf16(o[i][0] * inv_lo, o[i][1] * inv_lo);
+    for (int i = 0; i < DVTILES; ++i) {
+      const float2 f = out_factors(a.ho, tok, head, i * 8 + c);
+      *(uint32_t*)(dst + i * 8 + c) = pack_bf16(o[i][0] * inv_lo * f.x, o[i][1] * inv_lo * f.y);
+    }
   }
   if (r_hi < nt) {
-    bf16* dst = a.out + ((size_t)(q_begin + t0 + r_hi) * a.nq + head) * DV;
+    const size_t tok = q_begin + t0 + r_hi;
+    bf16* dst = a.out + tok * a.ho.out_ld + head * DV;
 #pragma unroll
-    for (int i = 0; i < DVTILES; ++i) *(uint32_t*)(dst + i * 8 + c) = pack_bf16(o[i][2] * inv_hi, o[i][3] * inv_hi);
+    for (int i = 0; i < DVTILES; ++i) {
+      const float2 f = out_factors(a.ho, tok, head, i * 8 + c);
+      *(uint32_t*)(dst + i * 8 + c) = pack_bf16(o[i][2] * inv_hi * f.x, o[i][3] * inv_hi * f.y);
+    }
   }
 }
 
@@ -327,6 +394,10 @@ attention_capped_decode_kernel(CappedDecodeArgs da) {
   for (int i = 0; i < DVTILES; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
   const float two_over_cap = a.softcap > 0.f ? 2.f / a.softcap : 0.f;
+  const bool has_rel = a.rel.table != nullptr;
+  const float* rel_lo = has_rel && r_lo < heads_here ? a.rel.table + (size_t)(head0 + r_lo) * a.rel.n : nullptr;
+  const float* rel_hi = has_rel && r_hi < heads_here ? a.rel.table + (size_t)(head0 + r_hi) * a.rel.n : nullptr;
+  const float far_lo = rel_lo ? rel_lo[a.rel.n - 1] : 0.f, far_hi = rel_hi ? rel_hi[a.rel.n - 1] : 0.f;
 
   auto issue = [&](int tile) {
     uint8_t* st = smem + (size_t)((tile - tile_begin) % STAGES) * (K_BYTES + V_BYTES);
@@ -363,6 +434,17 @@ attention_capped_decode_kernel(CappedDecodeArgs da) {
         s[i][1] = v1 ? shape_score(s[i][1], a.scale, a.softcap, two_over_cap) : -INFINITY;
         s[i][2] = v0 ? shape_score(s[i][2], a.scale, a.softcap, two_over_cap) : -INFINITY;
         s[i][3] = v1 ? shape_score(s[i][3], a.scale, a.softcap, two_over_cap) : -INFINITY;
+        if (has_rel) {
+          const int n0 = pos - kj, end = a.rel.n - 1;
+          float b[4] = {far_lo, far_lo, far_hi, far_hi};
+          if (n0 - 1 < end) {
+            const int i0 = min(max(n0, 0), end), i1 = min(max(n0 - 1, 0), end);
+            if (rel_lo) { b[0] = rel_lo[i0]; b[1] = rel_lo[i1]; }
+            if (rel_hi) { b[2] = rel_hi[i0]; b[3] = rel_hi[i1]; }
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[i][e] = fmaf(b[e], LOG2E, s[i][e]);
+        }
         mx_lo = fmaxf(mx_lo, fmaxf(s[i][0], s[i][1]));
         mx_hi = fmaxf(mx_hi, fmaxf(s[i][2], s[i][3]));
       }
@@ -429,12 +511,12 @@ attention_capped_decode_kernel(CappedDecodeArgs da) {
     if (da.splits == 1) {
       float inv = L > 0.f ? 1.f / L : 0.f;
       if (a.sink) inv = sink_inverse_log2(M, L);
-      bf16* dst = a.out + ((size_t)tok * a.nq + head) * DV;
+      bf16* dst = a.out + (size_t)tok * a.ho.out_ld + head * DV;
       for (int dd = lane; dd < DV; dd += 32) {
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < WARPS; ++w) v += wgt[w] * mg[((size_t)w * 16 + row) * RS + dd];
-        dst[dd] = __float2bfloat16_rn(v * inv);
+        dst[dd] = __float2bfloat16_rn(v * inv * head_out_factor<bf16>(a.ho, tok, head, DV, dd));
       }
     } else {
       // partial in the natural-log domain of the combine kernel: max * ln 2
@@ -452,7 +534,7 @@ attention_capped_decode_kernel(CappedDecodeArgs da) {
 
 // Merge the partials of one (token, head): out = sum_s e^(m_s - M) acc_s / sum_s e^(m_s - M) l_s, splits in order.
 __global__ void attention_capped_combine_kernel(const float* __restrict__ partial, bf16* __restrict__ out, int splits,
-                                                int sink) {
+                                                int sink, int nq, HeadOut ho) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int RS = DV + 2;
@@ -473,7 +555,9 @@ __global__ void attention_capped_combine_kernel(const float* __restrict__ partia
       const float ms = p[s * RS + DV];
       if (ms != -INFINITY) v += expf(ms - M) * p[s * RS + dd];
     }
-    out[row * DV + dd] = __float2bfloat16_rn(v * inv);
+    const size_t tok = row / nq;
+    const int h = (int)(row % nq);
+    out[tok * ho.out_ld + h * DV + dd] = __float2bfloat16_rn(v * inv * head_out_factor<bf16>(ho, tok, h, DV, dd));
   }
 }
 
@@ -484,7 +568,7 @@ extern "C" int odi_attention_capped_decode(const CappedAttnArgs* args, float* pa
   const CappedAttnArgs& a = da.base;
   if (a.n_seqs <= 0) return 0;
   if (a.nkv <= 0 || a.nq % a.nkv != 0 || a.n_seqs > 65535 || a.window < 0 || a.ring_pages < 0 || a.keep < 0 || splits < 1) return ODI_ERR_UNSUPPORTED;
-  if (((uintptr_t)a.q | (uintptr_t)a.k_pool | (uintptr_t)a.v_pool | (uintptr_t)a.out) % 16 != 0) return ODI_ERR_UNSUPPORTED;
+  if (((uintptr_t)a.q | (uintptr_t)a.k_pool | (uintptr_t)a.v_pool) % 16 != 0) return ODI_ERR_UNSUPPORTED;
   if (splits > 1 && partial == nullptr) return ODI_ERR_ARGUMENT;
   da.partial = partial;
   da.splits = splits;
@@ -503,7 +587,7 @@ extern "C" int odi_attention_capped_decode(const CappedAttnArgs* args, float* pa
   if (rc != 0 || splits == 1) return rc;
   const int rows = a.n_seqs * a.nq;
   const int threads = DV >= 128 ? 128 : (DV >= 64 ? 64 : 32);
-  odi_rc = launch_pdl(attention_capped_combine_kernel, dim3(rows), dim3(threads), 0, stream, (const float*)partial, a.out, splits, a.sink);
+  odi_rc = launch_pdl(attention_capped_combine_kernel, dim3(rows), dim3(threads), 0, stream, (const float*)partial, a.out, splits, a.sink, a.nq, a.ho);
   return launch_status();
 }
 
@@ -511,18 +595,21 @@ extern "C" int odi_attention_capped_dims(int* d, int* dv) { *d = D; *dv = DV; re
 
 // max_q_len: the longest q_len of the batch (sizes the grid).
 extern "C" int odi_attention_capped(const CappedAttnArgs* args, int max_q_len, cudaStream_t stream) {
-  const CappedAttnArgs a = *args;
+  CappedAttnArgs a = *args;
   if (a.n_seqs <= 0 || max_q_len <= 0) return 0;
   if (a.nkv <= 0 || a.nq % a.nkv != 0 || a.n_seqs > 65535 || a.window < 0 || a.ring_pages < 0 || a.keep < 0) return ODI_ERR_UNSUPPORTED;
-  if (((uintptr_t)a.q | (uintptr_t)a.k_pool | (uintptr_t)a.v_pool | (uintptr_t)a.out) % 16 != 0) return ODI_ERR_UNSUPPORTED;
+  if (((uintptr_t)a.q | (uintptr_t)a.k_pool | (uintptr_t)a.v_pool) % 16 != 0 || (uintptr_t)a.out % 4 != 0 || a.ho.out_ld % 2 != 0) return ODI_ERR_UNSUPPORTED;
   const int q_tiles = (max_q_len + 63) / 64;
   if (q_tiles > 65535) return ODI_ERR_UNSUPPORTED;
-  const size_t smem = (size_t)STAGES * (K_BYTES + V_BYTES);
-  static bool configured = false;
-  if (!configured) {
+  size_t smem = (size_t)STAGES * (K_BYTES + V_BYTES);
+  const size_t rel_bytes = sizeof(float) * ((size_t)a.rel.n + 2 * REL_PAD);
+  a.rel_staged = a.rel.table != nullptr && a.rel.n <= REL_STAGED_MAX && smem + rel_bytes <= 227 * 1024;
+  if (a.rel_staged) smem += rel_bytes;
+  static size_t configured = 0;
+  if (configured < smem) {
     const cudaError_t e = cudaFuncSetAttribute(attention_capped_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    configured = true;
+    configured = smem;
   }
   odi_rc = launch_pdl(attention_capped_kernel, dim3(a.nq, a.n_seqs, q_tiles), dim3(WARPS * 32), smem, stream, a);
   return launch_status();

@@ -17,6 +17,8 @@
 // With mixed = 1 a query head has nkv * D lanes, one query of D lanes for every key head, and its score is the sum of
 // their dot products with all key heads of the position (heads that mix their scores; the values stay grouped).
 // With softcap c > 0 a score s (already times scale) becomes c tanh(s / c) before the softmax.
+// With a distance bias its entry for the key's distance is added to the score behind scale and cap.  The output may go to
+// rows of its own width, times a constant and a gate (HeadOut).
 // With sink = 1 the softmax has one more term, of score 0 and without a value: p_j = e^(s_j) / (1 + sum e^(s_k)).
 //
 // With splits > 1 every split writes an un-normalised partial (acc[d], max, sum) and
@@ -65,6 +67,8 @@ struct AttnArgs {
   int keep;             // > 0 with a window: keys 0..keep-1 stay visible beyond the window
   int chunk;            // > 0: keys of the query's own chunk of this many positions
   int mixed;            // 1: q is [n_tokens, nq, nkv, D]; a score sums over the key heads
+  HeadOut ho;
+  DistanceBias rel;
 };
 
 // 1 / (l + e^-m) for sums l taken relative to the maximum m: the denominator with the sink's term, without overflow.
@@ -128,12 +132,14 @@ attention_simt_kernel(AttnArgs a) {
 
   float m[RW], l[RW], acc[RW][NACC];
   int rpos[RW], rold[RW];       // position of the row's query, and the oldest key of its window or chunk
+  const float* rrel[RW];        // the row's head in the table of distance biases
 #pragma unroll
   for (int r = 0; r < RW; ++r) {
     m[r] = -INFINITY; l[r] = 0.f;
     const int row = warp * RW + r;
     rpos[r] = row < nrows ? past + t0 + row / hpb : -1;
     rold[r] = a.window > 0 ? rpos[r] - a.window + 1 : (a.chunk > 0 && rpos[r] >= 0 ? rpos[r] - rpos[r] % a.chunk : 0);
+    rrel[r] = a.rel.table != nullptr && row < nrows ? a.rel.table + (size_t)(hk * g + chunk * 16 + row % hpb) * a.rel.n : nullptr;
 #pragma unroll
     for (int i = 0; i < NACC; ++i) acc[r][i] = 0.f;
   }
@@ -210,6 +216,7 @@ attention_simt_kernel(AttnArgs a) {
       const bool vis = rpos[r] >= 0 && kj <= rpos[r] && (kj >= rold[r] || kj < a.keep);
       float sc = s[r] * a.scale;
       if (a.softcap > 0.f) sc = a.softcap * tanhf(sc / a.softcap);
+      if (vis && rrel[r] != nullptr) sc += rrel[r][min(rpos[r] - kj, a.rel.n - 1)];
       if (!vis) sc = -INFINITY;
       const float mx = warp_max(sc);
       const float m_new = fmaxf(m[r], mx);
@@ -257,11 +264,11 @@ attention_simt_kernel(AttnArgs a) {
     if (a.splits == 1) {
       float inv = l[r] > 0.f ? 1.f / l[r] : 0.f;
       if (a.sink) inv = sink_inverse(m[r], l[r]);
-      T* o = (T*)a.out + ((size_t)tok * a.nq + h) * DV;
+      T* o = (T*)a.out + (size_t)tok * a.ho.out_ld + h * DV;
 #pragma unroll
       for (int i = 0; i < NACC; ++i) {
         const int dd = lane + 32 * i;
-        if (dd < DV) o[dd] = from_f<T>(acc[r][i] * inv);
+        if (dd < DV) o[dd] = from_f<T>(acc[r][i] * inv * head_out_factor<T>(a.ho, tok, h, DV, dd));
       }
     } else {
       float* o = a.partial + (((size_t)tok * a.nq + h) * a.splits + split) * (DV + 2);
@@ -277,7 +284,7 @@ attention_simt_kernel(AttnArgs a) {
 
 // Merge the partials of one (token, head): out = sum_s e^(m_s - M) acc_s / sum_s e^(m_s - M) l_s.
 template <typename T>
-__global__ void attention_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, int splits, int sink) {
+__global__ void attention_combine_kernel(const float* __restrict__ partial, T* __restrict__ out, int splits, int sink, int nq, HeadOut ho) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t row = blockIdx.x;  // token * nq + head
@@ -297,7 +304,9 @@ __global__ void attention_combine_kernel(const float* __restrict__ partial, T* _
       const float ms = p[s * (DV + 2) + DV];
       if (ms != -INFINITY) v += expf(ms - M) * p[s * (DV + 2) + dd];
     }
-    out[row * DV + dd] = from_f<T>(v * inv);
+    const size_t tok = row / nq;
+    const int h = (int)(row % nq);
+    out[tok * ho.out_ld + h * DV + dd] = from_f<T>(v * inv * head_out_factor<T>(ho, tok, h, DV, dd));
   }
 }
 
@@ -337,7 +346,7 @@ extern "C" int odi_attention_simt(const AttnArgs* args, int max_q_len, int n_tok
   if (rc != 0 || a.splits == 1) return rc;
   const int rows = n_tokens * a.nq;
   const int threads = DV >= 128 ? 128 : (DV >= 64 ? 64 : 32);
-  if (dtype == 0) odi_rc = launch_pdl((attention_combine_kernel<float>), dim3(rows), dim3(threads), 0, stream, a.partial, (float*)a.out, a.splits, a.sink);
-  else odi_rc = launch_pdl((attention_combine_kernel<bf16>), dim3(rows), dim3(threads), 0, stream, a.partial, (bf16*)a.out, a.splits, a.sink);
+  if (dtype == 0) odi_rc = launch_pdl((attention_combine_kernel<float>), dim3(rows), dim3(threads), 0, stream, a.partial, (float*)a.out, a.splits, a.sink, a.nq, a.ho);
+  else odi_rc = launch_pdl((attention_combine_kernel<bf16>), dim3(rows), dim3(threads), 0, stream, a.partial, (bf16*)a.out, a.splits, a.sink, a.nq, a.ho);
   return launch_status();
 }

@@ -46,7 +46,10 @@
 // key head, so a page's key heads pass one after the other through a ring of their own (KRING slots) while the CTA's
 // query rows of all key heads stay in shared memory.  When shared memory does not hold 128 rows of all key heads a CTA
 // takes 64 (QROWS): the products keep their 128 lanes, of which the upper half reads whatever lies behind the 64 rows and
-// is never looked at (lanes of a product do not mix), and two of the four softmax warps have nothing to do.  Compile with -DODI_HEAD_DIM=64 or 128.
+// is never looked at (lanes of a product do not mix), and two of the four softmax warps have nothing to do.  A learned bias by
+// distance (DistanceBias) is added to the scores behind scale and cap; the head's table lies in shared memory, with copies
+// of its last entry behind it so that a row reads a tile's 64 distances without clamping each.  The finished heads may go
+// to rows of their own width, times a constant and a gate (HeadOut).  Compile with -DODI_HEAD_DIM=64 or 128.
 //
 // Every wait on an mbarrier is bounded (about two seconds of SM clock): a role that gives up
 // records a code in `status`, raises the CTA's abort flag, and all roles fall through to the
@@ -101,7 +104,11 @@ struct TcAttnArgs {
   int keep;               // > 0 with a window: keys 0..keep-1 stay visible beyond the window; their tiles come first in the walk
   int chunk;              // > 0: keys of the query's own chunk of this many positions
   int mixed;              // 1: a score sums over the key heads (q has nkv rows of D lanes a head)
+  HeadOut ho;
+  DistanceBias rel;       // with one head per CTA
 };
+
+#define REL_PAD 64        // entries in front of and behind a head's biases in shared memory
 
 // ------------------------------------------------------------------------------ PTX wrappers
 
@@ -277,12 +284,26 @@ struct RowState { float m_used, l; };
 __device__ __forceinline__ bool softmax_keys64(uint32_t s_addr, uint32_t p_addr, uint32_t o_addr, int kbase, int pos, float sl2,
                                                int n, uint32_t pv_done, RowState& st, volatile int* abort_ptr,
                                                int oldest = 0, float scale = 1.f, float cap = 0.f, float two_over_cap = 0.f,
-                                               int keep = 0) {
+                                               int keep = 0, const float* rel = nullptr, int rel_n = 0) {
   float s[BNK];
   tmem_ld64(s_addr, s);
   if (cap > 0.f) {
 #pragma unroll
     for (int i = 0; i < BNK; ++i) s[i] = cap * (1.f - __fdividef(2.f, __expf(s[i] * scale * two_over_cap) + 1.f));
+  }
+  if (rel != nullptr) {
+    // entry REL_PAD + n of `rel` is the bias of distance n in log2 units; sl2 is 1, the scores' factor is `pre`
+    const float pre = cap > 0.f ? LOG2E : scale * LOG2E;
+    if (__all_sync(0xffffffffu, pos - (kbase + BNK - 1) >= rel_n - 1)) {
+      const float far = rel[REL_PAD + rel_n - 1];
+#pragma unroll
+      for (int i = 0; i < BNK; ++i) s[i] = fmaf(s[i], pre, far);
+    } else {
+      // keys behind the diagonal are masked below; farther than the copies reach every entry is the last one
+      const float* b = rel + REL_PAD + min(max(pos - kbase, 0), rel_n + REL_PAD - 2);
+#pragma unroll
+      for (int i = 0; i < BNK; ++i) s[i] = fmaf(s[i], pre, b[-i]);
+    }
   }
   float mx = -INFINITY;
   if (kbase + BNK - 1 <= pos && kbase >= oldest) {
@@ -339,8 +360,13 @@ __device__ __forceinline__ bool softmax_keys64(uint32_t s_addr, uint32_t p_addr,
 }
 
 // The finished row of O, divided by the row's sum, as bf16 to dst (D elements).
-__device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, bool valid) {
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+__device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, bool valid, const HeadOut& ho, size_t tok, int head) {
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  const bf16* gate = nullptr;              // a gate per lane: this head's lanes of the token's gate row
+  if (valid) {
+    if (ho.gate != nullptr && !ho.gate_per_head) { gate = (const bf16*)ho.gate + tok * ho.gate_ld + head * D; inv *= ho.scale; }
+    else inv *= head_out_factor<bf16>(ho, tok, head, D, 0);
+  }
 #pragma unroll 1
   for (int c = 0; c < D; c += 32) {
     float v[32];
@@ -349,6 +375,16 @@ __device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, b
 #pragma unroll
       for (int i = 0; i < 32; i += 8) {
         uint32_t w[4];
+        if (gate != nullptr) {
+          const uint4 raw = *(const uint4*)(gate + c + i);
+          const __nv_bfloat162* z = (const __nv_bfloat162*)&raw;
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float2 f = __bfloat1622float2(z[k]);
+            v[i + 2 * k] /= 1.f + __expf(-f.x);
+            v[i + 2 * k + 1] /= 1.f + __expf(-f.y);
+          }
+        }
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
           __nv_bfloat162 pr = __floats2bfloat162_rn(v[i + 2 * k] * inv, v[i + 2 * k + 1] * inv);
@@ -402,6 +438,12 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const int KH = MIXED ? a.nkv : 1;                          // key heads a score sums over
   uint8_t* k_smem = smem + TILES * KH * Q_TILE;              // ring of K pages
   uint8_t* v_smem = k_smem + KRING * KV_BYTES;            // ring of V pages
+  const bool has_rel = TILES == 1 && a.rel.table != nullptr;
+  float* rel_smem = (float*)(v_smem + RING * KV_BYTES);      // the head's biases by distance, in log2 units
+  if (has_rel) {
+    const float* src = a.rel.table + (size_t)head0 * a.rel.n;       // a weight: no earlier kernel writes it
+    for (int i = threadIdx.x; i < a.rel.n + 2 * REL_PAD; i += blockDim.x) rel_smem[i] = src[min(max(i - REL_PAD, 0), a.rel.n - 1)] * LOG2E;
+  }
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < BARS; ++i) mbar_init(bar0 + 8 * i, 1);
@@ -512,7 +554,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int row = lane_group * 32 + lane;          // query row inside the tile
     const int pos = past + t0 + row;
     const uint32_t lane_addr = (uint32_t)(lane_group * 32) << 16;
-    const float sl2 = a.softcap > 0.f ? LOG2E : a.scale * LOG2E;
+    const float sl2 = has_rel ? 1.f : (a.softcap > 0.f ? LOG2E : a.scale * LOG2E);
     const float two_over_cap = a.softcap > 0.f ? 2.f / a.softcap : 0.f;
     const int oldest = a.window > 0 ? pos - a.window + 1 : (a.chunk > 0 ? pos - pos % a.chunk : 0);
     // a sink is a key of score 0 and value 0 ahead of all others: the row starts from its maximum and its weight
@@ -528,7 +570,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       const uint32_t s_addr = tmem_base + lane_addr + S_COL(tile, b);
       // P_j goes over the first 32 columns of this row's scores
       if (!softmax_keys64(s_addr, s_addr, o_addr, tile_of(j) * BNK, pos, sl2, j, my_pv_done, st, abort_ptr, oldest, a.scale,
-                          a.softcap, two_over_cap, a.keep)) { ok = false; break; }
+                          a.softcap, two_over_cap, a.keep, has_rel ? rel_smem : nullptr, a.rel.n)) { ok = false; break; }
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(my_p_full + 8 * b);
@@ -536,7 +578,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     if (ok && !mbar_wait(my_pv_done, (uint32_t)(n_tiles - 1) & 1u, abort_ptr)) ok = false;
     tc_fence_after();
     if (!ok && lane == 0) atomicCAS(a.status, 0, ATT_ERR_SOFTMAX);
-    if (ok) write_row(o_addr, a.out + ((size_t)(q_begin + t0 + row) * a.nq + head) * D, st.l, row < nt);
+    if (ok) write_row(o_addr, a.out + (size_t)(q_begin + t0 + row) * a.ho.out_ld + head * D, st.l, row < nt, a.ho, q_begin + t0 + row, head);
     tc_fence_before();
   }
   __syncthreads();
@@ -589,12 +631,16 @@ static int mixed_rows(int nkv) {
 }
 extern "C" int odi_attention_tcgen05_mixed_rows(int nkv) { return mixed_rows(nkv); }
 
+// Entries of a head's table of biases by distance that shared memory holds beside everything else.
+extern "C" int odi_attention_tcgen05_bias_entries() { return (SMEM_LIMIT - (Q_BYTES + 2 * RING * KV_BYTES + 1024)) / 4 - 2 * REL_PAD; }
+
 // q [n_tokens, nq * D] bf16; k_pool, v_pool [pool_pages, nkv, 64, D] bf16; out [n_tokens, nq * D].
 // heads_per_cta: 2 = two heads of a key/value group per CTA (needs an even group size), 1 = one, 0 = choose.
 template <int TILES, bool MIXED, int QROWS = BM>
 static int launch_attention(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnArgs& a,
                             int max_q_len, cudaStream_t stream) {
-  const int smem = TILES * (MIXED ? a.nkv : 1) * (KB * QROWS * 128) + ((MIXED ? MIXED_KEY_RING : RING) + RING) * KV_BYTES + 1024;
+  const int smem = TILES * (MIXED ? a.nkv : 1) * (KB * QROWS * 128) + ((MIXED ? MIXED_KEY_RING : RING) + RING) * KV_BYTES + 1024 +
+                   (a.rel.table != nullptr ? (a.rel.n + 2 * REL_PAD) * 4 : 0);
   if (smem > SMEM_LIMIT) return ODI_ERR_UNSUPPORTED;
   auto kernel = attention_tcgen05_kernel<TILES, MIXED, QROWS>;
   static int configured = 0;
@@ -618,6 +664,10 @@ extern "C" int odi_attention_tcgen05(const void* q, const void* k_pool, const vo
     return ODI_ERR_UNSUPPORTED;
   if (pool_pages * a.nkv * BNK > 0x7fffffffL) return ODI_ERR_UNSUPPORTED;    // row coordinates are 32-bit
   if ((max_q_len + 63) / 64 > 65535) return ODI_ERR_UNSUPPORTED;
+  if (a.rel.table != nullptr && (a.rel.n < 1 || a.rel.n > odi_attention_tcgen05_bias_entries())) return ODI_ERR_UNSUPPORTED;
+  if (a.ho.out_ld % 8 != 0 || (a.ho.gate != nullptr && !a.ho.gate_per_head && (a.ho.gate_ld % 8 != 0 || ((uintptr_t)a.ho.gate & 15))))
+    return ODI_ERR_UNSUPPORTED;
+  if (a.rel.table != nullptr && heads_per_cta == 2) return ODI_ERR_UNSUPPORTED;
   if (heads_per_cta < 0 || heads_per_cta > 2 || a.chunk < 0 || (a.chunk > 0 && (a.window > 0 || a.keep > 0))) return ODI_ERR_ARGUMENT;
   if (a.mixed && heads_per_cta == 2) return ODI_ERR_UNSUPPORTED;
   if (heads_per_cta == 2 && (a.nq / a.nkv) % 2 != 0) return ODI_ERR_ARGUMENT;
@@ -628,7 +678,7 @@ extern "C" int odi_attention_tcgen05(const void* q, const void* k_pool, const vo
   if (rc == 0) rc = make_map(&mk, k_pool, pool_pages * a.nkv * BNK, D, BNK);
   if (rc == 0) rc = make_map(&mv, v_pool, pool_pages * a.nkv * BNK, D, BNK);
   if (rc != 0) return rc;
-  if (heads_per_cta == 0) heads_per_cta = ODI_ATT_DEFAULT_HEADS_PER_CTA;
+  if (heads_per_cta == 0) heads_per_cta = a.rel.table != nullptr ? 1 : ODI_ATT_DEFAULT_HEADS_PER_CTA;
   if (a.mixed)
     return q_rows == BM ? launch_attention<1, true>(mq, mk, mv, a, max_q_len, stream)
                         : launch_attention<1, true, 64>(mq, mk, mv, a, max_q_len, stream);

@@ -3,7 +3,7 @@
 //
 //  * rot_unit_prep: per (token, head) the rotation of neighbouring-lane pairs over the first rot_dim lanes, the
 //    division by sqrt(mean of squares + eps), optionally times a weight per lane (one for all query heads, one for
-//    all key heads), and the write of q to the query buffer, k and v to their cache pages (v has a width of its own);
+//    all key heads), the queries' factor 1 + coef ln(floor((p + 1) / every) + 1) at position p, and the write of q to the query buffer, k and v to their cache pages (v has a width of its own);
 //  * activation: out = act(x), act the exact (erf) GELU, its tanh form or the square of max(x, 0), fp32 arithmetic,
 //    one rounding;
 //  * gated_activation: out = act(gate) * up for rows of [gate | up], act one of the same forms;
@@ -16,7 +16,7 @@
 #include "common.cuh"
 
 struct RotUnitArgs {
-  const void* qkv;      // [n_tokens, nq * d + nkv * d + nkv * dv]
+  const void* qkv;      // [n_tokens, ld]: nq * d + nkv * d + nkv * dv lanes of every row
   void* q_out;          // [n_tokens, nq * d_store]
   void* k_pool;         // [pages, nkv, page_size, d_store]
   void* v_pool;         // [pages, nkv, page_size, dv]
@@ -32,7 +32,14 @@ struct RotUnitArgs {
   int v_from_k;         // 1: there are no v lanes in `qkv`; the value of a head is its key as projected, before the rotation (dv == d)
   const float* q_w;     // null, or [d]: after the division every query head is multiplied by it lane by lane
   const float* k_w;     // the same for the key heads
+  int ld;               // lanes of a row of `qkv`
+  float temp_coef;      // with temp_every > 0: queries are multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
+  int temp_every;
 };
+
+__device__ __forceinline__ float query_factor(const RotUnitArgs& a, int pos) {
+  return a.temp_every > 0 ? fmaf(a.temp_coef, logf((float)((pos + 1) / a.temp_every + 1)), 1.f) : 1.f;
+}
 
 // One warp per (token, head).  Lane i % 32 holds element i in register i / 32, so the partner of lane 2i
 // (lane 2i + 1) is the neighbouring lane of the same register.
@@ -46,7 +53,7 @@ __global__ void rot_unit_prep_kernel(RotUnitArgs a) {
   if (item >= (long)a.n_tokens * heads) return;
   const int t = (int)(item / heads), h = (int)(item % heads);
   const int d = a.d;
-  const size_t row = (size_t)(a.nq + a.nkv) * d + (a.v_from_k ? (size_t)0 : (size_t)a.nkv * a.dv);
+  const size_t row = a.ld;
   const int kind = h < a.nq ? 0 : (h < a.nq + a.nkv ? 1 : 2);  // 0 q, 1 k, 2 v
   const int pos = a.tok_pos[t];
   const T* src;
@@ -102,6 +109,11 @@ __global__ void rot_unit_prep_kernel(RotUnitArgs a) {
       x[r] *= (w != nullptr && i < d) ? inv * w[i] : inv;
     }
   }
+  if (kind == 0 && a.temp_every > 0) {
+    const float f = query_factor(a, pos);
+#pragma unroll
+    for (int r = 0; r < MAXP; ++r) x[r] *= f;
+  }
 #pragma unroll
   for (int r = 0; r < MAXP; ++r) {
     const int i = lane + 32 * r;
@@ -123,7 +135,7 @@ __global__ void rot_unit_prep_vec_kernel(RotUnitArgs a, int heads_per_warp) {
   if (item >= (long)a.n_tokens * groups) return;
   const int t = (int)(item / groups), h_begin = (int)(item % groups) * heads_per_warp;
   const int d = a.d, half = a.rot_dim >> 1;
-  const size_t row = (size_t)(a.nq + a.nkv) * d + (a.v_from_k ? (size_t)0 : (size_t)a.nkv * a.dv);
+  const size_t row = a.ld;
   const bf16* base = (const bf16*)a.qkv + (size_t)t * row;
   const int pos = a.tok_pos[t];
   size_t at = 0;
@@ -177,6 +189,7 @@ __global__ void rot_unit_prep_vec_kernel(RotUnitArgs a, int heads_per_warp) {
       inv = 1.0f / sqrtf(ss / (float)d + a.eps);
       w = kind == 0 ? a.q_w : a.k_w;
     }
+    if (kind == 0) inv *= query_factor(a, pos);
 #pragma unroll
     for (int r = 0; r < MAXP4; ++r) {
       const int i = 4 * lane + 128 * r;
@@ -196,10 +209,11 @@ extern "C" int odi_rot_unit_prep(const RotUnitArgs* args, int dtype, cudaStream_
   RotUnitArgs a = *args;
   if (a.n_tokens <= 0) return 0;
   if (a.v_from_k && a.dv != a.d) return ODI_ERR_ARGUMENT;
+  if (a.ld < (a.nq + a.nkv) * a.d + (a.v_from_k ? 0 : a.nkv * a.dv)) return ODI_ERR_ARGUMENT;
   if (!a.unit && (a.q_w != nullptr || a.k_w != nullptr)) return ODI_ERR_ARGUMENT;
   if (((uintptr_t)a.q_w | (uintptr_t)a.k_w) % 16 != 0) return ODI_ERR_UNSUPPORTED;
   if (dtype == 1 && a.d == a.d_store && a.d % 4 == 0 && a.d <= 512 && a.d > 0 && a.dv > 0 && !(a.rot_dim & 1) && a.rot_dim <= a.d &&
-      ((uintptr_t)a.qkv | (uintptr_t)a.q_out | (uintptr_t)a.k_pool) % 8 == 0 && (a.v_from_k || (a.nkv * a.dv) % 4 == 0)) {
+      ((uintptr_t)a.qkv | (uintptr_t)a.q_out | (uintptr_t)a.k_pool) % 8 == 0 && a.ld % 4 == 0) {
     const int heads = a.nq + (a.write_kv ? 2 * a.nkv : 0);
     // few tokens: a warp per head for parallelism; many tokens: a warp takes a quarter of a token's heads
     const int hpw = a.n_tokens >= 256 ? (heads + 3) / 4 : 1;

@@ -142,6 +142,29 @@ __device__ __forceinline__ int merge_used_splits(const int* plan, int splits, in
   return (n_tiles + per - 1) / per;
 }
 
+// What happens to an attention's finished heads on their way out: rows of `out_ld` elements (a head's lanes at head * dv),
+// times `scale`, times the logistic function of a gate that another product computed (null: none).
+struct HeadOut {
+  const void* gate;       // in T; a token's gate row starts at gate + tok * gate_ld
+  int gate_ld;
+  int gate_per_head;      // 1: one number per head; 0: one per lane of the heads
+  int out_ld;
+  float scale;
+};
+template <typename T>
+__device__ __forceinline__ float head_out_factor(const HeadOut& o, size_t tok, int head, int dv, int lane) {
+  if (o.gate == nullptr) return o.scale;
+  const float g = to_f<T>(((const T*)o.gate)[tok * o.gate_ld + (o.gate_per_head ? head : head * dv + lane)]);
+  return o.scale / (1.f + expf(-g));
+}
+
+// A learned bias of the scores by distance: what the query at position p adds to its score with key j is
+// table[head * n + min(p - j, n - 1)].
+struct DistanceBias {
+  const float* table;     // [nq, n], or null
+  int n;
+};
+
 // Position of key `pos` inside a sequence's page list.  A group that keeps every key
 // has ring_pages == 0; a windowed group keeps a ring of ring_pages pages per sequence.
 // A windowed group that also keeps a sequence's first positions for good puts the pages of those

@@ -5,25 +5,28 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------------
-// Embedding: hidden[t, :] = table[ids[t], :], widened to the fp32 residual stream.
+// Embedding: hidden[t, :] = table[ids[t], :] * scale, widened to the fp32 residual stream, `copies` times side by side.
 // ---------------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                             float* __restrict__ hidden, int H) {
+                             float* __restrict__ hidden, int H, int copies, float scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
   const T* row = table + (size_t)ids[t] * H;
-  float* out = hidden + (size_t)t * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] = to_f<T>(row[i]);
+  float* out = hidden + (size_t)t * copies * H;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float v = to_f<T>(row[i]) * scale;
+    for (int c = 0; c < copies; ++c) out[(size_t)c * H + i] = v;
+  }
 }
 
-extern "C" int odi_embed(const void* table, const int* ids, float* hidden, int n, int H, int dtype,
+extern "C" int odi_embed(const void* table, const int* ids, float* hidden, int n, int H, int copies, float scale, int dtype,
                          cudaStream_t stream) {
   if (n <= 0) return 0;
   const int threads = H >= 1024 ? 256 : 128;
-  if (dtype == 0) odi_rc = launch_pdl((embed_kernel<float>), dim3(n), dim3(threads), 0, stream, (const float*)table, ids, hidden, H);
-  else odi_rc = launch_pdl((embed_kernel<bf16>), dim3(n), dim3(threads), 0, stream, (const bf16*)table, ids, hidden, H);
+  if (dtype == 0) odi_rc = launch_pdl((embed_kernel<float>), dim3(n), dim3(threads), 0, stream, (const float*)table, ids, hidden, H, copies, scale);
+  else odi_rc = launch_pdl((embed_kernel<bf16>), dim3(n), dim3(threads), 0, stream, (const bf16*)table, ids, hidden, H, copies, scale);
   return launch_status();
 }
 

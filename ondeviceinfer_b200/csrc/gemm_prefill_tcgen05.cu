@@ -52,6 +52,7 @@
 #define EPI_HEAD_PREP 4    // the rows of w are q, k and v heads of 128: per-head norm, rotation, cache write
 #define EPI_GELU 5         // bf16 out = gelu(acc), the exact (erf) form
 #define EPI_GEGLU 6        // bf16 out = gelu(acc_gate) * acc_up, the tanh form of GELU; weight rows as for EPI_SWIGLU
+#define EPI_RELU2 7        // out_bf16[token, n] = max(acc, 0)^2
 #define EPI_IS_GATED(e) ((e) == EPI_SWIGLU || (e) == EPI_GEGLU)
 
 #define BM 128             // token rows per CTA (the lanes of its tensor memory); a tile has 2 * BM
@@ -155,6 +156,7 @@ __device__ __forceinline__ float silu_f(float g) { return g / (1.f + __expf(-g))
 __device__ __forceinline__ float gelu_tanh_f(float g) {
   return g / (1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * g * g, g, g)));
 }
+__device__ __forceinline__ float relu2_f(float z) { const float r = fmaxf(z, 0.f); return r * r; }
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f)); }
 
 // ------------------------------------------------------------------------------ the kernel
@@ -476,8 +478,8 @@ gemm_prefill_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 #pragma unroll
               for (int i = 0; i < 4; ++i) {
                 const int e = 8 * q + 2 * i;
-                const float lo = GATE ? (EPI == EPI_GEGLU ? gelu_tanh_f(v[e]) : silu_f(v[e])) * u[e] : (EPI == EPI_GELU ? gelu_erf_f(v[e]) : v[e]);
-                const float hi = GATE ? (EPI == EPI_GEGLU ? gelu_tanh_f(v[e + 1]) : silu_f(v[e + 1])) * u[e + 1] : (EPI == EPI_GELU ? gelu_erf_f(v[e + 1]) : v[e + 1]);
+                const float lo = GATE ? (EPI == EPI_GEGLU ? gelu_tanh_f(v[e]) : silu_f(v[e])) * u[e] : (EPI == EPI_GELU ? gelu_erf_f(v[e]) : EPI == EPI_RELU2 ? relu2_f(v[e]) : v[e]);
+                const float hi = GATE ? (EPI == EPI_GEGLU ? gelu_tanh_f(v[e + 1]) : silu_f(v[e + 1])) * u[e + 1] : (EPI == EPI_GELU ? gelu_erf_f(v[e + 1]) : EPI == EPI_RELU2 ? relu2_f(v[e + 1]) : v[e + 1]);
                 __nv_bfloat162 pr = __floats2bfloat162_rn(lo, hi);
                 w[i] = *(uint32_t*)&pr;
               }
@@ -660,6 +662,7 @@ extern "C" int odi_gemm_prefill_bf16(const void* x, const void* w, void* out, in
   switch (epi) {
     case EPI_STORE_BF16: return launch<EPI_STORE_BF16>(mx, mw, mo, a, sms, stream);
     case EPI_GELU: return launch<EPI_GELU>(mx, mw, mo, a, sms, stream);
+    case EPI_RELU2: return launch<EPI_RELU2>(mx, mw, mo, a, sms, stream);
     case EPI_STORE_F32: return launch<EPI_STORE_F32>(mx, mw, mo, a, sms, stream);
     case EPI_RESIDUAL: return launch<EPI_RESIDUAL>(mx, mw, mo, a, sms, stream);
     case EPI_SWIGLU: return launch<EPI_SWIGLU>(mx, mw, mo, a, sms, stream);

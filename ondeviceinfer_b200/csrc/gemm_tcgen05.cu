@@ -37,6 +37,7 @@
 #define EPI_HEAD_PREP 4    // the rows are q, k and v heads of 128: per-head norm, rotation, cache write
 #define EPI_GELU 5         // out_bf16[token, n] = gelu(acc), the exact (erf) form
 #define EPI_GEGLU 6        // out_bf16[token, n] = gelu(acc_gate) * acc_up, the tanh form of GELU   (DUAL)
+#define EPI_RELU2 7        // out_bf16[token, n] = max(acc, 0)^2
 
 #define BM 128             // features per tile (UMMA M)
 #define BK 64              // k per stage: 64 bf16 = one 128-byte swizzle row
@@ -277,6 +278,7 @@ __device__ __forceinline__ float emit(const GemmArgs& a, int token, int n, float
   else if (EPI == EPI_RESIDUAL) { const float r = ((float*)a.out)[at] + v; ((float*)a.out)[at] = r; return r; }
   else if (EPI == EPI_SWIGLU) ((bf16*)a.out)[at] = __float2bfloat16_rn(silu_f(v) * v2);
   else if (EPI == EPI_GEGLU) ((bf16*)a.out)[at] = __float2bfloat16_rn(gelu_tanh_f(v) * v2);
+  else if (EPI == EPI_RELU2) { const float r = fmaxf(v, 0.f); ((bf16*)a.out)[at] = __float2bfloat16_rn(r * r); }
   else if (EPI == EPI_GELU) ((bf16*)a.out)[at] = __float2bfloat16_rn(0.5f * v * (1.0f + erff(v * 0.70710678118654752440f)));
   return 0.f;
 }
@@ -900,6 +902,7 @@ static int dispatch_epi(int epi, const CUtensorMap& mw, const CUtensorMap& mx, c
   switch (epi) {
     case EPI_STORE_BF16: return launch<BN, false, EPI_STORE_BF16, CLUSTER>(mw, mx, a, grid, stream);
     case EPI_GELU: return launch<BN, false, EPI_GELU, CLUSTER>(mw, mx, a, grid, stream);
+    case EPI_RELU2: return launch<BN, false, EPI_RELU2, CLUSTER>(mw, mx, a, grid, stream);
     case EPI_STORE_F32: return launch<BN, false, EPI_STORE_F32, CLUSTER>(mw, mx, a, grid, stream);
     case EPI_RESIDUAL: return launch<BN, false, EPI_RESIDUAL, CLUSTER>(mw, mx, a, grid, stream);
     case EPI_SWIGLU:

@@ -85,16 +85,16 @@ def _require(t: torch.Tensor, name: str, dtype=None, ndim=None) -> None:
 # ------------------------------------------------------------------------------ elementwise
 
 
-def embed(table: torch.Tensor, ids: torch.Tensor, hidden: torch.Tensor) -> None:
-    """hidden[t, :] = table[ids[t], :] into the fp32 residual stream."""
+def embed(table: torch.Tensor, ids: torch.Tensor, hidden: torch.Tensor, scale: float = 1.0, copies: int = 1) -> None:
+    """hidden[t, :] = table[ids[t], :] * scale into the fp32 residual stream, ``copies`` times side by side."""
     _require(table, "table", ndim=2)
     _require(ids, "ids", torch.int32, 1)
     _require(hidden, "hidden", torch.float32, 2)
-    if hidden.shape != (ids.numel(), table.shape[1]):
-        raise KernelError(f"hidden is {tuple(hidden.shape)}, expected {(ids.numel(), table.shape[1])}")
+    if hidden.shape != (ids.numel(), copies * table.shape[1]):
+        raise KernelError(f"hidden is {tuple(hidden.shape)}, expected {(ids.numel(), copies * table.shape[1])}")
     lib = load_library("elementwise")
     _check(lib.odi_embed(_ptr(table), _ptr(ids), _ptr(hidden), c_int(ids.numel()), c_int(table.shape[1]),
-                         c_int(dtype_code(table.dtype)), _stream()), "embed")
+                         c_int(copies), c_float(scale), c_int(dtype_code(table.dtype)), _stream()), "embed")
 
 
 def embed_sinusoid(table: torch.Tensor, ids: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor, hidden: torch.Tensor,
@@ -280,7 +280,7 @@ def gemm_f32(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, residual: Opti
                             c_int(K), c_int(K), c_int(N), c_int(N), _stream()), "gemm_f32")
 
 
-EPI_STORE_BF16, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU, EPI_HEAD_PREP, EPI_GELU, EPI_GEGLU = 0, 1, 2, 3, 4, 5, 6
+EPI_STORE_BF16, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU, EPI_HEAD_PREP, EPI_GELU, EPI_GEGLU, EPI_RELU2 = 0, 1, 2, 3, 4, 5, 6, 7
 EPI_GATED = (EPI_SWIGLU, EPI_GEGLU)      # two weight rows a feature: the gate rows, then the up rows
 
 _gemm_state = {}
@@ -417,7 +417,7 @@ def gemm_bf16(x: Optional[torch.Tensor], w: torch.Tensor, out: Optional[torch.Te
     ``EPI_STORE_BF16`` / ``EPI_STORE_F32``: out [tokens, rows]; ``EPI_RESIDUAL``: out (fp32) += product;
     ``EPI_SWIGLU`` / ``EPI_GEGLU``: w holds the gate rows then the up rows, out [tokens, rows / 2] = silu(gate) * up
     resp. gelu(gate) * up (the tanh form);
-    ``EPI_GELU``: out [tokens, rows] = gelu(product) in bf16 (the exact erf form).
+    ``EPI_GELU``: out [tokens, rows] = gelu(product) in bf16 (the exact erf form); ``EPI_RELU2``: max(product, 0)^2.
     ``cluster``: let 2..8 K splits exchange their partials inside a thread-block cluster (else, and for
     more splits, through global scratch and a ticket).
     ``norm = (rows, weight, parts, eps)`` instead of ``x``: the operand is RMSNorm(rows) * weight with the
@@ -475,7 +475,7 @@ def gemm_bf16(x: Optional[torch.Tensor], w: torch.Tensor, out: Optional[torch.Te
         if w.shape[1] != K:
             raise KernelError(f"gemm sizes disagree: x {tuple(x_like.shape)}, w {tuple(w.shape)}")
     else:
-        _require(out, "out", torch.bfloat16 if epi in (EPI_STORE_BF16, EPI_SWIGLU, EPI_GELU, EPI_GEGLU) else torch.float32, 2)
+        _require(out, "out", torch.bfloat16 if epi in (EPI_STORE_BF16, EPI_SWIGLU, EPI_GELU, EPI_GEGLU, EPI_RELU2) else torch.float32, 2)
         if w.shape[1] != K or out.shape != (tokens, n_out) or (epi in EPI_GATED and w_rows % 2):
             raise KernelError(f"gemm sizes disagree: x {tuple(x_like.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
     if sumsq_out is not None:
@@ -565,9 +565,9 @@ def gemm_prefill_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tens
         if not gemm_bf16_supported(x, w):
             raise KernelError(f"gemm_prefill_tcgen05 needs K a multiple of 8 and 16-byte aligned operands (K={K})")
     else:
-        if epi not in (EPI_STORE_BF16, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU, EPI_GELU, EPI_GEGLU):
+        if epi not in (EPI_STORE_BF16, EPI_STORE_F32, EPI_RESIDUAL, EPI_SWIGLU, EPI_GELU, EPI_GEGLU, EPI_RELU2):
             raise KernelError(f"gemm_prefill_bf16 has no epilogue {epi}")
-        _require(out, "out", torch.bfloat16 if epi in (EPI_STORE_BF16, EPI_SWIGLU, EPI_GELU, EPI_GEGLU) else torch.float32, 2)
+        _require(out, "out", torch.bfloat16 if epi in (EPI_STORE_BF16, EPI_SWIGLU, EPI_GELU, EPI_GEGLU, EPI_RELU2) else torch.float32, 2)
         if w.shape[1] != K or out.shape != (tokens, n_out) or (epi in EPI_GATED and w_rows % 2):
             raise KernelError(f"gemm sizes disagree: x {tuple(x.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
         if not gemm_prefill_supported(x, w, n_out, out.dtype):
@@ -588,13 +588,55 @@ def gemm_prefill_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tens
 # ------------------------------------------------------------------------------ attention
 
 
+class _HeadOutArgs(Structure):
+    _fields_ = [("gate", c_void_p), ("gate_ld", c_int), ("gate_per_head", c_int), ("out_ld", c_int), ("scale", c_float)]
+
+
+class _DistanceBiasArgs(Structure):
+    _fields_ = [("table", c_void_p), ("n", c_int)]
+
+
+def _at_column(t: torch.Tensor, col: int) -> c_void_p:
+    """Address of column ``col`` of the first row of a contiguous 2-D tensor."""
+    return c_void_p(t.data_ptr() + col * t.element_size())
+
+
+def _head_out(out: torch.Tensor, n_tokens: int, width: int, out_col: int, scale: float, gate, dtype, heads: int) -> tuple:
+    """(argument block, address of the first head's first lane) for heads of ``width`` lanes in all that go to the columns
+    from ``out_col`` on of ``out`` [tokens, >= out_col + width], times ``scale`` and, with ``gate`` = (tensor, column,
+    per_head), times the logistic function of the tensor's columns (one per lane, or one per head)."""
+    if out_col == 0 and out.numel() == n_tokens * width:
+        ld = width
+    else:
+        if out.dim() != 2 or out.shape[0] != n_tokens or out_col < 0 or out_col + width > out.shape[1]:
+            raise KernelError("q and out disagree")
+        ld = out.shape[1]
+    if gate is None:
+        return _HeadOutArgs(None, 0, 0, ld, scale), _at_column(out, out_col)
+    tensor, col, per_head = gate
+    _require(tensor, "gate", dtype, 2)
+    if tensor.shape[0] != n_tokens or col < 0 or col + (heads if per_head else width) > tensor.shape[1]:
+        raise KernelError(f"the gate's columns do not fit {tuple(tensor.shape)}")
+    return _HeadOutArgs(_at_column(tensor, col), tensor.shape[1], 1 if per_head else 0, ld, scale), _at_column(out, out_col)
+
+
+def _distance_bias(rel: Optional[torch.Tensor], nq: int) -> _DistanceBiasArgs:
+    """``rel`` fp32 [nq, n]: what a score gets for the distance of its key, the last entry for n - 1 and everything beyond."""
+    if rel is None:
+        return _DistanceBiasArgs(None, 0)
+    _require(rel, "rel", torch.float32, 2)
+    if rel.shape[0] != nq or rel.shape[1] < 1:
+        raise KernelError(f"rel is {tuple(rel.shape)}, expected one row per query head")
+    return _DistanceBiasArgs(_ptr(rel), rel.shape[1])
+
+
 class _AttnArgs(Structure):
     _fields_ = [("q", c_void_p), ("k_pool", c_void_p), ("v_pool", c_void_p), ("out", c_void_p),
                 ("partial", c_void_p), ("cu_q", c_void_p), ("past", c_void_p), ("page_start", c_void_p),
                 ("page_ids", c_void_p), ("n_seqs", c_int), ("nq", c_int), ("nkv", c_int), ("page_size", c_int),
                 ("ring_pages", c_int), ("window", c_int), ("splits", c_int), ("bq", c_int),
                 ("head_chunks", c_int), ("scale", c_float), ("softcap", c_float), ("sink", c_int), ("keep", c_int),
-                ("chunk", c_int), ("mixed", c_int)]
+                ("chunk", c_int), ("mixed", c_int), ("ho", _HeadOutArgs), ("rel", _DistanceBiasArgs)]
 
 
 SIMT_HEAD_DIMS = tuple(range(16, 513, 16))
@@ -604,7 +646,8 @@ def attention_simt(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, 
                    nq: int, nkv: int, d: int, page_size: int, ring_pages: int, window: int, scale: float,
                    splits: int = 1, partial: Optional[torch.Tensor] = None, dv: Optional[int] = None,
                    shared_kv: bool = False, softcap: float = 0.0, sink: bool = False, keep: int = 0, chunk: int = 0,
-                   mixed: bool = False) -> None:
+                   mixed: bool = False, rel: Optional[torch.Tensor] = None, gate=None, out_scale: float = 1.0,
+                   out_col: int = 0) -> None:
     """Causal GQA over the paged cache for any mixture of prompt and decode sequences.  ``softcap`` c > 0:
     scores (times ``scale``) become c tanh(score / c) before the softmax.  ``sink``: the softmax has one more
     term of score 0 and no value, p_j = exp(s_j) / (1 + sum_k exp(s_k)).  ``keep`` > 0 with a window: the first
@@ -612,6 +655,11 @@ def attention_simt(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, 
 
     ``chunk`` c > 0 (instead of a window): position p sees the keys of its own chunk of c positions only.
     ``mixed``: q is [tokens, nq, nkv, d] and a score is the sum over the key heads of q . k (see :func:`mixed_prep`).
+
+    ``rel`` (fp32 [nq, n]): rel[h, min(distance, n - 1)] is added to a score behind scale and cap.  ``out`` may be wider
+    than the heads ([tokens, >= out_col + nq dv]): they go to its columns from ``out_col`` on, times ``out_scale`` and,
+    with ``gate`` = (tensor, column, per_head), times the logistic function of those columns of the tensor, one per
+    lane or one per head.
 
     ``dv`` (default ``d``): width of the value rows and of the output.  ``shared_kv``: a cached row is key and
     value at once (the value is its first ``dv`` lanes; ``v_pool`` is None), as in attention over a latent
@@ -632,15 +680,14 @@ def attention_simt(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, 
     else:
         _require(v_pool, "v_pool", q.dtype)
     n_tokens = q.numel() // (nq * d * (nkv if mixed else 1))
-    if out.numel() != n_tokens * nq * dv:
-        raise KernelError("q and out disagree")
+    ho, out_ptr = _head_out(out, n_tokens, nq * dv, out_col, out_scale, gate, q.dtype, nq)
     if splits > 1:
         need = n_tokens * nq * splits * (dv + 2)
         if partial is None or partial.numel() < need or partial.dtype != torch.float32:
             raise KernelError(f"splits={splits} needs an fp32 partial buffer of {need} elements")
-    args = _AttnArgs(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(partial), _ptr(cu_q), _ptr(past),
+    args = _AttnArgs(_ptr(q), _ptr(k_pool), _ptr(v_pool), out_ptr, _ptr(partial), _ptr(cu_q), _ptr(past),
                      _ptr(page_start), _ptr(page_ids), n_seqs, nq, nkv, page_size, ring_pages, window, splits,
-                     0, 0, scale, softcap, 1 if sink else 0, keep, chunk, 1 if mixed else 0)
+                     0, 0, scale, softcap, 1 if sink else 0, keep, chunk, 1 if mixed else 0, ho, _distance_bias(rel, nq))
     defines = {"ODI_HEAD_DIM": d}
     if not plain:
         defines.update({"ODI_VALUE_DIM": dv, "ODI_SHARED_KV": 1 if shared_kv else 0})
@@ -884,7 +931,7 @@ class _TcAttnArgs(Structure):
     _fields_ = [("out", c_void_p), ("cu_q", c_void_p), ("past", c_void_p), ("page_start", c_void_p),
                 ("page_ids", c_void_p), ("status", c_void_p), ("n_seqs", c_int), ("nq", c_int), ("nkv", c_int),
                 ("scale", c_float), ("window", c_int), ("ring_pages", c_int), ("softcap", c_float), ("sink", c_int),
-                ("keep", c_int), ("chunk", c_int), ("mixed", c_int)]
+                ("keep", c_int), ("chunk", c_int), ("mixed", c_int), ("ho", _HeadOutArgs), ("rel", _DistanceBiasArgs)]
 
 
 TCGEN05_ATTENTION_HEAD_DIMS = (64, 128)
@@ -893,7 +940,8 @@ TCGEN05_ATTENTION_HEAD_DIMS = (64, 128)
 def attention_tcgen05(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, n_seqs: int, max_q_len: int,
                       nq: int, nkv: int, d: int, page_size: int, scale: float, heads_per_cta: int = 0, window: int = 0,
                       ring_pages: int = 0, softcap: float = 0.0, sink: bool = False, keep: int = 0, chunk: int = 0,
-                      mixed: bool = False) -> None:
+                      mixed: bool = False, rel: Optional[torch.Tensor] = None, gate=None, out_scale: float = 1.0,
+                      out_col: int = 0) -> None:
     """bf16 causal GQA for prefill on tcgen05: scores and outputs in tensor memory, TMA-fed pages.
     ``sink``: one more term of score 0 and no value in the softmax.
     ``window`` > 0 keeps the last ``window`` keys visible (``ring_pages`` > 0: the page lists are rings);
@@ -901,6 +949,8 @@ def attention_tcgen05(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, 
     ``chunk`` c > 0 (instead of a window): position p sees the keys of its own chunk of c positions only.
     ``mixed``: q is [tokens, nq, nkv, d] and a score is the sum over the key heads of q . k (see :func:`mixed_prep`;
     :func:`attention_tcgen05_mixed_rows` says for how many key heads).
+    ``rel``, ``gate``, ``out_scale``, ``out_col``: as for :func:`attention_simt` (:func:`attention_tcgen05_takes` says
+    which tables and columns).
     ``heads_per_cta``: 1, or 2 (two heads of a key/value group share a CTA and its K/V pages; needs an
     even group size), or 0 for the library's choice."""
     if d not in TCGEN05_ATTENTION_HEAD_DIMS:
@@ -910,15 +960,27 @@ def attention_tcgen05(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, 
     for name, t in (("q", q), ("out", out), ("k_pool", k_pool), ("v_pool", v_pool)):
         _require(t, name, torch.bfloat16)
     n_tokens = q.numel() // (nq * d * (nkv if mixed else 1))
-    if out.numel() != n_tokens * nq * d or k_pool.shape != v_pool.shape or k_pool.dim() != 4:
-        raise KernelError("attention_tcgen05: q/out or the pools disagree")
+    if k_pool.shape != v_pool.shape or k_pool.dim() != 4:
+        raise KernelError("attention_tcgen05: the pools disagree")
+    ho, out_ptr = _head_out(out, n_tokens, nq * d, out_col, out_scale, gate, q.dtype, nq)
     _, _, status = _gemm_buffers(q.device, 0)
-    args = _TcAttnArgs(_ptr(out), _ptr(cu_q), _ptr(past), _ptr(page_start), _ptr(page_ids), _ptr(status),
-                       n_seqs, nq, nkv, scale, window, ring_pages, softcap, 1 if sink else 0, keep, chunk, 1 if mixed else 0)
+    args = _TcAttnArgs(out_ptr, _ptr(cu_q), _ptr(past), _ptr(page_start), _ptr(page_ids), _ptr(status),
+                       n_seqs, nq, nkv, scale, window, ring_pages, softcap, 1 if sink else 0, keep, chunk, 1 if mixed else 0,
+                       ho, _distance_bias(rel, nq))
     lib = load_library("attention_tcgen05", {"ODI_HEAD_DIM": d})
     _check(lib.odi_attention_tcgen05(_ptr(q), _ptr(k_pool), _ptr(v_pool), byref(args), c_int(n_tokens),
                                      c_int(max_q_len), c_long(k_pool.shape[0]), c_int(heads_per_cta), _stream()),
            "attention_tcgen05")
+
+
+def attention_tcgen05_takes(d: int, *, bias_entries: int = 0, out_ld: int = 0, out_col: int = 0, gate=None) -> bool:
+    """Whether :func:`attention_tcgen05` takes heads of ``d`` lanes with a table of ``bias_entries`` biases a head, rows of
+    ``out_ld`` columns written from ``out_col`` on, and this gate (a tensor's columns, 16-byte aligned unless per head)."""
+    if d not in TCGEN05_ATTENTION_HEAD_DIMS or out_ld % 8 or out_col % 8:
+        return False
+    if gate is not None and not gate[2] and (gate[0].shape[1] % 8 or gate[1] % 8):
+        return False
+    return bias_entries == 0 or bias_entries <= int(load_library("attention_tcgen05", {"ODI_HEAD_DIM": d}).odi_attention_tcgen05_bias_entries())
 
 
 def attention_tcgen05_mixed_rows(d: int, nkv: int) -> int:
@@ -1290,13 +1352,14 @@ class _RotUnitArgs(Structure):
                 ("page_start", c_void_p), ("page_ids", c_void_p), ("n_tokens", c_int), ("nq", c_int), ("nkv", c_int),
                 ("d", c_int), ("dv", c_int), ("rot_dim", c_int), ("page_size", c_int), ("ring_pages", c_int),
                 ("write_kv", c_int), ("unit", c_int), ("d_store", c_int), ("eps", c_float), ("v_from_k", c_int),
-                ("q_w", c_void_p), ("k_w", c_void_p)]
+                ("q_w", c_void_p), ("k_w", c_void_p), ("ld", c_int), ("temp_coef", c_float), ("temp_every", c_int)]
 
 
 def rot_unit_prep(qkv, q_out, k_pool, v_pool, cos_t, sin_t, tok_seq, tok_pos, page_start, page_ids, *, nq: int,
                   nkv: int, d: int, dv: int, rot_dim: int, page_size: int, ring_pages: int, write_kv: bool,
                   unit_eps: Optional[float], d_store: Optional[int] = None, v_from_k: bool = False,
-                  q_weight: Optional[torch.Tensor] = None, k_weight: Optional[torch.Tensor] = None) -> None:
+                  q_weight: Optional[torch.Tensor] = None, k_weight: Optional[torch.Tensor] = None,
+                  q_temperature: Optional[Tuple[float, int]] = None, col: int = 0) -> None:
     """Head preparation of an attention that rotates first and norms afterwards: q and k heads (``d`` lanes) of
     ``qkv`` [tokens, nq d + nkv d + nkv dv] are rotated over their first ``rot_dim`` lanes (lane 2i with 2i + 1;
     ``cos_t`` None: not at all) and, with ``unit_eps`` not None, divided by sqrt(mean of squares + eps); q goes to
@@ -1304,7 +1367,9 @@ def rot_unit_prep(qkv, q_out, k_pool, v_pool, cos_t, sin_t, tok_seq, tok_pos, pa
     and k heads have ``d_store`` >= ``d`` lanes (default ``d``), the ones beyond ``d`` zero.  ``v_from_k``: ``qkv``
     holds no v lanes ([tokens, nq d + nkv d]); the value of a head is its key as projected, before the rotation.
     ``q_weight`` / ``k_weight`` (fp32 [d], with ``unit_eps``): after the division every query resp. key head is
-    multiplied by it lane by lane (an RMS norm per head with a weight that the heads share)."""
+    multiplied by it lane by lane (an RMS norm per head with a weight that the heads share).  ``q_temperature`` = (coef,
+    every): queries at position p are also multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  ``qkv`` may be
+    wider than the heads: theirs are the columns from ``col`` on."""
     d_store = d if d_store is None else d_store
     for name, w in (("q_weight", q_weight), ("k_weight", k_weight)):
         if w is not None:
@@ -1316,7 +1381,7 @@ def rot_unit_prep(qkv, q_out, k_pool, v_pool, cos_t, sin_t, tok_seq, tok_pos, pa
     _require(qkv, "qkv", ndim=2)
     _require(q_out, "q_out", qkv.dtype, 2)
     n = qkv.shape[0]
-    if qkv.shape[1] != (nq + nkv) * d + (0 if v_from_k else nkv * dv) or q_out.shape != (n, nq * d_store):
+    if col < 0 or qkv.shape[1] < col + (nq + nkv) * d + (0 if v_from_k else nkv * dv) or q_out.shape != (n, nq * d_store):
         raise KernelError(f"rot_unit_prep sizes disagree: qkv {tuple(qkv.shape)}, q_out {tuple(q_out.shape)}, "
                           f"nq={nq}, nkv={nkv}, d={d}, dv={dv}")
     if write_kv:
@@ -1329,10 +1394,13 @@ def rot_unit_prep(qkv, q_out, k_pool, v_pool, cos_t, sin_t, tok_seq, tok_pos, pa
         _require(sin_t, "sin_t", torch.float32, 2)
         if cos_t.shape != (n, rot_dim // 2) or sin_t.shape != cos_t.shape:
             raise KernelError("rope tables must be [tokens, rot_dim / 2]")
-    args = _RotUnitArgs(_ptr(qkv), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(cos_t), _ptr(sin_t), _ptr(tok_seq),
+    coef, every = (0.0, 0) if q_temperature is None else q_temperature
+    if q_temperature is not None and every <= 0:
+        raise KernelError("q_temperature: every must be positive")
+    args = _RotUnitArgs(_at_column(qkv, col), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _ptr(cos_t), _ptr(sin_t), _ptr(tok_seq),
                         _ptr(tok_pos), _ptr(page_start), _ptr(page_ids), n, nq, nkv, d, dv, rot_dim, page_size, ring_pages,
                         1 if write_kv else 0, 0 if unit_eps is None else 1, d_store, 0.0 if unit_eps is None else unit_eps,
-                        1 if v_from_k else 0, _ptr(q_weight), _ptr(k_weight))
+                        1 if v_from_k else 0, _ptr(q_weight), _ptr(k_weight), qkv.shape[1], coef, every)
     lib = load_library("capped")
     _check(lib.odi_rot_unit_prep(byref(args), c_int(dtype_code(qkv.dtype)), _stream()), "rot_unit_prep")
 
@@ -1341,7 +1409,7 @@ class _CappedAttnArgs(Structure):
     _fields_ = [("q", c_void_p), ("k_pool", c_void_p), ("v_pool", c_void_p), ("out", c_void_p), ("cu_q", c_void_p),
                 ("past", c_void_p), ("page_start", c_void_p), ("page_ids", c_void_p), ("n_seqs", c_int), ("nq", c_int),
                 ("nkv", c_int), ("ring_pages", c_int), ("window", c_int), ("scale", c_float), ("softcap", c_float),
-                ("sink", c_int), ("keep", c_int)]
+                ("sink", c_int), ("keep", c_int), ("ho", _HeadOutArgs), ("rel", _DistanceBiasArgs), ("rel_staged", c_int)]
 
 
 def attention_capped_supported(dtype: torch.dtype, d: int, dv: int) -> bool:
@@ -1351,11 +1419,13 @@ def attention_capped_supported(dtype: torch.dtype, d: int, dv: int) -> bool:
 
 def attention_capped(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, n_seqs: int, max_q_len: int, nq: int,
                      nkv: int, d: int, dv: int, page_size: int, ring_pages: int, window: int, scale: float,
-                     softcap: float = 0.0, sink: bool = False, keep: int = 0) -> None:
+                     softcap: float = 0.0, sink: bool = False, keep: int = 0, rel: Optional[torch.Tensor] = None, gate=None,
+                     out_scale: float = 1.0, out_col: int = 0) -> None:
     """bf16 causal GQA on the tensor cores with squashed scores (``softcap`` c > 0: c tanh(score / c)), a window
     (0: none; the cache may be a ring of pages) and value rows of ``dv`` lanes, for any mixture of sequences.
     ``sink``: one more term of score 0 and no value in the softmax.  ``keep`` > 0 with a window: the first ``keep``
-    positions of a sequence stay visible beyond the window."""
+    positions of a sequence stay visible beyond the window.  ``rel``, ``gate``, ``out_scale``, ``out_col``: as for
+    :func:`attention_simt`."""
     if not attention_capped_supported(q.dtype, d, dv) or page_size != 64:
         raise KernelError(f"attention_capped takes bfloat16 heads in steps of 16 up to 256 and pages of 64 (d={d}, dv={dv})")
     _require(q, "q", torch.bfloat16)
@@ -1363,10 +1433,12 @@ def attention_capped(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *
     _require(k_pool, "k_pool", torch.bfloat16)
     _require(v_pool, "v_pool", torch.bfloat16)
     n_tokens = q.numel() // (nq * d)
-    if out.numel() != n_tokens * nq * dv or k_pool.shape[-1] != d or v_pool.shape[-1] != dv:
+    if k_pool.shape[-1] != d or v_pool.shape[-1] != dv:
         raise KernelError("attention_capped sizes disagree")
-    args = _CappedAttnArgs(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(cu_q), _ptr(past), _ptr(page_start),
-                           _ptr(page_ids), n_seqs, nq, nkv, ring_pages, window, scale, softcap, 1 if sink else 0, keep)
+    ho, out_ptr = _head_out(out, n_tokens, nq * dv, out_col, out_scale, gate, q.dtype, nq)
+    args = _CappedAttnArgs(_ptr(q), _ptr(k_pool), _ptr(v_pool), out_ptr, _ptr(cu_q), _ptr(past), _ptr(page_start),
+                           _ptr(page_ids), n_seqs, nq, nkv, ring_pages, window, scale, softcap, 1 if sink else 0, keep,
+                           ho, _distance_bias(rel, nq), 0)
     lib = load_library("attention_capped_mma", {"ODI_HEAD_DIM": d, "ODI_VALUE_DIM": dv})
     _check(lib.odi_attention_capped(byref(args), c_int(max_q_len), _stream()), "attention_capped")
 
@@ -1374,7 +1446,8 @@ def attention_capped(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *
 def attention_capped_decode(q, k_pool, v_pool, out, cu_q, past, page_start, page_ids, *, n_seqs: int, nq: int, nkv: int,
                             d: int, dv: int, page_size: int, ring_pages: int, window: int, scale: float,
                             softcap: float = 0.0, splits: int = 1, partial: Optional[torch.Tensor] = None,
-                            sink: bool = False, keep: int = 0) -> None:
+                            sink: bool = False, keep: int = 0, rel: Optional[torch.Tensor] = None, gate=None,
+                            out_scale: float = 1.0, out_col: int = 0) -> None:
     """:func:`attention_capped` for steps in which every sequence brings one token: each sequence's visible keys
     are cut into ``splits`` ranges that blocks of their own take; ``partial`` (fp32, tokens * nq * splits * (dv + 2))
     holds their results for the combine kernel."""
@@ -1384,14 +1457,16 @@ def attention_capped_decode(q, k_pool, v_pool, out, cu_q, past, page_start, page
     _require(out, "out", torch.bfloat16)
     _require(k_pool, "k_pool", torch.bfloat16)
     _require(v_pool, "v_pool", torch.bfloat16)
-    if q.numel() != n_seqs * nq * d or out.numel() != n_seqs * nq * dv or k_pool.shape[-1] != d or v_pool.shape[-1] != dv:
+    if q.numel() != n_seqs * nq * d or k_pool.shape[-1] != d or v_pool.shape[-1] != dv:
         raise KernelError("attention_capped_decode sizes disagree (one token per sequence)")
+    ho, out_ptr = _head_out(out, n_seqs, nq * dv, out_col, out_scale, gate, q.dtype, nq)
     if splits > 1:
         need = n_seqs * nq * splits * (dv + 2)
         if partial is None or partial.numel() < need or partial.dtype != torch.float32:
             raise KernelError(f"splits={splits} needs an fp32 partial buffer of {need} elements")
-    args = _CappedAttnArgs(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(cu_q), _ptr(past), _ptr(page_start),
-                           _ptr(page_ids), n_seqs, nq, nkv, ring_pages, window, scale, softcap, 1 if sink else 0, keep)
+    args = _CappedAttnArgs(_ptr(q), _ptr(k_pool), _ptr(v_pool), out_ptr, _ptr(cu_q), _ptr(past), _ptr(page_start),
+                           _ptr(page_ids), n_seqs, nq, nkv, ring_pages, window, scale, softcap, 1 if sink else 0, keep,
+                           ho, _distance_bias(rel, nq), 0)
     lib = load_library("attention_capped_mma", {"ODI_HEAD_DIM": d, "ODI_VALUE_DIM": dv})
     _check(lib.odi_attention_capped_decode(byref(args), _ptr(partial), c_int(splits), _stream()), "attention_capped_decode",
            2 if splits > 1 else 1)
@@ -1980,3 +2055,110 @@ def ssd_mix(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, dt_b
                     norm_groups, eps)
     lib = load_library("ssd")
     _check(lib.odi_ssd(byref(args), c_int(dtype_code(proj.dtype)), _stream()), "ssd_mix", 4 if taps > 1 else 3)
+
+
+# ------------------------------------------------------------------------------ parallel residual streams
+
+
+class _StreamMixArgs(Structure):
+    _fields_ = [("x", c_void_p), ("y", c_void_p), ("mix", c_void_p), ("out_c", c_void_p), ("in_c", c_void_p),
+                ("weight", c_void_p), ("bias", c_void_p), ("out", c_void_p), ("rows", c_void_p), ("n", c_int), ("S", c_int),
+                ("W", c_int), ("m", c_float), ("eps", c_float)]
+
+
+STREAM_MIX_MAX_STREAMS, STREAM_MIX_MAX_WIDTH = 16, 50 * 1024
+
+
+def stream_mix(x: torch.Tensor, *, streams: int, y: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+               out_coef: Optional[torch.Tensor] = None, m: float = 1.0, in_coef: Optional[torch.Tensor] = None,
+               weight: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None, eps: float = 0.0,
+               out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> None:
+    """Parallel streams x [tokens, streams * W] (fp32, side by side), up to two things in one pass over a row:
+
+    * with ``y`` (fp32 [tokens, W]): x_t <- sum_s mix[s, t] x_s + m out_coef[t] y, all from the old streams, in place;
+    * with ``out`` [rows, W]: u = sum_s in_coef[s] x_s of the (new) streams, out = cast((u - mean) / sqrt(var + eps) *
+      weight + bias), var the mean of the squared deviations.
+
+    Coefficients (fp32) that are None stand for the identity: every stream keeps itself, ones.  ``rows`` (int32, without
+    ``y``): the rows of x that are read."""
+    _require(x, "x", torch.float32, 2)
+    n, width = x.shape
+    if streams < 1 or width % streams:
+        raise KernelError(f"{streams} streams do not divide rows of {width}")
+    W = width // streams
+    for name, t, shape in (("mix", mix, (streams, streams)), ("out_coef", out_coef, (streams,)), ("in_coef", in_coef, (streams,)),
+                           ("weight", weight, (W,)), ("bias", bias, (W,))):
+        if t is not None:
+            _require(t, name, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"stream_mix: {name} is {tuple(t.shape)}, expected {shape}")
+    if y is not None:
+        _require(y, "y", torch.float32, 2)
+        if y.shape != (n, W) or rows is not None:
+            raise KernelError("stream_mix: y has a row for every row of x")
+    if rows is not None:
+        _require(rows, "rows", torch.int32, 1)
+        n = rows.numel()
+    if out is not None:
+        _require(out, "out", ndim=2)
+        if out.shape != (n, W) or weight is None or bias is None:
+            raise KernelError("stream_mix: out has a row for every row read, and goes with a weight and a bias")
+    args = _StreamMixArgs(_ptr(x), _ptr(y), _ptr(mix), _ptr(out_coef), _ptr(in_coef), _ptr(weight), _ptr(bias), _ptr(out),
+                          _ptr(rows), n, streams, W, m, eps)
+    lib = load_library("stream_mix")
+    _check(lib.odi_stream_mix(byref(args), c_int(0 if out is None else dtype_code(out.dtype)), _stream()), "stream_mix")
+
+
+# ------------------------------------------------------------------------------ retention
+
+
+class _RetentionArgs(Structure):
+    _fields_ = [("proj", c_void_p), ("cos_t", c_void_p), ("sin_t", c_void_p), ("decay", c_void_p), ("state", c_void_p),
+                ("chunks", c_void_p), ("o", c_void_p), ("out", c_void_p), ("cu_q", c_void_p), ("tok_seq", c_void_p),
+                ("slots", c_void_p), ("n_tokens", c_int), ("n_seqs", c_int), ("max_q_len", c_int), ("ld", c_int),
+                ("heads", c_int), ("d", c_int), ("dv", c_int), ("rot", c_int), ("interleaved", c_int), ("out_ld", c_int),
+                ("norm", c_int), ("eps", c_float), ("k_scale", c_float), ("out_scale", c_float)]
+
+
+RETENTION_MAX_DIM = 1024
+RETENTION_CHUNK = 64             # tokens of a chunk of the form for prompts
+RETENTION_MIN_CHUNK_TOKENS = 8   # shorter portions take the tokens in order
+
+
+def retention(proj: torch.Tensor, cos_t, sin_t, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, cu_q, tok_seq, slots, *,
+              n_seqs: int, max_q_len: int, heads: int, d: int, dv: int, rot: int, interleaved: bool, eps: Optional[float],
+              out_scale: float = 1.0, col: int = 0, out_col: int = 0, chunked: Optional[bool] = None) -> None:
+    """Retention between its products (``csrc/retention.cu``): the columns of ``proj`` from ``col`` on are q (heads d), k
+    (heads d), v (heads dv) and the gate's logits (heads dv); q and k are rotated over their first ``rot`` lanes
+    (``cos_t`` None: not at all), k is multiplied by d^-1/2, S <- decay_h S + k v^T, o = S^T q, then o / rms(o) per head
+    (``eps`` None: as it is), times silu(gate) and ``out_scale``, to the columns of ``out`` from ``out_col`` on.  ``state``
+    [slots, heads, d, dv] is fp32 rows of the cache, advanced in place over all tokens that each sequence brings.
+    ``chunked``: take chunks of 64 tokens side by side (bf16; default: for portions of 8 tokens and more)."""
+    _require(proj, "proj", ndim=2)
+    _require(out, "out", proj.dtype, 2)
+    _require(decay, "decay", torch.float32, 1)
+    _require(state, "state", torch.float32)
+    n = proj.shape[0]
+    if (col < 0 or proj.shape[1] < col + 2 * heads * (d + dv) or out.shape[0] != n or out_col < 0 or out.shape[1] < out_col + heads * dv
+            or decay.numel() != heads or tuple(state.shape[1:]) != (heads, d, dv)):
+        raise KernelError(f"retention sizes disagree: proj {tuple(proj.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
+    if cos_t is not None:
+        _require(cos_t, "cos_t", torch.float32, 2)
+        _require(sin_t, "sin_t", torch.float32, 2)
+        if cos_t.shape != (n, rot // 2) or sin_t.shape != cos_t.shape:
+            raise KernelError("rope tables must be [tokens, rot / 2]")
+    lib = load_library("retention")
+    if chunked is None:
+        chunked = max_q_len >= RETENTION_MIN_CHUNK_TOKENS
+    chunked = chunked and proj.dtype == torch.bfloat16 and bool(lib.odi_retention_takes_chunks(c_int(d), c_int(dv)))
+    chunks = o = None
+    if chunked:
+        chunks = torch.empty((n // RETENTION_CHUNK + n_seqs, heads, d, dv), dtype=torch.float32, device=proj.device)
+    elif max_q_len > 1:
+        o = torch.empty((n, heads * dv), dtype=torch.float32, device=proj.device)
+    args = _RetentionArgs(_at_column(proj, col), _ptr(cos_t), _ptr(sin_t), _ptr(decay), _ptr(state), _ptr(chunks), _ptr(o),
+                          _at_column(out, out_col), _ptr(cu_q), _ptr(tok_seq), _ptr(slots), n, n_seqs, max_q_len, proj.shape[1],
+                          heads, d, dv, rot if cos_t is not None else 0, 1 if interleaved else 0, out.shape[1],
+                          0 if eps is None else 1, 0.0 if eps is None else eps, d ** -0.5, out_scale)
+    _check(lib.odi_retention(byref(args), c_int(1 if chunked else 0), c_int(dtype_code(proj.dtype)), _stream()), "retention",
+           3 if chunked else (2 if max_q_len > 1 else 1))

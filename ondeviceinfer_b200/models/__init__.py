@@ -4,6 +4,7 @@ from ..config.lemesun import LemesunConfig
 from ..config.losivik import LosivikConfig
 from ..config.noganex import NoganexConfig
 from ..config.nulalorn import NulalornConfig
+from ..config.pukinex import PukinexConfig
 from ..config.qwen3 import Qwen3Config
 from ..config.zigivik import ZigivikConfig
 from ..registry import register_architecture
@@ -13,4 +14,5 @@ register_architecture("Lemesun", LemesunConfig)
 register_architecture("Losivik", LosivikConfig)
 register_architecture("Noganex", NoganexConfig)
 register_architecture("Nulalorn", NulalornConfig)
+register_architecture("Pukinex", PukinexConfig)
 register_architecture("Zigivik", ZigivikConfig)

@@ -64,6 +64,16 @@ context how (``ctx.key_splits(blocks_per_cut) -> (tiles_per_split, splits)``): t
 that a block takes, as one int32 on the device that follows the step's sequences (also under graph replay,
 where the host refreshes it), and a bound on the cuts of one sequence, which is what a captured graph fixes.
 
+Also optional: mixers that read the same input may share their products (``parts/side_by_side.py``).  A mixer with
+``joins = True`` keeps, after ``load``, its input rows as ``w_in`` [rows, hidden] with ``b_in`` (fp32 or None), a multiple
+of 8 rows, and its output matrix as ``w_o`` [hidden, lanes]; ``heads_into(proj, col, ctx, view, out, out_col, scale)``
+does everything between the two products: it reads its input product in the columns of ``proj`` from ``col`` on and
+writes its ``lanes`` columns, times ``scale``, to those of ``out`` from ``out_col`` on.
+
+A block of several parallel residual streams (``parts/block.py: StreamMixBlock``) works on [tokens, streams * hidden]
+and leaves its last update pending as a ``StreamUpdate`` (``parts/linear.py``), which the next norm of such a block or
+``flush_residual_add`` finishes.
+
 Parts are chosen by the *type* of their spec.  ``register_part(SpecType, PartClass)``
 adds a kind; nothing else in the library has to change for it.
 """

@@ -5,7 +5,8 @@ from __future__ import annotations
 import torch
 
 from ..cache import StateNeed
-from ..config.specs import GatedPostNormBlockSpec, ParallelBlockSpec, PreNormBlockSpec, ReinjectSpec, SandwichBlockSpec, ScaledParallelBlockSpec
+from ..config.specs import GatedPostNormBlockSpec, ParallelBlockSpec, PreNormBlockSpec, ReinjectSpec, SandwichBlockSpec, ScaledParallelBlockSpec, StreamMixBlockSpec
+from ..kernels.ops import STREAM_MIX_MAX_STREAMS, STREAM_MIX_MAX_WIDTH
 from ..weights.tensors import TensorDecl
 from .base import Part, build_part, register_part
 
@@ -401,6 +402,92 @@ class ScaledParallelBlock(Part):
                 self.after.forward(hidden, ctx)
 
 
+class StreamMixBlock(Part):
+    """Parallel residual streams (hyper-connections): u = sum_s in[s] x_s; y = sublayer(norm(u)); then, all at once,
+    x_t <- sum_s mix[s, t] x_s + m out[t] y; the mixer first, then the feed-forward.
+
+    ``hidden`` is [tokens, streams * hidden].  A sublayer's fp32 output is left pending (:class:`~.linear.StreamUpdate`) and
+    the next norm, of this or the following block of this kind, mixes the streams, sums its input and norms it in one
+    pass (``ops.stream_mix``); the model finishes the last one.  A part that says ``returns_output`` returns its output;
+    any other adds into a zeroed buffer."""
+
+    finishes_residual_adds = True     # its norms take over an update that the block before left pending
+
+    def __init__(self, spec: StreamMixBlockSpec) -> None:
+        super().__init__(spec)
+        has = spec.ffn is not None
+        if has != (spec.ffn_norm is not None) or (not has and spec.ffn_names is not None):
+            raise ValueError("a feed-forward comes with its norm (and perhaps its stream coefficients), or none of them")
+        if spec.streams < 1 or spec.streams > STREAM_MIX_MAX_STREAMS or spec.hidden_size > STREAM_MIX_MAX_WIDTH:
+            raise ValueError(f"the stream kernel takes 1 to {STREAM_MIX_MAX_STREAMS} streams of up to {STREAM_MIX_MAX_WIDTH} lanes")
+        if spec.streams > 1 and (spec.mixer_names is None or (has and spec.ffn_names is None)):
+            raise ValueError("several streams need their coefficients' tensors")
+        self.mixer_norm = build_part(spec.mixer_norm)
+        self.mixer = build_part(spec.mixer)
+        self.ffn_norm = build_part(spec.ffn_norm) if has else None
+        self.ffn = build_part(spec.ffn) if has else None
+        for norm in (self.mixer_norm, self.ffn_norm):
+            if norm is not None and not (hasattr(norm.spec, "bias_name") and norm.spec.streams == 1):
+                raise TypeError("this block's norms are layer norms of one stream's width")
+
+    def _children(self):
+        return tuple(part for part in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if part is not None)
+
+    def tensor_decls(self):
+        s = self.spec
+        decls = [d for part in self._children() for d in part.tensor_decls()]
+        for named in (s.mixer_names, s.ffn_names):
+            if named is not None:
+                decls += [TensorDecl(named[0], (s.streams,), "one_plus_normal"), TensorDecl(named[1], (s.streams,), "one_plus_normal"),
+                          TensorDecl(named[2], (s.streams, s.streams))]
+        return decls
+
+    def load(self, fetch, runtime) -> None:
+        self.runtime = runtime
+        for part in self._children():
+            part.load(fetch, runtime)
+        coefficients = lambda named: (None, None, None) if named is None else tuple(fetch.vector(name) for name in named)
+        self.mixer_coef, self.ffn_coef = coefficients(self.spec.mixer_names), coefficients(self.spec.ffn_names)
+
+    def cache_needs(self):
+        return tuple(self.mixer.cache_needs())
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(part, "graph_safe", False) for part in self._children())
+
+    def _half(self, hidden, ctx, part, norm, coefficients, call):
+        from ..kernels import ops
+        from .linear import StreamUpdate, flush_residual_add
+        s = self.spec
+        in_coef, out_coef, mix = coefficients
+        n = hidden.shape[0]
+        x = torch.empty((n, s.hidden_size), dtype=self.runtime.dtype, device=hidden.device)
+        read = dict(in_coef=in_coef, weight=norm.weight, bias=norm.bias, eps=norm.spec.eps, out=x)
+        pending = ctx.pending_residual_add
+        if isinstance(pending, StreamUpdate) and pending.hidden is hidden:
+            ctx.pending_residual_add = None
+            pending.finish(**read)
+        else:
+            flush_residual_add(ctx)
+            ops.stream_mix(hidden, streams=s.streams, **read)
+        if getattr(part, "returns_output", False):
+            y = call(x, None)
+        else:
+            y = torch.zeros((n, s.hidden_size), dtype=torch.float32, device=hidden.device)
+            call(x, y)
+        ctx.residual_sumsq = None
+        ctx.pending_residual_add = StreamUpdate(hidden, y, s.streams, mix, out_coef, s.residual_mult)
+
+    def forward(self, hidden, ctx, view) -> None:
+        ctx.defers_residual_add = False        # the parts' own products add (or return) at once
+        self._half(hidden, ctx, self.mixer, self.mixer_norm, self.mixer_coef,
+                   lambda x, residual: self.mixer.forward(x, ctx, view, residual))
+        if self.ffn is not None:
+            self._half(hidden, ctx, self.ffn, self.ffn_norm, self.ffn_coef,
+                       lambda x, residual: self.ffn.forward(x, ctx, residual))
+
+
 class Reinject(Part):
     """h <- W [h ; e] + steps[index], e the embedding's output (``ctx.embedded``): what opens a pass of a looped
     stack.  It keeps no cache and returns the new stream (the model goes on with what a layer returns)."""
@@ -435,4 +522,5 @@ register_part(SandwichBlockSpec, SandwichBlock)
 register_part(GatedPostNormBlockSpec, GatedPostNormBlock)
 register_part(ParallelBlockSpec, ParallelBlock)
 register_part(ScaledParallelBlockSpec, ScaledParallelBlock)
+register_part(StreamMixBlockSpec, StreamMixBlock)
 register_part(ReinjectSpec, Reinject)

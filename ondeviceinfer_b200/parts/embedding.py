@@ -26,13 +26,16 @@ class TokenEmbedding(Part):
     then pass it, in fp32 (a norm that scales in fp32).  With ``sinusoid_base`` in the spec the rows are multiplied
     by ``scale`` and get an absolute sinusoidal position vector in the same kernel: the frequencies
     base^(-2i / hidden) are computed here in double and rounded once, the angle position * frequency and its sine
-    and cosine are fp32 on the device."""
+    and cosine are fp32 on the device.  With ``streams`` in the spec a row is written that many times side by side."""
 
     graph_safe = True
 
     def __init__(self, spec) -> None:
         super().__init__(spec)
         self.norm = build_part(spec.norm) if getattr(spec, "norm", None) is not None else None
+        self.streams = int(getattr(spec, "streams", 1))
+        if self.streams < 1 or (self.streams > 1 and (self.norm is not None or getattr(spec, "sinusoid_base", None) is not None)):
+            raise ValueError("parallel streams go with a plain embedding (no positions, no norm)")
 
     def tensor_decls(self):
         decls = [TensorDecl(self.spec.weight_name, (self.spec.vocab_size, self.spec.hidden_size))]
@@ -50,15 +53,13 @@ class TokenEmbedding(Part):
             H = self.spec.hidden_size
             self.inv_freq = torch.tensor([float(base) ** (-2.0 * i / H) for i in range((H + 1) // 2)],
                                          dtype=torch.float64).to(torch.float32).to(runtime.device)
-        elif self.scale != 1.0:
-            raise ValueError("a scaled embedding without positions is not implemented")
 
     def forward(self, ctx) -> torch.Tensor:
-        hidden = torch.empty((ctx.n_tokens, self.spec.hidden_size), dtype=torch.float32, device=self.runtime.device)
+        hidden = torch.empty((ctx.n_tokens, self.streams * self.spec.hidden_size), dtype=torch.float32, device=self.runtime.device)
         if self.inv_freq is not None:
             ops.embed_sinusoid(self.table, ctx.token_ids, ctx.tok_pos, self.inv_freq, hidden, self.scale)
         else:
-            ops.embed(self.table, ctx.token_ids, hidden)
+            ops.embed(self.table, ctx.token_ids, hidden, self.scale, self.streams)
         if self.norm is not None:
             return self.norm(hidden, out_dtype=torch.float32)
         return hidden

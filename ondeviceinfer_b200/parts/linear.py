@@ -17,7 +17,7 @@ kernels.  The library also takes shapes the tcgen05 kernels refuse (K not a mult
 
 from __future__ import annotations
 
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 
@@ -49,7 +49,7 @@ def _persistent(tokens: int, weight: torch.Tensor, x: torch.Tensor, epi: int, bi
         return False
     if PREFILL_GEMM == "own":
         return True
-    fused = biased or epi in (ops.EPI_SWIGLU, ops.EPI_GEGLU, ops.EPI_RESIDUAL, ops.EPI_GELU)      # a bias is a fused epilogue too
+    fused = biased or epi in (ops.EPI_SWIGLU, ops.EPI_GEGLU, ops.EPI_RESIDUAL, ops.EPI_GELU, ops.EPI_RELU2)      # a bias is a fused epilogue too
     return tokens >= (PERSISTENT_MIN_TOKENS_FUSED if fused else PERSISTENT_MIN_TOKENS_PLAIN)
 
 
@@ -248,14 +248,32 @@ def linear(x, weight: torch.Tensor, *, bias: Optional[torch.Tensor] = None, resi
     return y
 
 
+class StreamUpdate(NamedTuple):
+    """An update of parallel residual streams that is still to be done: x_t <- sum_s mix[s, t] x_s + m out_coef[t] y for the
+    streams side by side in ``hidden`` (None coefficients: the identity)."""
+
+    hidden: torch.Tensor
+    y: torch.Tensor
+    streams: int
+    mix: Optional[torch.Tensor]
+    out_coef: Optional[torch.Tensor]
+    m: float
+
+    def finish(self, **norm) -> None:
+        """Do it; ``norm`` (in_coef, weight, bias, eps, out): with the layer norm that reads the new streams."""
+        ops.stream_mix(self.hidden, streams=self.streams, y=self.y, mix=self.mix, out_coef=self.out_coef, m=self.m, **norm)
+
+
 def flush_residual_add(ctx) -> None:
     """Do a residual add that was left pending on ``ctx`` (nothing if there is none): ``(residual, product)`` from
     :func:`linear`, or ``(residual, output, weight, eps)`` from a block that norms a sublayer's fp32 output before
-    it adds it (residual += output * rsqrt(mean(output^2) + eps) * weight)."""
+    it adds it (residual += output * rsqrt(mean(output^2) + eps) * weight), or a :class:`StreamUpdate`."""
     pending = getattr(ctx, "pending_residual_add", None)
     if pending is not None:
         ctx.pending_residual_add = None
-        if len(pending) == 4:
+        if isinstance(pending, StreamUpdate):
+            pending.finish()
+        elif len(pending) == 4:
             ops.rmsnorm_add(*pending)
         else:
             ops.residual_add(*pending)
@@ -315,18 +333,19 @@ def project_heads(x, weight_qkv: torch.Tensor, head_prep, bias: Optional[torch.T
 
 
 def activated_linear(x: torch.Tensor, weight: torch.Tensor, kind: str) -> torch.Tensor:
-    """act(x W^T) in the dtype of ``x``; ``kind`` "gelu_erf" or "gelu_tanh".  The exact GELU of bfloat16 products
-    is the epilogue of the tensor-core kernels (taken on the fp32 sum, one rounding); otherwise the product is
-    followed by the activation kernel."""
+    """act(x W^T) in the dtype of ``x``; ``kind`` "gelu_erf", "gelu_tanh" or "relu2".  The exact GELU and the squared ReLU
+    of bfloat16 products are the epilogue of the tensor-core kernels (taken on the fp32 sum, one rounding); otherwise the
+    product is followed by the activation kernel."""
     n, N = x.shape[0], weight.shape[0]
-    if kind == "gelu_erf" and x.dtype == torch.bfloat16:
+    epi = {"gelu_erf": ops.EPI_GELU, "relu2": ops.EPI_RELU2}.get(kind)
+    if epi is not None and x.dtype == torch.bfloat16:
         if _own(x, weight):
             out = torch.empty((n, N), dtype=torch.bfloat16, device=x.device)
-            ops.gemm_bf16(x, weight, out, ops.EPI_GELU)
+            ops.gemm_bf16(x, weight, out, epi)
             return out
-        if _persistent(n, weight, x, ops.EPI_GELU):
+        if _persistent(n, weight, x, epi):
             out = torch.empty((n, N), dtype=torch.bfloat16, device=x.device)
-            ops.gemm_prefill_bf16(x, weight, out, ops.EPI_GELU)
+            ops.gemm_prefill_bf16(x, weight, out, epi)
             return out
     out = linear(x, weight)
     ops.activation(out, out, kind)

@@ -4,7 +4,7 @@ from __future__ import annotations
 
 import torch
 
-from ..config.specs import RMSNormSpec
+from ..config.specs import LayerNormSpec, RMSNormSpec
 from ..kernels import ops
 from ..weights.tensors import TensorDecl
 from .base import Part, register_part
@@ -67,4 +67,28 @@ class RMSNorm(Part):
         return out
 
 
+class LayerNorm(Part):
+    """(x - mean) / sqrt(var + eps) * weight + bias of each row, or of the sum of the ``streams`` that a row holds side by
+    side; all in fp32, rounded once (``csrc/stream_mix.cu``)."""
+
+    graph_safe = True
+
+    def tensor_decls(self):
+        return [TensorDecl(self.spec.weight_name, (self.spec.size,), "one_plus_normal"),
+                TensorDecl(self.spec.bias_name, (self.spec.size,))]
+
+    def load(self, fetch, runtime) -> None:
+        self.runtime = runtime
+        self.weight, self.bias = fetch.vector(self.spec.weight_name), fetch.vector(self.spec.bias_name)
+        if self.spec.output_scale != 1.0:
+            self.weight, self.bias = self.weight * self.spec.output_scale, self.bias * self.spec.output_scale
+
+    def __call__(self, x: torch.Tensor, rows=None, out_dtype=None) -> torch.Tensor:
+        n = x.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, self.spec.size), dtype=out_dtype or self.runtime.dtype, device=x.device)
+        ops.stream_mix(x, streams=self.spec.streams, weight=self.weight, bias=self.bias, eps=self.spec.eps, out=out, rows=rows)
+        return out
+
+
 register_part(RMSNormSpec, RMSNorm)
+register_part(LayerNormSpec, LayerNorm)

@@ -61,6 +61,8 @@ class Rotary(Part):
         super().__init__(spec)
         if spec.dim % 2 != 0 or spec.dim > spec.head_dim or spec.dim <= 0:
             raise ValueError(f"rotary_dim must be even and at most head_dim, got {spec.dim} of {spec.head_dim}")
+        if spec.linear_factor is not None and (spec.scaling is not None or spec.index_ramp is not None or spec.linear_factor <= 0):
+            raise ValueError("linear_factor is positive and goes without the other ways to slow the frequencies")
         self.rot_dim = spec.dim
         self.interleaved = spec.interleaved     # which lanes pair up; the tables are the same either way
 
@@ -76,6 +78,9 @@ class Rotary(Part):
             exact = [float(self.spec.theta) ** (-2.0 * i / self.rot_dim) for i in range(self.rot_dim // 2)]
             ramped, self.magnitude = ramped_frequencies(exact, float(self.spec.theta), self.rot_dim, self.spec.index_ramp)
             inv_freq = torch.tensor(ramped, dtype=torch.float64).to(torch.float32)
+        if self.spec.linear_factor is not None:
+            inv_freq = torch.tensor([float(self.spec.theta) ** (-2.0 * i / self.rot_dim) / self.spec.linear_factor
+                                     for i in range(self.rot_dim // 2)], dtype=torch.float64).to(torch.float32)
         self.inv_freq = inv_freq.to(runtime.device)
 
     def rotary_tables(self, ctx):
