@@ -34,7 +34,7 @@ lengths and with temperature sampling.  One JSON line is printed:
 on the same configuration, and prints the same line with ``"impl": "reference"``.  Nothing of
 this library is imported in that arm.
 
-``--design lemesun`` (or ``nulalorn``, ``zigivik``, ``losivik``, ``noganex``) leaves the default workload alone and measures that architecture instead: prefill and
+``--design lemesun`` (or ``nulalorn``, ``zigivik``, ``losivik``, ``noganex``, ``pukinex``) leaves the default workload alone and measures that architecture instead: prefill and
 decode throughput at layer sizes like a real model's beside the dense model of equal width, one JSON line
 (``run_design_points``).
 
@@ -661,6 +661,28 @@ def _noganex_config(width, heads, kv_heads, dim, chunk, delta_heads, delta_kv, d
             "layers": [attention, delta, attention, delta]}
 
 
+def _pukinex_config(width, heads, kv_heads, dim, ret_heads, ret_dim, bias_max, ff, vocab):
+    """Four layers: biased attention beside retention, attention whose values are its keys, and both once more; two residual
+    streams, no loop (so that the weights read are those of four layers)."""
+    pair = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff},
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "bias_rows": 32,
+                               "bias_max": bias_max, "q_temp": {"coef": 0.1, "every": 1024}},
+                      "right": {"heads": ret_heads, "dim": ret_dim, "vdim": ret_dim, "rot": {"base": 10000.0, "dims": ret_dim},
+                                "decay": [1.0 - 2.0 ** (-5.0 - 4.0 * i / ret_heads) for i in range(ret_heads)]},
+                      "left_scale": 0.5, "right_scale": 0.5}}
+    attention = {"type": "attention", "mlp": {"kind": "dense", "ff": ff},
+                 "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
+                           "rot": {"base": 10000.0, "dims": dim // 2, "scaling": {"factor": 4.0}}}}
+    return {"architecture": "Pukinex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "residual_mult": 0.5, "streams": 2, "logit_scale": 0.5, "logit_softcap": 30.0, "layers": [pair, attention, pair, attention]}
+
+
+# the dense model's gated feed-forward has three matrices a layer, this design's two: half as wide again they weigh the same
+PUKINEX_POINTS = {
+    "w2048": (_pukinex_config(2048, 16, 4, 128, 16, 128, 512, 7680, 32768), _dense_config(2048, 16, 5 * 1024, 4, 32768)),
+    "w4096": (_pukinex_config(4096, 32, 8, 128, 32, 128, 512, 18432, 32768), _dense_config(4096, 32, 12288, 4, 32768)),
+}
+
 NOGANEX_POINTS = {
     "w2048": (_noganex_config(2048, 16, 4, 128, 1024, 16, 8, 128, 32, 4, 1024, 1024, 5 * 1024, 32768),
               _dense_config(2048, 16, 5 * 1024, 4, 32768)),
@@ -734,7 +756,7 @@ def _time_parts(model, cache, slots, runs, torch):
 
 
 def run_design_points(args) -> int:
-    """``--design lemesun|nulalorn|zigivik|losivik|noganex``: prefill and decode throughput of that design at layer sizes like a real model's
+    """``--design lemesun|nulalorn|zigivik|losivik|noganex|pukinex``: prefill and decode throughput of that design at layer sizes like a real model's
     (random weights), each beside the dense Qwen3 model of equal width, heads, layer executions and active
     feed-forward width, with the device time of every mixer and feed-forward call.  One JSON line; the default
     workload is untouched."""
@@ -752,7 +774,8 @@ def run_design_points(args) -> int:
     points = {}
     sampler = ClockSampler()
     sampler.start()
-    design_points = {"nulalorn": NULALORN_POINTS, "zigivik": ZIGIVIK_POINTS, "losivik": LOSIVIK_POINTS, "noganex": NOGANEX_POINTS}.get(args.design, DESIGN_POINTS)
+    design_points = {"nulalorn": NULALORN_POINTS, "zigivik": ZIGIVIK_POINTS, "losivik": LOSIVIK_POINTS, "noganex": NOGANEX_POINTS,
+                     "pukinex": PUKINEX_POINTS}.get(args.design, DESIGN_POINTS)
     for name, configs in design_points.items():
         if args.design_points and name not in args.design_points.split(","):
             continue
@@ -837,7 +860,7 @@ def main() -> int:
     parser.add_argument("--prompt-range", default=None, metavar="LOW,HIGH",
                         help="unequal prompts: lengths uniform in [LOW, HIGH] from --seed instead of --prompt-len")
     parser.add_argument("--context", type=int, default=None, help="cache positions per sequence (default 4096, or what the prompt needs)")
-    parser.add_argument("--design", default=None, choices=["lemesun", "nulalorn", "zigivik", "losivik", "noganex"],
+    parser.add_argument("--design", default=None, choices=["lemesun", "nulalorn", "zigivik", "losivik", "noganex", "pukinex"],
                         help="instead of the default workload: this design at real layer sizes beside the dense model of equal size")
     parser.add_argument("--design-points", default=None, help="which of the design's sizes, with commas (default: all)")
     args = parser.parse_args()

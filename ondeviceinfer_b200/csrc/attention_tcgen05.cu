@@ -105,7 +105,7 @@ struct TcAttnArgs {
   int chunk;              // > 0: keys of the query's own chunk of this many positions
   int mixed;              // 1: a score sums over the key heads (q has nkv rows of D lanes a head)
   HeadOut ho;
-  DistanceBias rel;       // with one head per CTA
+  DistanceBias rel;       // (with a gate or a bias: one head per CTA, heads unmixed)
 };
 
 #define REL_PAD 64        // entries in front of and behind a head's biases in shared memory
@@ -281,6 +281,7 @@ __device__ __forceinline__ void umma_a_tmem(uint32_t d_tmem, uint32_t a_tmem, ui
 // `oldest` is the first key the row still sees (0 without a window).  With a cap (two_over_cap > 0) the score
 // times `scale` is squashed first, as c (1 - 2 / (e^(2 x / c) + 1)) = c tanh(x / c), and sl2 is log2(e) alone.
 struct RowState { float m_used, l; };
+template <bool REL>
 __device__ __forceinline__ bool softmax_keys64(uint32_t s_addr, uint32_t p_addr, uint32_t o_addr, int kbase, int pos, float sl2,
                                                int n, uint32_t pv_done, RowState& st, volatile int* abort_ptr,
                                                int oldest = 0, float scale = 1.f, float cap = 0.f, float two_over_cap = 0.f,
@@ -291,7 +292,7 @@ __device__ __forceinline__ bool softmax_keys64(uint32_t s_addr, uint32_t p_addr,
 #pragma unroll
     for (int i = 0; i < BNK; ++i) s[i] = cap * (1.f - __fdividef(2.f, __expf(s[i] * scale * two_over_cap) + 1.f));
   }
-  if (rel != nullptr) {
+  if (REL) {
     // entry REL_PAD + n of `rel` is the bias of distance n in log2 units; sl2 is 1, the scores' factor is `pre`
     const float pre = cap > 0.f ? LOG2E : scale * LOG2E;
     if (__all_sync(0xffffffffu, pos - (kbase + BNK - 1) >= rel_n - 1)) {
@@ -360,10 +361,12 @@ __device__ __forceinline__ bool softmax_keys64(uint32_t s_addr, uint32_t p_addr,
 }
 
 // The finished row of O, divided by the row's sum, as bf16 to dst (D elements).
+template <bool GATED>
 __device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, bool valid, const HeadOut& ho, size_t tok, int head) {
   float inv = l > 0.f ? 1.f / l : 0.f;
   const bf16* gate = nullptr;              // a gate per lane: this head's lanes of the token's gate row
-  if (valid) {
+  if (!GATED) inv *= ho.scale;
+  else if (valid) {
     if (ho.gate != nullptr && !ho.gate_per_head) { gate = (const bf16*)ho.gate + tok * ho.gate_ld + head * D; inv *= ho.scale; }
     else inv *= head_out_factor<bf16>(ho, tok, head, D, 0);
   }
@@ -375,7 +378,7 @@ __device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, b
 #pragma unroll
       for (int i = 0; i < 32; i += 8) {
         uint32_t w[4];
-        if (gate != nullptr) {
+        if (GATED && gate != nullptr) {
           const uint4 raw = *(const uint4*)(gate + c + i);
           const __nv_bfloat162* z = (const __nv_bfloat162*)&raw;
 #pragma unroll
@@ -396,7 +399,8 @@ __device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, b
   }
 }
 
-template <int TILES, bool MIXED, int QROWS>
+// SHAPED: the scores may have a bias by distance and the output a gate (a form of its own: both take registers).
+template <int TILES, bool MIXED, int QROWS, bool SHAPED>
 __global__ void __launch_bounds__(64 + 128 * TILES, TILES == 1 && !MIXED ? 2 : 1)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                          const __grid_constant__ CUtensorMap map_v, const TcAttnArgs a) {
@@ -438,7 +442,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const int KH = MIXED ? a.nkv : 1;                          // key heads a score sums over
   uint8_t* k_smem = smem + TILES * KH * Q_TILE;              // ring of K pages
   uint8_t* v_smem = k_smem + KRING * KV_BYTES;            // ring of V pages
-  const bool has_rel = TILES == 1 && a.rel.table != nullptr;
+  const bool has_rel = SHAPED && a.rel.table != nullptr;
   float* rel_smem = (float*)(v_smem + RING * KV_BYTES);      // the head's biases by distance, in log2 units
   if (has_rel) {
     const float* src = a.rel.table + (size_t)head0 * a.rel.n;       // a weight: no earlier kernel writes it
@@ -569,8 +573,14 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       tc_fence_after();
       const uint32_t s_addr = tmem_base + lane_addr + S_COL(tile, b);
       // P_j goes over the first 32 columns of this row's scores
-      if (!softmax_keys64(s_addr, s_addr, o_addr, tile_of(j) * BNK, pos, sl2, j, my_pv_done, st, abort_ptr, oldest, a.scale,
-                          a.softcap, two_over_cap, a.keep, has_rel ? rel_smem : nullptr, a.rel.n)) { ok = false; break; }
+      if (SHAPED && has_rel) {
+        ok = softmax_keys64<true>(s_addr, s_addr, o_addr, tile_of(j) * BNK, pos, sl2, j, my_pv_done, st, abort_ptr, oldest, a.scale,
+                                  a.softcap, two_over_cap, a.keep, rel_smem, a.rel.n);
+      } else {
+        ok = softmax_keys64<false>(s_addr, s_addr, o_addr, tile_of(j) * BNK, pos, sl2, j, my_pv_done, st, abort_ptr, oldest, a.scale,
+                                   a.softcap, two_over_cap, a.keep);
+      }
+      if (!ok) break;
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(my_p_full + 8 * b);
@@ -578,7 +588,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     if (ok && !mbar_wait(my_pv_done, (uint32_t)(n_tiles - 1) & 1u, abort_ptr)) ok = false;
     tc_fence_after();
     if (!ok && lane == 0) atomicCAS(a.status, 0, ATT_ERR_SOFTMAX);
-    if (ok) write_row(o_addr, a.out + (size_t)(q_begin + t0 + row) * a.ho.out_ld + head * D, st.l, row < nt, a.ho, q_begin + t0 + row, head);
+    if (ok) write_row<SHAPED>(o_addr, a.out + (size_t)(q_begin + t0 + row) * a.ho.out_ld + head * D, st.l, row < nt, a.ho, q_begin + t0 + row, head);
     tc_fence_before();
   }
   __syncthreads();
@@ -636,13 +646,13 @@ extern "C" int odi_attention_tcgen05_bias_entries() { return (SMEM_LIMIT - (Q_BY
 
 // q [n_tokens, nq * D] bf16; k_pool, v_pool [pool_pages, nkv, 64, D] bf16; out [n_tokens, nq * D].
 // heads_per_cta: 2 = two heads of a key/value group per CTA (needs an even group size), 1 = one, 0 = choose.
-template <int TILES, bool MIXED, int QROWS = BM>
+template <int TILES, bool MIXED, int QROWS = BM, bool SHAPED = false>
 static int launch_attention(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnArgs& a,
                             int max_q_len, cudaStream_t stream) {
   const int smem = TILES * (MIXED ? a.nkv : 1) * (KB * QROWS * 128) + ((MIXED ? MIXED_KEY_RING : RING) + RING) * KV_BYTES + 1024 +
                    (a.rel.table != nullptr ? (a.rel.n + 2 * REL_PAD) * 4 : 0);
   if (smem > SMEM_LIMIT) return ODI_ERR_UNSUPPORTED;
-  auto kernel = attention_tcgen05_kernel<TILES, MIXED, QROWS>;
+  auto kernel = attention_tcgen05_kernel<TILES, MIXED, QROWS, SHAPED>;
   static int configured = 0;
   if (configured < smem) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -667,7 +677,8 @@ extern "C" int odi_attention_tcgen05(const void* q, const void* k_pool, const vo
   if (a.rel.table != nullptr && (a.rel.n < 1 || a.rel.n > odi_attention_tcgen05_bias_entries())) return ODI_ERR_UNSUPPORTED;
   if (a.ho.out_ld % 8 != 0 || (a.ho.gate != nullptr && !a.ho.gate_per_head && (a.ho.gate_ld % 8 != 0 || ((uintptr_t)a.ho.gate & 15))))
     return ODI_ERR_UNSUPPORTED;
-  if (a.rel.table != nullptr && heads_per_cta == 2) return ODI_ERR_UNSUPPORTED;
+  const bool shaped = a.rel.table != nullptr || a.ho.gate != nullptr;
+  if (shaped && (heads_per_cta == 2 || a.mixed)) return ODI_ERR_UNSUPPORTED;
   if (heads_per_cta < 0 || heads_per_cta > 2 || a.chunk < 0 || (a.chunk > 0 && (a.window > 0 || a.keep > 0))) return ODI_ERR_ARGUMENT;
   if (a.mixed && heads_per_cta == 2) return ODI_ERR_UNSUPPORTED;
   if (heads_per_cta == 2 && (a.nq / a.nkv) % 2 != 0) return ODI_ERR_ARGUMENT;
@@ -678,10 +689,11 @@ extern "C" int odi_attention_tcgen05(const void* q, const void* k_pool, const vo
   if (rc == 0) rc = make_map(&mk, k_pool, pool_pages * a.nkv * BNK, D, BNK);
   if (rc == 0) rc = make_map(&mv, v_pool, pool_pages * a.nkv * BNK, D, BNK);
   if (rc != 0) return rc;
-  if (heads_per_cta == 0) heads_per_cta = a.rel.table != nullptr ? 1 : ODI_ATT_DEFAULT_HEADS_PER_CTA;
+  if (heads_per_cta == 0) heads_per_cta = shaped ? 1 : ODI_ATT_DEFAULT_HEADS_PER_CTA;
   if (a.mixed)
     return q_rows == BM ? launch_attention<1, true>(mq, mk, mv, a, max_q_len, stream)
                         : launch_attention<1, true, 64>(mq, mk, mv, a, max_q_len, stream);
+  if (shaped) return launch_attention<1, false, BM, true>(mq, mk, mv, a, max_q_len, stream);
   return heads_per_cta == 2 ? launch_attention<2, false>(mq, mk, mv, a, max_q_len, stream)
                             : launch_attention<1, false>(mq, mk, mv, a, max_q_len, stream);
 }

@@ -169,6 +169,8 @@ ALL_SOURCES = {
     "ssd": [{}],
     "mixed": [{}],
     "delta_head": [{}],
+    "retention": [{}],
+    "stream_mix": [{}],
     "attention_mixed_mma": [{"ODI_HEAD_DIM": 128, "ODI_VALUE_DIM": 128}],
     "attention_capped_mma": [{"ODI_HEAD_DIM": 128, "ODI_VALUE_DIM": 128}],
     "attention_latent_mma": [{"ODI_HEAD_DIM": 576, "ODI_VALUE_DIM": 512}],      # a latent cache, on the tensor cores

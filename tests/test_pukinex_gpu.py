@@ -1,0 +1,668 @@
+"""The Pukinex design in the engine against its plain restatement (``plain_pukinex``): each mechanism alone, whole prompts,
+token-by-token decoding, portions, batches of unequal requests, slots and pages used again, far keys, page borders, the
+edges of distance buckets, the first tokens, long decoding, looped layers, sizes off every multiple, and greedy
+generation through ``generate`` and the command line.
+
+float32 is compared strictly, bfloat16 by the error of a row relative to the row's size."""
+
+import copy
+import json
+import math
+import subprocess
+import sys
+from pathlib import Path
+
+import pytest
+import torch
+
+import ondeviceinfer_b200 as odi
+import plain_pukinex as plain
+from helpers import F32_ATOL, F32_RTOL, write_model_folder
+from ondeviceinfer_b200.kernels import ops
+from ondeviceinfer_b200.parts.capped_attention import distance_entries
+from ondeviceinfer_b200.parts.linear import activated_linear, flush_residual_add
+
+pytestmark = pytest.mark.gpu
+DTYPES = ["float32", "bfloat16"]
+KINDS = [torch.float32, torch.bfloat16]
+CONFIGS = {"A": (plain.TINY_A, 71), "B": (plain.TINY_B, 72), "C": (plain.TINY_C, 73), "D": (plain.TINY_D, 74),
+           "sharp": (plain.SHARP, 75)}
+SHARPEN = {"sharp": 4.0}
+_MODELS, _PLAIN = {}, {}
+
+
+def weights_of(case):
+    return plain.random_weights(*CONFIGS[case], sharpen=SHARPEN.get(case, 1.0))
+
+
+def engine(case, dtype, tmp_path_factory):
+    if (case, dtype) not in _MODELS:
+        folder = write_model_folder(tmp_path_factory.mktemp(f"pukinex_{case}"), CONFIGS[case][0], weights_of(case))
+        _MODELS[(case, dtype)] = odi.load_resident_model(folder, dtype=dtype)
+    return _MODELS[(case, dtype)]
+
+
+def expected(case, tokens):
+    key = (case, tuple(tokens))
+    if key not in _PLAIN:
+        _PLAIN[key] = plain.forward(CONFIGS[case][0], weights_of(case), list(tokens)).float()
+    return _PLAIN[key]
+
+
+def close(actual, reference, dtype, what, atol=None):
+    """float32: |d| <= ``atol``, or the helpers' bound plus a term for the size of the logits.  bfloat16: row error relative
+    to the row's size: of ten rows and more the median at most 2.5e-2 and nine in ten within 6e-2, and every row within
+    4e-1: a retention read-out of a sequence's first positions is a sum of few terms, and where they nearly cancel its norm
+    magnifies the roundings of the projections."""
+    actual, reference = actual.float().cpu(), reference.float().cpu()
+    assert actual.shape == reference.shape and torch.isfinite(actual).all(), what
+    if dtype == "float32":
+        gap = (actual - reference).abs()
+        bound = F32_ATOL + F32_RTOL * reference.abs() + 1e-5 * float(reference.abs().max()) if atol is None else torch.tensor(atol)
+        assert not (gap > bound).any(), f"{what}: fp32 max |d| = {float(gap.max()):.3e} at logits up to {float(reference.abs().max()):.1f}"
+        return
+    error = (actual - reference).norm(dim=-1) / reference.norm(dim=-1).clamp_min(1e-6)
+    ranked = error.sort().values
+    high = ranked[int(0.9 * len(ranked))] if len(ranked) >= 10 else ranked[-1]
+    assert (len(ranked) < 10 or (float(error.median()) <= 2.5e-2 and float(high) <= 6e-2)) and float(ranked[-1]) <= 4e-1, \
+        f"{what}: bfloat16 row errors median {float(error.median()):.3e}, high {float(high):.3e}, max {float(ranked[-1]):.3e}"
+
+
+def ints(*values):
+    return torch.tensor(values, dtype=torch.int32, device="cuda")
+
+
+def tol(dtype):
+    return dict(atol=2e-5, rtol=1e-5) if dtype == torch.float32 else dict(atol=2e-2, rtol=2e-2)
+
+
+# ----------------------------------------------------------------------------- kernels against plain functions
+
+
+@pytest.mark.parametrize("dtype", KINDS)
+@pytest.mark.parametrize("rows,width,streams", [(1, 4, 1), (5, 37, 2), (9, 192, 2), (3, 2052, 3), (2, 9000, 4), (4, 4096, 4), (6, 104, 5),
+                                                (3, 1030, 16), (7, 8192, 2), (2, 12288, 1)])
+def test_streams_are_mixed_and_the_sum_normed(dtype, rows, width, streams):
+    gen = torch.Generator().manual_seed(rows * width)
+    X = torch.randn(streams, rows, width, generator=gen) * 3.0 + 1.5
+    X[:, 0] *= 1e-3            # eps decides beside the variance
+    y = torch.randn(rows, width, generator=gen) * 2.0
+    mix, out_c, in_c = torch.randn(streams, streams, generator=gen), torch.randn(streams, generator=gen), torch.randn(streams, generator=gen)
+    w, b = 1 + 0.3 * torch.randn(width, generator=gen), torch.randn(width, generator=gen)
+    side_by_side = lambda t: t.permute(1, 0, 2).reshape(rows, -1).contiguous()
+    D = lambda t: t.double()
+    dev = dict(mix=mix.cuda(), out_coef=out_c.cuda(), in_coef=in_c.cuda())
+    for identity in (False, True):
+        new = plain.stream_update(D(X), torch.eye(streams).double() if identity else D(mix), torch.ones(streams).double() if identity else D(out_c),
+                                  0.7, D(y))
+        u = plain.stream_input(new, torch.ones(streams).double() if identity else D(in_c))
+        stream, normed = side_by_side(X).cuda(), torch.empty(rows, width, dtype=dtype, device="cuda")
+        coef = {} if identity else dev
+        ops.stream_mix(stream, streams=streams, y=y.cuda(), m=0.7, weight=w.cuda(), bias=b.cuda(), eps=1e-5, out=normed, **coef)
+        torch.testing.assert_close(stream.cpu().double(), side_by_side(new), atol=1e-4, rtol=1e-5)
+        want = plain.layer_norm(u, D(w), D(b), 1e-5)
+        torch.testing.assert_close(normed.cpu().double(), want, **(dict(atol=1e-3, rtol=1e-4) if dtype == torch.float32 else tol(dtype)))
+        # the update alone, then the read alone, of every row and of some
+        apart = side_by_side(X).cuda()
+        ops.stream_mix(apart, streams=streams, y=y.cuda(), m=0.7, **{k: v for k, v in coef.items() if k != "in_coef"})
+        assert torch.equal(apart, stream)
+        again, some = torch.empty_like(normed), torch.empty(2, width, dtype=dtype, device="cuda")
+        read = dict(streams=streams, in_coef=coef.get("in_coef"), weight=w.cuda(), bias=b.cuda(), eps=1e-5)
+        ops.stream_mix(apart, out=again, **read)
+        torch.testing.assert_close(again, normed, atol=1e-3 if dtype == torch.float32 else 2e-2, rtol=1e-2)
+        ops.stream_mix(apart, out=some, rows=ints(rows - 1, 0), **read)
+        assert torch.equal(some, again[[rows - 1, 0]])
+        assert torch.equal(apart, stream)
+
+
+@pytest.mark.parametrize("dtype", KINDS)
+def test_scaled_embedding_rows_side_by_side(dtype):
+    gen = torch.Generator().manual_seed(2)
+    table = torch.randn(11, 37, generator=gen).to(dtype)
+    ids = [3, 10, 0, 3]
+    for copies, scale in ((1, 1.0), (2, 5.7), (3, 0.5)):
+        out = torch.empty(4, copies * 37, device="cuda")
+        ops.embed(table.cuda(), ints(*ids), out, scale, copies)
+        torch.testing.assert_close(out.cpu(), (table[ids].float() * scale).repeat(1, copies), atol=0, rtol=1e-6)
+
+
+@pytest.mark.parametrize("dtype", KINDS)
+@pytest.mark.parametrize("tokens,K,F", [(1, 64, 40), (3, 36, 50), (33, 96, 72), (200, 128, 136), (1100, 128, 200), (7, 512, 1000)])
+def test_squared_relu_products(dtype, tokens, K, F):
+    """Every form of the product: few tokens, split K, the many-token kernel, sizes that the tensor-core kernels refuse."""
+    gen = torch.Generator().manual_seed(tokens + K)
+    x = torch.randn(tokens, K, generator=gen).to(dtype)
+    w = (1.5 * torch.randn(F, K, generator=gen) / math.sqrt(K)).to(dtype)
+    want = torch.clamp(x.double() @ w.double().T, min=0) ** 2
+    torch.testing.assert_close(activated_linear(x.cuda(), w.cuda(), "relu2").cpu().double(), want,
+                               **(tol(dtype) if dtype == torch.float32 else dict(atol=4e-2, rtol=3e-2)))
+
+
+def _tables(rot, base, factor, positions):
+    if not rot:
+        return None, None
+    f = torch.tensor([base ** (-2.0 * i / rot) / factor for i in range(rot // 2)], dtype=torch.float64).float().cuda()
+    cos, sin = torch.empty(len(positions), rot // 2, device="cuda"), torch.empty(len(positions), rot // 2, device="cuda")
+    ops.rope_table(f, ints(*positions), cos, sin)
+    return cos, sin
+
+
+@pytest.mark.parametrize("dtype", KINDS)
+@pytest.mark.parametrize("d,dv,nq,nkv,rot", [(16, 8, 4, 2, 0), (6, 5, 3, 1, 4), (48, 64, 2, 2, 20), (20, 20, 12, 2, 20), (160, 160, 8, 1, 64)])
+def test_head_preparation_with_a_temperature_in_columns_of_a_wider_product(dtype, d, dv, nq, nkv, rot):
+    gen = torch.Generator().manual_seed(d)
+    n, eps, pos0, factor = 6, 1e-5, 61, 3.0                # over a page border and over edges of the temperature's steps
+    v_from_k = d == dv
+    width = (nq + nkv) * d + (0 if v_from_k else nkv * dv)
+    for col, extra, every in ((0, 0, 9), (8, 24, 64), (3, 2, 1)):
+        wide = torch.randn(n, col + width + extra, generator=gen).to(dtype)
+        x = wide[:, col:col + width].double()
+        qw, kw = 1 + 0.3 * torch.randn(d, generator=gen), 1 + 0.3 * torch.randn(d, generator=gen)
+        cos, sin = _tables(rot, 500.0, factor, range(pos0, pos0 + n))
+        q, k = x[:, :nq * d].view(n, nq, d), x[:, nq * d:(nq + nkv) * d].view(n, nkv, d)
+        v = k if v_from_k else x[:, (nq + nkv) * d:].view(n, nkv, dv)
+        if rot:
+            q, k = (plain.rotate(t, rot, 500.0, factor, first=pos0) for t in (q, k))
+        q, k = plain.rms(q, eps) * qw.double(), plain.rms(k, eps) * kw.double()
+        q = q * plain.temperature(range(pos0, pos0 + n), 0.4, every)[:, None, None]
+        lanes = -(-d // 4) * 4
+        q_out = torch.full((n, nq * lanes), 7.0, dtype=dtype, device="cuda")
+        k_pool = torch.full((2, nkv, 64, lanes), 7.0, dtype=dtype, device="cuda")
+        v_pool = torch.full((2, nkv, 64, dv), 7.0, dtype=dtype, device="cuda")
+        ops.rot_unit_prep(wide.cuda(), q_out, k_pool, v_pool, cos, sin, ints(*[0] * n), ints(*range(pos0, pos0 + n)), ints(0, 2), ints(1, 0),
+                          nq=nq, nkv=nkv, d=d, dv=dv, rot_dim=rot, page_size=64, ring_pages=0, write_kv=True, unit_eps=eps, d_store=lanes,
+                          v_from_k=v_from_k, q_weight=qw.cuda(), k_weight=kw.cuda(), q_temperature=(0.4, every), col=col)
+        got = q_out.cpu().double().view(n, nq, lanes)
+        torch.testing.assert_close(got[..., :d], q, **tol(dtype))
+        assert float(got[..., d:].abs().sum()) == 0
+        for i in range(n):
+            page, at = [1, 0][(pos0 + i) // 64], (pos0 + i) % 64
+            torch.testing.assert_close(k_pool[page, :, at, :d].cpu().double(), k[i], **tol(dtype))
+            torch.testing.assert_close(v_pool[page, :, at].cpu().double(), v[i], atol=0, rtol=0)
+
+
+# ----------------------------------------------------------------------------- attention with a sink, a distance bias and a gate
+
+
+def _pools(keys, values, n_extra_pages=3):
+    L, nkv, d = keys.shape
+    n_pages = -(-L // 64)
+    order = torch.randperm(n_pages + n_extra_pages).tolist()[:n_pages]
+    k_pool = torch.full((n_pages + n_extra_pages, nkv, 64, d), 9.0, dtype=keys.dtype)      # what nobody wrote is loud
+    v_pool = torch.full((n_pages + n_extra_pages, nkv, 64, values.shape[-1]), 9.0, dtype=values.dtype)
+    for pos in range(L):
+        k_pool[order[pos // 64], :, pos % 64] = keys[pos]
+        v_pool[order[pos // 64], :, pos % 64] = values[pos]
+    return k_pool.cuda(), v_pool.cuda(), order
+
+
+BIAS_CASES = [  # rows and reach of the table, total length, tokens of the step, splits
+    (16, 100, 150, 150, 1), (16, 100, 150, 1, 1), (16, 100, 500, 1, 4), (2, 5, 130, 130, 1), (2, 5, 65, 1, 2), (40, 300, 700, 200, 1),
+    (40, 300, 700, 1, 3), (64, 63, 257, 100, 1), (32, 4000, 400, 399, 1), (16, 100, 20, 17, 1), (16, 100, 3, 3, 1), (16, 100, 1, 1, 1),
+    (0, 0, 200, 140, 1), (0, 0, 200, 1, 2), (128, 9000, 300, 33, 1), (24000, 12001, 200, 150, 1), (24000, 12001, 200, 1, 2)]
+
+
+@pytest.mark.parametrize("kind,dtype", [("cores", torch.float32), ("cores", torch.bfloat16), ("tensor", torch.bfloat16),
+                                        ("tensor memory", torch.bfloat16)])
+@pytest.mark.parametrize("rows,reach,L,T,splits", BIAS_CASES)
+def test_attention_with_a_distance_bias_a_sink_and_a_gate(kind, dtype, rows, reach, L, T, splits):
+    """Random biases of the size of the scores at every distance, so that a key that reads its neighbour's bias moves the
+    output; outputs in columns of a wider buffer, times a factor and a gate per lane, per head or none."""
+    if kind == "tensor memory" and (T == 1 or rows > 20000):
+        pytest.skip("the form for prompts, with tables that fit shared memory")
+    gen = torch.Generator().manual_seed(rows * 1000 + L + T)
+    nq, nkv, d, dv = {"tensor memory": (4, 2, 64, 64)}.get(kind, (6, 3, 32, 16) if L % 2 else (20, 2, 16, 48))
+    past, rep, scale, cap = L - T, nq // nkv, 0.3, 8.0 if L % 3 == 0 else None
+    keys, values = torch.randn(L, nkv, d, generator=gen).to(dtype), torch.randn(L, nkv, dv, generator=gen).to(dtype)
+    q = torch.randn(T, nq, d, generator=gen).to(dtype)
+    table = 2.0 * torch.randn(max(rows, 1), nq, generator=gen)
+    rel = bias = None
+    if rows:
+        rel = table[torch.tensor(distance_entries(rows, reach))].t().contiguous().cuda()
+        bias = plain.distance_bias(table.double(), range(past, L), range(L), reach)
+    want = plain.sink_attend(q.double(), keys.double(), values.double(), scale, cap, bias)
+    gates = torch.randn(T, 8 + nq * dv + 8, generator=gen).to(dtype)
+    k_pool, v_pool, pages = _pools(keys, values)
+    partial = torch.empty(T * nq * splits * (dv + 2), device="cuda") if splits > 1 else None
+    for per_head, factor in ((None, 1.0), (True, 0.7), (False, -1.3)):
+        out = torch.full((T, 16 + nq * dv + 8), 5.0, dtype=dtype, device="cuda")
+        gate = None if per_head is None else (gates.cuda(), 8, per_head)
+        args = (q.reshape(T, -1).cuda(), k_pool, v_pool, out, ints(0, T), ints(past), ints(0, len(pages)), ints(*pages))
+        common = dict(n_seqs=1, nq=nq, nkv=nkv, d=d, page_size=64, ring_pages=0, window=0, scale=scale, softcap=cap or 0.0, sink=True,
+                      rel=rel, gate=gate, out_scale=factor, out_col=16)
+        if kind == "cores":
+            ops.attention_simt(*args, max_q_len=T, dv=dv, splits=splits, partial=partial, **common)
+        elif kind == "tensor memory":
+            assert ops.attention_tcgen05_takes(d, bias_entries=0 if rel is None else rel.shape[1], out_ld=out.shape[1], out_col=16, gate=gate)
+            ops.attention_tcgen05(*args, max_q_len=T, **common)
+        elif T == 1:
+            ops.attention_capped_decode(*args, dv=dv, splits=splits, partial=partial, **common)
+        else:
+            ops.attention_capped(*args, max_q_len=T, dv=dv, **common)
+        torch.cuda.synchronize()
+        ops.raise_on_kernel_fault()
+        z = gates.double()[:, 8:]
+        g = 1.0 if per_head is None else (torch.sigmoid(z[:, :nq])[:, :, None] if per_head else torch.sigmoid(z[:, :nq * dv]).view(T, nq, dv))
+        got = out.cpu().double()
+        assert float((got[:, 16:16 + nq * dv].view(T, nq, dv) - factor * g * want).abs().max()) < (1e-4 if dtype == torch.float32 else 4e-2)
+        assert float((got[:, :16] - 5.0).abs().max()) == 0 and float((got[:, 16 + nq * dv:] - 5.0).abs().max()) == 0
+    if 2 < rows < 1000 and T > 1 and L > rows:      # the setup shows a bias read one distance off, and a softmax without its sink
+        moved = plain.distance_bias(table.double(), range(past + 1, L + 1), range(L), reach)
+        assert float((plain.sink_attend(q.double(), keys.double(), values.double(), scale, cap, moved) - want).abs().max()) > 0.1
+        plain_softmax = torch.cat([torch.zeros(nq, T, 0).double(), bias], -1)
+        s = torch.einsum("phd,khd->hpk", q.double(), keys.double().repeat_interleave(rep, 1)) * scale
+        s = (cap * torch.tanh(s / cap) if cap else s) + plain_softmax
+        s = s.masked_fill(torch.arange(L)[None, None] > torch.arange(past, L)[None, :, None], float("-inf"))
+        bare = torch.einsum("hpk,khd->phd", torch.softmax(s, -1), values.double().repeat_interleave(rep, 1))
+        assert past > 100 or float((bare - want).abs().max()) > 0.1
+
+
+@pytest.mark.parametrize("kind", ["cores", "tensor", "tensor memory"])
+@pytest.mark.parametrize("nq,nkv,d", [(8, 4, 128), (6, 3, 64), (4, 4, 128)])
+def test_attention_of_unequal_sequences_in_one_launch(kind, nq, nkv, d):
+    gen = torch.Generator().manual_seed(3)
+    dtype, rows, reach = torch.bfloat16, 16, 120
+    table = torch.randn(rows, nq, generator=gen)
+    rel = table[torch.tensor(distance_entries(rows, reach))].t().contiguous().cuda()
+    runs, pasts = [70, 1, 200, 33], [0, 99, 40, 300]
+    seqs, qs, pools = [], [], []
+    for T, past in zip(runs, pasts):
+        L = T + past
+        keys = torch.randn(L, nkv, d, generator=gen).to(dtype)
+        values = torch.randn(L, nkv, d, generator=gen).to(dtype)
+        q = torch.randn(T, nq, d, generator=gen).to(dtype)
+        seqs.append(plain.sink_attend(q.double(), keys.double(), values.double(), d ** -0.5, None,
+                                      plain.distance_bias(table.double(), range(past, L), range(L), reach)))
+        qs.append(q)
+        pools.append(_pools(keys, values, 0))
+    starts, cu = [0], [0]
+    for T, (_, _, order) in zip(runs, pools):
+        starts.append(starts[-1] + len(order))
+        cu.append(cu[-1] + T)
+    ids = [starts[i] + page for i, (_, _, order) in enumerate(pools) for page in order]
+    out = torch.empty(cu[-1], nq * d, dtype=dtype, device="cuda")
+    args = (torch.cat(qs).reshape(cu[-1], -1).cuda(), torch.cat([p[0] for p in pools]), torch.cat([p[1] for p in pools]), out, ints(*cu),
+            ints(*pasts), ints(*starts), ints(*ids))
+    common = dict(n_seqs=4, max_q_len=200, nq=nq, nkv=nkv, d=d, page_size=64, ring_pages=0, window=0, scale=d ** -0.5, sink=True, rel=rel)
+    if kind == "cores":
+        ops.attention_simt(*args, dv=d, **common)
+    elif kind == "tensor":
+        ops.attention_capped(*args, dv=d, **common)
+    else:
+        ops.attention_tcgen05(*args, **common)
+    torch.cuda.synchronize()
+    ops.raise_on_kernel_fault()
+    assert float((out.cpu().double().view(-1, nq, d) - torch.cat(seqs)).abs().max()) < 4e-2
+
+
+# ----------------------------------------------------------------------------- retention
+
+
+@pytest.mark.parametrize("dtype,chunked", [(torch.float32, False), (torch.bfloat16, False), (torch.bfloat16, True)])
+@pytest.mark.parametrize("decay,d,dv,rot,inter", [((0.9, 0.99, 0.5), 32, 48, 32, False), ((0.97,), 10, 7, 6, False), ((0.999, 0.0), 24, 40, 8, True),
+                                                  ((1.0, 0.95), 64, 33, 0, False), ((0.98, 0.9), 128, 128, 128, False), ((0.99,), 130, 5, 64, False),
+                                                  ((0.9, 0.8, 0.99, 0.7), 16, 130, 16, False), ((0.95,), 256, 64, 128, False),
+                                                  ((0.96,), 96, 200, 48, False)])
+def test_retention_over_cut_sequences(dtype, chunked, decay, d, dv, rot, inter):
+    """Three sequences cut into unequal runs (single tokens, short portions, several chunks, chunks with tokens left over),
+    stepped together with states in slots of their own, in columns of wider buffers, against the recurrence over each whole
+    sequence.  The chunked form in bfloat16 is held to more than bfloat16's accuracy before its one rounding."""
+    gen = torch.Generator().manual_seed(d + dv)
+    H = len(decay)
+    m = {"heads": H, "dim": d, "vdim": dv, "decay": decay}
+    lengths, col, out_col, eps = [233, 3, 99], 8, 16, 1e-5
+    width = 2 * H * (d + dv)
+    projs = [torch.randn(L, col + width + 8, generator=gen).to(dtype) for L in lengths]
+    want = []
+    for p in projs:
+        x = p.double()[:, col:]
+        T = len(x)
+        q, k = x[:, :H * d].view(T, H, d), x[:, H * d:2 * H * d].view(T, H, d)
+        if rot:
+            q, k = (plain.rotate(t, rot, 700.0, 1.0, neighbours=inter) for t in (q, k))
+        o, S = plain.retention_recurrence(q, k * d ** -0.5, x[:, 2 * H * d:2 * H * d + H * dv].reshape(T, H, dv), torch.tensor(decay).double())
+        want.append((plain.rms(o, eps).reshape(T, H * dv) * plain.silu(x[:, 2 * H * d + H * dv:width]) * 0.8, S))
+    slots = [4, 0, 2]
+    state = torch.zeros(6, H, d, dv, device="cuda")
+    state[1].fill_(7.0)          # a slot of somebody else: must stay as it is
+    cuts = [[1, 1, 150, 66, 15], [1, 1, 1], [64, 1, 3, 31]]
+    got, at = [[] for _ in lengths], [0, 0, 0]
+    for step in range(5):
+        live = [s for s in range(3) if step < len(cuts[s])]
+        runs = [projs[s][at[s]:at[s] + cuts[s][step]] for s in live]
+        positions = [at[s] + i for s, r in zip(live, runs) for i in range(len(r))]
+        cu = [0]
+        for r in runs:
+            cu.append(cu[-1] + len(r))
+        proj = torch.cat(runs).cuda()
+        cos, sin = _tables(rot, 700.0, 1.0, positions)
+        out = torch.full((cu[-1], out_col + H * dv + 8), 5.0, dtype=dtype, device="cuda")
+        ops.retention(proj, cos, sin, torch.tensor(decay, device="cuda"), state, out, ints(*cu),
+                      ints(*[i for i, r in enumerate(runs) for _ in range(len(r))]), ints(*[slots[s] for s in live]), n_seqs=len(live),
+                      max_q_len=max(len(r) for r in runs), heads=H, d=d, dv=dv, rot=rot, interleaved=inter, eps=eps, out_scale=0.8,
+                      col=col, out_col=out_col, chunked=chunked)
+        got_rows = out.cpu()
+        assert float((got_rows[:, :out_col].float() - 5).abs().max()) == 0 and float((got_rows[:, out_col + H * dv:].float() - 5).abs().max()) == 0
+        for i, s in enumerate(live):
+            got[s].append(got_rows[cu[i]:cu[i + 1], out_col:out_col + H * dv])
+            at[s] += cuts[s][step]
+    assert at == lengths and float((state[1] - 7.0).abs().max()) == 0
+    for s in range(3):
+        torch.testing.assert_close(torch.cat(got[s]).double(), want[s][0], **(dict(atol=2e-4, rtol=2e-4) if dtype == torch.float32
+                                                                              else dict(atol=2e-3, rtol=6e-3)))
+        S = state[slots[s]].cpu().double()
+        assert float((S - want[s][1]).abs().max()) <= (3e-5 if not chunked else 1e-4) * max(1.0, float(want[s][1].abs().max()))
+
+
+def test_prompts_of_bfloat16_take_the_chunks_where_shared_memory_holds_them():
+    from ctypes import c_int
+    from ondeviceinfer_b200.kernels.build import load_library
+    takes = load_library("retention").odi_retention_takes_chunks
+    assert takes(c_int(128), c_int(128)) and takes(c_int(32), c_int(64)) and takes(c_int(256), c_int(128))
+    assert not takes(c_int(1024), c_int(64))
+
+
+@pytest.mark.parametrize("dtype", KINDS)
+def test_retention_of_large_heads_goes_in_order(dtype):
+    """Heads whose chunks do not fit shared memory, and more columns than a block has threads."""
+    gen = torch.Generator().manual_seed(5)
+    H, d, dv, L = 1, 600, 300, 20
+    proj = torch.randn(L, 2 * H * (d + dv), generator=gen).to(dtype)
+    m = {"heads": H, "dim": d, "vdim": dv, "decay": (0.9,)}
+    x = proj.double()
+    want, S = plain.retention_core(m, x[:, :d], x[:, d:2 * d], x[:, 2 * d:2 * d + dv], x[:, 2 * d + dv:], 1e-5)
+    state, rows = torch.zeros(1, H, d, dv, device="cuda"), []
+    for lo, hi in ((0, 12), (12, 13), (13, 20)):
+        out = torch.empty(hi - lo, dv, dtype=dtype, device="cuda")
+        ops.retention(proj[lo:hi].cuda(), None, None, torch.tensor([0.9], device="cuda"), state, out, ints(0, hi - lo), ints(*[0] * (hi - lo)),
+                      ints(0), n_seqs=1, max_q_len=hi - lo, heads=H, d=d, dv=dv, rot=0, interleaved=False, eps=1e-5)
+        rows.append(out.cpu())
+    torch.testing.assert_close(torch.cat(rows).double(), want, **(dict(atol=2e-4, rtol=2e-4) if dtype == torch.float32 else dict(atol=2e-3, rtol=6e-3)))
+    torch.testing.assert_close(state[0].cpu().double(), S, atol=2e-4, rtol=2e-4)
+
+
+# ----------------------------------------------------------------------------- two mixers that share their products
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("case,layer", [("A", 0), ("B", 0), ("B", 2), ("C", 1)])
+def test_mixers_side_by_side_share_their_products(case, layer, dtype, tmp_path_factory):
+    """The joined form against the plain sum of the two mixers, as a part by itself."""
+    model = engine(case, dtype, tmp_path_factory)
+    cfg = CONFIGS[case][0]
+    mixer = model.decoder.layers[layer].mixer
+    assert mixer.joined and mixer.left.w_in is None and mixer.right.w_o is None
+    m, p = cfg["layers"][layer]["mixer"], f"l{layer}.mix."
+    gen = torch.Generator().manual_seed(9)
+    x = torch.randn(100, cfg["width"], generator=gen).to(getattr(torch, dtype))
+    w = {k: v.double() for k, v in weights_of(case).items()}
+    want = plain.parallel(w, p, m, x.double(), cfg["norm"]["eps"])
+    cache = model.make_cache(max_tokens=128, max_seqs=1)
+    slot = cache.alloc()
+    from ondeviceinfer_b200.engine.step import StepContext
+    cache.reserve([slot], [100])
+    ctx = StepContext(cache, [slot], [[0] * 100], [], model.device)
+    entry = next(i for i, e in enumerate(model.decoder.plan.order) if e.layer == layer)
+    got = mixer.forward(x.cuda(), ctx, cache.view(entry), None)
+    error = (got.cpu().double() - want).norm(dim=-1) / want.norm(dim=-1)
+    assert float(error.median()) < (1e-5 if dtype == "float32" else 1e-2) and float(error.max()) < (1e-4 if dtype == "float32" else 1e-1)
+
+
+# ----------------------------------------------------------------------------- whole models
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("case", ["A", "B", "C", "D"])
+def test_whole_prompts_and_their_first_tokens(case, dtype, tmp_path_factory):
+    model = engine(case, dtype, tmp_path_factory)
+    cfg = CONFIGS[case][0]
+    cache = model.make_cache(max_tokens=512, max_seqs=2)
+    for n in (1, 2, 3, 150):
+        tokens = plain.random_prompts(cfg, [n], n)[0]
+        slot = cache.alloc()
+        got = model.step(cache, [slot], [tokens], "all")
+        cache.free(slot)
+        close(got, expected(case, tokens), dtype, f"{case} whole prompt of {n}")
+    cache.check()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("case", ["A", "B", "C", "D"])
+def test_sum_of_the_streams_after_every_layer(case, dtype, tmp_path_factory):
+    model = engine(case, dtype, tmp_path_factory)
+    cfg = CONFIGS[case][0]
+    tokens = plain.random_prompts(cfg, [40], 2)[0]
+    want = plain.forward(cfg, weights_of(case), tokens, keep_layers=True)[1].float()
+    seen, blocks = [], list(model.decoder.layers)
+    originals = [block.forward for block in blocks]
+    try:
+        for block, original in zip(blocks, originals):
+            def record(hidden, ctx, view, original=original):
+                result = original(hidden, ctx, view)
+                flush_residual_add(ctx)              # the update that the next norm would have finished
+                seen.append(hidden.view(len(tokens), -1, cfg["width"]).sum(1))
+                return result
+            block.forward = record
+        cache = model.make_cache(max_tokens=64, max_seqs=1)
+        model.step(cache, [cache.alloc()], [tokens], "last")
+    finally:
+        for block, original in zip(blocks, originals):
+            block.forward = original
+    assert len(seen) == want.shape[0] == len(plain.layer_runs(cfg))
+    for run, (got, ref) in enumerate(zip(seen, want)):
+        gap, size = float((got.cpu() - ref).abs().max()), float(ref.abs().max())
+        assert gap < (1e-5 if dtype == "float32" else 3e-2) * max(size, 1.0), (run, gap, size)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("case", ["A", "B", "C", "D"])
+def test_prompt_then_single_tokens_over_page_borders(case, dtype, tmp_path_factory):
+    model = engine(case, dtype, tmp_path_factory)
+    cfg = CONFIGS[case][0]
+    tokens = plain.random_prompts(cfg, [150], 4)[0]
+    want = expected(case, tokens)
+    cache = model.make_cache(max_tokens=192, max_seqs=1)
+    slot = cache.alloc()
+    rows = [model.step(cache, [slot], [tokens[:50]], "all")]
+    rows += [model.step(cache, [slot], [[t]], "last") for t in tokens[50:]]
+    close(torch.cat(rows), want, dtype, f"{case} decoded")
+    cache.free(slot)
+    slot = cache.alloc()                                                            # the same slot and pages again
+    rows = [model.step(cache, [slot], [[t]], "last") for t in tokens[:80]]          # from the very first token
+    close(torch.cat(rows), want[:80], dtype, f"{case} decoded from the first token")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("case", ["A", "B", "C", "D"])
+def test_portions_of_several_sizes_down_to_two_tokens(case, dtype, tmp_path_factory):
+    model = engine(case, dtype, tmp_path_factory)
+    cfg = CONFIGS[case][0]
+    tokens = plain.random_prompts(cfg, [200], 5)[0]
+    want = expected(case, tokens)
+    for sizes in ([2] * 40 + [120], [63, 2, 64, 1, 70], [7, 129, 64], [199, 1], [1, 2, 1, 196]):
+        cache = model.make_cache(max_tokens=256, max_seqs=1)
+        slot, at, rows = cache.alloc(), 0, []
+        for size in sizes:
+            rows.append(model.step(cache, [slot], [tokens[at:at + size]], "all"))
+            at += size
+        close(torch.cat(rows), want, dtype, f"{case} portions {sizes[:4]}")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("case", ["A", "B", "C", "D"])
+def test_unequal_batches_on_slots_and_pages_used_again(case, dtype, tmp_path_factory):
+    model = engine(case, dtype, tmp_path_factory)
+    cfg = CONFIGS[case][0]
+    requests = plain.random_prompts(cfg, [90, 1, 33, 70, 5, 129], 8)
+    cache = model.make_cache(max_tokens=448, max_seqs=3)
+    got = {r: [] for r in range(len(requests))}
+    for batch in ([0, 1, 2], [3, 4, 5]):          # the second batch takes the slots and pages the first gave back
+        slots = {r: cache.alloc() for r in batch}
+        cut = {r: max(1, len(requests[r]) - 4 - 2 * (r % 3)) for r in batch}
+        logits = model.step(cache, [slots[r] for r in batch], [requests[r][:cut[r]] for r in batch], "all")
+        at = 0
+        for r in batch:
+            got[r].append(logits[at:at + cut[r]])
+            at += cut[r]
+        live = list(batch)
+        while live:
+            for r in [r for r in live if cut[r] == len(requests[r])]:
+                cache.free(slots.pop(r))
+                live.remove(r)
+            if not live:
+                break
+            logits = model.step(cache, [slots[r] for r in live], [[requests[r][cut[r]]] for r in live], "last")
+            for i, r in enumerate(live):
+                got[r].append(logits[i:i + 1])
+                cut[r] += 1
+        cache.check()
+    for r, tokens in enumerate(requests):
+        close(torch.cat(got[r]), expected(case, tokens), dtype, f"{case} batched request {r}")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_batch_rows_do_not_depend_on_their_neighbours(dtype, tmp_path_factory):
+    model = engine("A", dtype, tmp_path_factory)
+    requests = plain.random_prompts(plain.TINY_A, [77, 12, 140], 6)
+    cache = model.make_cache(max_tokens=512, max_seqs=4)
+    alone = []
+    for tokens in requests:
+        slot = cache.alloc()
+        alone.append(model.step(cache, [slot], [tokens], "all"))
+        cache.free(slot)
+    together = model.step(cache, [cache.alloc() for _ in requests], requests, "all")
+    gap = float((together - torch.cat(alone)).abs().max())
+    assert gap < (2e-5 if dtype == "float32" else 0.3)          # bfloat16: tiles of other sizes round otherwise
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_sharp_attention_finds_far_keys_in_prompts_and_in_decoding(dtype, tmp_path_factory):
+    """Sharpened queries make both softmaxes pick single keys anywhere in 700 positions, so a key that is lost or read from
+    the wrong page moves the logits.  float32 is held to the plain implementation; bfloat16 (whose rounded scores such a
+    scale magnifies) to its own whole-prompt run, which the decoded run must repeat from the cache."""
+    model = engine("sharp", dtype, tmp_path_factory)
+    tokens = plain.random_prompts(plain.SHARP, [700], 9)[0]
+    cache = model.make_cache(max_tokens=1536, max_seqs=2)
+    whole = cache.alloc()
+    whole_logits = model.step(cache, [whole], [tokens], "all")
+    want = expected("sharp", tokens) if dtype == "float32" else whole_logits
+    if dtype == "float32":
+        close(whole_logits, want, dtype, "sharp whole", atol=5e-4)      # the effects looked for below are above 2e-2
+    decoded = cache.alloc()
+    rows = [model.step(cache, [decoded], [tokens[:500]], "all")]
+    rows += [model.step(cache, [decoded], [[t]], "last") for t in tokens[500:]]
+    close(torch.cat(rows), want, dtype, "sharp decoded", atol=5e-4)
+    if dtype == "float32":
+        weights = weights_of("sharp")
+
+        def moved(change=lambda c: None, since=500, **tensors):
+            cfg = copy.deepcopy(plain.SHARP)
+            change(cfg["layers"])
+            return float((plain.forward(cfg, {**weights, **tensors}, tokens).float()[since:] - want[since:]).abs().max())
+
+        # the plain logits of decoded positions really depend on each mechanism's constants
+        left, right = (lambda L: L[0]["mixer"]["left"]), (lambda L: L[0]["mixer"]["right"])
+        assert moved(lambda L: left(L).update(bias_max=280)) > 0.02
+        assert moved(lambda L: left(L)["q_temp"].update(every=65)) > 0.02
+        assert moved(lambda L: left(L)["q_temp"].update(coef=0.32)) > 0.02
+        assert moved(lambda L: right(L).update(decay=[0.9975, 0.99])) > 0.02
+        assert moved(lambda L: right(L)["rot"].update(base=2e4)) > 0.02
+        assert moved(lambda L: L[1]["mixer"].update(softcap=38.0)) > 0.02
+        assert moved(lambda L: L[1]["mixer"]["rot"]["scaling"].update(factor=3.1)) > 0.02
+        # ... on the last row of the distance table, and on the state carried from the first tokens on
+        rel = weights["l0.mix.left.rel"].clone()
+        rel[-1] += 1.0
+        assert moved(**{"l0.mix.left.rel": rel}) > 0.02
+        later = plain.forward(plain.SHARP, weights, tokens[400:]).float()
+        assert float((later[-50:] - want[-50:]).abs().max()) > 0.02
+
+
+@pytest.mark.parametrize("case", ["A", "B"])
+def test_long_decoding(case, tmp_path_factory):
+    """700 single-token steps: the state is carried through all of them, distances run far beyond the tables' reach and the
+    temperature takes many steps."""
+    model = engine(case, "float32", tmp_path_factory)
+    tokens = plain.random_prompts(CONFIGS[case][0], [720], 11)[0]
+    cache = model.make_cache(max_tokens=768, max_seqs=1)
+    slot = cache.alloc()
+    rows = [model.step(cache, [slot], [tokens[:20]], "all")]
+    rows += [model.step(cache, [slot], [[t]], "last") for t in tokens[20:]]
+    close(torch.cat(rows), expected(case, tokens), "float32", "long decoding", atol=2e-4)
+
+
+def test_decode_steps_are_captured_as_graphs(tmp_path_factory):
+    assert engine("A", "bfloat16", tmp_path_factory).decoder.graph_safe
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_greedy_generation_through_the_entry_point(dtype, tmp_path_factory):
+    for case in ("A", "B", "C"):
+        model = engine(case, dtype, tmp_path_factory)
+        cfg = CONFIGS[case][0]
+        prompts = plain.random_prompts(cfg, [9, 60, 3], 10)
+        weights = weights_of(case)
+        for use_graphs in (False, True):              # the step function, then the captured decode steps
+            result = model.generate(prompts, max_new_tokens=6, use_graphs=use_graphs)
+            for prompt, produced in zip(prompts, result.generated_ids):
+                assert len(produced) == 6
+                ids = list(prompt)
+                for token in produced:
+                    logits = plain.forward(cfg, weights, ids)[-1]
+                    slack = 1e-4 if dtype == "float32" else 0.05 * float(logits.abs().max())
+                    assert float(logits.max() - logits[token]) < slack, "the generated token is not the plain argmax"
+                    ids.append(token)
+
+
+def test_command_line_writes_a_random_model_and_generates_from_it(tmp_path):
+    cfg = plain.TINY_B
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    root = Path(__file__).resolve().parent.parent
+    run = lambda *a: subprocess.run([sys.executable, "-m", "ondeviceinfer_b200", *a], cwd=root, text=True,
+                                    capture_output=True, timeout=600)
+    made = run("random-model", "--config", str(tmp_path / "config.json"), "--seed", "3", "--out", str(tmp_path / "model"))
+    assert made.returncode == 0, made.stderr
+    done = run("generate", "--model", str(tmp_path / "model"), "--prompt-ids", "5,9,2,40,7", "--dtype", "float32",
+               "--max-new-tokens", "4", "--warmup-runs", "0", "--repeats", "1", "--output", str(tmp_path / "report.json"))
+    assert done.returncode == 0, done.stderr
+    report = json.loads((tmp_path / "report.json").read_text())
+    from ondeviceinfer_b200.weights import SafetensorsSource
+    source = SafetensorsSource(tmp_path / "model")
+    weights = {n: source.fetch(n) for n in source.stored()}
+    ids = [5, 9, 2, 40, 7]
+    for token in report["measurements"][0]["output_token_ids"]:
+        logits = plain.forward(cfg, weights, ids)[-1]
+        assert float(logits.max() - logits[token]) < 1e-4
+        ids.append(token)
+    assert len(ids) == 9
+
+
+def test_a_table_whose_rows_only_the_checkpoint_gives(tmp_path):
+    cfg = copy.deepcopy(plain.TINY_A)
+    weights = plain.random_weights(cfg, 5)
+    for i in (0, 2):
+        cfg["layers"][i]["mixer"]["left"].pop("bias_rows")
+    model = odi.load_resident_model(write_model_folder(tmp_path / "model", cfg, weights), dtype="float32")
+    tokens = plain.random_prompts(cfg, [70], 1)[0]
+    cache = model.make_cache(max_tokens=128, max_seqs=1)
+    close(model.step(cache, [cache.alloc()], [tokens], "all"), plain.forward(cfg, weights, tokens), "float32", "rows from the checkpoint")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("seed", range(16))
+def test_models_of_random_odd_sizes(seed, dtype, tmp_path):
+    """Configurations drawn from odd sizes: a prompt, then single tokens, then a portion, on a cache that a shorter
+    request used before."""
+    cfg = plain.random_config(seed)
+    weights = plain.random_weights(cfg, 300 + seed)
+    model = odi.load_resident_model(write_model_folder(tmp_path / "model", cfg, weights), dtype=dtype)
+    tokens = plain.random_prompts(cfg, [150], seed)[0]
+    want = plain.forward(cfg, weights, tokens).float()
+    cache = model.make_cache(max_tokens=192, max_seqs=1)
+    slot = cache.alloc()
+    model.step(cache, [slot], [tokens[:37]], "none")
+    cache.free(slot)
+    slot = cache.alloc()
+    rows = [model.step(cache, [slot], [tokens[:100]], "all")]
+    rows += [model.step(cache, [slot], [[t]], "last") for t in tokens[100:130]]
+    rows.append(model.step(cache, [slot], [tokens[130:]], "all"))
+    close(torch.cat(rows), want, dtype, f"random sizes {seed}: {json.dumps(cfg)[:300]}")
