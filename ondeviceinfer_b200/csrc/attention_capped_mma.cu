@@ -217,20 +217,32 @@ attention_capped_kernel(CappedAttnArgs a) {
           mma_bf16(s[np * 2 + 1], qf[ks], b2, b3);
         }
       }
-      // scale, cap, bias, mask, running maximum (log2 domain)
-      if (has_rel) {
-        const float pre = a.softcap > 0.f ? 1.f : a.scale;
-        if (a.softcap > 0.f) {
+      // cap, scale, bias (log2 domain), mask, running maximum
+      const float pre = (a.softcap > 0.f ? a.softcap : a.scale) * LOG2E;
+      if (a.softcap > 0.f) {               // tanh of the score over the cap: a polynomial while all of the warp's are small
+        float top = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) { s[i][e] *= 0.5f * a.scale * two_over_cap; top = fmaxf(top, fabsf(s[i][e])); }
+        if (__all_sync(0xffffffffu, top <= TANH_SMALL)) {
 #pragma unroll
           for (int i = 0; i < 8; ++i)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) s[i][e] = a.softcap * (1.f - __fdividef(2.f, __expf(s[i][e] * a.scale * two_over_cap) + 1.f));
+            for (int e = 0; e < 4; ++e) s[i][e] *= tanh_ratio(s[i][e] * s[i][e]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[i][e] = 1.f - __fdividef(2.f, __expf(2.f * s[i][e]) + 1.f);
         }
+      }
+      if (has_rel) {
         if (warp_first - (kbase + KT - 1) >= a.rel.n - 1) {          // every pair is beyond the table's last distance
 #pragma unroll
           for (int i = 0; i < 8; ++i)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) s[i][e] = fmaf(s[i][e], pre * LOG2E, rel_far);
+            for (int e = 0; e < 4; ++e) s[i][e] = fmaf(s[i][e], pre, rel_far);
         } else if (a.rel_staged) {
           const int last = a.rel.n - 1 + REL_PAD, k0 = kbase + (lane & 3) * 2;
           // distances of this lane's first key, no farther than the copies reach; those behind the diagonal are masked below
@@ -238,8 +250,8 @@ attention_capped_kernel(CappedAttnArgs a) {
           const float* b_hi = rel_s + REL_PAD + min(max(pos_hi - k0, 0), last - 1);
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            s[i][0] = fmaf(s[i][0], pre * LOG2E, b_lo[-8 * i]); s[i][1] = fmaf(s[i][1], pre * LOG2E, b_lo[-8 * i - 1]);
-            s[i][2] = fmaf(s[i][2], pre * LOG2E, b_hi[-8 * i]); s[i][3] = fmaf(s[i][3], pre * LOG2E, b_hi[-8 * i - 1]);
+            s[i][0] = fmaf(s[i][0], pre, b_lo[-8 * i]); s[i][1] = fmaf(s[i][1], pre, b_lo[-8 * i - 1]);
+            s[i][2] = fmaf(s[i][2], pre, b_hi[-8 * i]); s[i][3] = fmaf(s[i][3], pre, b_hi[-8 * i - 1]);
           }
         } else {
 #pragma unroll
@@ -247,19 +259,23 @@ attention_capped_kernel(CappedAttnArgs a) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const int dist = (e < 2 ? pos_lo : pos_hi) - (kbase + i * 8 + (lane & 3) * 2 + (e & 1));
-              s[i][e] = fmaf(s[i][e], pre * LOG2E, rel_g[min(max(dist, 0), a.rel.n - 1)] * LOG2E);
+              s[i][e] = fmaf(s[i][e], pre, rel_g[min(max(dist, 0), a.rel.n - 1)] * LOG2E);
             }
         }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[i][e] *= pre;
       }
-      auto shaped = [&](float x) { return has_rel ? x : shape_score(x, a.scale, a.softcap, two_over_cap); };
       float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int kj = kbase + i * 8 + (lane & 3) * 2;
-        s[i][0] = (kj <= pos_lo && (kj >= old_lo || kj < a.keep)) ? shaped(s[i][0]) : -INFINITY;
-        s[i][1] = (kj + 1 <= pos_lo && (kj + 1 >= old_lo || kj + 1 < a.keep)) ? shaped(s[i][1]) : -INFINITY;
-        s[i][2] = (kj <= pos_hi && (kj >= old_hi || kj < a.keep)) ? shaped(s[i][2]) : -INFINITY;
-        s[i][3] = (kj + 1 <= pos_hi && (kj + 1 >= old_hi || kj + 1 < a.keep)) ? shaped(s[i][3]) : -INFINITY;
+        s[i][0] = (kj <= pos_lo && (kj >= old_lo || kj < a.keep)) ? s[i][0] : -INFINITY;
+        s[i][1] = (kj + 1 <= pos_lo && (kj + 1 >= old_lo || kj + 1 < a.keep)) ? s[i][1] : -INFINITY;
+        s[i][2] = (kj <= pos_hi && (kj >= old_hi || kj < a.keep)) ? s[i][2] : -INFINITY;
+        s[i][3] = (kj + 1 <= pos_hi && (kj + 1 >= old_hi || kj + 1 < a.keep)) ? s[i][3] : -INFINITY;
         mx_lo = fmaxf(mx_lo, fmaxf(s[i][0], s[i][1]));
         mx_hi = fmaxf(mx_hi, fmaxf(s[i][2], s[i][3]));
       }

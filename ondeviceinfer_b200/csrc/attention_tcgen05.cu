@@ -278,8 +278,9 @@ __device__ __forceinline__ void umma_a_tmem(uint32_t d_tmem, uint32_t a_tmem, ui
 // pairs, 32 columns at p_addr) against the row's running maximum; n counts this head's PV products
 // (the one that will read this P is product n), kbase is the first key's position.  Returns false if a
 // wait gave up.  The caller signals P afterwards.
-// `oldest` is the first key the row still sees (0 without a window).  With a cap (two_over_cap > 0) the score
-// times `scale` is squashed first, as c (1 - 2 / (e^(2 x / c) + 1)) = c tanh(x / c), and sl2 is log2(e) alone.
+// `oldest` is the first key the row still sees (0 without a window).  With a cap c the score x (times `scale`) is squashed
+// first: s becomes tanh(x / c), by the polynomial of common.cuh when all of the warp's scores are small enough, else as
+// 1 - 2 / (e^(2 x / c) + 1); sl2 is then c log2(e).
 struct RowState { float m_used, l; };
 template <bool REL>
 __device__ __forceinline__ bool softmax_keys64(uint32_t s_addr, uint32_t p_addr, uint32_t o_addr, int kbase, int pos, float sl2,
@@ -289,12 +290,20 @@ __device__ __forceinline__ bool softmax_keys64(uint32_t s_addr, uint32_t p_addr,
   float s[BNK];
   tmem_ld64(s_addr, s);
   if (cap > 0.f) {
+    float top = 0.f;
 #pragma unroll
-    for (int i = 0; i < BNK; ++i) s[i] = cap * (1.f - __fdividef(2.f, __expf(s[i] * scale * two_over_cap) + 1.f));
+    for (int i = 0; i < BNK; ++i) { s[i] *= 0.5f * scale * two_over_cap; top = fmaxf(top, fabsf(s[i])); }
+    if (__all_sync(0xffffffffu, top <= TANH_SMALL)) {
+#pragma unroll
+      for (int i = 0; i < BNK; ++i) s[i] *= tanh_ratio(s[i] * s[i]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < BNK; ++i) s[i] = 1.f - __fdividef(2.f, __expf(2.f * s[i]) + 1.f);
+    }
   }
   if (REL) {
     // entry REL_PAD + n of `rel` is the bias of distance n in log2 units; sl2 is 1, the scores' factor is `pre`
-    const float pre = cap > 0.f ? LOG2E : scale * LOG2E;
+    const float pre = (cap > 0.f ? cap : scale) * LOG2E;
     if (__all_sync(0xffffffffu, pos - (kbase + BNK - 1) >= rel_n - 1)) {
       const float far = rel[REL_PAD + rel_n - 1];
 #pragma unroll
@@ -360,17 +369,22 @@ __device__ __forceinline__ bool softmax_keys64(uint32_t s_addr, uint32_t p_addr,
   return true;
 }
 
-// The finished row of O, divided by the row's sum, as bf16 to dst (D elements).
+// A token's gates for one head: 64 numbers of the lanes from `c` on, all in flight together.
+__device__ __forceinline__ void load_gates64(const HeadOut& ho, size_t tok, int head, int c, uint4* raw) {
+  const uint4* src = (const uint4*)((const bf16*)ho.gate + tok * ho.gate_ld + head * D + c);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) raw[i] = src[i];
+}
+
+// The finished row of O, divided by the row's sum, as bf16 to dst (D elements); `gates`: its first 64 gates (with a gate
+// per lane), requested before the last product was waited for.
 template <bool GATED>
-__device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, bool valid, const HeadOut& ho, size_t tok, int head) {
+__device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, bool valid, const HeadOut& ho, size_t tok, int head,
+                                          bool gated, uint4* gates) {
   float inv = l > 0.f ? 1.f / l : 0.f;
-  const bf16* gate = nullptr;              // a gate per lane: this head's lanes of the token's gate row
-  if (!GATED) inv *= ho.scale;
-  else if (valid) {
-    if (ho.gate != nullptr && !ho.gate_per_head) { gate = (const bf16*)ho.gate + tok * ho.gate_ld + head * D; inv *= ho.scale; }
-    else inv *= head_out_factor<bf16>(ho, tok, head, D, 0);
-  }
-#pragma unroll 1
+  if (!GATED || gated) inv *= ho.scale;
+  else if (valid) inv *= head_out_factor<bf16>(ho, tok, head, D, 0);
+#pragma unroll
   for (int c = 0; c < D; c += 32) {
     float v[32];
     tmem_ld32(o_addr + c, v);                    // every thread of the warp loads
@@ -378,14 +392,13 @@ __device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, b
 #pragma unroll
       for (int i = 0; i < 32; i += 8) {
         uint32_t w[4];
-        if (GATED && gate != nullptr) {
-          const uint4 raw = *(const uint4*)(gate + c + i);
-          const __nv_bfloat162* z = (const __nv_bfloat162*)&raw;
+        if (GATED && gated) {
+          const __nv_bfloat162* z = (const __nv_bfloat162*)&gates[(c % 64 + i) / 8];
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
             const float2 f = __bfloat1622float2(z[k]);
-            v[i + 2 * k] /= 1.f + __expf(-f.x);
-            v[i + 2 * k + 1] /= 1.f + __expf(-f.y);
+            v[i + 2 * k] = __fdividef(v[i + 2 * k], 1.f + __expf(-f.x));
+            v[i + 2 * k + 1] = __fdividef(v[i + 2 * k + 1], 1.f + __expf(-f.y));
           }
         }
 #pragma unroll
@@ -395,6 +408,7 @@ __device__ __forceinline__ void write_row(uint32_t o_addr, bf16* dst, float l, b
         }
         *(uint4*)(dst + c + i) = make_uint4(w[0], w[1], w[2], w[3]);
       }
+      if (GATED && gated && c % 64 == 32 && c + 32 < D) load_gates64(ho, tok, head, c + 32, gates);
     }
   }
 }
@@ -558,7 +572,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int row = lane_group * 32 + lane;          // query row inside the tile
     const int pos = past + t0 + row;
     const uint32_t lane_addr = (uint32_t)(lane_group * 32) << 16;
-    const float sl2 = has_rel ? 1.f : (a.softcap > 0.f ? LOG2E : a.scale * LOG2E);
+    const float sl2 = has_rel ? 1.f : (a.softcap > 0.f ? a.softcap : a.scale) * LOG2E;
     const float two_over_cap = a.softcap > 0.f ? 2.f / a.softcap : 0.f;
     const int oldest = a.window > 0 ? pos - a.window + 1 : (a.chunk > 0 ? pos - pos % a.chunk : 0);
     // a sink is a key of score 0 and value 0 ahead of all others: the row starts from its maximum and its weight
@@ -585,10 +599,14 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
       __syncwarp();
       if (lane == 0) mbar_arrive(my_p_full + 8 * b);
     }
+    const size_t tok = q_begin + t0 + row;
+    const bool gated = SHAPED && a.ho.gate != nullptr && !a.ho.gate_per_head;
+    uint4 gates[8];
+    if (gated && row < nt) load_gates64(a.ho, tok, head, 0, gates);
     if (ok && !mbar_wait(my_pv_done, (uint32_t)(n_tiles - 1) & 1u, abort_ptr)) ok = false;
     tc_fence_after();
     if (!ok && lane == 0) atomicCAS(a.status, 0, ATT_ERR_SOFTMAX);
-    if (ok) write_row<SHAPED>(o_addr, a.out + (size_t)(q_begin + t0 + row) * a.ho.out_ld + head * D, st.l, row < nt, a.ho, q_begin + t0 + row, head);
+    if (ok) write_row<SHAPED>(o_addr, a.out + tok * a.ho.out_ld + head * D, st.l, row < nt, a.ho, tok, head, gated, gates);
     tc_fence_before();
   }
   __syncthreads();

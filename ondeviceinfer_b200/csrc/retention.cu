@@ -27,7 +27,8 @@ struct RetentionArgs {
   const float* sin_t;
   const float* decay;     // [heads]
   float* state;           // [slots, heads, d, dv]
-  float* chunks;          // chunk form: [n_tokens / 64 + n_seqs, heads, d, dv] scratch
+  float* chunks;          // chunk form: [n_tokens / 64 + n_seqs, heads, d, dv rounded up to 8] scratch
+  void* qk;               // chunk form: [n_tokens, heads, 4, d rounded up to 16] bf16 scratch
   float* o;               // walk form: [n_tokens, heads dv] scratch
   void* out;              // [n_tokens, out_ld] in T, from this mixer's first column on
   const int* cu_q;
@@ -51,29 +52,12 @@ __device__ __forceinline__ float rt_lane(const RetentionArgs& a, const T* row, i
   return first ? fmaf(-y, sn, x * cs) : fmaf(y, sn, x * cs);
 }
 
-// Eight neighbouring lanes (bf16, aligned rows; a rotation in halves whose halves are multiples of 8 lanes, or none).
+// Eight neighbouring bf16 numbers.
 __device__ __forceinline__ void rt_unpack8(const uint4 raw, float* v) {
   const __nv_bfloat162* h = (const __nv_bfloat162*)&raw;
 #pragma unroll
   for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(h[e]); v[2 * e] = f.x; v[2 * e + 1] = f.y; }
 }
-__device__ __forceinline__ void rt_lanes8(const RetentionArgs& a, const bf16* row, int i, int t, float* v) {
-  rt_unpack8(*(const uint4*)(row + i), v);
-  if (i >= a.rot) return;
-  const int half = a.rot >> 1;
-  const bool first = i < half;
-  const int pair = first ? i : i - half;
-  float y[8], cs[8], sn[8];
-  rt_unpack8(*(const uint4*)(row + (first ? i + half : i - half)), y);
-  const float4* cp = (const float4*)(a.cos_t + (size_t)t * half + pair);
-  const float4* sp = (const float4*)(a.sin_t + (size_t)t * half + pair);
-  const float4 c0 = cp[0], c1 = cp[1], s0 = sp[0], s1 = sp[1];
-  cs[0] = c0.x; cs[1] = c0.y; cs[2] = c0.z; cs[3] = c0.w; cs[4] = c1.x; cs[5] = c1.y; cs[6] = c1.z; cs[7] = c1.w;
-  sn[0] = s0.x; sn[1] = s0.y; sn[2] = s0.z; sn[3] = s0.w; sn[4] = s1.x; sn[5] = s1.y; sn[6] = s1.z; sn[7] = s1.w;
-#pragma unroll
-  for (int e = 0; e < 8; ++e) v[e] = first ? fmaf(-y[e], sn[e], v[e] * cs[e]) : fmaf(y[e], sn[e], v[e] * cs[e]);
-}
-
 // g^n by squaring (n < 2^16; 0^0 = 1).
 __device__ __forceinline__ float rt_power(float g, int n) {
   float r = 1.f;
@@ -269,170 +253,231 @@ __device__ __forceinline__ bool rt_chunk(const RetentionArgs& a, int seq, int c,
   return true;
 }
 
-// One head's q or k rows of a chunk, rotated and times `scale` (and g^(n-1-row) with `weights`), split, into
-// [64][W] rows of high and low parts; lanes from d on and rows from n on are zero.
-__device__ __forceinline__ void rt_stage_rows(const RetentionArgs& a, bf16* high, bf16* low, int W, const bf16* src, int t0, int n,
-                                              float scale, const float* weights, int vec, int tid, int threads) {
-  const int d16 = (a.d + 15) & ~15;
-  const int pieces = d16 / 8;
-  for (int i = tid; i < RT_CHUNK * pieces; i += threads) {
-    const int r = i / pieces, e0 = 8 * (i % pieces);
-    float v[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = 0.f;
-    if (r < n) {
-      const bf16* row = src + (size_t)(t0 + r) * a.ld;
-      if (vec) { if (e0 < a.d) rt_lanes8(a, row, e0, t0 + r, v); }
-      else {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) if (e0 + e < a.d) v[e] = rt_lane<bf16>(a, row, e0 + e, t0 + r);
-      }
-      const float w = weights != nullptr ? scale * weights[n - 1 - r] : scale;
-#pragma unroll
-      for (int e = 0; e < 8; ++e) v[e] *= w;
-    }
-    uint4 hi, lo;
-    rt_split2(v[0], v[1], hi.x, lo.x); rt_split2(v[2], v[3], hi.y, lo.y);
-    rt_split2(v[4], v[5], hi.z, lo.z); rt_split2(v[6], v[7], hi.w, lo.w);
-    *(uint4*)(high + r * W + e0) = hi;
-    *(uint4*)(low + r * W + e0) = lo;
-  }
+// 16 bytes of split numbers: the high and the low parts of eight.
+__device__ __forceinline__ void rt_split8(const float* v, uint4& hi, uint4& lo) {
+  rt_split2(v[0], v[1], hi.x, lo.x); rt_split2(v[2], v[3], hi.y, lo.y);
+  rt_split2(v[4], v[5], hi.z, lo.z); rt_split2(v[6], v[7], hi.w, lo.w);
 }
+__device__ __forceinline__ void rt_cp16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(rt_addr(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void rt_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void rt_cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// `cols` columns (a multiple of 16) of the head's values from column c0 on into [64][W] rows; the rest is zero.
-__device__ __forceinline__ void rt_stage_values(const RetentionArgs& a, bf16* dst, int W, int c0, int cols, const bf16* src, int t0,
-                                                int n, int vec, int tid, int threads) {
+// The head's values of a chunk into [64][W] rows; rows from n on and columns from dv to `cols` (a multiple of 16) are zero.
+// With `vec` by asynchronous copies (the caller commits and waits).
+__device__ __forceinline__ void rt_stage_values(const RetentionArgs& a, bf16* dst, int W, int cols, const bf16* src, int t0, int n,
+                                                int vec, int tid) {
   const int pieces = cols / 8;
-  for (int i = tid; i < RT_CHUNK * pieces; i += threads) {
-    const int r = i / pieces, e0 = 8 * (i % pieces);
+  for (int i = tid; i < RT_CHUNK * pieces; i += 256) {
+    const int r = i / pieces, c = 8 * (i % pieces);
+    const bf16* row = src + (size_t)(t0 + r) * a.ld + c;
+    bf16* to = dst + r * W + c;
+    if (vec && r < n && c < a.dv) { rt_cp16(to, row); continue; }
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < n) {
-      const bf16* row = src + (size_t)(t0 + r) * a.ld;
-      if (vec) { if (c0 + e0 < a.dv) v = *(const uint4*)(row + c0 + e0); }
-      else {
-        bf16* p = (bf16*)&v;
+    if (!vec && r < n) {
+      bf16* p = (bf16*)&v;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) if (c0 + e0 + e < a.dv) p[e] = row[c0 + e0 + e];
-      }
+      for (int e = 0; e < 8; ++e) if (c + e < a.dv) p[e] = row[e];
     }
-    *(uint4*)(dst + r * W + e0) = v;
+    *(uint4*)to = v;
   }
 }
 
-#define RT_CB 64            // columns of the values per block of chunk_sums and per turn of chunk_outputs
+#define RT_CB 64            // columns of the values per turn
 
-// U of a chunk, RT_CB columns of it: rows are key lanes, 16 a warp at a time.
-__global__ void __launch_bounds__(256)
+// A chunk of one head: q and k rotated, k scaled, both split, into `qk` for rt_chunk_outputs; and the sum of its k v^T, each
+// token weighed by g^(tokens behind it), into `chunks`.  A block's 8 warps take 16 key lanes each at a time.
+__global__ void __launch_bounds__(256, 2)
 rt_chunk_sums_kernel(RetentionArgs a, int vec) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) uint8_t rt_bytes[];
   __shared__ float pw[RT_CHUNK + 1];
-  const int seq = blockIdx.z, col_blocks = (a.dv + RT_CB - 1) / RT_CB;
-  const int h = blockIdx.y / col_blocks, c0 = blockIdx.y % col_blocks * RT_CB;
+  const int seq = blockIdx.z, h = blockIdx.y;
   int t0, n;
   size_t place;
   if (!rt_chunk(a, seq, blockIdx.x, t0, n, place)) return;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d16 = (a.d + 15) & ~15, WK = d16 + 8, WV = RT_CB + 8;
-  bf16* kh = (bf16*)rt_bytes;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = a.d, d16 = (d + 15) & ~15, WK = d16 + 8;
+  const int dvp = (a.dv + 7) & ~7, turns = (a.dv + RT_CB - 1) / RT_CB, WV = turns * RT_CB + 8;
+  bf16* kh = (bf16*)rt_bytes;                      // weighted k, high and low [64][WK]
   bf16* kl = kh + RT_CHUNK * WK;
-  bf16* vs = kl + RT_CHUNK * WK;
+  bf16* vs = kl + RT_CHUNK * WK;                   // [64][WV]
+  const bf16* base = (const bf16*)a.proj;
+  rt_stage_values(a, vs, WV, turns * RT_CB, base + (size_t)2 * a.heads * d + (size_t)h * a.dv, t0, n, vec, tid);
+  rt_cp_commit();
   if (tid <= RT_CHUNK) pw[tid] = rt_power(a.decay[h], tid);
   __syncthreads();
-  const bf16* base = (const bf16*)a.proj;
-  rt_stage_rows(a, kh, kl, WK, base + (size_t)(a.heads + h) * a.d, t0, n, a.k_scale, pw, vec, tid, 256);
-  rt_stage_values(a, vs, WV, c0, RT_CB, base + (size_t)2 * a.heads * a.d + (size_t)h * a.dv, t0, n, vec, tid, 256);
-  __syncthreads();
-  float* U = a.chunks + (place * a.heads + h) * a.d * a.dv;
-  const int m = lane >> 3, r = lane & 7;
-  for (int row0 = warp * 16; row0 < d16; row0 += 8 * 16) {
-    float acc[RT_CB / 8][4] = {};
+  const bf16* q_src = base + (size_t)h * d;
+  const bf16* k_src = base + (size_t)(a.heads + h) * d;
+  bf16* split = (bf16*)a.qk + ((size_t)t0 * a.heads + h) * 4 * d16;      // a token's rows: q high, q low, k high, k low
+  auto put = [&](int r, int c, const float* q, const float* k) {  // eight lanes of token r (k scaled)
+    uint4 hi, lo;
+    bf16* dst = split + (size_t)r * a.heads * 4 * d16 + c;
+    rt_split8(q, hi, lo);
+    *(uint4*)dst = hi; *(uint4*)(dst + d16) = lo;
+    rt_split8(k, hi, lo);
+    *(uint4*)(dst + 2 * d16) = hi; *(uint4*)(dst + 3 * d16) = lo;
+    float w[8];
+    const float g = pw[n - 1 - r];
 #pragma unroll
-    for (int kk = 0; kk < RT_CHUNK / 16; ++kk) {
-      // A = k^T: matrices (lanes row0 .. + 7, tokens kk*16 .. + 7), (lanes + 8, same tokens), (lanes, tokens + 8), (both + 8)
-      uint32_t ah[4], al[4];
-      const int at = (kk * 16 + (m >> 1) * 8 + r) * WK + row0 + (m & 1) * 8;
-      rt_ldm_trans(rt_addr(kh + at), ah);
-      rt_ldm_trans(rt_addr(kl + at), al);
+    for (int e = 0; e < 8; ++e) w[e] = k[e] * g;
+    rt_split8(w, hi, lo);
+    *(uint4*)(kh + r * WK + c) = hi; *(uint4*)(kl + r * WK + c) = lo;
+  };
+  if (vec) {
+    // an item: eight lanes of the first half and their partners in the second, or eight lanes that do not turn
+    const int half = a.rot >> 1, pairs = half / 8, items = pairs + (d16 - a.rot) / 8;
+    for (int i = tid; i < n * items; i += 256) {
+      const int r = i / items, x = i % items;
+      const bf16* q_row = q_src + (size_t)(t0 + r) * a.ld;
+      const bf16* k_row = k_src + (size_t)(t0 + r) * a.ld;
+      if (x < pairs) {
+        const int c = 8 * x;
+        const uint4 qa = *(const uint4*)(q_row + c), qb = *(const uint4*)(q_row + c + half);
+        const uint4 ka = *(const uint4*)(k_row + c), kb = *(const uint4*)(k_row + c + half);
+        const float4* cp = (const float4*)(a.cos_t + (size_t)(t0 + r) * half + c);
+        const float4* sp = (const float4*)(a.sin_t + (size_t)(t0 + r) * half + c);
+        float cs[8], sn[8], u[8], v[8], q1[8], q2[8], k1[8], k2[8];
+        *(float4*)cs = cp[0]; *(float4*)(cs + 4) = cp[1];
+        *(float4*)sn = sp[0]; *(float4*)(sn + 4) = sp[1];
+        rt_unpack8(qa, u); rt_unpack8(qb, v);
 #pragma unroll
-      for (int np = 0; np < RT_CB / 16; ++np) {
-        uint32_t b[4];
-        rt_ldm_trans(rt_addr(vs + (kk * 16 + (m & 1) * 8 + r) * WV + np * 16 + (m >> 1) * 8), b);
-        rt_mma(acc[2 * np], ah, b[0], b[1]);
-        rt_mma(acc[2 * np], al, b[0], b[1]);
-        rt_mma(acc[2 * np + 1], ah, b[2], b[3]);
-        rt_mma(acc[2 * np + 1], al, b[2], b[3]);
+        for (int e = 0; e < 8; ++e) { q1[e] = fmaf(-v[e], sn[e], u[e] * cs[e]); q2[e] = fmaf(u[e], sn[e], v[e] * cs[e]); }
+        rt_unpack8(ka, u); rt_unpack8(kb, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          k1[e] = fmaf(-v[e], sn[e], u[e] * cs[e]) * a.k_scale;
+          k2[e] = fmaf(u[e], sn[e], v[e] * cs[e]) * a.k_scale;
+        }
+        put(r, c, q1, k1);
+        put(r, c + half, q2, k2);
+      } else {
+        const int c = a.rot + 8 * (x - pairs);
+        float q[8] = {}, k[8] = {};
+        if (c < d) {
+          rt_unpack8(*(const uint4*)(q_row + c), q);
+          rt_unpack8(*(const uint4*)(k_row + c), k);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) k[e] *= a.k_scale;
+        put(r, c, q, k);
       }
     }
-    const int lo = row0 + (lane >> 2), c = c0 + (lane & 3) * 2;
-    const bool pair = (a.dv & 1) == 0;
+  } else {
+    const int pieces = d16 / 8;
+    for (int i = tid; i < n * pieces; i += 256) {
+      const int r = i / pieces, c = 8 * (i % pieces);
+      float q[8], k[8];
 #pragma unroll
-    for (int i = 0; i < RT_CB / 8; ++i) {
-      const int cc = c + 8 * i;
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int row = lo + 8 * half;
-        if (row >= a.d || cc >= a.dv) continue;
-        float* dst = U + (size_t)row * a.dv + cc;
-        if (pair) *(float2*)dst = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
-        else { dst[0] = acc[i][2 * half]; if (cc + 1 < a.dv) dst[1] = acc[i][2 * half + 1]; }
+      for (int e = 0; e < 8; ++e) {
+        q[e] = c + e < d ? rt_lane<bf16>(a, q_src + (size_t)(t0 + r) * a.ld, c + e, t0 + r) : 0.f;
+        k[e] = c + e < d ? rt_lane<bf16>(a, k_src + (size_t)(t0 + r) * a.ld, c + e, t0 + r) * a.k_scale : 0.f;
       }
+      put(r, c, q, k);
+    }
+  }
+  for (int i = tid; i < (RT_CHUNK - n) * (WK / 8); i += 256) {    // rows behind the chunk's tokens
+    const int r = n + i / (WK / 8), c = 8 * (i % (WK / 8));
+    *(uint4*)(kh + r * WK + c) = make_uint4(0u, 0u, 0u, 0u);
+    *(uint4*)(kl + r * WK + c) = make_uint4(0u, 0u, 0u, 0u);
+  }
+  rt_cp_wait<0>();
+  __syncthreads();
+  float* U = a.chunks + (place * a.heads + h) * d * dvp;
+  const int m = lane >> 3, r = lane & 7;
+  for (int row0 = warp * 16; row0 < d16; row0 += 8 * 16) {
+    // A = k^T: matrices (lanes row0 .. + 7, tokens kk*16 .. + 7), (lanes + 8, same tokens), (lanes, tokens + 8), (both + 8)
+    uint32_t ah[RT_CHUNK / 16][4], al[RT_CHUNK / 16][4];
+#pragma unroll
+    for (int kk = 0; kk < RT_CHUNK / 16; ++kk) {
+      const int at = (kk * 16 + (m >> 1) * 8 + r) * WK + row0 + (m & 1) * 8;
+      rt_ldm_trans(rt_addr(kh + at), ah[kk]);
+      rt_ldm_trans(rt_addr(kl + at), al[kk]);
+    }
+    for (int c0 = 0; c0 < a.dv; c0 += RT_CB) {
+      float acc[RT_CB / 8][4] = {};
+#pragma unroll
+      for (int kk = 0; kk < RT_CHUNK / 16; ++kk) {
+#pragma unroll
+        for (int np = 0; np < RT_CB / 16; ++np) {
+          uint32_t b[4];
+          rt_ldm_trans(rt_addr(vs + (kk * 16 + (m & 1) * 8 + r) * WV + c0 + np * 16 + (m >> 1) * 8), b);
+          rt_mma(acc[2 * np], ah[kk], b[0], b[1]);
+          rt_mma(acc[2 * np], al[kk], b[0], b[1]);
+          rt_mma(acc[2 * np + 1], ah[kk], b[2], b[3]);
+          rt_mma(acc[2 * np + 1], al[kk], b[2], b[3]);
+        }
+      }
+      const int lo = row0 + (lane >> 2), c = c0 + (lane & 3) * 2;
+#pragma unroll
+      for (int i = 0; i < RT_CB / 8; ++i)
+        if (c + 8 * i < dvp) {
+          if (lo < d) *(float2*)(U + (size_t)lo * dvp + c + 8 * i) = make_float2(acc[i][0], acc[i][1]);
+          if (lo + 8 < d) *(float2*)(U + (size_t)(lo + 8) * dvp + c + 8 * i) = make_float2(acc[i][2], acc[i][3]);
+        }
     }
   }
 }
 
-// The state in front of every chunk in place of its sum, and the sequence's new state.
-template <int V>
+// The state in front of every chunk in place of its sum, and the sequence's new state.  A thread takes eight neighbouring
+// columns of a row; what it leaves in their 32 bytes are the eight high parts and then the eight low parts of the state.
 __global__ void __launch_bounds__(128)
 rt_chunk_scan_kernel(RetentionArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  const int seq = blockIdx.z, h = blockIdx.y, size = a.d * a.dv;
-  const int i = V * (blockIdx.x * blockDim.x + threadIdx.x);
-  if (i >= size) return;
+  const int seq = blockIdx.z, h = blockIdx.y, dvp = (a.dv + 7) & ~7;
+  const int i = 8 * (blockIdx.x * blockDim.x + threadIdx.x);
+  if (i >= a.d * dvp) return;
   const int q_begin = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q_begin;
   if (q_len <= 0) return;
-  const int n_chunks = (q_len + RT_CHUNK - 1) / RT_CHUNK;
-  const size_t step = (size_t)a.heads * size;
-  float* p = a.chunks + ((size_t)(q_begin / RT_CHUNK + seq) * a.heads + h) * size + i;
-  float* st = a.state + ((size_t)a.slots[seq] * a.heads + h) * size + i;
+  const int n_chunks = (q_len + RT_CHUNK - 1) / RT_CHUNK, row = i / dvp, c0 = i % dvp;
+  const size_t step = (size_t)a.heads * a.d * dvp;
+  float* p = a.chunks + ((size_t)(q_begin / RT_CHUNK + seq) * a.heads + h) * a.d * dvp + i;
+  float* st = a.state + (((size_t)a.slots[seq] * a.heads + h) * a.d + row) * a.dv + c0;
   const float g = a.decay[h], gc = rt_power(g, RT_CHUNK), gl = rt_power(g, q_len - (n_chunks - 1) * RT_CHUNK);
-  float S[V];
-  auto load = [&](const float* src, float* v) {
-    if (V == 4) { const float4 f = *(const float4*)src; v[0] = f.x; v[1 % V] = f.y; v[2 % V] = f.z; v[3 % V] = f.w; }
-    else v[0] = src[0];
+  const bool whole = (a.dv & 3) == 0 && c0 + 8 <= a.dv && ((uintptr_t)a.state & 15) == 0;
+  float S[8];
+  if (whole) { *(float4*)S = *(const float4*)st; *(float4*)(S + 4) = *(const float4*)(st + 4); }
+  else {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) S[e] = c0 + e < a.dv ? st[e] : 0.f;
+  }
+  auto turn = [&](float* at, const float* u, float w) {
+    uint4 hi, lo;
+    rt_split8(S, hi, lo);
+    *(uint4*)at = hi; *(uint4*)(at + 4) = lo;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) S[e] = fmaf(w, S[e], u[e]);
   };
-  auto store = [&](float* dst, const float* v) {
-    if (V == 4) *(float4*)dst = make_float4(v[0], v[1 % V], v[2 % V], v[3 % V]);
-    else dst[0] = v[0];
-  };
-  load(st, S);
   int c = 0;
-  for (; c + 8 < n_chunks; c += 8) {            // eight loads in flight
-    float u[8][V];
+  for (; c + 4 < n_chunks; c += 4) {            // four chunks' loads in flight
+    float u[4][8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) load(p + (size_t)(c + j) * step, u[j]);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      store(p + (size_t)(c + j) * step, S);
-#pragma unroll
-      for (int e = 0; e < V; ++e) S[e] = fmaf(gc, S[e], u[j][e]);
+    for (int j = 0; j < 4; ++j) {
+      *(float4*)u[j] = *(const float4*)(p + (size_t)(c + j) * step);
+      *(float4*)(u[j] + 4) = *(const float4*)(p + (size_t)(c + j) * step + 4);
     }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) turn(p + (size_t)(c + j) * step, u[j], gc);
   }
   for (; c < n_chunks; ++c) {
-    float u[V];
-    load(p + (size_t)c * step, u);
-    store(p + (size_t)c * step, S);
-    const float w = c + 1 < n_chunks ? gc : gl;
-#pragma unroll
-    for (int e = 0; e < V; ++e) S[e] = fmaf(w, S[e], u[e]);
+    float u[8];
+    *(float4*)u = *(const float4*)(p + (size_t)c * step);
+    *(float4*)(u + 4) = *(const float4*)(p + (size_t)c * step + 4);
+    turn(p + (size_t)c * step, u, c + 1 < n_chunks ? gc : gl);
   }
-  store(st, S);
+  if (whole) { *(float4*)st = *(const float4*)S; *(float4*)(st + 4) = *(const float4*)(S + 4); }
+  else {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) if (c0 + e < a.dv) st[e] = S[e];
+  }
 }
 
 // The read-outs of a chunk's tokens for one head: 8 warps, warp w takes token rows 16 (w % 4) .. + 15 and half w / 4 of the
-// keys (scores) and of the columns of a turn (read-outs).
-__global__ void __launch_bounds__(256)
+// keys (scores) and of the columns of a turn (read-outs).  TURNS turns of 64 columns stay in registers until the norm.
+template <int TURNS>
+__global__ void __launch_bounds__(256, TURNS <= 2 ? 2 : 1)
 rt_chunk_outputs_kernel(RetentionArgs a, int vec) {
   pdl_launch_dependents();
   pdl_wait();
@@ -443,21 +488,32 @@ rt_chunk_outputs_kernel(RetentionArgs a, int vec) {
   size_t place;
   if (!rt_chunk(a, seq, blockIdx.x, t0, n, place)) return;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = a.d, dv = a.dv, d16 = (d + 15) & ~15, WQ = d16 + 8;
-  constexpr int WV = RT_CB + 8, WP = RT_CHUNK + 8;
-  const int turns = (dv + RT_CB - 1) / RT_CB, WO = turns * RT_CB + 4;
+  constexpr int WP = RT_CHUNK + 8, WS = RT_CB + 8, WV = TURNS * RT_CB + 8;
+  const int dvp = (dv + 7) & ~7;
   bf16* qh = (bf16*)rt_bytes;                      // q, high and low [64][WQ]
   bf16* ql = qh + RT_CHUNK * WQ;
   bf16* ph = ql + RT_CHUNK * WQ;                   // decayed scores [64][WP]
   bf16* pl = ph + RT_CHUNK * WP;
-  bf16* vs = pl + RT_CHUNK * WP;                   // a turn's values [64][WV]
-  bf16* un = vs + RT_CHUNK * WV;                   // k [64][WQ] twice, then a turn's state [d16][WV] twice
-  const int un_elems = max(2 * RT_CHUNK * WQ, 2 * d16 * WV);
-  float* o = (float*)(un + un_elems);              // [64][WO]
-  if (tid <= RT_CHUNK) pw[tid] = rt_power(a.decay[h], tid);
-  const bf16* base = (const bf16*)a.proj;
+  bf16* vs = pl + RT_CHUNK * WP;                   // values [64][WV]
+  bf16* un = vs + RT_CHUNK * WV;                   // k [64][WQ] twice, then a turn's state [d16][WS] twice
   bf16 *kh = un, *kl = un + RT_CHUNK * WQ;
-  rt_stage_rows(a, qh, ql, WQ, base + (size_t)h * d, t0, n, 1.f, nullptr, vec, tid, 256);
-  rt_stage_rows(a, kh, kl, WQ, base + (size_t)(a.heads + h) * d, t0, n, a.k_scale, nullptr, vec, tid, 256);
+  const bf16* base = (const bf16*)a.proj;
+  const bf16* v_src = base + (size_t)2 * a.heads * d + (size_t)h * dv;
+  {
+    const bf16* split = (bf16*)a.qk + ((size_t)t0 * a.heads + h) * 4 * d16;
+    const int pieces = d16 / 8;
+    for (int i = tid; i < RT_CHUNK * 4 * pieces; i += 256) {
+      const int r = i / (4 * pieces), x = i % (4 * pieces), which = x / pieces, c = 8 * (x % pieces);
+      bf16* dst = (which < 2 ? qh + which * RT_CHUNK * WQ : kh + (which - 2) * RT_CHUNK * WQ) + r * WQ + c;
+      if (r < n) rt_cp16(dst, split + ((size_t)r * a.heads * 4 + which) * d16 + c);
+      else *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
+    }
+    rt_cp_commit();
+  }
+  rt_stage_values(a, vs, WV, TURNS * RT_CB, v_src, t0, n, vec, tid);
+  rt_cp_commit();
+  if (tid <= RT_CHUNK) pw[tid] = rt_power(a.decay[h], tid);
+  rt_cp_wait<1>();
   __syncthreads();
   const int m = lane >> 3, r = lane & 7, row0 = (warp & 3) * 16, part = warp >> 2;
   const int lo = row0 + (lane >> 2), hi = lo + 8, cq = (lane & 3) * 2;
@@ -497,34 +553,27 @@ rt_chunk_outputs_kernel(RetentionArgs a, int vec) {
       *(uint32_t*)(pl + hi * WP + j) = l2;
     }
   }
-  const float* S = a.chunks + (place * a.heads + h) * d * dv;
-  const bf16* v_src = base + (size_t)2 * a.heads * d + (size_t)h * dv;
-  bf16 *sh = un, *sl = un + d16 * WV;
+  const bf16* S = (const bf16*)(a.chunks + (place * a.heads + h) * d * dvp);     // per eight columns: high parts, low parts
+  bf16 *sh = un, *sl = un + d16 * WS;
+  float out_acc[TURNS][4][4];
   float ss_lo = 0.f, ss_hi = 0.f;
-  for (int turn = 0; turn < turns; ++turn) {
+#pragma unroll
+  for (int turn = 0; turn < TURNS; ++turn) {
     const int c0 = turn * RT_CB;
-    __syncthreads();                               // the scores are written; the turn before has left vs and the state
-    rt_stage_values(a, vs, WV, c0, RT_CB, v_src, t0, n, vec, tid, 256);
+    __syncthreads();                               // the scores are written; k, or the turn before, is done with `un`
     for (int i = tid; i < d16 * (RT_CB / 4); i += 256) {
-      const int row = i / (RT_CB / 4), c = c0 + 4 * (i % (RT_CB / 4));
-      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (row < d) {
-        const float* src = S + (size_t)row * dv + c;
-        if ((dv & 3) == 0) { if (c < dv) f = *(const float4*)src; }
-        else {
-          if (c < dv) f.x = src[0];
-          if (c + 1 < dv) f.y = src[1];
-          if (c + 2 < dv) f.z = src[2];
-          if (c + 3 < dv) f.w = src[3];
-        }
-      }
-      uint2 h2, l2;
-      rt_split2(f.x, f.y, h2.x, l2.x); rt_split2(f.z, f.w, h2.y, l2.y);
-      *(uint2*)(sh + row * WV + c - c0) = h2;
-      *(uint2*)(sl + row * WV + c - c0) = l2;
+      const int row = i / (RT_CB / 4), x = i % (RT_CB / 4), c = 8 * (x >> 1);
+      bf16* dst = ((x & 1) ? sl : sh) + row * WS + c;
+      if (row < d && c0 + c < dvp) rt_cp16(dst, S + 2 * ((size_t)row * dvp + c0 + c) + 8 * (x & 1));
+      else *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
     }
+    rt_cp_commit();
+    rt_cp_wait<0>();
     __syncthreads();
-    float acc[4][4] = {};
+    float (&acc)[4][4] = out_acc[turn];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f; }
+#pragma unroll 2
     for (int ks = 0; ks < d16 / 16; ++ks) {        // S^T q
       uint32_t ah[4], al[4];
       const int at = (row0 + (m & 1) * 8 + r) * WQ + ks * 16 + (m >> 1) * 8;
@@ -533,7 +582,7 @@ rt_chunk_outputs_kernel(RetentionArgs a, int vec) {
 #pragma unroll
       for (int np = 0; np < 2; ++np) {
         uint32_t bh[4], bl[4];
-        const int bt = (ks * 16 + (m & 1) * 8 + r) * WV + part * 32 + np * 16 + (m >> 1) * 8;
+        const int bt = (ks * 16 + (m & 1) * 8 + r) * WS + part * 32 + np * 16 + (m >> 1) * 8;
         rt_ldm_trans(rt_addr(sh + bt), bh);
         rt_ldm_trans(rt_addr(sl + bt), bl);
 #pragma unroll
@@ -555,7 +604,7 @@ rt_chunk_outputs_kernel(RetentionArgs a, int vec) {
 #pragma unroll
       for (int np = 0; np < 2; ++np) {
         uint32_t b[4];
-        rt_ldm_trans(rt_addr(vs + (kk * 16 + (m & 1) * 8 + r) * WV + part * 32 + np * 16 + (m >> 1) * 8), b);
+        rt_ldm_trans(rt_addr(vs + (kk * 16 + (m & 1) * 8 + r) * WV + c0 + part * 32 + np * 16 + (m >> 1) * 8), b);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           rt_mma(acc[2 * np + e], ah, b[2 * e], b[2 * e + 1]);
@@ -565,9 +614,6 @@ rt_chunk_outputs_kernel(RetentionArgs a, int vec) {
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {                  // columns from dv on are zero
-      const int c = c0 + part * 32 + i * 8 + cq;
-      *(float2*)(o + lo * WO + c) = make_float2(acc[i][0], acc[i][1]);
-      *(float2*)(o + hi * WO + c) = make_float2(acc[i][2], acc[i][3]);
       ss_lo = fmaf(acc[i][0], acc[i][0], fmaf(acc[i][1], acc[i][1], ss_lo));
       ss_hi = fmaf(acc[i][2], acc[i][2], fmaf(acc[i][3], acc[i][3], ss_hi));
     }
@@ -579,45 +625,46 @@ rt_chunk_outputs_kernel(RetentionArgs a, int vec) {
   }
   if ((lane & 3) == 0) { sums[part][lo] = ss_lo; sums[part][hi] = ss_hi; }
   __syncthreads();
-  const bf16* gate = v_src + (size_t)a.heads * dv;
-  bf16* out = (bf16*)a.out + (size_t)h * dv;
-  auto factor = [&](int row) {
-    return a.norm ? a.out_scale / sqrtf((sums[0][row] + sums[1][row]) / (float)dv + a.eps) : a.out_scale;
-  };
-  if (vec) {
-    const int pieces = dv / 8;
-    for (int i = tid; i < n * pieces; i += 256) {
-      const int row = i / pieces, c = 8 * (i % pieces);
-      const float inv = factor(row);
-      float z[8];
-      rt_unpack8(*(const uint4*)(gate + (size_t)(t0 + row) * a.ld + c), z);
-      const float* x = o + row * WO + c;
-      const float4 x0 = *(const float4*)x, x1 = *(const float4*)(x + 4);
-      uint4 p;
-      __nv_bfloat162* p2 = (__nv_bfloat162*)&p;
-      p2[0] = __floats2bfloat162_rn(x0.x * inv * rt_silu(z[0]), x0.y * inv * rt_silu(z[1]));
-      p2[1] = __floats2bfloat162_rn(x0.z * inv * rt_silu(z[2]), x0.w * inv * rt_silu(z[3]));
-      p2[2] = __floats2bfloat162_rn(x1.x * inv * rt_silu(z[4]), x1.y * inv * rt_silu(z[5]));
-      p2[3] = __floats2bfloat162_rn(x1.z * inv * rt_silu(z[6]), x1.w * inv * rt_silu(z[7]));
-      *(uint4*)(out + (size_t)(t0 + row) * a.out_ld + c) = p;
-    }
-  } else {
-    for (int i = tid; i < n * dv; i += 256) {
-      const int row = i / dv, c = i % dv;
-      out[(size_t)(t0 + row) * a.out_ld + c] =
-          __float2bfloat16_rn(o[row * WO + c] * factor(row) * rt_silu(__bfloat162float(gate[(size_t)(t0 + row) * a.ld + c])));
-    }
+  // two columns a lane: four lanes write 16 neighbouring bytes
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int row = e ? hi : lo;
+    if (row >= n) continue;
+    const float inv = a.norm ? a.out_scale / sqrtf((sums[0][row] + sums[1][row]) / (float)dv + a.eps) : a.out_scale;
+    const bf16* gate = v_src + (size_t)a.heads * dv + (size_t)(t0 + row) * a.ld;
+    bf16* out = (bf16*)a.out + (size_t)(t0 + row) * a.out_ld + (size_t)h * dv;
+#pragma unroll
+    for (int turn = 0; turn < TURNS; ++turn)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int c = turn * RT_CB + part * 32 + i * 8 + cq;
+        const float x = out_acc[turn][i][2 * e] * inv, y = out_acc[turn][i][2 * e + 1] * inv;
+        if (vec) {
+          if (c < dv) {
+            const float2 z = __bfloat1622float2(*(const __nv_bfloat162*)(gate + c));
+            *(__nv_bfloat162*)(out + c) = __floats2bfloat162_rn(x * rt_silu(z.x), y * rt_silu(z.y));
+          }
+        } else {
+          if (c < dv) out[c] = __float2bfloat16_rn(x * rt_silu(__bfloat162float(gate[c])));
+          if (c + 1 < dv) out[c + 1] = __float2bfloat16_rn(y * rt_silu(__bfloat162float(gate[c + 1])));
+        }
+      }
   }
 }
 
-static size_t rt_sums_smem(int d) {
+// Turns that chunk_outputs is compiled for.
+static int rt_turns(int dv) {
+  const int t = (dv + RT_CB - 1) / RT_CB;
+  return t <= 1 ? 1 : (t <= 2 ? 2 : (t <= 4 ? 4 : 8));
+}
+static size_t rt_sums_smem(int d, int dv) {
   const int d16 = (d + 15) & ~15;
-  return sizeof(bf16) * (size_t)RT_CHUNK * (2 * (d16 + 8) + RT_CB + 8);
+  return sizeof(bf16) * (size_t)RT_CHUNK * (2 * (d16 + 8) + (dv + RT_CB - 1) / RT_CB * RT_CB + 8);
 }
 static size_t rt_outputs_smem(int d, int dv) {
-  const int d16 = (d + 15) & ~15, WQ = d16 + 8, turns = (dv + RT_CB - 1) / RT_CB;
-  const size_t un = 2 * (size_t)RT_CHUNK * WQ > 2 * (size_t)d16 * (RT_CB + 8) ? 2 * (size_t)RT_CHUNK * WQ : 2 * (size_t)d16 * (RT_CB + 8);
-  return sizeof(bf16) * ((size_t)RT_CHUNK * (2 * WQ + 2 * (RT_CHUNK + 8) + RT_CB + 8) + un) + sizeof(float) * (size_t)RT_CHUNK * (turns * RT_CB + 4);
+  const int d16 = (d + 15) & ~15, WQ = d16 + 8;
+  const size_t k = 2 * (size_t)RT_CHUNK * WQ, state = 2 * (size_t)d16 * (RT_CB + 8);
+  return sizeof(bf16) * ((size_t)RT_CHUNK * (2 * WQ + 2 * (RT_CHUNK + 8) + rt_turns(dv) * RT_CB + 8) + (k > state ? k : state));
 }
 #define RT_SMEM_LIMIT (220 * 1024)
 
@@ -631,7 +678,9 @@ static int rt_walk_columns(int d, int dv) {
 }
 
 // Whether prompts of these heads can take the chunk form (bf16).
-extern "C" int odi_retention_takes_chunks(int d, int dv) { return rt_outputs_smem(d, dv) <= RT_SMEM_LIMIT && d <= 1024; }
+extern "C" int odi_retention_takes_chunks(int d, int dv) {
+  return dv <= 8 * RT_CB && rt_outputs_smem(d, dv) <= RT_SMEM_LIMIT && rt_sums_smem(d, dv) <= RT_SMEM_LIMIT;
+}
 
 template <typename K>
 static int rt_configure(K kernel, size_t smem) {
@@ -659,23 +708,30 @@ static int launch_in_order(const RetentionArgs& a, cudaStream_t stream) {
   return rc;
 }
 
+template <int TURNS>
+static int launch_outputs(const RetentionArgs& a, int n_chunks, int vec, cudaStream_t stream) {
+  const size_t smem = rt_outputs_smem(a.d, a.dv);
+  const int rc = rt_configure(rt_chunk_outputs_kernel<TURNS>, smem);
+  return rc != 0 ? rc : launch_pdl(rt_chunk_outputs_kernel<TURNS>, dim3(n_chunks, a.heads, a.n_seqs), dim3(256), smem, stream, a, vec);
+}
+
 static int launch_chunks(const RetentionArgs& a, cudaStream_t stream) {
-  const int half = a.rot / 2, n_chunks = (a.max_q_len + RT_CHUNK - 1) / RT_CHUNK, col_blocks = (a.dv + RT_CB - 1) / RT_CB;
+  const int half = a.rot / 2, n_chunks = (a.max_q_len + RT_CHUNK - 1) / RT_CHUNK;
   const int vec = a.d % 8 == 0 && a.dv % 8 == 0 && a.ld % 8 == 0 && a.out_ld % 8 == 0 &&
                   (a.cos_t == nullptr || (!a.interleaved && half % 8 == 0)) &&
                   (((uintptr_t)a.proj | (uintptr_t)a.out | (uintptr_t)a.cos_t | (uintptr_t)a.sin_t) & 15) == 0;
-  const size_t s1 = rt_sums_smem(a.d), s3 = rt_outputs_smem(a.d, a.dv);
+  const size_t s1 = rt_sums_smem(a.d, a.dv);
   int rc = rt_configure(rt_chunk_sums_kernel, s1);
-  if (rc == 0) rc = rt_configure(rt_chunk_outputs_kernel, s3);
-  if (rc == 0) rc = launch_pdl(rt_chunk_sums_kernel, dim3(n_chunks, a.heads * col_blocks, a.n_seqs), dim3(256), s1, stream, a, vec);
-  const int size = a.d * a.dv;
-  const bool wide = size % 4 == 0 && (((uintptr_t)a.chunks | (uintptr_t)a.state) & 15) == 0;
-  const int items = wide ? size / 4 : size;
-  if (rc == 0)
-    rc = launch_pdl(wide ? rt_chunk_scan_kernel<4> : rt_chunk_scan_kernel<1>, dim3((items + 127) / 128, a.heads, a.n_seqs), dim3(128), 0,
-                    stream, a);
-  if (rc == 0) rc = launch_pdl(rt_chunk_outputs_kernel, dim3(n_chunks, a.heads, a.n_seqs), dim3(256), s3, stream, a, vec);
-  return rc;
+  if (rc == 0) rc = launch_pdl(rt_chunk_sums_kernel, dim3(n_chunks, a.heads, a.n_seqs), dim3(256), s1, stream, a, vec);
+  const int items = a.d * ((a.dv + 7) / 8);
+  if (rc == 0) rc = launch_pdl(rt_chunk_scan_kernel, dim3((items + 127) / 128, a.heads, a.n_seqs), dim3(128), 0, stream, a);
+  if (rc != 0) return rc;
+  switch (rt_turns(a.dv)) {
+    case 1: return launch_outputs<1>(a, n_chunks, vec, stream);
+    case 2: return launch_outputs<2>(a, n_chunks, vec, stream);
+    case 4: return launch_outputs<4>(a, n_chunks, vec, stream);
+    default: return launch_outputs<8>(a, n_chunks, vec, stream);
+  }
 }
 
 // form 0: tokens in order; 1: chunks side by side (bf16; `chunks` holds their states).
@@ -684,9 +740,9 @@ extern "C" int odi_retention(const RetentionArgs* args, int form, int dtype, cud
   if (a.n_tokens <= 0 || a.n_seqs <= 0) return 0;
   if (a.heads <= 0 || a.d <= 0 || a.dv <= 0 || a.rot < 0 || a.rot > a.d || (a.rot & 1)) return ODI_ERR_ARGUMENT;
   if (a.cos_t == nullptr) a.rot = 0;
-  if (a.heads > 65535 || a.n_seqs > 65535 || (long)a.heads * ((a.dv + RT_CB - 1) / RT_CB) > 65535) return ODI_ERR_UNSUPPORTED;
+  if (a.heads > 65535 || a.n_seqs > 65535) return ODI_ERR_UNSUPPORTED;
   if (form == 1) {
-    if (dtype != 1 || a.chunks == nullptr || !odi_retention_takes_chunks(a.d, a.dv)) return ODI_ERR_UNSUPPORTED;
+    if (dtype != 1 || a.chunks == nullptr || a.qk == nullptr || !odi_retention_takes_chunks(a.d, a.dv)) return ODI_ERR_UNSUPPORTED;
     odi_rc = launch_chunks(a, stream);
   } else {
     if (a.max_q_len > 1 && a.o == nullptr) return ODI_ERR_ARGUMENT;

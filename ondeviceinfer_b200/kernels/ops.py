@@ -2114,8 +2114,8 @@ def stream_mix(x: torch.Tensor, *, streams: int, y: Optional[torch.Tensor] = Non
 
 class _RetentionArgs(Structure):
     _fields_ = [("proj", c_void_p), ("cos_t", c_void_p), ("sin_t", c_void_p), ("decay", c_void_p), ("state", c_void_p),
-                ("chunks", c_void_p), ("o", c_void_p), ("out", c_void_p), ("cu_q", c_void_p), ("tok_seq", c_void_p),
-                ("slots", c_void_p), ("n_tokens", c_int), ("n_seqs", c_int), ("max_q_len", c_int), ("ld", c_int),
+                ("chunks", c_void_p), ("qk", c_void_p), ("o", c_void_p), ("out", c_void_p), ("cu_q", c_void_p),
+                ("tok_seq", c_void_p), ("slots", c_void_p), ("n_tokens", c_int), ("n_seqs", c_int), ("max_q_len", c_int), ("ld", c_int),
                 ("heads", c_int), ("d", c_int), ("dv", c_int), ("rot", c_int), ("interleaved", c_int), ("out_ld", c_int),
                 ("norm", c_int), ("eps", c_float), ("k_scale", c_float), ("out_scale", c_float)]
 
@@ -2151,12 +2151,13 @@ def retention(proj: torch.Tensor, cos_t, sin_t, decay: torch.Tensor, state: torc
     if chunked is None:
         chunked = max_q_len >= RETENTION_MIN_CHUNK_TOKENS
     chunked = chunked and proj.dtype == torch.bfloat16 and bool(lib.odi_retention_takes_chunks(c_int(d), c_int(dv)))
-    chunks = o = None
+    chunks = qk = o = None
     if chunked:
-        chunks = torch.empty((n // RETENTION_CHUNK + n_seqs, heads, d, dv), dtype=torch.float32, device=proj.device)
+        chunks = torch.empty((n // RETENTION_CHUNK + n_seqs, heads, d, -(-dv // 8) * 8), dtype=torch.float32, device=proj.device)
+        qk = torch.empty((n, heads, 4, -(-d // 16) * 16), dtype=torch.bfloat16, device=proj.device)
     elif max_q_len > 1:
         o = torch.empty((n, heads * dv), dtype=torch.float32, device=proj.device)
-    args = _RetentionArgs(_at_column(proj, col), _ptr(cos_t), _ptr(sin_t), _ptr(decay), _ptr(state), _ptr(chunks), _ptr(o),
+    args = _RetentionArgs(_at_column(proj, col), _ptr(cos_t), _ptr(sin_t), _ptr(decay), _ptr(state), _ptr(chunks), _ptr(qk), _ptr(o),
                           _at_column(out, out_col), _ptr(cu_q), _ptr(tok_seq), _ptr(slots), n, n_seqs, max_q_len, proj.shape[1],
                           heads, d, dv, rot if cos_t is not None else 0, 1 if interleaved else 0, out.shape[1],
                           0 if eps is None else 1, 0.0 if eps is None else eps, d ** -0.5, out_scale)

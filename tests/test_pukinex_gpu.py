@@ -302,7 +302,7 @@ def test_attention_of_unequal_sequences_in_one_launch(kind, nq, nkv, d):
 @pytest.mark.parametrize("decay,d,dv,rot,inter", [((0.9, 0.99, 0.5), 32, 48, 32, False), ((0.97,), 10, 7, 6, False), ((0.999, 0.0), 24, 40, 8, True),
                                                   ((1.0, 0.95), 64, 33, 0, False), ((0.98, 0.9), 128, 128, 128, False), ((0.99,), 130, 5, 64, False),
                                                   ((0.9, 0.8, 0.99, 0.7), 16, 130, 16, False), ((0.95,), 256, 64, 128, False),
-                                                  ((0.96,), 96, 200, 48, False)])
+                                                  ((0.96,), 96, 200, 48, False), ((0.9,), 24, 300, 16, False)])
 def test_retention_over_cut_sequences(dtype, chunked, decay, d, dv, rot, inter):
     """Three sequences cut into unequal runs (single tokens, short portions, several chunks, chunks with tokens left over),
     stepped together with states in slots of their own, in columns of wider buffers, against the recurrence over each whole
