@@ -138,6 +138,7 @@ __global__ void rot_unit_prep_vec_kernel(RotUnitArgs a, int heads_per_warp) {
   const size_t row = a.ld;
   const bf16* base = (const bf16*)a.qkv + (size_t)t * row;
   const int pos = a.tok_pos[t];
+  const bool wide_v = a.dv % 4 == 0 && ((uintptr_t)a.v_pool & 7) == 0;
   size_t at = 0;
   if (a.write_kv) {
     const int s = a.tok_seq[t];
@@ -150,7 +151,8 @@ __global__ void rot_unit_prep_vec_kernel(RotUnitArgs a, int heads_per_warp) {
       const int hk = h - a.nq - a.nkv;
       const bf16* src = a.v_from_k ? base + (size_t)(a.nq + hk) * d : base + (size_t)(a.nq + a.nkv) * d + (size_t)hk * a.dv;
       bf16* dst = (bf16*)a.v_pool + (at + (size_t)hk * a.page_size) * a.dv;
-      for (int i = lane; i < a.dv; i += 32) dst[i] = src[i];
+      if (wide_v) { for (int i = 4 * lane; i < a.dv; i += 128) *(uint2*)(dst + i) = *(const uint2*)(src + i); }
+      else { for (int i = lane; i < a.dv; i += 32) dst[i] = src[i]; }
       continue;
     }
     const int hk = h - a.nq;

@@ -20,6 +20,7 @@
 #include "common.cuh"
 
 #define RT_CHUNK 64
+#define RT_CB 64            // columns of the values per turn
 
 struct RetentionArgs {
   const void* proj;       // [n_tokens, ld] in T, from this mixer's first column on: q (H d), k (H d), v (H dv), gate (H dv)
@@ -69,9 +70,12 @@ __device__ __forceinline__ float rt_silu(float z) { return z / (1.f + expf(-z));
 
 // ------------------------------------------------------------------------------ one token per sequence
 
-// V columns a thread per access; threads tid / (dv / V) take the rows in turn.
-template <typename T, int V>
-__global__ void __launch_bounds__(256)
+#define RT_STEP_ROWS 8      // rows of the state that a thread has in flight
+
+// V columns a thread per access; the threads of a column take its rows in turn.  What the block needs from memory (rows of
+// the state, values, gates, q and k) is requested before anything waits.
+template <typename T, int V, int THREADS>
+__global__ void __launch_bounds__(THREADS)
 rt_step_kernel(RetentionArgs a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -81,56 +85,77 @@ rt_step_kernel(RetentionArgs a) {
   const int t = a.cu_q[seq], slot = a.slots[seq];
   float* qs = rt_smem;                   // [d]
   float* ks = qs + d;                    // [d]
-  float* part = ks + d + ((4 - (2 * d & 3)) & 3);      // [row groups][columns], aligned
+  float* part = ks + d;                  // [row groups][columns]
   const T* base = (const T*)a.proj + (size_t)t * a.ld;
-  for (int i = tid; i < 2 * d; i += blockDim.x) {
-    const bool is_k = i >= d;
-    const T* row = base + (size_t)((is_k ? a.heads : 0) + h) * d;
-    const float x = rt_lane<T>(a, row, is_k ? i - d : i, t);
-    if (is_k) ks[i - d] = x * a.k_scale; else qs[i] = x;
-  }
   const T* v_row = base + (size_t)2 * a.heads * d + (size_t)h * dv;
   const T* gate = v_row + (size_t)a.heads * dv;
   float* S = a.state + ((size_t)slot * a.heads + h) * d * dv;
+  // columns in passes of at most one access a thread
+  const int nc = (dv + V - 1) / V, cols = min(nc, THREADS), groups = THREADS / cols, grp = tid / cols;
   const float g = a.decay[h];
-  __syncthreads();
-  // columns in passes of at most `cols` accesses, so that every thread has one
-  const int nc = (dv + V - 1) / V, cols = min(nc, (int)blockDim.x), groups = blockDim.x / cols;
-  float ss = 0.f;
+  const float z0 = tid < dv ? to_f<T>(gate[tid]) : 0.f;
+  auto load = [&](float (&x)[RT_STEP_ROWS][V], int c, int r0) {
+#pragma unroll
+    for (int j = 0; j < RT_STEP_ROWS; ++j) {
+      const int r = r0 + j * groups;
+      if (r < d) {
+        const float* p = S + (size_t)r * dv + c * V;
+        if (V == 4) { const float4 f = *(const float4*)p; x[j][0] = f.x; x[j][1 % V] = f.y; x[j][2 % V] = f.z; x[j][3 % V] = f.w; }
+        else x[j][0] = p[0];
+      }
+    }
+  };
   for (int c0 = 0; c0 < nc; c0 += cols) {
-    const int c = c0 + tid % cols, grp = tid / cols;
+    const int c = c0 + tid % cols;
     const bool live = c < nc && grp < groups;
-    float o[V] = {}, v[V];
+    float x[RT_STEP_ROWS][V], o[V] = {}, v[V];
     if (live) {
+      load(x, c, grp);
 #pragma unroll
       for (int e = 0; e < V; ++e) v[e] = to_f<T>(v_row[c * V + e]);
-#pragma unroll 8
-      for (int r = grp; r < d; r += groups) {
-        float* p = S + (size_t)r * dv + c * V;
-        float x[V];
-        if (V == 4) { const float4 f = *(const float4*)p; x[0] = f.x; x[1 % V] = f.y; x[2 % V] = f.z; x[3 % V] = f.w; }
-        else x[0] = p[0];
-        const float k = ks[r], q = qs[r];
+    }
+    if (c0 == 0) {
+      for (int i = tid; i < 2 * d; i += THREADS) {
+        const bool is_k = i >= d;
+        const T* row = base + (size_t)((is_k ? a.heads : 0) + h) * d;
+        const float y = rt_lane<T>(a, row, is_k ? i - d : i, t);
+        if (is_k) ks[i - d] = y * a.k_scale; else qs[i] = y;
+      }
+      __syncthreads();
+    }
+    if (live) {
+      for (int r0 = grp; r0 < d; r0 += RT_STEP_ROWS * groups) {
+        if (r0 != grp) load(x, c, r0);
 #pragma unroll
-        for (int e = 0; e < V; ++e) { x[e] = fmaf(g, x[e], k * v[e]); o[e] = fmaf(q, x[e], o[e]); }
-        if (V == 4) *(float4*)p = make_float4(x[0], x[1 % V], x[2 % V], x[3 % V]);
-        else p[0] = x[0];
+        for (int j = 0; j < RT_STEP_ROWS; ++j) {
+          const int r = r0 + j * groups;
+          if (r < d) {
+            float* p = S + (size_t)r * dv + c * V;
+            const float k = ks[r], q = qs[r];
+#pragma unroll
+            for (int e = 0; e < V; ++e) { x[j][e] = fmaf(g, x[j][e], k * v[e]); o[e] = fmaf(q, x[j][e], o[e]); }
+            if (V == 4) *(float4*)p = make_float4(x[j][0], x[j][1 % V], x[j][2 % V], x[j][3 % V]);
+            else p[0] = x[j][0];
+          }
+        }
       }
 #pragma unroll
       for (int e = 0; e < V; ++e) part[((size_t)grp * nc + c) * V + e] = o[e];
     }
   }
   __syncthreads();
-  for (int i = tid; i < dv; i += blockDim.x) {
+  float ss = 0.f, first = 0.f;           // a thread's first column stays in a register
+  for (int i = tid; i < dv; i += THREADS) {
     float x = part[i];
     for (int r = 1; r < groups; ++r) x += part[(size_t)r * nc * V + i];
-    part[i] = x;
+    if (i == tid) first = x; else part[i] = x;
     ss = fmaf(x, x, ss);
   }
   float inv = a.out_scale;
   if (a.norm) inv *= 1.0f / sqrtf(block_sum(ss, scratch) / (float)dv + a.eps);
   T* out = (T*)a.out + (size_t)t * a.out_ld + (size_t)h * dv;
-  for (int i = tid; i < dv; i += blockDim.x) out[i] = from_f<T>(part[i] * inv * rt_silu(to_f<T>(gate[i])));
+  for (int i = tid; i < dv; i += THREADS)
+    out[i] = from_f<T>((i == tid ? first : part[i]) * inv * rt_silu(i == tid ? z0 : to_f<T>(gate[i])));
 }
 
 // ------------------------------------------------------------------------------ tokens in order
@@ -265,10 +290,11 @@ __device__ __forceinline__ void rt_cp_commit() { asm volatile("cp.async.commit_g
 template <int N> __device__ __forceinline__ void rt_cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // The head's values of a chunk into [64][W] rows; rows from n on and columns from dv to `cols` (a multiple of 16) are zero.
-// With `vec` by asynchronous copies (the caller commits and waits).
+// With `vec` by asynchronous copies (the caller commits and waits).  TURNS > 0: `cols` is TURNS * RT_CB.
+template <int TURNS>
 __device__ __forceinline__ void rt_stage_values(const RetentionArgs& a, bf16* dst, int W, int cols, const bf16* src, int t0, int n,
                                                 int vec, int tid) {
-  const int pieces = cols / 8;
+  const int pieces = TURNS > 0 ? TURNS * (RT_CB / 8) : cols / 8;
   for (int i = tid; i < RT_CHUNK * pieces; i += 256) {
     const int r = i / pieces, c = 8 * (i % pieces);
     const bf16* row = src + (size_t)(t0 + r) * a.ld + c;
@@ -283,8 +309,6 @@ __device__ __forceinline__ void rt_stage_values(const RetentionArgs& a, bf16* ds
     *(uint4*)to = v;
   }
 }
-
-#define RT_CB 64            // columns of the values per turn
 
 // A chunk of one head: q and k rotated, k scaled, both split, into `qk` for rt_chunk_outputs; and the sum of its k v^T, each
 // token weighed by g^(tokens behind it), into `chunks`.  A block's 8 warps take 16 key lanes each at a time.
@@ -304,7 +328,7 @@ rt_chunk_sums_kernel(RetentionArgs a, int vec) {
   bf16* kl = kh + RT_CHUNK * WK;
   bf16* vs = kl + RT_CHUNK * WK;                   // [64][WV]
   const bf16* base = (const bf16*)a.proj;
-  rt_stage_values(a, vs, WV, turns * RT_CB, base + (size_t)2 * a.heads * d + (size_t)h * a.dv, t0, n, vec, tid);
+  rt_stage_values<0>(a, vs, WV, turns * RT_CB, base + (size_t)2 * a.heads * d + (size_t)h * a.dv, t0, n, vec, tid);
   rt_cp_commit();
   if (tid <= RT_CHUNK) pw[tid] = rt_power(a.decay[h], tid);
   __syncthreads();
@@ -487,30 +511,30 @@ rt_chunk_outputs_kernel(RetentionArgs a, int vec) {
   int t0, n;
   size_t place;
   if (!rt_chunk(a, seq, blockIdx.x, t0, n, place)) return;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = a.d, dv = a.dv, d16 = (d + 15) & ~15, WQ = d16 + 8;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = a.d, dv = a.dv, d16 = (d + 15) & ~15, WQ = 2 * d16 + 8;
   constexpr int WP = RT_CHUNK + 8, WS = RT_CB + 8, WV = TURNS * RT_CB + 8;
   const int dvp = (dv + 7) & ~7;
-  bf16* qh = (bf16*)rt_bytes;                      // q, high and low [64][WQ]
-  bf16* ql = qh + RT_CHUNK * WQ;
-  bf16* ph = ql + RT_CHUNK * WQ;                   // decayed scores [64][WP]
+  bf16* qh = (bf16*)rt_bytes;                      // q, high and then low parts in a row [64][WQ]
+  bf16* ql = qh + d16;
+  bf16* ph = qh + RT_CHUNK * WQ;                   // decayed scores [64][WP]
   bf16* pl = ph + RT_CHUNK * WP;
   bf16* vs = pl + RT_CHUNK * WP;                   // values [64][WV]
-  bf16* un = vs + RT_CHUNK * WV;                   // k [64][WQ] twice, then a turn's state [d16][WS] twice
-  bf16 *kh = un, *kl = un + RT_CHUNK * WQ;
+  bf16* un = vs + RT_CHUNK * WV;                   // k [64][WQ] like q, then a turn's state [d16][WS] twice
+  bf16 *kh = un, *kl = un + d16;
   const bf16* base = (const bf16*)a.proj;
   const bf16* v_src = base + (size_t)2 * a.heads * d + (size_t)h * dv;
   {
     const bf16* split = (bf16*)a.qk + ((size_t)t0 * a.heads + h) * 4 * d16;
-    const int pieces = d16 / 8;
-    for (int i = tid; i < RT_CHUNK * 4 * pieces; i += 256) {
-      const int r = i / (4 * pieces), x = i % (4 * pieces), which = x / pieces, c = 8 * (x % pieces);
-      bf16* dst = (which < 2 ? qh + which * RT_CHUNK * WQ : kh + (which - 2) * RT_CHUNK * WQ) + r * WQ + c;
-      if (r < n) rt_cp16(dst, split + ((size_t)r * a.heads * 4 + which) * d16 + c);
-      else *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
-    }
+    const int half = d16 / 4;                      // 16-byte pieces of q (and of k) in a token's row
+    for (int r = warp; r < RT_CHUNK; r += 8)
+      for (int x = lane; x < 2 * half; x += 32) {
+        bf16* dst = (x < half ? qh + 8 * x : kh + 8 * (x - half)) + r * WQ;
+        if (r < n) rt_cp16(dst, split + (size_t)r * a.heads * 4 * d16 + 8 * x);
+        else *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
+      }
     rt_cp_commit();
   }
-  rt_stage_values(a, vs, WV, TURNS * RT_CB, v_src, t0, n, vec, tid);
+  rt_stage_values<TURNS>(a, vs, WV, TURNS * RT_CB, v_src, t0, n, vec, tid);
   rt_cp_commit();
   if (tid <= RT_CHUNK) pw[tid] = rt_power(a.decay[h], tid);
   rt_cp_wait<1>();
@@ -662,9 +686,9 @@ static size_t rt_sums_smem(int d, int dv) {
   return sizeof(bf16) * (size_t)RT_CHUNK * (2 * (d16 + 8) + (dv + RT_CB - 1) / RT_CB * RT_CB + 8);
 }
 static size_t rt_outputs_smem(int d, int dv) {
-  const int d16 = (d + 15) & ~15, WQ = d16 + 8;
-  const size_t k = 2 * (size_t)RT_CHUNK * WQ, state = 2 * (size_t)d16 * (RT_CB + 8);
-  return sizeof(bf16) * ((size_t)RT_CHUNK * (2 * WQ + 2 * (RT_CHUNK + 8) + rt_turns(dv) * RT_CB + 8) + (k > state ? k : state));
+  const int d16 = (d + 15) & ~15, WQ = 2 * d16 + 8;
+  const size_t k = (size_t)RT_CHUNK * WQ, state = 2 * (size_t)d16 * (RT_CB + 8);
+  return sizeof(bf16) * ((size_t)RT_CHUNK * (WQ + 2 * (RT_CHUNK + 8) + rt_turns(dv) * RT_CB + 8) + (k > state ? k : state));
 }
 #define RT_SMEM_LIMIT (220 * 1024)
 
@@ -691,13 +715,14 @@ static int rt_configure(K kernel, size_t smem) {
 template <typename T>
 static int launch_in_order(const RetentionArgs& a, cudaStream_t stream) {
   if (a.max_q_len == 1) {
-    const bool vec = a.dv % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
-    const int V = vec ? 4 : 1, nc = (a.dv + V - 1) / V, cols = nc < 256 ? nc : 256, groups = 256 / cols;
-    const size_t smem = sizeof(float) * (2 * (size_t)a.d + 4 + (size_t)groups * nc * V);
+    const bool vec = a.dv % 4 == 0 && ((uintptr_t)a.state & 15) == 0, big = vec && (long)a.d * a.dv > 8192;
+    const int V = vec ? 4 : 1, threads = big ? 512 : 256, nc = (a.dv + V - 1) / V, cols = nc < threads ? nc : threads,
+              groups = threads / cols;
+    const size_t smem = sizeof(float) * (2 * (size_t)a.d + (size_t)groups * nc * V);
     if (smem > 200 * 1024) return ODI_ERR_UNSUPPORTED;
-    auto kernel = vec ? rt_step_kernel<T, 4> : rt_step_kernel<T, 1>;
+    auto kernel = big ? rt_step_kernel<T, 4, 512> : vec ? rt_step_kernel<T, 4, 256> : rt_step_kernel<T, 1, 256>;
     const int rc = rt_configure(kernel, smem);
-    return rc != 0 ? rc : launch_pdl(kernel, dim3(a.heads, a.n_seqs), dim3(256), smem, stream, a);
+    return rc != 0 ? rc : launch_pdl(kernel, dim3(a.heads, a.n_seqs), dim3(threads), smem, stream, a);
   }
   const int cb = rt_walk_columns(a.d, a.dv);
   if (cb == 0) return ODI_ERR_UNSUPPORTED;
