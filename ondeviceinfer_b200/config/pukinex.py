@@ -194,7 +194,9 @@ class PukinexConfig:
         layers: List[StreamMixBlockSpec] = []
         ignored: List[str] = []
         streams = self.streams or 1
-        mix = lambda i, q: None if self.streams is None else tuple(f"l{i}.hc{q}.{role}" for role in ("in", "out", "mix"))
+        # one stream may come without coefficients: the plain residual sum
+        plain = self.streams is None or (self.streams == 1 and bool(stored) and not any(".hc1." in name for name in stored))
+        mix = lambda i, q: None if plain else tuple(f"l{i}.hc{q}.{role}" for role in ("in", "out", "mix"))
         for i, layer in enumerate(self.layers):
             mlp = self._mlp(i, layer)
             has = mlp is not None

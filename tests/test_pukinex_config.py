@@ -79,6 +79,15 @@ def test_the_checkpoint_gives_the_rows_of_a_distance_table():
     assert config.to_plan().layers[0].mixer.left.bias_rows == 32
 
 
+def test_one_stream_comes_with_or_without_coefficients():
+    cfg = dict(copy.deepcopy(plain.TINY_C), streams=1)
+    stored_of = lambda c: {name: StoredTensor(shape=shape, dtype=torch.bfloat16) for name, shape in plain.tensor_shapes(c).items()}
+    with_them = config_from_dict(cfg).plan_for(stored_of(cfg))
+    assert with_them.layers[0].mixer_names == ("l0.hc1.in", "l0.hc1.out", "l0.hc1.mix")
+    assert config_from_dict(cfg).plan_for(stored_of(plain.TINY_C)).layers[0].mixer_names is None
+    assert config_from_dict(cfg).to_plan().layers[0].mixer_names is not None
+
+
 def test_every_pass_of_a_loop_keeps_a_cache_of_its_own():
     model = DecoderModel(config_from_dict(plain.TINY_A).to_plan())
     assert model.layers[0].cache_needs() == (KVNeed(2, 32, None, value_dim=24), StateNeed((3, 24, 40), torch.float32, "retention state"))
