@@ -266,7 +266,7 @@ TINY_B = _config(97, 90, [
     (_parallel(_left(5, 1, 18, 30, 0.2, 2, 9, (0.5, 7)), _right((0.7,), 33, 5), 1.0, 1.0), 10)],
     streams=3, scale=2.0, logit_scale=1.9, eps=1e-6)
 # one plain stream, heads of 64 lanes, nothing optional
-TINY_C = _config(120, 64, [(_attention(4, 2, 64, 0.12), 48), (_parallel(_left(4, 2, 64, 64, 0.13, 16, 100), _right((0.98, 0.9), 32, 64)), 40),
+TINY_C = _config(120, 64, [(_attention(4, 2, 64, 0.12), 48), (_parallel(_left(4, 2, 64, 64, 0.13, 16, 100), _right((0.98, 0.9), 40, 96)), 40),
                            (_attention(2, 2, 64, 0.1, 10.0, _rot(10000.0, 32, 2.0)), None)])
 # heads of 128, 96 and 80 lanes, six streams, a loop over everything
 TINY_D = _config(200, 160, [

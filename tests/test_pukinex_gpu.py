@@ -261,7 +261,7 @@ def test_attention_with_a_distance_bias_a_sink_and_a_gate(kind, dtype, rows, rea
 @pytest.mark.parametrize("nq,nkv,d", [(8, 4, 128), (6, 3, 64), (4, 4, 128)])
 def test_attention_of_unequal_sequences_in_one_launch(kind, nq, nkv, d):
     gen = torch.Generator().manual_seed(3)
-    dtype, rows, reach = torch.bfloat16, 16, 120
+    dtype, rows, reach = torch.bfloat16, 18, 110
     table = torch.randn(rows, nq, generator=gen)
     rel = table[torch.tensor(distance_entries(rows, reach))].t().contiguous().cuda()
     runs, pasts = [70, 1, 200, 33], [0, 99, 40, 300]
@@ -358,7 +358,7 @@ def test_prompts_of_bfloat16_take_the_chunks_where_shared_memory_holds_them():
     from ctypes import c_int
     from ondeviceinfer_b200.kernels.build import load_library
     takes = load_library("retention").odi_retention_takes_chunks
-    assert takes(c_int(128), c_int(128)) and takes(c_int(32), c_int(64)) and takes(c_int(256), c_int(128))
+    assert takes(c_int(128), c_int(128)) and takes(c_int(48), c_int(96)) and takes(c_int(256), c_int(128))
     assert not takes(c_int(1024), c_int(64))
 
 
